@@ -695,13 +695,25 @@ B200_API int b200_sink_attn_prepare(float* q_out, const void* q_in, const void* 
                                     const int32_t* positions, const int32_t* slots, int64_t rows, int64_t H, int64_t G,
                                     int64_t dim, int64_t vdim, float eps, float temp_coef, int64_t temp_every,
                                     int dtype, b200_stream_t stream);
+/* Per token: q = q_in / sqrt(mean(q_in^2) + eps) * q_weight over ALL H * dim channels at once, k likewise over its
+ * G * dim; then the first rot_dims channels of every head turn (channel t with t + rot_dims / 2, angle position *
+ * inv_freq[t], fp32).  q_out fp32 [rows, H, dim]; k and v_in (unchanged) go to the cache rows `slots`.  q_in / k_in /
+ * v_in: column blocks of one matrix (row stride ld); weights fp32. */
+B200_API int b200_sink_attn_prepare_turned(float* q_out, const void* q_in, const void* k_in, const void* v_in, int64_t ld,
+                                           const float* q_weight, const float* k_weight,
+                                           const float* inv_freq /*nullable*/, void* k_cache, void* v_cache,
+                                           const int32_t* positions, const int32_t* slots, int64_t rows, int64_t H,
+                                           int64_t G, int64_t dim, int64_t vdim, int64_t rot_dims, float eps, int dtype,
+                                           b200_stream_t stream);
 /* out[row, h] = sum_j p_j v_j over the cached rows j <= position i of the row (paged), p_j = exp(s_j) /
  * (exp(sink[h]) + sum_j' exp(s_j')), s_j = scale q . k_j - r1[h] ln(1 + r2[h] (i - j)).  r1 / r2 (both or
- * neither) and sink are fp32 [H], nullable.  q fp32 [rows, H, dim]; caches [slots, G, dim] and [slots, G, vdim]
+ * neither) and sink are fp32 [H], nullable.  What is stored is out_mul * out * sigmoid(gate[row, h * vdim + c]) (gate:
+ * rows of type T with stride ld_gate, nullable).  q fp32 [rows, H, dim]; caches [slots, G, dim] and [slots, G, vdim]
  * of type `dtype`; CUDA cores, any sizes. */
 B200_API int b200_sink_attn(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache,
                             const float* r1 /*nullable*/, const float* r2 /*nullable*/,
-                            const float* sink /*nullable*/, const int32_t* q_cu_lens, const int32_t* kv_cu_lens,
+                            const float* sink /*nullable*/, const void* gate /*nullable*/, int64_t ld_gate,
+                            float out_mul, const int32_t* q_cu_lens, const int32_t* kv_cu_lens,
                             const int32_t* block_tables, const int32_t* cu_block_lens, const int32_t* token_seq,
                             int64_t rows, int64_t H, int64_t G, int64_t dim, int64_t vdim, int64_t block_size,
                             float scale, int dtype, b200_stream_t stream);
@@ -710,8 +722,8 @@ B200_API int b200_sink_attn(void* out, int64_t ldo, const float* q, const void* 
 B200_API int b200_sink_attn_prefill_supported(int64_t dim, int64_t vdim, int dtype);
 B200_API int b200_sink_attn_prefill(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache,
                                     const float* r1 /*nullable*/, const float* r2 /*nullable*/,
-                                    const float* sink /*nullable*/, const int32_t* q_cu_lens,
-                                    const int32_t* kv_cu_lens, const int32_t* block_tables,
+                                    const float* sink /*nullable*/, const void* gate /*nullable*/, int64_t ld_gate,
+                                    float out_mul, const int32_t* q_cu_lens, const int32_t* kv_cu_lens, const int32_t* block_tables,
                                     const int32_t* cu_block_lens, int64_t n_seq, int64_t q_max, int64_t H, int64_t G,
                                     int64_t dim, int64_t vdim, int64_t block_size, float scale, int dtype,
                                     b200_stream_t stream);
@@ -722,8 +734,8 @@ B200_API int b200_sink_attn_prefill(void* out, int64_t ldo, const float* q, cons
  * n_splits * (2 + vdim) floats). */
 B200_API int b200_sink_attn_decode_tc(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache,
                                       const float* r1 /*nullable*/, const float* r2 /*nullable*/,
-                                      const float* sink /*nullable*/, const int32_t* q_cu_lens,
-                                      const int32_t* kv_cu_lens, const int32_t* block_tables,
+                                      const float* sink /*nullable*/, const void* gate /*nullable*/, int64_t ld_gate,
+                                      float out_mul, const int32_t* q_cu_lens, const int32_t* kv_cu_lens, const int32_t* block_tables,
                                       const int32_t* cu_block_lens, const int32_t* token_seq, int64_t rows, int64_t H,
                                       int64_t G, int64_t dim, int64_t vdim, int64_t block_size, float scale,
                                       int64_t n_splits, float* workspace /*nullable*/, int64_t workspace_floats,
@@ -822,6 +834,54 @@ B200_API int b200_branch_norm_residual(float* x_out, void* h_out /*nullable*/, c
 /* out [rows, n] = max(in, 0)^2 for the first n columns of rows with stride ld_in. */
 B200_API int b200_relu_squared(void* out, const void* in, int64_t rows, int64_t n, int64_t ld_in, int dtype,
                                b200_stream_t stream);
+
+/* ---- input side of pre-norm sublayers with short causal filters, linear recurrences with a matrix state whose decay
+ * does not look at the state (filters.cu, linear_scan.cu).  The reference has no such operators; each entry states its
+ * arithmetic.  Filters are fp32, state rows hold the last taps - 1 inputs [slot, taps - 1, channels] fp32, oldest
+ * first; q_max: the longest portion of the step; n_seq: its sequences. ---- */
+/* x_out = x_in + y ; n = x_out / sqrt(mean(x_out^2) + eps) * weight ; h_out[t] = n_t (filter null), or n_t +
+ * sum_i filter[i] n_{t - (taps - 1) + i} per channel with zeros before the start of the sequence (filter [taps, W]).
+ * y: rows of T (stride ldy), or the split-K partials [n_slots][rows][W] of the product that makes it (plan6:
+ * b200_dense_splitk_plan; their sum is rounded to T first), or neither (then x_in is normalised and x_out unused).
+ * x_out must not be x_in. */
+B200_API int b200_prenorm(float* x_out /*nullable*/, void* h_out, const float* x_in, const void* y /*nullable*/,
+                          int64_t ldy, const float* partials /*nullable*/, int64_t n_slots,
+                          const int32_t* plan6 /*nullable*/, const float* weight, const float* filter /*nullable*/,
+                          int64_t taps, float* filter_state /*nullable*/, const int32_t* q_cu_lens /*nullable*/,
+                          const int32_t* positions /*nullable*/, const int32_t* state_slots /*nullable*/,
+                          int64_t n_seq, int64_t q_max, int64_t rows, int64_t W, float eps, int dtype,
+                          b200_stream_t stream);
+/* out_t = act(bias + sum_i filter[i] in_{t - (taps - 1) + i}) per channel; silu: 1 for act = silu, 0 for none.
+ * filter [taps, channels]. */
+B200_API int b200_causal_filter(void* out, int64_t ldo, const void* in, int64_t ld, const float* filter,
+                                const float* bias /*nullable*/, int64_t taps, float* filter_state /*nullable*/,
+                                const int32_t* q_cu_lens, const int32_t* positions, const int32_t* state_slots,
+                                int64_t n_seq, int64_t q_max, int64_t rows, int64_t channels, int silu, int dtype,
+                                b200_stream_t stream);
+/* Column parts a head of value size V is walked in (1: its CTA holds the whole head). */
+B200_API int b200_linear_scan_parts(int64_t N, int64_t V);
+/* Per head and token, S [N x V] fp32 in state[slot, h]:  f = low + (1 - low) sigmoid(f_in + f_bias) ;
+ * S <- diag(f) S + (1 - f) v^T ; o = S^T silu(q_in) ; out[row, h] = mul * o / sqrt(mean(o^2) + eps) * norm_weight.
+ * q / f / v: column blocks of one matrix (row stride ld), heads in order; f_bias, f_low fp32 [H * N]; norm_weight
+ * fp32 [V].  raw (fp32 [rows, H * V]) is required where b200_linear_scan_parts > 1.  bf16 or fp32. */
+B200_API int b200_forget_scan(void* out, int64_t ldo, const void* q, const void* f, const void* v, int64_t ld,
+                              const float* f_bias, const float* f_low, const float* norm_weight, float* state,
+                              const int32_t* q_cu_lens, const int32_t* positions, const int32_t* state_slots,
+                              int64_t n_seq, int64_t q_max, int64_t rows, int64_t H, int64_t N, int64_t V, float eps,
+                              float mul, float* raw /*nullable*/, int dtype, b200_stream_t stream);
+/* Per head h (group h / (H / G)) and token, S [N x V] fp32 in state[slot, h]:  d = softplus(dt + dt_bias) ;
+ * S <- exp(-exp(a_log) d) S + d B x^T ; y[row, h] = S^T C + skip x  (fp32 [rows, H * V]).  x / B / C: column blocks of
+ * one matrix (row stride ld); dt: row stride ld_dt; dt_bias, a_log, skip fp32 [H].  bf16 or fp32. */
+B200_API int b200_ssd_scan(float* y, const void* x, const void* B, const void* C, int64_t ld, const void* dt,
+                           int64_t ld_dt, const float* dt_bias, const float* a_log, const float* skip, float* state,
+                           const int32_t* q_cu_lens, const int32_t* positions, const int32_t* state_slots,
+                           int64_t n_seq, int64_t q_max, int64_t rows, int64_t H, int64_t G, int64_t N, int64_t V,
+                           int dtype, b200_stream_t stream);
+/* u = y silu(z) ; out = u / sqrt(mean_part(u^2) + eps) * weight, the row of n channels in `parts` equal parts.  y fp32
+ * [rows, n]; z rows of T (stride ldz).  bf16 or fp32. */
+B200_API int b200_gated_part_norm(void* out, int64_t ldo, const float* y, const void* z, int64_t ldz,
+                                  const float* weight, int64_t rows, int64_t n, int64_t parts, float eps, int dtype,
+                                  b200_stream_t stream);
 
 #ifdef __cplusplus
 } /* extern "C" */

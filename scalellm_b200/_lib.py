@@ -153,12 +153,14 @@ SIGNATURES = {
     "b200_softcap": (_int, [_vp, _vp, _i64, _f32, _int, _vp]),
     "b200_sink_attn_prepare": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _i64, _f32, _vp, _vp, _vp, _vp, _i64, _i64, _i64,
                                       _i64, _i64, _f32, _f32, _i64, _int, _vp]),
-    "b200_sink_attn": (_int, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64,
+    "b200_sink_attn_prepare_turned": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64,
+                                             _i64, _i64, _i64, _i64, _f32, _int, _vp]),
+    "b200_sink_attn": (_int, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _f32, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64,
                               _i64, _i64, _f32, _int, _vp]),
     "b200_sink_attn_prefill_supported": (_int, [_i64, _i64, _int]),
-    "b200_sink_attn_decode_tc": (_int, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64,
+    "b200_sink_attn_decode_tc": (_int, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _f32, _vp, _vp, _vp, _vp, _vp, _i64, _i64,
                                         _i64, _i64, _i64, _i64, _f32, _i64, _vp, _i64, _int, _vp]),
-    "b200_sink_attn_prefill": (_int, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64,
+    "b200_sink_attn_prefill": (_int, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _f32, _vp, _vp, _vp, _vp, _i64, _i64, _i64,
                                       _i64, _i64, _i64, _i64, _f32, _int, _vp]),
     # sigmoid attention in blocks of positions with a head mix, gated delta rule with input filters, softmax router
     # with group limits, branch norms (sigmoid_attn.cu, delta_rule.cu, moe.cu, postnorm.cu)
@@ -181,6 +183,17 @@ SIGNATURES = {
     "b200_branch_norm_residual": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i64, _f32,
                                          _int, _vp]),
     "b200_relu_squared": (_int, [_vp, _vp, _i64, _i64, _i64, _int, _vp]),
+    # pre-norm input side with short causal filters, linear recurrences with a matrix state (filters.cu, linear_scan.cu)
+    "b200_prenorm": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i64,
+                            _i64, _i64, _f32, _int, _vp]),
+    "b200_causal_filter": (_int, [_vp, _i64, _vp, _i64, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _int,
+                                  _int, _vp]),
+    "b200_linear_scan_parts": (_int, [_i64, _i64]),
+    "b200_forget_scan": (_int, [_vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64,
+                                _i64, _i64, _i64, _f32, _f32, _vp, _int, _vp]),
+    "b200_ssd_scan": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64,
+                             _i64, _i64, _i64, _i64, _int, _vp]),
+    "b200_gated_part_norm": (_int, [_vp, _i64, _vp, _vp, _i64, _vp, _i64, _i64, _i64, _f32, _int, _vp]),
 }
 
 # Which source files a partial library needs for a group of entry points.  The whole library
@@ -188,7 +201,7 @@ SIGNATURES = {
 # just the sources a model asks for into a library of its own.
 ALL_SOURCES = ("runtime.cu", "elementwise.cu", "sampling.cu", "paged_attn.cu", "prefill_attn.cu", "w4a16.cu",
                "dense.cu", "allreduce.cu", "hyper.cu", "latent_attn.cu", "delta_rule.cu", "moe.cu", "postnorm.cu", "mingru.cu",
-               "diff_attn.cu", "sink_attn.cu", "sigmoid_attn.cu")
+               "diff_attn.cu", "sink_attn.cu", "sigmoid_attn.cu", "filters.cu", "linear_scan.cu")
 
 _lib: Optional[C.CDLL] = None
 _lib_sources: frozenset = frozenset()

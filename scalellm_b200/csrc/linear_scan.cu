@@ -1,0 +1,467 @@
+// linear_scan.cu — linear recurrences with a matrix state per head whose decay does not look at the state.
+//
+//     S_t = diag(a_t) S_{t-1} + k_t v_t^T ,   o_t = S_t^T q_t           S [N (key) x V (value)], fp32, per head
+//
+//   forget : a = f, k = 1 - f, f = low + (1 - low) sigmoid(fl + b) per head and key channel, q = silu(ql);
+//            out = mul * o / sqrt(mean_head(o^2) + eps) * w                              (what is forgotten is written)
+//   ssd    : a = exp(-exp(A_h) d) for the whole head, k = d B, q = C (one B, C per group of heads),
+//            d = softplus(dl + bias_h);  y = o + D_h v                                   (state-space duality form)
+//
+// The elements of S do not meet except in o's sum over the key channels, so a thread keeps a tile of RL key rows x 4
+// value columns in registers (packed pairs of key rows: two multiply-adds an instruction) and LP neighbouring lanes
+// share a column group; a warp walks 128 / LP columns.  One CTA per (sequence, head[, column part]); up to 16 tokens
+// at a time are turned into fp32 decay / key / query rows in shared memory by all threads (so no transcendental sits
+// in the walk), then the walk runs with no barrier, its read-outs collected in shared memory for the norm.
+// A portion that starts at position 0 starts from S = 0 instead of reading the slot.
+//
+//   part_norm : out = u / sqrt(mean_part(u^2) + eps) * w, u = y silu(z), the row in equal parts    (after the ssd walk)
+#include "common.cuh"
+
+namespace b200 {
+namespace {
+
+constexpr int kScanTokens = 16;
+constexpr int kScanWarps = 8;
+
+enum { MODE_FORGET = 0, MODE_SSD = 1 };
+
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float lo, float hi) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float2 unpack2(f32x2 v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float softplus_f(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
+
+template <typename T>
+struct ScanArgs {
+  T* out;                  // forget: rows of stride ldo (when the CTA holds the whole head)
+  int64_t ldo;
+  float* raw;              // fp32 [rows, H * V]: read-outs before the norm (forget in column parts), or y (ssd)
+  const T *q, *k, *v;      // forget: query, forget and value logits; ssd: C, B, x
+  int64_t ld;
+  const float *f_bias, *f_low, *norm_w;
+  const T* dt;
+  int64_t ld_dt;
+  const float *dt_bias, *a_log, *skip;
+  float* state;            // [slot][H][N][V]
+  const int *q_cu, *positions, *state_slots;
+  int H, G, N, V, CB, chunk;
+  float eps, mul;
+  int vec_in, vec_state;
+};
+
+template <typename T>
+__device__ __forceinline__ void get4c(const T* __restrict__ p, float (&v)[4], int n, bool vec) {
+  if (vec) {
+    load4<T>(p, v);
+  } else {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) v[i] = i < n ? Num<T>::to_f(p[i]) : 0.0f;
+  }
+}
+
+template <typename T, int MODE, int RL, int LP>
+__global__ void __launch_bounds__(kScanWarps * 32)
+linear_scan_kernel(const ScanArgs<T> a) {
+  constexpr int NP = RL * LP;                             // key rows, padded
+  extern __shared__ __align__(16) float sm[];
+  const int CH = a.chunk, CBP = (int)(blockDim.x >> 5) * (128 / LP);
+  float* k_s = sm;                                        // [CH][NP]
+  float* q_s = k_s + CH * NP;                             // [CH][NP]
+  float* a_s = q_s + CH * NP;                             // forget: [CH][NP]; ssd: [CH] (rounded up to 4)
+  float* v_s = a_s + (MODE == MODE_FORGET ? CH * NP : (CH + 3) / 4 * 4);   // [CH][CBP]
+  float* o_s = v_s + CH * CBP;                            // [CH][CBP]
+  const int seq = blockIdx.x, h = blockIdx.y, cb0 = (int)blockIdx.z * a.CB;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+  const int t0 = a.q_cu[seq], t1 = a.q_cu[seq + 1];
+  if (t0 >= t1) return;
+  const int N = a.N, V = a.V;
+  const int ncol = V - cb0 < a.CB ? V - cb0 : a.CB;
+  const int p = lane % LP, cq = warp * (32 / LP) + lane / LP;
+  const int c0 = cq * 4;                                  // this thread's columns c0 .. c0 + 3 of the part
+  float* Sg = a.state + (((size_t)a.state_slots[seq] * a.H + h) * N) * V + cb0;
+  const bool fresh = a.positions[t0] == 0;
+  f32x2 S[RL / 2][4];                                     // pairs of key rows
+#pragma unroll
+  for (int i = 0; i < RL / 4; ++i) {
+    const int n0 = p * 4 + i * 4 * LP;
+#pragma unroll
+    for (int jj = 0; jj < 2; ++jj) {
+      float lo[4] = {0.0f, 0.0f, 0.0f, 0.0f}, hi[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+      const int n = n0 + jj * 2;
+      if (!fresh && c0 < ncol) {
+        if (n < N) get4c<float>(Sg + (size_t)n * V + c0, lo, ncol - c0, a.vec_state);
+        if (n + 1 < N) get4c<float>(Sg + (size_t)(n + 1) * V + c0, hi, ncol - c0, a.vec_state);
+      }
+#pragma unroll
+      for (int c = 0; c < 4; ++c) S[i * 2 + jj][c] = pack2(lo[c], hi[c]);
+    }
+  }
+  const int g = MODE == MODE_SSD ? h / (a.H / a.G) : h;
+  float neg_a = 0.0f, dbias = 0.0f, skip = 0.0f;
+  if constexpr (MODE == MODE_SSD) {
+    neg_a = -expf(a.a_log[h]);
+    dbias = a.dt_bias[h];
+    skip = a.skip[h];
+  }
+  for (int tc = t0; tc < t1; tc += CH) {
+    const int nt = t1 - tc < CH ? t1 - tc : CH;
+    __syncthreads();                                      // the read-outs and rows of the chunk before are done with
+    for (int tok = warp; tok < nt; tok += n_warps) {
+      const size_t row = (size_t)(tc + tok);
+      const T* qr = a.q + row * a.ld + (size_t)g * N;
+      const T* kr = a.k + row * a.ld + (size_t)g * N;
+      float dt = 0.0f;
+      if constexpr (MODE == MODE_SSD) {
+        dt = softplus_f(Num<T>::to_f(a.dt[row * a.ld_dt + h]) + dbias);
+        if (lane == 0) a_s[tok] = expf(neg_a * dt);
+      }
+      for (int c = lane * 4; c < NP; c += 128) {
+        float qv[4] = {0.0f, 0.0f, 0.0f, 0.0f}, kv[4] = {0.0f, 0.0f, 0.0f, 0.0f}, av[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+        if (c < N) {
+          get4c<T>(qr + c, qv, N - c, a.vec_in);
+          get4c<T>(kr + c, kv, N - c, a.vec_in);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            if constexpr (MODE == MODE_FORGET) {
+              if (c + i < N) {
+                const float l = a.f_low[h * N + c + i];
+                const float z = kv[i] + a.f_bias[h * N + c + i];
+                const float e = expf(-fabsf(z));          // sigmoid(z) and sigmoid(-z) without cancellation
+                const float big = 1.0f / (1.0f + e), small = e * big;
+                av[i] = l + (1.0f - l) * (z >= 0.0f ? big : small);
+                kv[i] = (1.0f - l) * (z >= 0.0f ? small : big);
+                qv[i] = qv[i] * sigmoid_f(qv[i]);
+              }
+            } else {
+              kv[i] *= dt;
+            }
+          }
+        }
+        *reinterpret_cast<float4*>(k_s + tok * NP + c) = make_float4(kv[0], kv[1], kv[2], kv[3]);
+        *reinterpret_cast<float4*>(q_s + tok * NP + c) = make_float4(qv[0], qv[1], qv[2], qv[3]);
+        if constexpr (MODE == MODE_FORGET)
+          *reinterpret_cast<float4*>(a_s + tok * NP + c) = make_float4(av[0], av[1], av[2], av[3]);
+      }
+      const T* vr = a.v + row * a.ld + (size_t)h * V + cb0;
+      for (int c = lane * 4; c < CBP; c += 128) {
+        float vv[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+        if (c < ncol) get4c<T>(vr + c, vv, ncol - c, a.vec_in);
+        *reinterpret_cast<float4*>(v_s + tok * CBP + c) = make_float4(vv[0], vv[1], vv[2], vv[3]);
+      }
+    }
+    __syncthreads();
+    for (int tok = 0; tok < nt; ++tok) {
+      const float4 vv = *reinterpret_cast<const float4*>(v_s + tok * CBP + c0);
+      const f32x2 v2[4] = {pack2(vv.x, vv.x), pack2(vv.y, vv.y), pack2(vv.z, vv.z), pack2(vv.w, vv.w)};
+      f32x2 o2[4];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) o2[c] = 0ull;
+      f32x2 da = 0ull;
+      if constexpr (MODE == MODE_SSD) da = pack2(a_s[tok], a_s[tok]);
+#pragma unroll
+      for (int i = 0; i < RL / 4; ++i) {
+        const int n0 = tok * NP + p * 4 + i * 4 * LP;
+        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(k_s + n0);
+        const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(q_s + n0);
+        ulonglong2 f2;
+        if constexpr (MODE == MODE_FORGET) f2 = *reinterpret_cast<const ulonglong2*>(a_s + n0);
+        else f2.x = f2.y = da;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          S[i * 2][c] = fma2(f2.x, S[i * 2][c], mul2(k2.x, v2[c]));
+          o2[c] = fma2(S[i * 2][c], q2.x, o2[c]);
+          S[i * 2 + 1][c] = fma2(f2.y, S[i * 2 + 1][c], mul2(k2.y, v2[c]));
+          o2[c] = fma2(S[i * 2 + 1][c], q2.y, o2[c]);
+        }
+      }
+      float o[4];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const float2 t = unpack2(o2[c]);
+        o[c] = t.x + t.y;
+      }
+      // sum over the LP lanes of the column group; two exchanges leave one column with each of four lanes
+      const bool b0 = p & 1, b1 = p & 2;
+      float s0 = b0 ? o[0] : o[2], s1 = b0 ? o[1] : o[3], r0 = b0 ? o[2] : o[0], r1 = b0 ? o[3] : o[1];
+      r0 += __shfl_xor_sync(0xffffffffu, s0, 1);
+      r1 += __shfl_xor_sync(0xffffffffu, s1, 1);
+      const float s = b1 ? r0 : r1;
+      float r = b1 ? r1 : r0;
+      r += __shfl_xor_sync(0xffffffffu, s, 2);
+#pragma unroll
+      for (int d = 4; d < LP; d <<= 1) r += __shfl_xor_sync(0xffffffffu, r, d);
+      if (p < 4) o_s[tok * CBP + c0 + (b0 ? 2 : 0) + (b1 ? 1 : 0)] = r;
+    }
+    __syncthreads();
+    for (int tok = warp; tok < nt; tok += n_warps) {
+      const size_t row = (size_t)(tc + tok);
+      const float* ot = o_s + tok * CBP;
+      if constexpr (MODE == MODE_SSD) {
+        float* dst = a.raw + row * (size_t)a.H * V + (size_t)h * V + cb0;
+        for (int c = lane; c < ncol; c += 32) dst[c] = ot[c] + skip * v_s[tok * CBP + c];
+      } else if (a.raw) {
+        float* dst = a.raw + row * (size_t)a.H * V + (size_t)h * V + cb0;
+        for (int c = lane; c < ncol; c += 32) dst[c] = ot[c];
+      } else {
+        float ss = 0.0f;
+        for (int c = lane; c < V; c += 32) ss += ot[c] * ot[c];
+        ss = warp_sum(ss);
+        const float inv = a.mul / sqrtf(ss / (float)V + a.eps);
+        T* dst = a.out + row * a.ldo + (size_t)h * V;
+        for (int c = lane; c < V; c += 32) dst[c] = Num<T>::from_f(ot[c] * inv * a.norm_w[c]);
+      }
+    }
+  }
+  if (c0 < ncol) {
+#pragma unroll
+    for (int i = 0; i < RL / 2; ++i) {
+      const int n = p * 4 + (i / 2) * 4 * LP + (i & 1) * 2;
+      float2 t[4];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) t[c] = unpack2(S[i][c]);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        if (n + e >= N) continue;
+        float* dst = Sg + (size_t)(n + e) * V + c0;
+        if (a.vec_state) {
+          *reinterpret_cast<float4*>(dst) = e == 0 ? make_float4(t[0].x, t[1].x, t[2].x, t[3].x)
+                                                   : make_float4(t[0].y, t[1].y, t[2].y, t[3].y);
+        } else {
+#pragma unroll
+          for (int c = 0; c < 4; ++c)
+            if (c0 + c < ncol) dst[c] = e == 0 ? t[c].x : t[c].y;
+        }
+      }
+    }
+  }
+}
+
+// out[row, h] = mul * raw / sqrt(mean(raw^2) + eps) * w: a warp per (row, head)
+template <typename T>
+__global__ void __launch_bounds__(256)
+head_norm_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict__ raw, const float* __restrict__ w,
+                 int64_t n_units, int H, int V, float eps, float mul) {
+  const int64_t u = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (u >= n_units) return;
+  const int64_t row = u / H;
+  const int h = (int)(u - row * H);
+  const float* r = raw + (size_t)u * V;
+  float ss = 0.0f;
+  for (int i = lane; i < V; i += 32) ss += r[i] * r[i];
+  ss = warp_sum(ss);
+  const float inv = mul / sqrtf(ss / (float)V + eps);
+  for (int i = lane; i < V; i += 32) out[(size_t)row * ldo + (size_t)h * V + i] = Num<T>::from_f(r[i] * inv * w[i]);
+}
+
+// out = u / sqrt(mean_part(u^2) + eps) * w, u = y silu(z); one CTA per row, the row in `parts` equal parts.  With
+// fewer parts than warps several warps share a part.
+constexpr int kPartThreads = 256;
+template <typename T>
+__global__ void __launch_bounds__(kPartThreads)
+gated_part_norm_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict__ y, const T* __restrict__ z,
+                       int64_t ldz, const float* __restrict__ w, int n, int parts, float eps, int vec) {
+  extern __shared__ __align__(16) float sm[];
+  float* u_s = sm;                                        // [n]
+  float* r_s = sm + (n + 3) / 4 * 4;                      // [units] partial sums of squares
+  constexpr int NW = kPartThreads / 32;
+  const size_t row = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int i = threadIdx.x * 4; i < n; i += kPartThreads * 4) {
+    float yv[4], zv[4];
+    get4c<float>(y + row * n + i, yv, n - i, vec);
+    get4c<T>(z + row * ldz + i, zv, n - i, vec);
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if (i + k < n) u_s[i + k] = yv[k] * zv[k] * sigmoid_f(zv[k]);
+  }
+  __syncthreads();
+  const int ps = n / parts;
+  const int per = parts >= NW ? 1 : NW / parts;           // warps of a part
+  for (int un = warp; un < parts * per; un += NW) {
+    const int part = un / per, sub = un - part * per;
+    float ss = 0.0f;
+    for (int i = sub * 32 + lane; i < ps; i += per * 32) {
+      const float v = u_s[part * ps + i];
+      ss += v * v;
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) r_s[un] = ss;
+  }
+  __syncthreads();
+  for (int part = threadIdx.x; part < parts; part += kPartThreads) {
+    float ss = 0.0f;
+    for (int k = 0; k < per; ++k) ss += r_s[part * per + k];
+    r_s[part * per] = 1.0f / sqrtf(ss / (float)ps + eps);
+  }
+  __syncthreads();
+  for (int i = threadIdx.x * 4; i < n; i += kPartThreads * 4) {
+    float wv[4], o[4];
+    get4c<float>(w + i, wv, n - i, vec);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) o[k] = i + k < n ? u_s[i + k] * r_s[(i + k) / ps * per] * wv[k] : 0.0f;
+    T* dst = out + row * ldo + i;
+    if (vec) {
+      if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
+      else *reinterpret_cast<uint2*>(dst) = make_uint2(Num<T>::pack(o[0], o[1]), Num<T>::pack(o[2], o[3]));
+    } else {
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+        if (i + k < n) dst[k] = Num<T>::from_f(o[k]);
+    }
+  }
+}
+
+int scan_col_parts(int N, int V) {
+  const int lp = N <= 128 ? 4 : (N <= 256 ? 8 : 16);
+  const int warps = (V + 128 / lp - 1) / (128 / lp);
+  return (warps + kScanWarps - 1) / kScanWarps;
+}
+
+template <typename T, int MODE, int RL, int LP>
+int launch_scan_n(ScanArgs<T>& a, int64_t n_seq, int64_t q_max, cudaStream_t st) {
+  constexpr int CW = 128 / LP;                            // columns of a warp
+  int warps = (a.V + CW - 1) / CW;
+  const int parts = scan_col_parts(a.N, a.V);
+  warps = (warps + parts - 1) / parts;
+  a.CB = warps * CW;
+  a.chunk = q_max < kScanTokens ? (int)q_max : kScanTokens;
+  constexpr int NP = RL * LP;
+  const size_t smem = ((size_t)a.chunk * (NP * (MODE == MODE_FORGET ? 3 : 2) + 2 * a.CB) +
+                       (MODE == MODE_FORGET ? 0 : (a.chunk + 3) / 4 * 4)) * sizeof(float);
+  auto kern = linear_scan_kernel<T, MODE, RL, LP>;
+  if (smem > 48 * 1024)
+    B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  kern<<<dim3((unsigned)n_seq, (unsigned)a.H, (unsigned)((a.V + a.CB - 1) / a.CB)), warps * 32, smem, st>>>(a);
+  B200_LAUNCH_OK("linear_scan_kernel");
+  return B200_OK;
+}
+
+template <typename T, int MODE>
+int launch_scan(ScanArgs<T>& a, int64_t n_seq, int64_t q_max, cudaStream_t st) {
+  if (a.N <= 16) return launch_scan_n<T, MODE, 4, 4>(a, n_seq, q_max, st);
+  if (a.N <= 32) return launch_scan_n<T, MODE, 8, 4>(a, n_seq, q_max, st);
+  if (a.N <= 64) return launch_scan_n<T, MODE, 16, 4>(a, n_seq, q_max, st);
+  if (a.N <= 128) return launch_scan_n<T, MODE, 32, 4>(a, n_seq, q_max, st);
+  if (a.N <= 256) return launch_scan_n<T, MODE, 32, 8>(a, n_seq, q_max, st);
+  return launch_scan_n<T, MODE, 32, 16>(a, n_seq, q_max, st);
+}
+
+}  // namespace
+}  // namespace b200
+
+using namespace b200;
+
+#define SCAN_DISPATCH(dtype, ...)                                                            \
+  switch (dtype) {                                                                           \
+    case B200_BF16: { using T = __nv_bfloat16; __VA_ARGS__; break; }                         \
+    case B200_FP32: { using T = float; __VA_ARGS__; break; }                                 \
+    default: return set_error(B200_ERR_INVALID_ARG, "linear_scan: bf16 or fp32, got %d", dtype); \
+  }
+
+extern "C" {
+
+int b200_linear_scan_parts(int64_t N, int64_t V) { return scan_col_parts((int)N, (int)V); }
+
+int b200_forget_scan(void* out, int64_t ldo, const void* q, const void* f, const void* v, int64_t ld,
+                     const float* f_bias, const float* f_low, const float* norm_weight, float* state,
+                     const int32_t* q_cu_lens, const int32_t* positions, const int32_t* state_slots, int64_t n_seq,
+                     int64_t q_max, int64_t rows, int64_t H, int64_t N, int64_t V, float eps, float mul, float* raw,
+                     int dtype, b200_stream_t stream) {
+  if (rows == 0 || n_seq == 0) return B200_OK;
+  B200_CHECK_ARG(out && q && f && v && f_bias && f_low && norm_weight && state && q_cu_lens && positions && state_slots,
+                 "forget_scan: null pointer");
+  B200_CHECK_ARG(rows > 0 && n_seq > 0 && q_max > 0 && H > 0 && H <= 65535 && N > 0 && N <= 512 && V > 0 && V <= 4096 &&
+                     ldo >= H * V && ld >= H * (N > V ? N : V),
+                 "forget_scan: bad shape (key size <= 512)");
+  B200_CHECK_ARG(raw || scan_col_parts((int)N, (int)V) == 1, "forget_scan: heads in several column parts need a workspace");
+  auto st = static_cast<cudaStream_t>(stream);
+  SCAN_DISPATCH(dtype, {
+    ScanArgs<T> a{};
+    a.out = static_cast<T*>(out); a.ldo = ldo; a.raw = raw;
+    a.q = static_cast<const T*>(q); a.k = static_cast<const T*>(f); a.v = static_cast<const T*>(v); a.ld = ld;
+    a.f_bias = f_bias; a.f_low = f_low; a.norm_w = norm_weight; a.state = state;
+    a.q_cu = q_cu_lens; a.positions = positions; a.state_slots = state_slots;
+    a.H = (int)H; a.G = (int)H; a.N = (int)N; a.V = (int)V; a.eps = eps; a.mul = mul;
+    a.vec_in = N % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && is_aligned(q, 4 * sizeof(T)) && is_aligned(f, 4 * sizeof(T)) &&
+               is_aligned(v, 4 * sizeof(T));
+    a.vec_state = V % 4 == 0 && is_aligned(state, 16);
+    const int rc = launch_scan<T, MODE_FORGET>(a, n_seq, q_max, st);
+    if (rc != B200_OK) return rc;
+    if (raw) {
+      const int64_t n_units = rows * H;
+      head_norm_kernel<T><<<(unsigned)((n_units + 7) / 8), 256, 0, st>>>(static_cast<T*>(out), ldo, raw, norm_weight,
+                                                                         n_units, (int)H, (int)V, eps, mul);
+      B200_LAUNCH_OK("head_norm_kernel");
+    }
+  });
+  return B200_OK;
+}
+
+int b200_ssd_scan(float* y, const void* x, const void* B, const void* Cm, int64_t ld, const void* dt, int64_t ld_dt,
+                  const float* dt_bias, const float* a_log, const float* skip, float* state, const int32_t* q_cu_lens,
+                  const int32_t* positions, const int32_t* state_slots, int64_t n_seq, int64_t q_max, int64_t rows,
+                  int64_t H, int64_t G, int64_t N, int64_t V, int dtype, b200_stream_t stream) {
+  if (rows == 0 || n_seq == 0) return B200_OK;
+  B200_CHECK_ARG(y && x && B && Cm && dt && dt_bias && a_log && skip && state && q_cu_lens && positions && state_slots,
+                 "ssd_scan: null pointer");
+  B200_CHECK_ARG(rows > 0 && n_seq > 0 && q_max > 0 && H > 0 && H <= 65535 && G > 0 && H % G == 0 && N > 0 && N <= 512 &&
+                     V > 0 && V <= 4096 && ld >= H * V && ld >= G * N && ld_dt >= H,
+                 "ssd_scan: bad shape (state size <= 512, heads a multiple of groups)");
+  auto st = static_cast<cudaStream_t>(stream);
+  SCAN_DISPATCH(dtype, {
+    ScanArgs<T> a{};
+    a.raw = y;
+    a.q = static_cast<const T*>(Cm); a.k = static_cast<const T*>(B); a.v = static_cast<const T*>(x); a.ld = ld;
+    a.dt = static_cast<const T*>(dt); a.ld_dt = ld_dt; a.dt_bias = dt_bias; a.a_log = a_log; a.skip = skip;
+    a.state = state; a.q_cu = q_cu_lens; a.positions = positions; a.state_slots = state_slots;
+    a.H = (int)H; a.G = (int)G; a.N = (int)N; a.V = (int)V; a.mul = 1.0f;
+    a.vec_in = N % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && is_aligned(x, 4 * sizeof(T)) && is_aligned(B, 4 * sizeof(T)) &&
+               is_aligned(Cm, 4 * sizeof(T));
+    a.vec_state = V % 4 == 0 && is_aligned(state, 16);
+    return (launch_scan<T, MODE_SSD>(a, n_seq, q_max, st));
+  });
+  return B200_OK;
+}
+
+int b200_gated_part_norm(void* out, int64_t ldo, const float* y, const void* z, int64_t ldz, const float* weight,
+                         int64_t rows, int64_t n, int64_t parts, float eps, int dtype, b200_stream_t stream) {
+  if (rows == 0) return B200_OK;
+  B200_CHECK_ARG(out && y && z && weight, "gated_part_norm: null pointer");
+  B200_CHECK_ARG(rows > 0 && n > 0 && parts > 0 && n % parts == 0 && ldo >= n && ldz >= n && (n + parts + 16) * 4 <= 200 * 1024,
+                 "gated_part_norm: bad shape (the row in equal parts, at most ~50K channels)");
+  auto st = static_cast<cudaStream_t>(stream);
+  const size_t smem = (size_t)((n + 3) / 4 * 4 + (parts < 8 ? 8 : parts)) * sizeof(float);
+  SCAN_DISPATCH(dtype, {
+    const int vec = n % 4 == 0 && ldo % 4 == 0 && ldz % 4 == 0 && is_aligned(out, 4 * sizeof(T)) &&
+                    is_aligned(z, 4 * sizeof(T)) && is_aligned(y, 16) && is_aligned(weight, 16);
+    if (smem > 48 * 1024)
+      B200_CUDA_OK(cudaFuncSetAttribute(gated_part_norm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    gated_part_norm_kernel<T><<<(unsigned)rows, kPartThreads, smem, st>>>(static_cast<T*>(out), ldo, y,
+                                                                          static_cast<const T*>(z), ldz, weight, (int)n,
+                                                                          (int)parts, eps, vec);
+  });
+  B200_LAUNCH_OK("gated_part_norm_kernel");
+  return B200_OK;
+}
+
+}  // extern "C"

@@ -6,9 +6,14 @@
 //     s_ij = scale q_i . k_j - r1_h ln(1 + r2_h (i - j))               j <= i                 (r1 absent: no bias)
 //     p_ij = exp(s_ij) / (exp(sink_h) + sum_j' exp(s_ij'))             the sink has no key and no value
 //     o_i  = sum_j p_ij v_j
+// On the way out a head's result may be multiplied by a number and, element by element, with sigmoid(gate): an output
+// gate and a branch weight cost no launch of their own.
 // Query head h reads key/value head h / (H / G).  Values may be blended with the values another layer made of the
 // same token before they are cached:  v <- (1 - lam) v + lam v_other.
 //
+//   turned prepare : instead of unit heads and the temperature, one root mean square over ALL heads of the queries (and
+//             one over all of the keys) with a weight per channel, then a rotary turn of the first rot_dims channels of
+//             every head: channel t with t + rot_dims / 2, angle position * inv_freq[t] (fp32)
 //   prepare : q rows -> fp32 [rows, H, dim]; k rows -> K cache [slots, G, dim]; v rows -> V cache [slots, G, vdim]
 //             (cache entries have the activation type T)
 //   attend  : CUDA cores, any type and size: one CTA per (row, key/value head, chunk of query heads); its warps are
@@ -16,6 +21,8 @@
 //   prefill : bf16 on the tensor cores (mma.sync m16n8k16): tiles of 16 consecutive tokens x 32 keys.
 //   decode  : bf16 on the tensor cores, single tokens: the 16 rows of a tile are the query heads of a key/value group.
 // Norms, temperature, scores, bias, softmax weights and sums are fp32.
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace b200 {
@@ -70,6 +77,107 @@ sink_attn_prepare_kernel(float* __restrict__ q_out, const T* __restrict__ q_in, 
   }
 }
 
+// Queries and keys normalised over their whole projection rows, turned, written out / into the cache.  One CTA per
+// row; V: channels a thread moves at once (4 where head sizes, turn and addresses allow it).
+constexpr int kTurnThreads = 256;
+template <typename T, int V>
+__global__ void __launch_bounds__(kTurnThreads)
+sink_attn_prepare_turned_kernel(float* __restrict__ q_out, const T* __restrict__ q_in, const T* __restrict__ k_in,
+                                const T* __restrict__ v_in, int64_t ld, const float* __restrict__ q_w,
+                                const float* __restrict__ k_w, const float* __restrict__ inv_freq,
+                                T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ positions,
+                                const int* __restrict__ slots, int H, int G, int dim, int vdim, int rot_dims,
+                                float eps) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float red_q[32], red_k[32];
+  const int nq = H * dim, nk = G * dim, nv = G * vdim, half = rot_dims / 2;
+  float* x_s = sm;                                       // [nq + nk] rows times their weights (before the norm's factor)
+  float* cos_s = x_s + (nq + nk + 3) / 4 * 4;            // [half]
+  float* sin_s = cos_s + (half + 3) / 4 * 4;             // [half]
+  const size_t row = blockIdx.x;
+  const int pos = positions[row];
+  const size_t slot = (size_t)slots[row];
+  for (int i = threadIdx.x; i < half; i += kTurnThreads) {
+    float sn, cs;
+    sincosf((float)pos * inv_freq[i], &sn, &cs);
+    cos_s[i] = cs;
+    sin_s[i] = sn;
+  }
+  float sq = 0.0f, sk = 0.0f;
+  for (int e = threadIdx.x * V; e < nq + nk; e += kTurnThreads * V) {
+    const bool is_q = e < nq;
+    const T* src = is_q ? q_in + row * ld + e : k_in + row * ld + (e - nq);
+    const float* w = is_q ? q_w + e : k_w + (e - nq);
+    float x[V], ss = 0.0f;
+    if constexpr (V == 4) load4<T>(src, x);
+    else x[0] = Num<T>::to_f(src[0]);
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      ss += x[k] * x[k];
+      x_s[e + k] = x[k] * w[k];
+    }
+    if (is_q) sq += ss;
+    else sk += ss;
+  }
+  const float rq = 1.0f / sqrtf(block_sum<kTurnThreads>(sq, red_q) / (float)nq + eps);
+  const float rk = 1.0f / sqrtf(block_sum<kTurnThreads>(sk, red_k) / (float)nk + eps);
+  for (int e = threadIdx.x * V; e < nq + nk; e += kTurnThreads * V) {
+    const bool is_q = e < nq;
+    const int d = (is_q ? e : e - nq) % dim;
+    const float r = is_q ? rq : rk;
+    float y[V];
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      const int t = d + k;
+      float v = x_s[e + k] * r;
+      if (t < half) v = v * cos_s[t] - x_s[e + k + half] * r * sin_s[t];
+      else if (t < 2 * half) v = v * cos_s[t - half] + x_s[e + k - half] * r * sin_s[t - half];
+      y[k] = v;
+    }
+    if (is_q) {
+      float* dst = q_out + row * nq + e;
+      if constexpr (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1], y[2], y[3]);
+      else dst[0] = y[0];
+    } else {
+      T* dst = k_cache + slot * nk + (e - nq);
+      if constexpr (V == 4 && sizeof(T) == 4) *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1], y[2], y[3]);
+      else if constexpr (V == 4)
+        *reinterpret_cast<uint2*>(dst) = make_uint2(Num<T>::pack(y[0], y[1]), Num<T>::pack(y[2], y[3]));
+      else dst[0] = Num<T>::from_f(y[0]);
+    }
+  }
+  const T* vs = v_in + row * ld;
+  T* vd = v_cache + slot * nv;
+  if constexpr (V == 4) {
+    using U = typename std::conditional<sizeof(T) == 4, uint4, uint2>::type;
+    for (int i = threadIdx.x * 4; i < nv; i += kTurnThreads * 4)
+      *reinterpret_cast<U*>(vd + i) = *reinterpret_cast<const U*>(vs + i);
+  } else {
+    for (int i = threadIdx.x; i < nv; i += kTurnThreads) vd[i] = vs[i];
+  }
+}
+
+template <typename T>
+int launch_prepare_turned(float* q_out, const void* q_in, const void* k_in, const void* v_in, int64_t ld,
+                          const float* q_w, const float* k_w, const float* inv_freq, void* k_cache, void* v_cache,
+                          const int* positions, const int* slots, int64_t rows, int H, int G, int dim, int vdim,
+                          int rot_dims, float eps, cudaStream_t st) {
+  const size_t smem = ((size_t)((H + G) * dim + 3) / 4 * 4 + (size_t)(rot_dims / 2 + 3) / 4 * 8) * sizeof(float);
+  B200_CHECK_ARG(smem <= 200 * 1024, "sink_attn_prepare_turned: %d + %d heads of %d do not fit in shared memory", H, G, dim);
+  const bool vec = dim % 4 == 0 && vdim % 4 == 0 && ld % 4 == 0 && is_aligned(q_in, 4 * sizeof(T)) &&
+                   is_aligned(k_in, 4 * sizeof(T)) && is_aligned(v_in, 4 * sizeof(T)) && is_aligned(k_cache, 16) &&
+                   is_aligned(v_cache, 16) && is_aligned(q_out, 16);
+  auto kern = vec ? sink_attn_prepare_turned_kernel<T, 4> : sink_attn_prepare_turned_kernel<T, 1>;
+  if (smem > 48 * 1024)
+    B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  kern<<<(unsigned)rows, kTurnThreads, smem, st>>>(q_out, static_cast<const T*>(q_in), static_cast<const T*>(k_in),
+                                                   static_cast<const T*>(v_in), ld, q_w, k_w, inv_freq,
+                                                   static_cast<T*>(k_cache), static_cast<T*>(v_cache), positions, slots, H,
+                                                   G, dim, vdim, rot_dims, eps);
+  B200_LAUNCH_OK("sink_attn_prepare_turned_kernel");
+  return B200_OK;
+}
+
 // The end of a head's walk: its softmax denominator takes the sink, a term exp(sink) with no value.
 __device__ __forceinline__ float sink_scale(float m, float l, const float* sink, int h) {
   // returns f with o_final = o * f, o accumulated relative to the running maximum m with sum l
@@ -80,13 +188,21 @@ __device__ __forceinline__ float sink_scale(float m, float l, const float* sink,
   return c / (l * c + expf(s - M));
 }
 
+// What leaves the kernels: mul * o * sigmoid(gate[i]) (gate absent: mul * o).
+template <typename T>
+__device__ __forceinline__ float gated_out(float o, const T* __restrict__ gate, size_t i, float mul) {
+  o *= mul;
+  return gate ? o / (1.0f + expf(-Num<T>::to_f(gate[i]))) : o;
+}
+
 // One CTA per (row, key/value head, chunk of RH query heads of that group); warp = (head r, key split sp).  Lane
 // owns value channels lane + 32 c, c < NC.
 template <typename T, int NC>
 __global__ void __launch_bounds__(kMaxWarps * 32)
 sink_attn_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict__ q, const T* __restrict__ k_cache,
                  const T* __restrict__ v_cache, const float* __restrict__ r1, const float* __restrict__ r2,
-                 const float* __restrict__ sink, const int* __restrict__ q_cu, const int* __restrict__ kv_cu,
+                 const float* __restrict__ sink, const T* __restrict__ gate, int64_t ld_gate, float out_mul,
+                 const int* __restrict__ q_cu, const int* __restrict__ kv_cu,
                  const int* __restrict__ block_tables, const int* __restrict__ cu_block_lens,
                  const int* __restrict__ token_seq, int H, int G, int dim, int vdim, int block_size, float scale,
                  int RH, int S) {
@@ -184,15 +300,17 @@ sink_attn_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict__ q, 
 #pragma unroll
   for (int c = 0; c < NC; ++c) {
     const int col = lane + 32 * c;
-    if (col < vdim) out[(size_t)row * ldo + (size_t)h * vdim + col] = Num<T>::from_f(o[c] * f);
+    if (col < vdim)
+      out[(size_t)row * ldo + (size_t)h * vdim + col] =
+          Num<T>::from_f(gated_out(o[c] * f, gate, (size_t)row * ld_gate + (size_t)h * vdim + col, out_mul));
   }
 }
 
 template <typename T, int NC>
 int launch_simt(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache, const float* r1,
-                const float* r2, const float* sink, const int* q_cu, const int* kv_cu, const int* tables,
-                const int* blk_cu, const int* token_seq, int64_t rows, int H, int G, int dim, int vdim,
-                int block_size, float scale, cudaStream_t st) {
+                const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul, const int* q_cu,
+                const int* kv_cu, const int* tables, const int* blk_cu, const int* token_seq, int64_t rows, int H, int G,
+                int dim, int vdim, int block_size, float scale, cudaStream_t st) {
   const int R = H / G;
   const int RH = R < kMaxWarps ? R : kMaxWarps;
   int S = kMaxWarps / RH;
@@ -206,19 +324,20 @@ int launch_simt(void* out, int64_t ldo, const float* q, const void* k_cache, con
     B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   dim3 grid((unsigned)rows, (unsigned)G, (unsigned)chunks);
   kern<<<grid, n_warps * 32, smem, st>>>(static_cast<T*>(out), ldo, q, static_cast<const T*>(k_cache),
-                                         static_cast<const T*>(v_cache), r1, r2, sink, q_cu, kv_cu, tables, blk_cu,
-                                         token_seq, H, G, dim, vdim, block_size, scale, RH, S);
+                                         static_cast<const T*>(v_cache), r1, r2, sink, static_cast<const T*>(gate),
+                                         ld_gate, out_mul, q_cu, kv_cu, tables, blk_cu, token_seq, H, G, dim, vdim,
+                                         block_size, scale, RH, S);
   B200_LAUNCH_OK("sink_attn_kernel");
   return B200_OK;
 }
 
 template <typename T>
 int dispatch_simt(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache, const float* r1,
-                  const float* r2, const float* sink, const int* q_cu, const int* kv_cu, const int* tables,
-                  const int* blk_cu, const int* token_seq, int64_t rows, int H, int G, int dim, int vdim,
-                  int block_size, float scale, cudaStream_t st) {
-#define SA_ARGS out, ldo, q, k_cache, v_cache, r1, r2, sink, q_cu, kv_cu, tables, blk_cu, token_seq, rows, H, G, dim, \
-                vdim, block_size, scale, st
+                  const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul, const int* q_cu,
+                  const int* kv_cu, const int* tables, const int* blk_cu, const int* token_seq, int64_t rows, int H,
+                  int G, int dim, int vdim, int block_size, float scale, cudaStream_t st) {
+#define SA_ARGS out, ldo, q, k_cache, v_cache, r1, r2, sink, gate, ld_gate, out_mul, q_cu, kv_cu, tables, blk_cu, \
+                token_seq, rows, H, G, dim, vdim, block_size, scale, st
   const int nc = (vdim + 31) / 32;
   if (nc <= 1) return launch_simt<T, 1>(SA_ARGS);
   if (nc <= 2) return launch_simt<T, 2>(SA_ARGS);
@@ -271,6 +390,7 @@ __global__ void __launch_bounds__(128, EXACT ? 4 : 1)
 sink_attn_prefill_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const float* __restrict__ q,
                          const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
                          const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink,
+                         const __nv_bfloat16* __restrict__ gate, int64_t ld_gate, float out_mul,
                          const int* __restrict__ q_cu, const int* __restrict__ kv_cu,
                          const int* __restrict__ block_tables, const int* __restrict__ cu_block_lens, int H, int G,
                          int dim_rt, int vdim_rt, int block_size, float scale, int RW, int chunks) {
@@ -438,17 +558,19 @@ sink_attn_prefill_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const flo
     const float f = sink_scale(mx[r2i], ls[r2i], sink, h);
     const size_t row = (size_t)q0 + row_t[r2i];
     __nv_bfloat16* dst = out + row * ldo + (size_t)h * vdim;
+    const size_t gi = row * ld_gate + (size_t)h * vdim + qc;
 #pragma unroll
     for (int n = 0; n < VT_MAX * 2; ++n)
       if (n < VT * 2)
         *reinterpret_cast<uint32_t*>(dst + n * 8 + qc) =
-            Num<__nv_bfloat16>::pack(o[n][r2i * 2] * f, o[n][r2i * 2 + 1] * f);
+            Num<__nv_bfloat16>::pack(gated_out(o[n][r2i * 2] * f, gate, gi + n * 8, out_mul),
+                                     gated_out(o[n][r2i * 2 + 1] * f, gate, gi + n * 8 + 1, out_mul));
   }
 }
 
 template <int KS_MAX, int VT_MAX, bool EXACT>
 int launch_prefill(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache, const float* r1,
-                   const float* r2, const float* sink, const int* q_cu, const int* kv_cu, const int* tables,
+                   const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul, const int* q_cu, const int* kv_cu, const int* tables,
                    const int* blk_cu, int64_t n_seq, int64_t q_max, int H, int G, int dim, int vdim, int block_size,
                    float scale, cudaStream_t st) {
   const int R = H / G;
@@ -461,7 +583,8 @@ int launch_prefill(void* out, int64_t ldo, const float* q, const void* k_cache, 
     B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   dim3 grid((unsigned)((q_max + BQ - 1) / BQ), (unsigned)n_seq, (unsigned)(G * chunks));
   kern<<<grid, 128, smem, st>>>(static_cast<__nv_bfloat16*>(out), ldo, q, static_cast<const __nv_bfloat16*>(k_cache),
-                                static_cast<const __nv_bfloat16*>(v_cache), r1, r2, sink, q_cu, kv_cu, tables, blk_cu,
+                                static_cast<const __nv_bfloat16*>(v_cache), r1, r2, sink,
+                                static_cast<const __nv_bfloat16*>(gate), ld_gate, out_mul, q_cu, kv_cu, tables, blk_cu,
                                 H, G, dim, vdim, block_size, scale, RW, chunks);
   B200_LAUNCH_OK("sink_attn_prefill_kernel");
   return B200_OK;
@@ -484,6 +607,7 @@ __global__ void __launch_bounds__(128)
 sink_attn_decode_tc_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const float* __restrict__ q,
                            const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
                            const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink,
+                           const __nv_bfloat16* __restrict__ gate, int64_t ld_gate, float out_mul,
                            const int* __restrict__ q_cu, const int* __restrict__ kv_cu,
                            const int* __restrict__ block_tables, const int* __restrict__ cu_block_lens,
                            const int* __restrict__ token_seq, int H, int G, int dim, int vdim, int block_size,
@@ -694,7 +818,9 @@ sink_attn_decode_tc_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const f
 #pragma unroll
     for (int c = 0; c < 4; ++c) {
       const int col = lane + 32 * c;
-      if (col < vdim) out[(size_t)row * ldo + (size_t)h * vdim + col] = __float2bfloat16_rn(x[c] * fo);
+      if (col < vdim)
+        out[(size_t)row * ldo + (size_t)h * vdim + col] = __float2bfloat16_rn(
+            gated_out(x[c] * fo, gate, (size_t)row * ld_gate + (size_t)h * vdim + col, out_mul));
     }
   }
 }
@@ -703,7 +829,8 @@ sink_attn_decode_tc_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const f
 // shares' maxima, sums and weighted sums and lets the sink into the denominator.
 __global__ void __launch_bounds__(128)
 sink_attn_merge_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const float* __restrict__ ws,
-                       const float* __restrict__ sink, int64_t n_pairs, int H, int vdim, int n_splits) {
+                       const float* __restrict__ sink, const __nv_bfloat16* __restrict__ gate, int64_t ld_gate,
+                       float out_mul, int64_t n_pairs, int H, int vdim, int n_splits) {
   const int64_t pair = (int64_t)blockIdx.x * 4 + (threadIdx.x >> 5);      // row * H + head
   const int lane = threadIdx.x & 31;
   if (pair >= n_pairs) return;
@@ -726,14 +853,16 @@ sink_attn_merge_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const float
 #pragma unroll
   for (int c = 0; c < 4; ++c) {
     const int col = lane + 32 * c;
-    if (col < vdim) out[row * ldo + (size_t)h * vdim + col] = __float2bfloat16_rn(x[c] * fo);
+    if (col < vdim)
+      out[row * ldo + (size_t)h * vdim + col] = __float2bfloat16_rn(
+          gated_out(x[c] * fo, gate, (size_t)row * ld_gate + (size_t)h * vdim + col, out_mul));
   }
 }
 
 template <int KS_MAX, int VT_MAX>
 int launch_decode_tc(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache, const float* r1,
-                     const float* r2, const float* sink, const int* q_cu, const int* kv_cu, const int* tables,
-                     const int* blk_cu, const int* token_seq, int64_t rows, int H, int G, int dim, int vdim,
+                     const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul,
+                     const int* q_cu, const int* kv_cu, const int* tables, const int* blk_cu, const int* token_seq, int64_t rows, int H, int G, int dim, int vdim,
                      int block_size, float scale, int n_splits, float* ws, cudaStream_t st) {
   const int R = H / G;
   const size_t tiles = ((size_t)kDS * kDK * (dim + 8) + (size_t)kDS * kDK * (vdim + 8)) * sizeof(__nv_bfloat16);
@@ -745,13 +874,15 @@ int launch_decode_tc(void* out, int64_t ldo, const float* q, const void* k_cache
     B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   dim3 grid((unsigned)(rows * n_splits), (unsigned)G, (unsigned)((R + 15) / 16));
   kern<<<grid, 128, smem, st>>>(static_cast<__nv_bfloat16*>(out), ldo, q, static_cast<const __nv_bfloat16*>(k_cache),
-                                static_cast<const __nv_bfloat16*>(v_cache), r1, r2, sink, q_cu, kv_cu, tables, blk_cu,
+                                static_cast<const __nv_bfloat16*>(v_cache), r1, r2, sink,
+                                static_cast<const __nv_bfloat16*>(gate), ld_gate, out_mul, q_cu, kv_cu, tables, blk_cu,
                                 token_seq, H, G, dim, vdim, block_size, scale, n_splits, n_splits > 1 ? ws : nullptr);
   B200_LAUNCH_OK("sink_attn_decode_tc_kernel");
   if (n_splits > 1) {
     const int64_t n_pairs = rows * H;
-    sink_attn_merge_kernel<<<(unsigned)((n_pairs + 3) / 4), 128, 0, st>>>(static_cast<__nv_bfloat16*>(out), ldo, ws,
-                                                                          sink, n_pairs, H, vdim, n_splits);
+    sink_attn_merge_kernel<<<(unsigned)((n_pairs + 3) / 4), 128, 0, st>>>(
+        static_cast<__nv_bfloat16*>(out), ldo, ws, sink, static_cast<const __nv_bfloat16*>(gate), ld_gate, out_mul, n_pairs,
+        H, vdim, n_splits);
     B200_LAUNCH_OK("sink_attn_merge_kernel");
   }
   return B200_OK;
@@ -792,22 +923,47 @@ int b200_sink_attn_prepare(float* q_out, const void* q_in, const void* k_in, con
   return B200_OK;
 }
 
+int b200_sink_attn_prepare_turned(float* q_out, const void* q_in, const void* k_in, const void* v_in, int64_t ld,
+                                  const float* q_weight, const float* k_weight, const float* inv_freq, void* k_cache,
+                                  void* v_cache, const int32_t* positions, const int32_t* slots, int64_t rows, int64_t H,
+                                  int64_t G, int64_t dim, int64_t vdim, int64_t rot_dims, float eps, int dtype,
+                                  b200_stream_t stream) {
+  if (rows == 0) return B200_OK;
+  B200_CHECK_ARG(q_out && q_in && k_in && v_in && q_weight && k_weight && k_cache && v_cache && positions && slots,
+                 "sink_attn_prepare_turned: null pointer");
+  B200_CHECK_ARG(rows > 0 && H > 0 && G > 0 && H % G == 0 && dim > 0 && vdim > 0 && ld >= H * dim && ld >= G * vdim &&
+                     rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim && (rot_dims == 0 || inv_freq),
+                 "sink_attn_prepare_turned: bad shape (an even number of turned channels, at most the head's)");
+  auto st = static_cast<cudaStream_t>(stream);
+#define SPT_CALL(T)                                                                                                  \
+  return launch_prepare_turned<T>(q_out, q_in, k_in, v_in, ld, q_weight, k_weight, inv_freq, k_cache, v_cache, positions, \
+                                  slots, rows, (int)H, (int)G, (int)dim, (int)vdim, (int)rot_dims, eps, st)
+  switch (dtype) {
+    case B200_BF16: SPT_CALL(__nv_bfloat16);
+    case B200_FP16: SPT_CALL(__half);
+    case B200_FP32: SPT_CALL(float);
+    default: return set_error(B200_ERR_INVALID_ARG, "bad dtype %d", dtype);
+  }
+#undef SPT_CALL
+}
+
 int b200_sink_attn(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache, const float* r1,
-                   const float* r2, const float* sink, const int32_t* q_cu_lens, const int32_t* kv_cu_lens,
-                   const int32_t* block_tables, const int32_t* cu_block_lens, const int32_t* token_seq, int64_t rows,
+                   const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul,
+                   const int32_t* q_cu_lens, const int32_t* kv_cu_lens, const int32_t* block_tables, const int32_t* cu_block_lens, const int32_t* token_seq, int64_t rows,
                    int64_t H, int64_t G, int64_t dim, int64_t vdim, int64_t block_size, float scale, int dtype,
                    b200_stream_t stream) {
   if (rows == 0) return B200_OK;
   B200_CHECK_ARG(out && q && k_cache && v_cache && q_cu_lens && kv_cu_lens && block_tables && cu_block_lens && token_seq,
                  "sink_attn: null pointer");
   B200_CHECK_ARG((r1 == nullptr) == (r2 == nullptr), "sink_attn: the distance bias takes both of its numbers");
+  B200_CHECK_ARG(!gate || ld_gate >= H * vdim, "sink_attn: gate rows shorter than the heads");
   B200_CHECK_ARG(rows > 0 && H > 0 && G > 0 && G <= 65535 && H % G == 0 && dim > 0 && vdim > 0 && vdim <= kMaxVdim &&
                      block_size > 0 && ldo >= H * vdim,
                  "sink_attn: bad shape (value heads of at most %d channels)", kMaxVdim);
   auto st = static_cast<cudaStream_t>(stream);
 #define SA_CALL(T)                                                                                                 \
-  return dispatch_simt<T>(out, ldo, q, k_cache, v_cache, r1, r2, sink, q_cu_lens, kv_cu_lens, block_tables,         \
-                          cu_block_lens, token_seq, rows, (int)H, (int)G, (int)dim, (int)vdim, (int)block_size, scale, st)
+  return dispatch_simt<T>(out, ldo, q, k_cache, v_cache, r1, r2, sink, gate, ld_gate, out_mul, q_cu_lens, kv_cu_lens, \
+                          block_tables, cu_block_lens, token_seq, rows, (int)H, (int)G, (int)dim, (int)vdim, (int)block_size, scale, st)
   switch (dtype) {
     case B200_BF16: SA_CALL(__nv_bfloat16);
     case B200_FP16: SA_CALL(__half);
@@ -822,14 +978,15 @@ int b200_sink_attn_prefill_supported(int64_t dim, int64_t vdim, int dtype) {
 }
 
 int b200_sink_attn_prefill(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache,
-                           const float* r1, const float* r2, const float* sink, const int32_t* q_cu_lens,
-                           const int32_t* kv_cu_lens, const int32_t* block_tables, const int32_t* cu_block_lens,
+                           const float* r1, const float* r2, const float* sink, const void* gate, int64_t ld_gate,
+                           float out_mul, const int32_t* q_cu_lens, const int32_t* kv_cu_lens, const int32_t* block_tables, const int32_t* cu_block_lens,
                            int64_t n_seq, int64_t q_max, int64_t H, int64_t G, int64_t dim, int64_t vdim,
                            int64_t block_size, float scale, int dtype, b200_stream_t stream) {
   if (n_seq == 0 || q_max == 0) return B200_OK;
   B200_CHECK_ARG(out && q && k_cache && v_cache && q_cu_lens && kv_cu_lens && block_tables && cu_block_lens,
                  "sink_attn_prefill: null pointer");
   B200_CHECK_ARG((r1 == nullptr) == (r2 == nullptr), "sink_attn_prefill: the distance bias takes both of its numbers");
+  B200_CHECK_ARG(!gate || ld_gate >= H * vdim, "sink_attn_prefill: gate rows shorter than the heads");
   B200_CHECK_ARG(b200_sink_attn_prefill_supported(dim, vdim, dtype),
                  "sink_attn_prefill: bf16 with head sizes that are multiples of 16 and at most 128");
   B200_CHECK_ARG(n_seq > 0 && n_seq <= 65535 && q_max > 0 && H > 0 && G > 0 && H % G == 0 && block_size > 0 &&
@@ -837,8 +994,8 @@ int b200_sink_attn_prefill(void* out, int64_t ldo, const float* q, const void* k
                      is_aligned(v_cache, 16) && G * ((H / G + 3) / 4) <= 65535,
                  "sink_attn_prefill: bad shape or alignment");
   auto st = static_cast<cudaStream_t>(stream);
-#define SPF_ARGS out, ldo, q, k_cache, v_cache, r1, r2, sink, q_cu_lens, kv_cu_lens, block_tables, cu_block_lens, n_seq, \
-                 q_max, (int)H, (int)G, (int)dim, (int)vdim, (int)block_size, scale, st
+#define SPF_ARGS out, ldo, q, k_cache, v_cache, r1, r2, sink, gate, ld_gate, out_mul, q_cu_lens, kv_cu_lens, \
+                 block_tables, cu_block_lens, n_seq, q_max, (int)H, (int)G, (int)dim, (int)vdim, (int)block_size, scale, st
   if (dim == 64 && vdim == 64) return launch_prefill<4, 4, true>(SPF_ARGS);
   if (dim == 128 && vdim == 128) return launch_prefill<8, 8, true>(SPF_ARGS);
   if (dim <= 64 && vdim <= 64) return launch_prefill<4, 4, false>(SPF_ARGS);
@@ -847,8 +1004,8 @@ int b200_sink_attn_prefill(void* out, int64_t ldo, const float* q, const void* k
 }
 
 int b200_sink_attn_decode_tc(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache,
-                             const float* r1, const float* r2, const float* sink, const int32_t* q_cu_lens,
-                             const int32_t* kv_cu_lens, const int32_t* block_tables, const int32_t* cu_block_lens,
+                             const float* r1, const float* r2, const float* sink, const void* gate, int64_t ld_gate,
+                             float out_mul, const int32_t* q_cu_lens, const int32_t* kv_cu_lens, const int32_t* block_tables, const int32_t* cu_block_lens,
                              const int32_t* token_seq, int64_t rows, int64_t H, int64_t G, int64_t dim, int64_t vdim,
                              int64_t block_size, float scale, int64_t n_splits, float* workspace,
                              int64_t workspace_floats, int dtype, b200_stream_t stream) {
@@ -856,6 +1013,7 @@ int b200_sink_attn_decode_tc(void* out, int64_t ldo, const float* q, const void*
   B200_CHECK_ARG(out && q && k_cache && v_cache && q_cu_lens && kv_cu_lens && block_tables && cu_block_lens && token_seq,
                  "sink_attn_decode_tc: null pointer");
   B200_CHECK_ARG((r1 == nullptr) == (r2 == nullptr), "sink_attn_decode_tc: the distance bias takes both of its numbers");
+  B200_CHECK_ARG(!gate || ld_gate >= H * vdim, "sink_attn_decode_tc: gate rows shorter than the heads");
   B200_CHECK_ARG(b200_sink_attn_prefill_supported(dim, vdim, dtype),
                  "sink_attn_decode_tc: bf16 with head sizes that are multiples of 16 and at most 128");
   B200_CHECK_ARG(rows > 0 && H > 0 && G > 0 && G <= 65535 && H % G == 0 && block_size > 0 && ldo >= H * vdim &&
@@ -864,8 +1022,8 @@ int b200_sink_attn_decode_tc(void* out, int64_t ldo, const float* q, const void*
   B200_CHECK_ARG(n_splits == 1 || (workspace && workspace_floats >= rows * H * n_splits * (2 + vdim)),
                  "sink_attn_decode_tc: workspace of rows * H * n_splits * (2 + vdim) floats required");
   auto st = static_cast<cudaStream_t>(stream);
-#define SDT_ARGS out, ldo, q, k_cache, v_cache, r1, r2, sink, q_cu_lens, kv_cu_lens, block_tables, cu_block_lens, \
-                 token_seq, rows, (int)H, (int)G, (int)dim, (int)vdim, (int)block_size, scale, (int)n_splits, workspace, st
+#define SDT_ARGS out, ldo, q, k_cache, v_cache, r1, r2, sink, gate, ld_gate, out_mul, q_cu_lens, kv_cu_lens, \
+                 block_tables, cu_block_lens, token_seq, rows, (int)H, (int)G, (int)dim, (int)vdim, (int)block_size, scale, (int)n_splits, workspace, st
   if (dim <= 64 && vdim <= 64) return launch_decode_tc<4, 4>(SDT_ARGS);
   return launch_decode_tc<8, 8>(SDT_ARGS);
 #undef SDT_ARGS

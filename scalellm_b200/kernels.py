@@ -1236,6 +1236,32 @@ def sink_attn_prepare(q_in: torch.Tensor, k_in: torch.Tensor, v_in: torch.Tensor
     return q
 
 
+def sink_attn_prepare_turned(q_in: torch.Tensor, k_in: torch.Tensor, v_in: torch.Tensor, q_weight: torch.Tensor,
+                             k_weight: torch.Tensor, inv_freq: Optional[torch.Tensor], k_cache: torch.Tensor,
+                             v_cache: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, H: int, G: int,
+                             dim: int, vdim: int, rot_dims: int, eps: float) -> torch.Tensor:
+    """Queries (fp32 [rows, H, dim]) and keys under one root mean square per projection row and a weight per channel,
+    then turned (the first rot_dims channels of a head, channel t with t + rot_dims / 2); keys and plain values go to
+    the cache rows `slots`.  q_in, k_in, v_in: column blocks of one projection matrix."""
+    _cuda(q_in, k_in, v_in, q_weight, k_weight, inv_freq, k_cache, v_cache)
+    _f32(q_weight, k_weight, inv_freq)
+    _check_i32(positions, slots)
+    rows, ld = q_in.shape[0], q_in.stride(0)
+    assert q_in.shape[1] == H * dim and k_in.shape[1] == G * dim and v_in.shape[1] == G * vdim
+    assert q_weight.numel() == H * dim and k_weight.numel() == G * dim
+    assert inv_freq is None or inv_freq.numel() == rot_dims // 2
+    for t in (q_in, k_in, v_in):
+        assert t.stride(1) == 1 and t.stride(0) == ld and t.dtype == q_in.dtype
+    assert k_cache.dtype == v_cache.dtype == q_in.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert k_cache.shape[1:] == (G, dim) and v_cache.shape[1:] == (G, vdim)
+    q = torch.empty((rows, H, dim), dtype=torch.float32, device=q_in.device)
+    check(_lib.load().b200_sink_attn_prepare_turned(_p(q), _p(q_in), _p(k_in), _p(v_in), ld, _p(q_weight),
+                                                    _p(k_weight), _p(inv_freq), _p(k_cache), _p(v_cache),
+                                                    _p(positions), _p(slots), rows, H, G, dim, vdim, rot_dims, eps,
+                                                    _dt(q_in), _stream()))
+    return q
+
+
 # a step whose longest portion has at least this many tokens runs the tensor-core kernel (bf16, fitting head sizes)
 SINK_ATTN_PREFILL_MIN_ROWS = 4
 # single tokens in bf16 with at least this many query heads per key/value head run as tensor-core tiles of heads
@@ -1245,25 +1271,33 @@ SINK_ATTN_DECODE_TC_MIN_GROUP = 2
 def sink_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, r1: Optional[torch.Tensor],
               r2: Optional[torch.Tensor], sink: Optional[torch.Tensor], q_cu: torch.Tensor, kv_cu: torch.Tensor,
               block_tables: torch.Tensor, cu_block_lens: torch.Tensor, token_seq: torch.Tensor, block_size: int,
-              scale: float, n_seq: int = 0, q_max: int = 0, kv_max: int = 0, n_splits: int = 0) -> torch.Tensor:
-    """[rows, H * vdim] in the cache's dtype: causal softmax attention with the score scale q . k - r1 ln(1 + r2
+              scale: float, n_seq: int = 0, q_max: int = 0, kv_max: int = 0, n_splits: int = 0,
+              gate: Optional[torch.Tensor] = None, out_mul: float = 1.0,
+              out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """[rows, H * vdim] in the cache's dtype (into `out` where given): causal softmax attention with the score scale q . k - r1 ln(1 + r2
     (i - j)) and exp(sink) added to the denominator (r1 / r2 / sink fp32 [H] or None).  With n_seq and q_max (the
     step's sequence count and longest portion, host numbers) a step with prompt portions in bf16 runs on the tensor
     cores where the head sizes allow it; single tokens in bf16 with grouped heads run as tensor-core tiles of heads,
     their keys shared out over several CTAs per row when the step has few rows (kv_max: an upper bound of the cached
-    lengths, sizes the split; n_splits forces it); fp32 and odd sizes run the CUDA-core kernel."""
-    _cuda(q, k_cache, v_cache, r1, r2, sink)
+    lengths, sizes the split; n_splits forces it); fp32 and odd sizes run the CUDA-core kernel.  What is stored is
+    out_mul * result * sigmoid(gate) (gate [rows, H * vdim], a column block, or None)."""
+    _cuda(q, k_cache, v_cache, r1, r2, sink, gate, out)
     _f32(q, r1, r2, sink)
     _check_i32(q_cu, kv_cu, block_tables, cu_block_lens, token_seq)
     rows, H, dim = q.shape
     G, vdim = v_cache.shape[1], v_cache.shape[2]
-    out = torch.empty((rows, H * vdim), dtype=k_cache.dtype, device=q.device)
+    if out is None:
+        out = torch.empty((rows, H * vdim), dtype=k_cache.dtype, device=q.device)
+    assert out.shape == (rows, H * vdim) and out.stride(1) == 1 and out.dtype == k_cache.dtype
+    assert gate is None or (gate.shape == out.shape and gate.stride(1) == 1 and gate.dtype == out.dtype)
+    ldo, ldg = out.stride(0), gate.stride(0) if gate is not None else 0
     lib = _lib.load()
     impl = os.environ.get("B200_SINK_ATTN_IMPL")      # "simt": CUDA cores throughout; "simt_decode": for single tokens
     if (n_seq > 0 and q_max >= SINK_ATTN_PREFILL_MIN_ROWS and impl != "simt"
+            and ldo % 2 == 0 and out.data_ptr() % 4 == 0
             and lib.b200_sink_attn_prefill_supported(dim, vdim, _dt(k_cache))):
-        check(lib.b200_sink_attn_prefill(_p(out), H * vdim, _p(q), _p(k_cache), _p(v_cache), _p(r1), _p(r2), _p(sink),
-                                         _p(q_cu), _p(kv_cu), _p(block_tables), _p(cu_block_lens), n_seq, q_max, H, G,
+        check(lib.b200_sink_attn_prefill(_p(out), ldo, _p(q), _p(k_cache), _p(v_cache), _p(r1), _p(r2), _p(sink),
+                                         _p(gate), ldg, out_mul, _p(q_cu), _p(kv_cu), _p(block_tables), _p(cu_block_lens), n_seq, q_max, H, G,
                                          dim, vdim, block_size, scale, _dt(k_cache), _stream()))
         return out
     if (impl not in ("simt", "simt_decode") and H // G >= SINK_ATTN_DECODE_TC_MIN_GROUP
@@ -1278,13 +1312,13 @@ def sink_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, r1:
         ws = None
         if n_splits > 1:
             ws = torch.empty(rows * H * n_splits * (2 + vdim), dtype=torch.float32, device=q.device)
-        check(lib.b200_sink_attn_decode_tc(_p(out), H * vdim, _p(q), _p(k_cache), _p(v_cache), _p(r1), _p(r2), _p(sink),
-                                           _p(q_cu), _p(kv_cu), _p(block_tables), _p(cu_block_lens), _p(token_seq),
+        check(lib.b200_sink_attn_decode_tc(_p(out), ldo, _p(q), _p(k_cache), _p(v_cache), _p(r1), _p(r2), _p(sink),
+                                           _p(gate), ldg, out_mul, _p(q_cu), _p(kv_cu), _p(block_tables), _p(cu_block_lens), _p(token_seq),
                                            rows, H, G, dim, vdim, block_size, scale, n_splits, _p(ws),
                                            ws.numel() if ws is not None else 0, _dt(k_cache), _stream()))
         return out
-    check(lib.b200_sink_attn(_p(out), H * vdim, _p(q), _p(k_cache), _p(v_cache), _p(r1), _p(r2), _p(sink), _p(q_cu),
-                             _p(kv_cu), _p(block_tables), _p(cu_block_lens), _p(token_seq), rows, H, G, dim, vdim,
+    check(lib.b200_sink_attn(_p(out), ldo, _p(q), _p(k_cache), _p(v_cache), _p(r1), _p(r2), _p(sink), _p(gate), ldg,
+                             out_mul, _p(q_cu), _p(kv_cu), _p(block_tables), _p(cu_block_lens), _p(token_seq), rows, H, G, dim, vdim,
                              block_size, scale, _dt(k_cache), _stream()))
     return out
 
@@ -1510,4 +1544,121 @@ def relu_squared(x: torch.Tensor) -> torch.Tensor:
     assert x.dim() == 2 and x.stride(1) == 1
     out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
     check(_lib.load().b200_relu_squared(_p(out), _p(x), x.shape[0], x.shape[1], x.stride(0), _dt(x), _stream()))
+    return out
+
+
+# ---------------------------------------------------------------------------
+# pre-norm input side with short causal filters (csrc/filters.cu), linear recurrences with a matrix state
+# (csrc/linear_scan.cu)
+# ---------------------------------------------------------------------------
+def prenorm(x: torch.Tensor, y, weight: torch.Tensor, eps: float, dtype: torch.dtype,
+            filter: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None,
+            q_cu: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None,
+            state_slots: Optional[torch.Tensor] = None, n_seq: int = 0, q_max: int = 0):
+    """x' = x + y (y: the rows of the sublayer before, the split-K partials of the product that makes them, or None),
+    h = x' / rms(x') * weight in `dtype`; with filter [taps, W] (fp32) h_t = n_t + sum_i filter[i] n_{t - taps + 1 + i}
+    over each sequence's rows, the lags before the step from state [slots, taps - 1, W] (which then takes the step's
+    last rows).  Returns (x' — x itself where y is None —, h)."""
+    partials = y.data if isinstance(y, W4Partials) else None
+    rows_y = None if partials is not None else y
+    _cuda(x, rows_y, partials, weight, filter, state)
+    _f32(x, weight, filter, state, partials)
+    rows, W = x.shape
+    assert x.is_contiguous() and weight.numel() == W
+    if rows_y is not None:
+        assert rows_y.shape == (rows, W) and rows_y.stride(1) == 1 and rows_y.dtype == dtype
+    if partials is not None:
+        assert partials.shape[1:] == (rows, W)
+    taps = 0
+    if filter is not None:
+        _check_i32(q_cu, positions, state_slots)
+        taps = filter.shape[0]
+        assert filter.shape == (taps, W) and filter.is_contiguous() and n_seq > 0 and q_max > 0
+        assert taps == 1 or (state.shape[1:] == (taps - 1, W) and state.is_contiguous())
+    out = torch.empty_like(x) if y is not None else x
+    h = torch.empty((rows, W), dtype=dtype, device=x.device)
+    check(_lib.load().b200_prenorm(_p(out) if y is not None else None, _p(h), _p(x), _p(rows_y),
+                                   rows_y.stride(0) if rows_y is not None else 0, _p(partials),
+                                   partials.shape[0] if partials is not None else 0,
+                                   splitk_plan(W, y.K) if partials is not None else None, _p(weight), _p(filter), taps,
+                                   _p(state), _p(q_cu), _p(positions), _p(state_slots), n_seq, q_max, rows, W, eps,
+                                   _DT[dtype], _stream()))
+    return out, h
+
+
+def causal_filter(x: torch.Tensor, filter: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor,
+                  q_cu: torch.Tensor, positions: torch.Tensor, state_slots: torch.Tensor, n_seq: int, q_max: int,
+                  silu: bool) -> torch.Tensor:
+    """act(bias + sum_i filter[i] x_{t - taps + 1 + i}) per channel over each sequence's rows (filter [taps, channels]
+    fp32); the lags before the step come from state [slots, taps - 1, channels] fp32, which then takes the step's last
+    rows.  x may be a column block."""
+    _cuda(x, filter, bias, state)
+    _f32(filter, bias, state)
+    _check_i32(q_cu, positions, state_slots)
+    rows, ch = x.shape
+    taps = filter.shape[0]
+    assert x.stride(1) == 1 and filter.shape == (taps, ch) and filter.is_contiguous()
+    assert bias is None or bias.numel() == ch
+    assert taps == 1 or (state.shape[1:] == (taps - 1, ch) and state.is_contiguous())
+    out = torch.empty((rows, ch), dtype=x.dtype, device=x.device)
+    check(_lib.load().b200_causal_filter(_p(out), ch, _p(x), x.stride(0), _p(filter), _p(bias), taps, _p(state),
+                                         _p(q_cu), _p(positions), _p(state_slots), n_seq, q_max, rows, ch,
+                                         1 if silu else 0, _dt(x), _stream()))
+    return out
+
+
+def forget_scan(q: torch.Tensor, f: torch.Tensor, v: torch.Tensor, f_bias: torch.Tensor, f_low: torch.Tensor,
+                norm_weight: torch.Tensor, state: torch.Tensor, q_cu: torch.Tensor, positions: torch.Tensor,
+                state_slots: torch.Tensor, n_seq: int, q_max: int, eps: float, out_mul: float = 1.0,
+                out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """f = low + (1 - low) sigmoid(f + bias) ; S <- diag(f) S + (1 - f) v^T ; o = S^T silu(q) ; out_mul * o / rms(o) *
+    norm_weight per head, into `out` (a column block may be given).  state [slots, H, N, V] fp32."""
+    _cuda(q, f, v, f_bias, f_low, norm_weight, state, out)
+    _f32(f_bias, f_low, norm_weight, state)
+    _check_i32(q_cu, positions, state_slots)
+    H, N, V = state.shape[1:]
+    rows, ld = q.shape[0], q.stride(0)
+    for t, n in ((q, H * N), (f, H * N), (v, H * V)):
+        assert t.shape == (rows, n) and t.stride(1) == 1 and t.stride(0) == ld and t.dtype == q.dtype
+    assert f_bias.numel() == f_low.numel() == H * N and norm_weight.numel() == V and state.is_contiguous()
+    if out is None:
+        out = torch.empty((rows, H * V), dtype=q.dtype, device=q.device)
+    assert out.shape == (rows, H * V) and out.stride(1) == 1 and out.dtype == q.dtype
+    lib = _lib.load()
+    raw = torch.empty((rows, H * V), dtype=torch.float32, device=q.device) if lib.b200_linear_scan_parts(N, V) > 1 else None
+    check(lib.b200_forget_scan(_p(out), out.stride(0), _p(q), _p(f), _p(v), ld, _p(f_bias), _p(f_low), _p(norm_weight),
+                               _p(state), _p(q_cu), _p(positions), _p(state_slots), n_seq, q_max, rows, H, N, V, eps,
+                               out_mul, _p(raw), _dt(q), _stream()))
+    return out
+
+
+def ssd_scan(x: torch.Tensor, B: torch.Tensor, C_: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor,
+             a_log: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, q_cu: torch.Tensor, positions: torch.Tensor,
+             state_slots: torch.Tensor, n_seq: int, q_max: int, groups: int) -> torch.Tensor:
+    """d = softplus(dt + bias) ; S <- exp(-exp(a_log) d) S + d B x^T ; y = S^T C + skip x per head (head h reads group
+    h / (H / groups)), fp32 [rows, H * V].  state [slots, H, N, V] fp32."""
+    _cuda(x, B, C_, dt, dt_bias, a_log, skip, state)
+    _f32(dt_bias, a_log, skip, state)
+    _check_i32(q_cu, positions, state_slots)
+    H, N, V = state.shape[1:]
+    rows, ld = x.shape[0], x.stride(0)
+    for t, n in ((x, H * V), (B, groups * N), (C_, groups * N)):
+        assert t.shape == (rows, n) and t.stride(1) == 1 and t.stride(0) == ld and t.dtype == x.dtype
+    assert dt.shape == (rows, H) and dt.stride(1) == 1 and dt.dtype == x.dtype and state.is_contiguous()
+    y = torch.empty((rows, H * V), dtype=torch.float32, device=x.device)
+    check(_lib.load().b200_ssd_scan(_p(y), _p(x), _p(B), _p(C_), ld, _p(dt), dt.stride(0), _p(dt_bias), _p(a_log),
+                                    _p(skip), _p(state), _p(q_cu), _p(positions), _p(state_slots), n_seq, q_max, rows,
+                                    H, groups, N, V, _dt(x), _stream()))
+    return y
+
+
+def gated_part_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, parts: int, eps: float) -> torch.Tensor:
+    """u = y silu(z) ; u / rms_part(u) * weight with one root mean square per equal part of the row, in z's dtype."""
+    _cuda(y, z, weight)
+    _f32(y, weight)
+    rows, n = y.shape
+    assert y.is_contiguous() and z.shape == (rows, n) and z.stride(1) == 1 and weight.numel() == n
+    out = torch.empty((rows, n), dtype=z.dtype, device=z.device)
+    check(_lib.load().b200_gated_part_norm(_p(out), n, _p(y), _p(z), z.stride(0), _p(weight), rows, n, parts, eps,
+                                           _dt(z), _stream()))
     return out

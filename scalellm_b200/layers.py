@@ -766,11 +766,14 @@ class GatedMLP:
         self.gate_up, self.down, self.act = Linear(torch.cat([gate, up], dim=0)), Linear(down), act
         self.ff = gate.shape[0]
 
-    def forward(self, h: torch.Tensor) -> torch.Tensor:
+    def forward(self, h: torch.Tensor, fusable_out: bool = False):
+        """The result, or (fusable_out) the down projection's split-K partials where a fused consumer can take them."""
         if (self.act == "silu" and h.dtype == torch.bfloat16 and self.ff % 64 == 0
                 and self.gate_up.supports_partials(h.shape[0]) and kernels.silu_mul_splitk_available()):
-            return self.down(kernels.silu_mul_splitk(self.gate_up.forward_partials(h), h.dtype))
-        return self.down(kernels.gated_act(self.gate_up(h), self.act))
+            a = kernels.silu_mul_splitk(self.gate_up.forward_partials(h), h.dtype)
+        else:
+            a = kernels.gated_act(self.gate_up(h), self.act)
+        return self.down.forward_fusable(a) if fusable_out else self.down(a)
 
     __call__ = forward
 
@@ -1227,5 +1230,151 @@ class GroupLimitedMoE:
         y = kernels.grouped_gemm(kernels.glu_clamped(gu, self.limit, self.slope), self.down, real, n)
         shared = self.shared(h, fusable_out=False) if self.shared is not None else None
         return kernels.moe_combine_weighted(y, pos_of_pair, ids, wts, self.n_real, h, shared, sg)
+
+    __call__ = forward
+
+
+# ---------------------------------------------------------------------------
+# Layers of pre-norm decoders whose mixers read their input through a short causal filter and mix tokens with a
+# state-space recurrence, or with softmax attention beside a recurrence whose forget gate also decides what is written.
+# ---------------------------------------------------------------------------
+class PreNormInput:
+    """x <- x + y on an fp32 residual, then what the next sublayer reads: h = n = x / rms(x) * w, or with a filter
+    [W, taps] h_t = n_t + sum_i filter[:, i] n_{t - (taps - 1) + i} over the sequence's own rows (csrc/filters.cu).  Per
+    sequence slot the last taps - 1 rows n are kept, fp32."""
+
+    def __init__(self, weight: torch.Tensor, eps: float, filter: Optional[torch.Tensor] = None, n_slots: int = 0):
+        self.weight, self.eps = weight.to(torch.float32).contiguous(), eps
+        self.filter = self.state = None
+        if filter is not None:
+            self.filter = filter.to(torch.float32).t().contiguous()           # [taps, W]
+            taps, W = self.filter.shape
+            self.state = torch.zeros((n_slots, taps - 1, W), dtype=torch.float32, device=weight.device)
+
+    def forward(self, x: torch.Tensor, y, dtype: torch.dtype, positions: torch.Tensor, params: InputParameters):
+        """y: what the sublayer before made (rows, split-K partials, or None).  Returns (new x, h in `dtype`)."""
+        if self.filter is None:
+            return kernels.prenorm(x, y, self.weight, self.eps, dtype)
+        return kernels.prenorm(x, y, self.weight, self.eps, dtype, self.filter, self.state, params.q_cu_seq_lens,
+                               positions, params.state_slots, params.num_sequences, params.q_max_seq_len)
+
+    __call__ = forward
+
+
+class TurnedSinkAttention:
+    """Causal softmax attention over a paged cache (csrc/sink_attn.cu) with a fixed sink, no biases:
+        q, k, v, g = maps of h ; q <- q / rms(q) * wq over the whole projection row (all heads at once), k likewise ;
+        the first rot_dims channels of every q and k head turn with the position (channel t with t + rot_dims / 2) ;
+        p_j = exp(scale q . k_j) / (exp(sink) + sum_j' exp(scale q . k_j')) ;
+        result = concat_h(sum_j p_j v_j) * sigmoid(g) (before the output map),  H / G query heads per key/value head.
+    The output map belongs to the caller (`out_weight`), who may join it with another mixer's."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], n_heads: int, n_kv_heads: int, dim: int, vdim: int, scale: float,
+                 sink: float, inv_freq: Optional[torch.Tensor], rot_dims: int, eps: float, dtype: torch.dtype, device):
+        self.H, self.G, self.dim, self.vd = n_heads, n_kv_heads, dim, vdim
+        self.scale, self.rot_dims, self.eps, self.dtype = scale, rot_dims, eps, dtype
+        self.inv_freq = None if inv_freq is None else inv_freq.to(torch.float32).to(device).contiguous()
+        self.in_weight = torch.cat([w["q"], w["k"], w["v"], w["g"]], dim=0)
+        self.n_in, self.n_out = self.in_weight.shape[0], n_heads * vdim
+        self.q_end = n_heads * dim
+        self.k_end = self.q_end + n_kv_heads * dim
+        self.v_end = self.k_end + n_kv_heads * vdim
+        f = lambda name: w[name].to(torch.float32).to(device).contiguous()
+        self.q_norm, self.k_norm = f("q.norm"), f("k.norm")
+        self.sink = torch.full((n_heads,), sink, dtype=torch.float32, device=device)
+        self.out_weight = w["o"]
+
+    def run(self, proj: torch.Tensor, positions: torch.Tensor, cache: KVCache, params: InputParameters, mul: float,
+            out: torch.Tensor) -> torch.Tensor:
+        """proj [rows, n_in]: this mixer's column block of the input product; mul times the result goes to `out`."""
+        q = kernels.sink_attn_prepare_turned(proj[:, : self.q_end], proj[:, self.q_end: self.k_end],
+                                             proj[:, self.k_end: self.v_end], self.q_norm, self.k_norm, self.inv_freq,
+                                             cache.key_cache, cache.value_cache, positions, params.new_cache_slots,
+                                             self.H, self.G, self.dim, self.vd, self.rot_dims, self.eps)
+        return kernels.sink_attn(q, cache.key_cache, cache.value_cache, None, None, self.sink, params.q_cu_seq_lens,
+                                 params.kv_cu_seq_lens, params.block_tables, params.cu_block_lens, params.token_seq,
+                                 cache.block_size(), self.scale, params.num_sequences, params.q_max_seq_len,
+                                 params.kv_max_seq_len, gate=proj[:, self.v_end: self.n_in], out_mul=mul, out=out)
+
+
+class ForgetWriteMixer:
+    """Linear recurrence whose forget gate also decides what is written (csrc/linear_scan.cu):
+        q = silu(Wq h), f = low + (1 - low) sigmoid(Wf h + b), v = Wv h ;
+        S <- diag(f) S + (1 - f) v^T ; o = S^T q per head (S [dim, vdim], fp32, one per sequence slot) ;
+        result = concat_h(o / rms(o) * norm) (before the output map, which belongs to the caller)."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], n_heads: int, dim: int, vdim: int, eps: float, n_slots: int,
+                 dtype: torch.dtype, device):
+        self.H, self.dim, self.vd, self.eps = n_heads, dim, vdim, eps
+        self.in_weight = torch.cat([w["q"], w["f"], w["v"]], dim=0)
+        self.n_in, self.n_out = self.in_weight.shape[0], n_heads * vdim
+        f = lambda name: w[name].to(torch.float32).to(device).contiguous()
+        self.f_bias, self.f_low, self.norm_weight = f("f.b"), f("lower"), f("norm")
+        self.state = torch.zeros((n_slots, n_heads, dim, vdim), dtype=torch.float32, device=device)
+        self.out_weight = w["o"]
+
+    def run(self, proj: torch.Tensor, positions: torch.Tensor, params: InputParameters, mul: float,
+            out: torch.Tensor) -> torch.Tensor:
+        n = self.H * self.dim
+        return kernels.forget_scan(proj[:, :n], proj[:, n: 2 * n], proj[:, 2 * n: self.n_in], self.f_bias, self.f_low,
+                                   self.norm_weight, self.state, params.q_cu_seq_lens, positions, params.state_slots,
+                                   params.num_sequences, params.q_max_seq_len, self.eps, mul, out)
+
+
+class ScaledPairMixer:
+    """Two mixers side by side on the same rows, one with a paged cache (`left`) and one with state slots (`right`):
+    left_scale * Wl left(h) + right_scale * Wr right(h).  Everything that reads h is ONE matrix product, and so is
+    everything that leaves: both mixers write their scaled results into one row, which meets [Wl | Wr]."""
+
+    def __init__(self, left, right, left_scale: float, right_scale: float):
+        self.left, self.right, self.left_scale, self.right_scale = left, right, left_scale, right_scale
+        self.in_proj = Linear(torch.cat([left.in_weight, right.in_weight], dim=0))
+        self.o_proj = Linear(torch.cat([left.out_weight, right.out_weight], dim=1))
+        left.in_weight = right.in_weight = left.out_weight = right.out_weight = None     # held once
+
+    def forward(self, h: torch.Tensor, positions: torch.Tensor, cache: KVCache, params: InputParameters):
+        """The result, or the output product's split-K partials where a fused consumer can take them."""
+        proj = self.in_proj(h)
+        n, nl, nr = self.left.n_in, self.left.n_out, self.right.n_out
+        ld = -(-(nl + nr) // 8) * 8                  # rows start on 16 bytes whatever the head sizes are
+        both = torch.empty((h.shape[0], ld), dtype=h.dtype, device=h.device)[:, : nl + nr]
+        self.left.run(proj[:, :n], positions, cache, params, self.left_scale, both[:, :nl])
+        self.right.run(proj[:, n:], positions, params, self.right_scale, both[:, nl:])
+        return self.o_proj.forward_fusable(both)
+
+    __call__ = forward
+
+
+class StateSpaceMixer:
+    """State-space recurrence with one decay per head (csrc/linear_scan.cu, csrc/filters.cu):
+        [z | x | B | C | dt] = Win h ; [x | B | C] <- silu(filter(.) + bias), filter [channels, taps] causal ;
+        d = softplus(dt + dt_bias) ; S <- exp(-exp(A_log) d) S + d B x^T ; y = S^T C + D x per head (S [state, vdim],
+        B and C shared by the heads of a group) ; result = Wo ((y silu(z)) / rms_part * norm), the row in equal parts.
+    Per sequence slot the layer keeps S and the last taps - 1 filter inputs, both fp32."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], n_heads: int, vdim: int, state: int, groups: int, parts: int,
+                 eps: float, n_slots: int, dtype: torch.dtype, device):
+        self.H, self.vd, self.N, self.groups, self.parts, self.eps = n_heads, vdim, state, groups, parts, eps
+        self.inner, self.gn = n_heads * vdim, groups * state
+        self.in_proj, self.o_proj = Linear(w["in"]), Linear(w["o"])
+        f = lambda name: w[name].to(torch.float32).to(device).contiguous()
+        self.filter, self.filter_bias = f("conv").t().contiguous(), f("conv.b")
+        self.dt_bias, self.a_log, self.skip, self.norm_weight = f("dt_bias"), f("A_log"), f("D"), f("norm")
+        taps, ch = self.filter.shape
+        self.filter_state = torch.zeros((n_slots, taps - 1, ch), dtype=torch.float32, device=device)
+        self.state = torch.zeros((n_slots, n_heads, state, vdim), dtype=torch.float32, device=device)
+
+    def forward(self, h: torch.Tensor, positions: torch.Tensor, params: InputParameters):
+        """The result, or the output product's split-K partials where a fused consumer can take them."""
+        proj = self.in_proj(h)
+        inner, gn = self.inner, self.gn
+        xbc_end = 2 * inner + 2 * gn
+        step = (params.q_cu_seq_lens, positions, params.state_slots, params.num_sequences, params.q_max_seq_len)
+        xbc = kernels.causal_filter(proj[:, inner: xbc_end], self.filter, self.filter_bias, self.filter_state, *step,
+                                    silu=True)
+        y = kernels.ssd_scan(xbc[:, :inner], xbc[:, inner: inner + gn], xbc[:, inner + gn:], proj[:, xbc_end:],
+                             self.dt_bias, self.a_log, self.skip, self.state, *step, self.groups)
+        return self.o_proj.forward_fusable(kernels.gated_part_norm(y, proj[:, :inner], self.norm_weight, self.parts,
+                                                                   self.eps))
 
     __call__ = forward

@@ -1,6 +1,6 @@
-"""Prefill and decode throughput of the Kigalix, Pokadra, Zomurax and Fesupel designs beside the Llama decoder (Zomurax
-and Fesupel also beside Kigalix, the design nearest to them) at equal size (`bench.py --arch
-kigalix|pokadra|zomurax|fesupel`), all through the serving engine, random weights, bf16.
+"""Prefill and decode throughput of the Kigalix, Pokadra, Zomurax, Fesupel and Gugalorn designs beside the Llama decoder
+(Zomurax and Fesupel also beside Kigalix, Gugalorn beside Fesupel: the designs nearest to them) at equal size (`bench.py
+--arch kigalix|pokadra|zomurax|fesupel|gugalorn`), all through the serving engine, random weights, bf16.
 
 Per size: tokens/s of a prompt step (B sequences of L tokens in one batch) and of decode steps (B sequences
 with L cached tokens, one token each), timed with CUDA events after warm-up; and, per kind of kernel, the
@@ -802,5 +802,195 @@ def run_fesupel(args) -> None:
         out["sizes"][name] = {"shape": s, "batch": batch, "seq_len": seqlen, "fesupel": f, "kigalix": k, "llama": l,
                               "kernel_rooflines": fesupel_rooflines(s, batch, seqlen, f, k, l, peaks),
                               "kernels_alone": fesupel_kernels_alone(s, peaks),
+                              "seconds": round(time.time() - t0, 1)}
+    print(json.dumps(out))
+
+
+# ---------------------------------------------------------------------------
+# Gugalorn beside Fesupel (attention and a recurrence side by side, short filters) and Llama
+# ---------------------------------------------------------------------------
+GUGALORN_EXTRA = {"w2048": dict(kv_heads=4, rheads=16, rdim=128, rvdim=128, taps=4, canon=4, mheads=64, mvdim=64,
+                                mstate=128, mgroups=8),
+                  "w4096": dict(kv_heads=8, rheads=32, rdim=128, rvdim=128, taps=4, canon=4, mheads=128, mvdim=64,
+                                mstate=128, mgroups=8)}
+GUGALORN_KERNELS = ["bigram_embed", "prenorm", "causal_filter", "ssd_scan", "gated_part_norm", "sink_attn_prepare_turned",
+                    "sink_attn", "forget_scan", "gated_act", "silu_mul_splitk"]
+
+
+def gugalorn_config(s: dict) -> dict:
+    """State-space layers without a feed-forward and layers of both mixers with one, in turn."""
+    left = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"],
+            "scale": s["dim"] ** -0.5, "rot": {"base": 10000.0, "dims": s["rot"]}}
+    right = {"heads": s["rheads"], "dim": s["rdim"], "vdim": s["rvdim"]}
+    pattern = [{"type": "mamba2", "mixer": {"heads": s["mheads"], "vdim": s["mvdim"], "state": s["mstate"],
+                                            "groups": s["mgroups"], "norm_groups": s["mgroups"], "conv": s["taps"]},
+                "mlp": None},
+               {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 0.7, "right_scale": 0.7},
+                "mlp": {"kind": "dense", "ff": s["ff"]}}]
+    return {"architecture": "Gugalorn", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-5},
+            "canon": {"taps": s["canon"]}, "embedding": {"scale": 1.0},
+            "layers": [pattern[i % 2] for i in range(s["layers"])]}
+
+
+def _forget_bytes(rows: int, batch: int, s: dict) -> int:
+    H, N, V = s["rheads"], s["rdim"], s["rvdim"]
+    return rows * H * (2 * N + 2 * V) * 2 + batch * 2 * H * N * V * 4
+
+
+def _ssd_bytes(rows: int, batch: int, s: dict) -> int:
+    H, N, V = s["mheads"], s["mstate"], s["mvdim"]
+    return rows * (H * V * (2 + 4) + 2 * s["mgroups"] * N * 2 + H * 2) + batch * 2 * H * N * V * 4
+
+
+def gugalorn_rooflines(s: dict, batch: int, seqlen: int, g: dict, f: dict, l: dict, peaks: dict) -> dict:
+    """As fesupel_rooflines: the design's kernels from the per-kernel times of one step of each model (all layers of that
+    kind together), each beside the like kernel of the nearest existing models."""
+    hbm, tf = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    L, W = s["layers"], s["width"]
+    n_ssd, n_par = (L + 1) // 2, L // 2
+    H, G, dim, vd = s["heads"], s["kv_heads"], s["dim"], s["vdim"]
+    inner, ch = s["mheads"] * s["mvdim"], s["mheads"] * s["mvdim"] + 2 * s["mgroups"] * s["mstate"]
+    RH, RG, rd, rv = s["rheads"], s["rkv"], s["rdim"], s["rvdim"]
+    out = {}
+    for phase in ("decode", "prefill"):
+        q_len = 1 if phase == "decode" else seqlen
+        ctx = seqlen + 1 if phase == "decode" else seqlen
+        rows = batch * q_len
+        gm, fm, lm = g[phase]["kernels_ms"], f[phase]["kernels_ms"], l[phase]["kernels_ms"]
+        pairs = batch * _visible_pairs(ctx, q_len, 0, 0)
+        fr = lambda ms, nbytes, flops: _frac(ms, nbytes, flops, hbm, tf)
+        out[f"gugalorn sink_attn (gated) {phase}"] = fr(
+            gm.get("sink_attn", 0.0), n_par * (batch * ctx * G * (dim + vd) * 2 + rows * H * (dim * 4 + vd * 4)),
+            n_par * pairs * H * 2 * (dim + vd))
+        Hl, Hkv = W // 128, max(1, W // 512)
+        out[f"llama paged attention {phase}"] = fr(
+            lm.get("paged_kv_varlen_mha", 0.0), L * (batch * ctx * 2 * Hkv * 128 * 2 + rows * Hl * 128 * 4),
+            L * pairs * Hl * 4 * 128)
+        blk = s["block"]
+        bpairs = batch * _block_pairs(ctx, q_len, blk)
+        touched = batch * (min(ctx, (ctx - 1) % blk + 1) if phase == "decode" else ctx)
+        out[f"fesupel sigmoid_attn (blocks of {blk}) {phase}"] = fr(
+            fm.get("sigmoid_attn", 0.0), L * (touched * G * (dim + vd) * 2 + rows * H * (dim * 4 + vd * 2)),
+            L * bpairs * H * 2 * (dim + vd))
+        out[f"gugalorn forget_scan {phase}"] = fr(gm.get("forget_scan", 0.0), n_par * _forget_bytes(rows, batch, s),
+                                                  n_par * rows * RH * 5 * rd * rv)
+        out[f"gugalorn ssd_scan {phase}"] = fr(gm.get("ssd_scan", 0.0), n_ssd * _ssd_bytes(rows, batch, s),
+                                               n_ssd * rows * s["mheads"] * 5 * s["mstate"] * s["mvdim"])
+        out[f"fesupel gated_delta_scan {phase}"] = fr(
+            fm.get("gated_delta_scan", 0.0),
+            L * (rows * (2 * RG * rd * 4 + RH * rd * 4 + RH * rv * 8) + batch * 2 * RH * rd * rv * 4),
+            L * rows * RH * 6 * rd * rv)
+        out[f"gugalorn causal_filter {phase}"] = fr(gm.get("causal_filter", 0.0), n_ssd * rows * ch * 4, 0)
+        out[f"gugalorn gated_part_norm {phase}"] = fr(gm.get("gated_part_norm", 0.0), n_ssd * rows * inner * 8, 0)
+        nch = 2 * RG * rd + RH * rv
+        out[f"fesupel gated_delta_prepare {phase}"] = fr(
+            fm.get("gated_delta_prepare", 0.0), L * rows * (nch * 2 + RH * rd * 2 + nch * 4 + RH * rd * 4), 0)
+        out[f"gugalorn sink_attn_prepare_turned {phase}"] = fr(
+            gm.get("sink_attn_prepare_turned", 0.0),
+            n_par * rows * ((H + G) * dim * 2 + G * vd * 2 + H * dim * 4 + G * (dim + vd) * 2), 0)
+        out[f"fesupel sigmoid_attn_prepare {phase}"] = fr(
+            fm.get("sigmoid_attn_prepare", 0.0),
+            L * rows * ((H + G) * dim * 2 + G * vd * 2 + H * dim * 4 + G * (dim + vd) * 2), 0)
+        # every sublayer but the first reads x (4) and a result (2) and writes x (4) and 16 bits
+        out[f"gugalorn prenorm {phase}"] = fr(gm.get("prenorm", 0.0), rows * W * ((n_ssd + 2 * n_par) * 12 + 6), 0)
+        out[f"fesupel branch_norm_residual {phase}"] = fr(fm.get("branch_norm_residual", 0.0), rows * W * L * (14 + 12), 0)
+        out[f"llama rms_norm_residual {phase}"] = fr(
+            lm.get("rms_norm_residual", 0.0) + lm.get("rms_norm", 0.0) + lm.get("rms_norm_residual_splitk", 0.0),
+            rows * W * (2 * L + 1) * 4 * 2, 0)
+    return out
+
+
+def gugalorn_kernels_alone(s: dict, peaks: dict, cases=((64, 4096, 1), (4, 2048, 2048))) -> dict:
+    """The design's attention and recurrence kernels alone beside their like kernels, on caches larger than L2: (batch,
+    cached length, new tokens per sequence) = decoding over long contexts and one prompt portion.  CUDA events around 10
+    launches after 3."""
+    from . import kernels
+    from .decode_step import BlockPool, StepBuffers, build_step_batch
+    dev = torch.device("cuda", torch.cuda.current_device())
+    hbm, tf = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    H, G, dim, vd = s["heads"], s["kv_heads"], s["dim"], s["vdim"]
+    RH, RG, rd, rv = s["rheads"], s["rkv"], s["rdim"], s["rvdim"]
+    MH, mv, mn, mg = s["mheads"], s["mvdim"], s["mstate"], s["mgroups"]
+    bs, out = 16, {}
+    for batch, ctx, q_len in cases:
+        n_blocks = batch * (-(-ctx // bs)) + 8
+        pool = BlockPool(n_blocks, bs, seed=1)
+        seqs = []
+        for _ in range(batch):
+            sq = pool.open_sequence()
+            pool.reserve(sq, ctx)
+            seqs.append(sq)
+        hb = build_step_batch(pool, seqs, [[0] * q_len] * batch, [ctx - q_len] * batch, list(range(batch)))
+        tokens, positions, prm = StepBuffers(dev, batch * q_len, batch, n_blocks).upload(hb)
+        rows = batch * q_len
+        g = torch.Generator(device=dev).manual_seed(0)
+        rnd = lambda *shape: torch.randn(shape, generator=g, device=dev, dtype=torch.float32).to(torch.bfloat16)
+        r32 = lambda *shape: torch.randn(shape, generator=g, device=dev, dtype=torch.float32)
+        step = (prm.q_cu_seq_lens, positions, prm.state_slots, batch, q_len)
+        kc, vc, q = rnd(n_blocks * bs, G, dim), rnd(n_blocks * bs, G, vd), r32(rows, H, dim)
+        gate, sink, bias = rnd(rows, H * vd), torch.zeros(H, device=dev), 0.1 + 0.3 * torch.rand(H, device=dev)
+        f_sink = lambda b, gt: (lambda: kernels.sink_attn(
+            q, kc, vc, b, b, sink, prm.q_cu_seq_lens, prm.kv_cu_seq_lens, prm.block_tables, prm.cu_block_lens,
+            prm.token_seq, bs, dim ** -0.5, batch, q_len, ctx, gate=gt, out_mul=0.7))
+        kl, vl = rnd(n_blocks * bs, G, dim), rnd(n_blocks * bs, G, dim)
+        ql, ol = rnd(rows, H, dim), torch.empty((rows, H, dim), dtype=torch.bfloat16, device=dev)
+        f_llama = lambda: kernels.paged_kv_varlen_mha(ol, ql, kl, vl, prm.q_cu_seq_lens, prm.kv_cu_seq_lens,
+                                                      prm.block_tables, prm.cu_block_lens, None, bs, q_len, ctx,
+                                                      dim ** -0.5, 0.0, -1)
+        n, nv = RH * rd, RH * rv
+        rp = rnd(rows, 2 * n + nv)
+        fb, low, wn = r32(n), torch.rand(n, device=dev), torch.ones(rv, device=dev)
+        st = torch.zeros((batch, RH, rd, rv), dtype=torch.float32, device=dev)
+        f_fs = lambda: kernels.forget_scan(rp[:, :n], rp[:, n:2 * n], rp[:, 2 * n:], fb, low, wn, st, *step, 1e-5, 0.7)
+        xbc, dt = rnd(rows, MH * mv + 2 * mg * mn), rnd(rows, MH)
+        h1 = torch.ones(MH, device=dev)
+        st2 = torch.zeros((batch, MH, mn, mv), dtype=torch.float32, device=dev)
+        f_ssd = lambda: kernels.ssd_scan(xbc[:, :MH * mv], xbc[:, MH * mv: MH * mv + mg * mn], xbc[:, MH * mv + mg * mn:],
+                                         dt, -4.0 * h1, h1, h1, st2, *step, mg)
+        dq, dk = (torch.nn.functional.normalize(r32(rows, RG, rd), dim=-1) for _ in range(2))
+        dv, dd, db = r32(rows, RH, rv), torch.sigmoid(r32(rows, RH, rd) + 3.0), torch.sigmoid(r32(rows, RH))
+        dg = rnd(rows, RH * rv)
+        st3 = torch.zeros((batch, RH, rd, rv), dtype=torch.float32, device=dev)
+        f_gd = lambda: kernels.gated_delta_scan(dq, dk, dv, dd, db, dg, wn, st3, prm.q_cu_seq_lens, positions,
+                                                prm.state_slots, 1e-5, q_len)
+        pairs = batch * _visible_pairs(ctx, q_len, 0, 0)
+        a_bytes = batch * ctx * G * (dim + vd) * 2 + rows * H * (dim * 4 + vd * 2)
+        for name, fn, nbytes, flops in (
+                ("gugalorn sink_attn, gated", f_sink(None, gate), a_bytes + rows * H * vd * 2, pairs * H * 2 * (dim + vd)),
+                ("zomurax sink_attn (with its distance bias)", f_sink(bias, None), a_bytes, pairs * H * 2 * (dim + vd)),
+                ("llama paged attention, same heads", f_llama, batch * ctx * 2 * G * dim * 2 + rows * H * dim * 4,
+                 pairs * H * 4 * dim),
+                ("gugalorn forget_scan", f_fs, _forget_bytes(rows, batch, s), rows * RH * 5 * rd * rv),
+                ("gugalorn ssd_scan", f_ssd, _ssd_bytes(rows, batch, s), rows * MH * 5 * mn * mv),
+                ("fesupel gated_delta_scan", f_gd,
+                 rows * (2 * RG * rd * 4 + RH * rd * 4 + RH * rv * 8) + batch * 2 * RH * rd * rv * 4,
+                 rows * RH * 6 * rd * rv)):
+            ms = _time_steps(fn, 3, 10)
+            out[f"{name}, {batch} x {ctx} cached, {q_len} new"] = _frac(ms, nbytes, flops, hbm, tf)
+        del kc, vc, kl, vl
+        torch.cuda.empty_cache()
+    return out
+
+
+def run_gugalorn(args) -> None:
+    torch.cuda.set_device(0)
+    torch.backends.cuda.matmul.allow_tf32 = False
+    peaks_path = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "MEASURED_PEAKS.json")
+    peaks = json.load(open(peaks_path)) if os.path.exists(peaks_path) else {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+    out = {"metric": "gugalorn_vs_fesupel_vs_llama_tokens_per_s", "unit": "tokens/s", "dtype": "bf16",
+           "data": "synthetic (random-init weights, random token ids)", "n_gpus": 1,
+           "peaks": {"hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"],
+                     "source": "measured" if os.path.exists(peaks_path) else "fallback"}, "sizes": {}}
+    names = [args.arch_size] if args.arch_size != "all" else list(SIZES)
+    for name in names:
+        s = dict(SIZES[name], **dict(FESUPEL_EXTRA[name], **GUGALORN_EXTRA[name]))
+        batch, seqlen = args.arch_batch, args.arch_seqlen
+        t0 = time.time()
+        g = _run_model(gugalorn_config(s), batch, seqlen, args.warmup, args.steps, GUGALORN_KERNELS)
+        f = _run_model(fesupel_config(s), batch, seqlen, args.warmup, args.steps, FESUPEL_KERNELS)
+        l = _run_model(llama_config(s), batch, seqlen, args.warmup, args.steps, LLAMA_KERNELS)
+        out["sizes"][name] = {"shape": s, "batch": batch, "seq_len": seqlen, "gugalorn": g, "fesupel": f, "llama": l,
+                              "kernel_rooflines": gugalorn_rooflines(s, batch, seqlen, g, f, l, peaks),
+                              "kernels_alone": gugalorn_kernels_alone(s, peaks),
                               "seconds": round(time.time() - t0, 1)}
     print(json.dumps(out))

@@ -860,6 +860,9 @@ B200_API int b200_causal_filter(void* out, int64_t ldo, const void* in, int64_t 
                                 b200_stream_t stream);
 /* Column parts a head of value size V is walked in (1: its CTA holds the whole head). */
 B200_API int b200_linear_scan_parts(int64_t N, int64_t V);
+/* Whether portions of heads of these sizes can be walked 16 tokens at a time on the tensor cores (bf16; tensor_cores = 1
+ * below; rows then start on 16 bytes: ld a multiple of 8). */
+B200_API int b200_linear_scan_tc_supported(int64_t N, int64_t V, int dtype);
 /* Per head and token, S [N x V] fp32 in state[slot, h]:  f = low + (1 - low) sigmoid(f_in + f_bias) ;
  * S <- diag(f) S + (1 - f) v^T ; o = S^T silu(q_in) ; out[row, h] = mul * o / sqrt(mean(o^2) + eps) * norm_weight.
  * q / f / v: column blocks of one matrix (row stride ld), heads in order; f_bias, f_low fp32 [H * N]; norm_weight
@@ -868,7 +871,7 @@ B200_API int b200_forget_scan(void* out, int64_t ldo, const void* q, const void*
                               const float* f_bias, const float* f_low, const float* norm_weight, float* state,
                               const int32_t* q_cu_lens, const int32_t* positions, const int32_t* state_slots,
                               int64_t n_seq, int64_t q_max, int64_t rows, int64_t H, int64_t N, int64_t V, float eps,
-                              float mul, float* raw /*nullable*/, int dtype, b200_stream_t stream);
+                              float mul, float* raw /*nullable*/, int tensor_cores, int dtype, b200_stream_t stream);
 /* Per head h (group h / (H / G)) and token, S [N x V] fp32 in state[slot, h]:  d = softplus(dt + dt_bias) ;
  * S <- exp(-exp(a_log) d) S + d B x^T ; y[row, h] = S^T C + skip x  (fp32 [rows, H * V]).  x / B / C: column blocks of
  * one matrix (row stride ld); dt: row stride ld_dt; dt_bias, a_log, skip fp32 [H].  bf16 or fp32. */
@@ -876,7 +879,7 @@ B200_API int b200_ssd_scan(float* y, const void* x, const void* B, const void* C
                            int64_t ld_dt, const float* dt_bias, const float* a_log, const float* skip, float* state,
                            const int32_t* q_cu_lens, const int32_t* positions, const int32_t* state_slots,
                            int64_t n_seq, int64_t q_max, int64_t rows, int64_t H, int64_t G, int64_t N, int64_t V,
-                           int dtype, b200_stream_t stream);
+                           int tensor_cores, int dtype, b200_stream_t stream);
 /* u = y silu(z) ; out = u / sqrt(mean_part(u^2) + eps) * weight, the row of n channels in `parts` equal parts.  y fp32
  * [rows, n]; z rows of T (stride ldz).  bf16 or fp32. */
 B200_API int b200_gated_part_norm(void* out, int64_t ldo, const float* y, const void* z, int64_t ldz,

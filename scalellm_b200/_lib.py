@@ -189,10 +189,11 @@ SIGNATURES = {
     "b200_causal_filter": (_int, [_vp, _i64, _vp, _i64, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _int,
                                   _int, _vp]),
     "b200_linear_scan_parts": (_int, [_i64, _i64]),
+    "b200_linear_scan_tc_supported": (_int, [_i64, _i64, _int]),
     "b200_forget_scan": (_int, [_vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64,
-                                _i64, _i64, _i64, _f32, _f32, _vp, _int, _vp]),
+                                _i64, _i64, _i64, _f32, _f32, _vp, _int, _int, _vp]),
     "b200_ssd_scan": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64,
-                             _i64, _i64, _i64, _i64, _int, _vp]),
+                             _i64, _i64, _i64, _i64, _int, _int, _vp]),
     "b200_gated_part_norm": (_int, [_vp, _i64, _vp, _vp, _i64, _vp, _i64, _i64, _i64, _f32, _int, _vp]),
 }
 

@@ -366,6 +366,468 @@ int launch_scan(ScanArgs<T>& a, int64_t n_seq, int64_t q_max, cudaStream_t st) {
   return launch_scan_n<T, MODE, 32, 16>(a, n_seq, q_max, st);
 }
 
+
+// ------------------------------------------------------------------------------------------------------------
+// Portions in bf16 on the tensor cores (mma.sync m16n8k16, fp32 accumulation): 16 tokens of a sequence at a time.
+// S^T [V x N] stays in fp32 accumulators over the whole portion, a warp holding 16 MT value rows: the accumulator
+// layout of S^T is the operand layout of S in  o_i = q_i . S,  so the state never passes through memory between tiles.
+// fp32 factors enter a product as two bf16 terms (hi + lo, 16 mantissa bits); inputs that are bf16 already enter as
+// they are.
+//   ssd    : with c_i = sum_{t <= i} log a_t inside the tile,  o_i = exp(c_i) (C_i . S) + sum_{j <= i} (C_i . B_j)
+//            exp(c_i - c_j) d_j x_j ;  S <- exp(c_last) S + sum_j exp(c_last - c_j) d_j B_j x_j^T    (exponents <= 0)
+//   forget : everything relative to the middle of the tile, per key channel: with r_t the product of the gates between
+//            token t and the middle, q and k become q / r, k r before it and q r, k / r after it; S is decayed to the
+//            middle, o = q . S + (masked q k^T) v, S <- S + k v^T, and S is decayed to the end.  Where a product of a
+//            half tile falls below kMinSpan the tile is cut to 4 tokens, and to one (which needs no division) if need be.
+// ------------------------------------------------------------------------------------------------------------
+constexpr int kTile = 16;
+constexpr float kMinSpan = 1e-16f;
+
+__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void split_bf16(float x, float y, uint32_t& hi, uint32_t& lo) {
+  hi = Num<__nv_bfloat16>::pack(x, y);
+  const float2 h = Num<__nv_bfloat16>::unpack(hi);
+  lo = Num<__nv_bfloat16>::pack(x - h.x, y - h.y);
+}
+
+// Shared-memory rows of a tile (bf16, 8 elements of padding per row).  forget: q hi, q lo, k hi, k lo; ssd: C, B, k hi,
+// k lo (k: B with its decay to the tile's end).
+template <int KN>
+struct TileRows {
+  static constexpr int NS = 16 * KN + 8;
+  static constexpr int kRows = 4 * kTile * NS;            // the four key-channel arrays
+};
+
+// One token of two neighbouring key channels of a forget tile: gates a, written shares k and silu(q) from the raw pairs.
+__device__ __forceinline__ void forget_token(uint32_t qraw, uint32_t fraw, float2 bias, float2 low, float2& q, float2& a,
+                                             float2& k) {
+  const float2 qv = Num<__nv_bfloat16>::unpack(qraw), fv = Num<__nv_bfloat16>::unpack(fraw);
+  auto gate = [](float z, float l, float& ga, float& gk) {
+    const float e = __expf(-fabsf(z));
+    const float big = __fdividef(1.0f, 1.0f + e), small = e * big;
+    ga = l + (1.0f - l) * (z >= 0.0f ? big : small);
+    gk = (1.0f - l) * (z >= 0.0f ? small : big);
+  };
+  gate(fv.x + bias.x, low.x, a.x, k.x);
+  gate(fv.y + bias.y, low.y, a.y, k.y);
+  q = make_float2(__fdividef(qv.x, 1.0f + __expf(-qv.x)), __fdividef(qv.y, 1.0f + __expf(-qv.y)));
+}
+
+// Channels c, c + 1 of one half of a forget tile of L tokens whose middle is after token HA - 1.  BEFORE: tokens
+// HA - 1 .. 0, else tokens HA .. 15 (zeros from L on).  FULL: HA = 8, L = 16, all loads in flight together.  Returns the
+// product of the half's gates.
+template <int KN, bool BEFORE, bool FULL>
+__device__ __forceinline__ float2 stage_forget_half(__nv_bfloat16* rows, const __nv_bfloat16* __restrict__ q,
+                                                    const __nv_bfloat16* __restrict__ f, int64_t ld, int c, bool live,
+                                                    float2 bias, float2 low, int HA_rt, int L_rt) {
+  constexpr int NS = TileRows<KN>::NS;
+  const int HA = FULL ? 8 : HA_rt, L = FULL ? kTile : L_rt;
+  float2 r = make_float2(1.0f, 1.0f);
+  auto put = [&](int t, uint32_t qraw, uint32_t fraw, bool ok) {
+    uint32_t qh = 0u, ql = 0u, kh = 0u, kl = 0u;
+    if (ok) {
+      float2 qs, a, k;
+      forget_token(qraw, fraw, bias, low, qs, a, k);
+      if constexpr (BEFORE) {
+        split_bf16(__fdividef(qs.x, r.x), __fdividef(qs.y, r.y), qh, ql);
+        split_bf16(k.x * r.x, k.y * r.y, kh, kl);
+        r.x *= a.x;
+        r.y *= a.y;
+      } else {
+        r.x *= a.x;
+        r.y *= a.y;
+        split_bf16(qs.x * r.x, qs.y * r.y, qh, ql);
+        split_bf16(__fdividef(k.x, r.x), __fdividef(k.y, r.y), kh, kl);
+      }
+    }
+    __nv_bfloat16* dst = rows + (size_t)t * NS + c;
+    *reinterpret_cast<uint32_t*>(dst) = qh;
+    *reinterpret_cast<uint32_t*>(dst + kTile * NS) = ql;
+    *reinterpret_cast<uint32_t*>(dst + 2 * kTile * NS) = kh;
+    *reinterpret_cast<uint32_t*>(dst + 3 * kTile * NS) = kl;
+  };
+  if constexpr (FULL) {
+    uint32_t qraw[8], fraw[8];
+#pragma unroll
+    for (int s = 0; s < 8; ++s) {
+      const int t = BEFORE ? 7 - s : 8 + s;
+      qraw[s] = live ? *reinterpret_cast<const uint32_t*>(q + (int64_t)t * ld + c) : 0u;
+      fraw[s] = live ? *reinterpret_cast<const uint32_t*>(f + (int64_t)t * ld + c) : 0u;
+    }
+#pragma unroll
+    for (int s = 0; s < 8; ++s) put(BEFORE ? 7 - s : 8 + s, qraw[s], fraw[s], live);
+  } else {
+    const int n = BEFORE ? HA : kTile - HA;
+    for (int s = 0; s < n; ++s) {
+      const int t = BEFORE ? HA - 1 - s : HA + s;
+      const bool ok = live && t < L;
+      put(t, ok ? *reinterpret_cast<const uint32_t*>(q + (int64_t)t * ld + c) : 0u,
+          ok ? *reinterpret_cast<const uint32_t*>(f + (int64_t)t * ld + c) : 0u, ok);
+    }
+  }
+  return r;
+}
+
+template <int MODE, int KN, int MT>
+__global__ void __launch_bounds__(MT == 1 ? 128 : kScanWarps * 32, MT == 1 ? (MODE == MODE_SSD ? 3 : 2) : 1)
+linear_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
+  using bf16 = __nv_bfloat16;
+  constexpr int NP = 16 * KN, NS = TileRows<KN>::NS;
+  extern __shared__ __align__(16) unsigned char smraw[];
+  const int N = a.N, V = a.V, VS = V + 8, OS = V + 4;
+  bf16* rows = reinterpret_cast<bf16*>(smraw);            // [4][16][NS]
+  bf16* v_s = rows + TileRows<KN>::kRows;                 // [16][VS]
+  float* e_s = reinterpret_cast<float*>(v_s + kTile * VS);   // forget: [2][NP] half products; ssd: [16] c_i, [16] d_i
+  float* c_s = e_s + (MODE == MODE_FORGET ? 2 * NP : 2 * kTile);   // forget: [2][NP] bias, lower bound
+  float* o_s = c_s + (MODE == MODE_FORGET ? 2 * NP : 0);           // forget: [16][OS]
+  const int seq = blockIdx.x, h = blockIdx.y;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+  const int t0 = a.q_cu[seq], t1 = a.q_cu[seq + 1];
+  if (t0 >= t1) return;
+  const int gr = lane >> 2, qc = (lane & 3) * 2;
+  const int v0 = warp * 16 * MT;                          // this warp's value rows v0 .. v0 + 16 MT - 1
+  float* Sg = a.state + (((size_t)a.state_slots[seq] * a.H + h) * N) * V;
+  const bool fresh = a.positions[t0] == 0;
+  float S[MT][2 * KN][4];
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < 2 * KN; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = nt * 8 + qc + (e & 1), v = v0 + mt * 16 + gr + (e >> 1) * 8;
+        S[mt][nt][e] = (!fresh && n < N && v < V) ? Sg[(size_t)n * V + v] : 0.0f;
+      }
+  const int g = MODE == MODE_SSD ? h / (a.H / a.G) : h;
+  float neg_a = 0.0f, dbias = 0.0f, skip = 0.0f;
+  if constexpr (MODE == MODE_SSD) {
+    neg_a = -expf(a.a_log[h]);
+    dbias = a.dt_bias[h];
+    skip = a.skip[h];
+  } else {
+    for (int i = threadIdx.x; i < NP; i += blockDim.x) {
+      c_s[i] = i < N ? a.f_bias[h * N + i] : 0.0f;
+      c_s[NP + i] = i < N ? a.f_low[h * N + i] : 1.0f;
+    }
+    __syncthreads();
+  }
+  int L = 0;
+  for (int tc = t0; tc < t1; tc += L) {
+    L = t1 - tc < kTile ? t1 - tc : kTile;
+    // ---- stage the tile
+    const bf16* vg = a.v + (size_t)tc * a.ld + (size_t)h * V;
+    if constexpr (MODE == MODE_FORGET) {
+      const bf16* qg = a.q + (size_t)tc * a.ld + (size_t)h * N;
+      const bf16* fg = a.k + (size_t)tc * a.ld + (size_t)h * N;
+      while (true) {
+        const int HA = (L + 1) / 2;
+        bool bad = false;
+        for (int u = threadIdx.x; u < NP; u += blockDim.x) {
+          const bool before = u < NP / 2;
+          const int c = (before ? u : u - NP / 2) * 2;
+          const bool live = c < N;
+          const float2 bias = *reinterpret_cast<const float2*>(c_s + c), low = *reinterpret_cast<const float2*>(c_s + NP + c);
+          float2 r;
+          if (L == kTile) {
+            r = before ? stage_forget_half<KN, true, true>(rows, qg, fg, a.ld, c, live, bias, low, HA, L)
+                       : stage_forget_half<KN, false, true>(rows, qg, fg, a.ld, c, live, bias, low, HA, L);
+          } else {
+            r = before ? stage_forget_half<KN, true, false>(rows, qg, fg, a.ld, c, live, bias, low, HA, L)
+                       : stage_forget_half<KN, false, false>(rows, qg, fg, a.ld, c, live, bias, low, HA, L);
+          }
+          *reinterpret_cast<float2*>(e_s + (before ? 0 : NP) + c) = r;
+          bad |= live && !(fminf(r.x, r.y) >= kMinSpan);
+        }
+        if (L == 1 || !__syncthreads_or(bad)) break;
+        L = L > 4 ? 4 : 1;
+      }
+    } else {
+      // the tile's decay exponents, by every warp for itself: lane t < 16 holds token t
+      const bool tok_ok = lane < L;
+      float d = 0.0f;
+      if (tok_ok) d = softplus_f(Num<bf16>::to_f(a.dt[(size_t)(tc + lane) * a.ld_dt + h]) + dbias);
+      float c = neg_a * d;
+#pragma unroll
+      for (int s = 1; s < kTile; s <<= 1) {
+        const float up = __shfl_up_sync(0xffffffffu, c, s);
+        if (lane >= s) c += up;
+      }
+      const float c_last = __shfl_sync(0xffffffffu, c, kTile - 1);     // (tokens past L add nothing)
+      if (warp == 0 && lane < kTile) {
+        e_s[lane] = c;
+        e_s[kTile + lane] = d;
+      }
+      const float wgt = d * expf(c_last - c);
+      const bf16* cg = a.q + (size_t)tc * a.ld + (size_t)g * N;
+      const bf16* bg = a.k + (size_t)tc * a.ld + (size_t)g * N;
+#pragma unroll 4
+      for (int t = warp; t < kTile; t += n_warps) {
+        const float wt = __shfl_sync(0xffffffffu, wgt, t);
+        for (int x = lane; x < NP / 4; x += 32) {          // 8 channels of C, or of B
+          const bool is_b = x >= NP / 8;
+          const int ch = (is_b ? x - NP / 8 : x) * 8;
+          uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+          if (t < L && ch < N) raw = *reinterpret_cast<const uint4*>((is_b ? bg : cg) + (size_t)t * a.ld + ch);
+          bf16* dst = rows + (size_t)t * NS + ch;
+          if (!is_b) {
+            *reinterpret_cast<uint4*>(dst) = raw;
+          } else {
+            *reinterpret_cast<uint4*>(dst + kTile * NS) = raw;
+            const uint32_t in[4] = {raw.x, raw.y, raw.z, raw.w};
+            uint32_t hi[4], lo[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const float2 b = Num<bf16>::unpack(in[i]);
+              split_bf16(b.x * wt, b.y * wt, hi[i], lo[i]);
+            }
+            *reinterpret_cast<uint4*>(dst + 2 * kTile * NS) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+            *reinterpret_cast<uint4*>(dst + 3 * kTile * NS) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+          }
+        }
+      }
+    }
+    for (int x = threadIdx.x; x < kTile * (V / 8); x += blockDim.x) {
+      const int t = x / (V / 8), ch = (x - t * (V / 8)) * 8;
+      uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+      if (t < L) raw = *reinterpret_cast<const uint4*>(vg + (size_t)t * a.ld + ch);
+      *reinterpret_cast<uint4*>(v_s + t * VS + ch) = raw;
+    }
+    __syncthreads();
+    // ---- products
+    const bf16* q_hi = rows;
+    const bf16* q_lo = rows + kTile * NS;                  // ssd: B
+    const bf16* k_hi = rows + 2 * kTile * NS;
+    const bf16* k_lo = rows + 3 * kTile * NS;
+    if constexpr (MODE == MODE_FORGET) {                   // to the middle of the tile
+#pragma unroll
+      for (int nt = 0; nt < 2 * KN; ++nt) {
+        const float2 e = *reinterpret_cast<const float2*>(e_s + nt * 8 + qc);
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt) {
+          S[mt][nt][0] *= e.x; S[mt][nt][1] *= e.y; S[mt][nt][2] *= e.x; S[mt][nt][3] *= e.y;
+        }
+      }
+    }
+    float sc[2][4], y[MT * 2][4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.0f;
+#pragma unroll
+    for (int i = 0; i < MT * 2; ++i) y[i][0] = y[i][1] = y[i][2] = y[i][3] = 0.0f;
+    const int a_off = (lane & 15) * NS + (lane >> 4) * 8;
+    const int b_off = ((lane & 7) + (lane >> 4) * 8) * NS + ((lane >> 3) & 1) * 8;
+#pragma unroll
+    for (int ks = 0; ks < KN; ++ks) {
+      uint32_t ah[4], b[4];
+      ldsm_x4(ah, q_hi + a_off + ks * 16);
+      if constexpr (MODE == MODE_FORGET) {
+        uint32_t al[4], bl[4];
+        ldsm_x4(al, q_lo + a_off + ks * 16);
+        ldsm_x4(b, k_hi + b_off + ks * 16);
+        ldsm_x4(bl, k_lo + b_off + ks * 16);
+        mma_bf16(sc[0], ah, b[0], b[1]);  mma_bf16(sc[1], ah, b[2], b[3]);
+        mma_bf16(sc[0], ah, bl[0], bl[1]); mma_bf16(sc[1], ah, bl[2], bl[3]);
+        mma_bf16(sc[0], al, b[0], b[1]);  mma_bf16(sc[1], al, b[2], b[3]);
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+          for (int hf = 0; hf < 2; ++hf) {
+            uint32_t h0, l0, h1, l1;
+            split_bf16(S[mt][2 * ks][2 * hf], S[mt][2 * ks][2 * hf + 1], h0, l0);
+            split_bf16(S[mt][2 * ks + 1][2 * hf], S[mt][2 * ks + 1][2 * hf + 1], h1, l1);
+            mma_bf16(y[mt * 2 + hf], ah, h0, h1);
+            mma_bf16(y[mt * 2 + hf], ah, l0, l1);
+            mma_bf16(y[mt * 2 + hf], al, h0, h1);
+          }
+      } else {
+        ldsm_x4(b, q_lo + b_off + ks * 16);
+        mma_bf16(sc[0], ah, b[0], b[1]);
+        mma_bf16(sc[1], ah, b[2], b[3]);
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+          for (int hf = 0; hf < 2; ++hf) {
+            uint32_t h0, l0, h1, l1;
+            split_bf16(S[mt][2 * ks][2 * hf], S[mt][2 * ks][2 * hf + 1], h0, l0);
+            split_bf16(S[mt][2 * ks + 1][2 * hf], S[mt][2 * ks + 1][2 * hf + 1], h1, l1);
+            mma_bf16(y[mt * 2 + hf], ah, h0, h1);
+            mma_bf16(y[mt * 2 + hf], ah, l0, l1);
+          }
+      }
+    }
+    float c_end = 0.0f;
+    if constexpr (MODE == MODE_SSD) {
+      const float ci[2] = {e_s[gr], e_s[gr + 8]};
+      const float gi[2] = {expf(ci[0]), expf(ci[1])};
+      c_end = expf(e_s[kTile - 1]);
+#pragma unroll
+      for (int i = 0; i < MT * 2; ++i) { y[i][0] *= gi[0]; y[i][1] *= gi[0]; y[i][2] *= gi[1]; y[i][3] *= gi[1]; }
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int i = gr + (e >> 1) * 8, j = n * 8 + qc + (e & 1);
+          sc[n][e] = j <= i ? sc[n][e] * (expf(ci[e >> 1] - e_s[j]) * e_s[kTile + j]) : 0.0f;
+        }
+    } else {
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (n * 8 + qc + (e & 1) > gr + (e >> 1) * 8) sc[n][e] = 0.0f;
+    }
+    uint32_t ph[4], pl[4];
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+      split_bf16(sc[n][0], sc[n][1], ph[n * 2], pl[n * 2]);
+      split_bf16(sc[n][2], sc[n][3], ph[n * 2 + 1], pl[n * 2 + 1]);
+    }
+    const int t_off = ((lane & 7) + ((lane >> 3) & 1) * 8);
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {
+      const int vc = v0 + mt * 16;
+      if (vc < V) {                                        // (the same for the whole warp)
+        uint32_t b[4];
+        ldsm_x4_t(b, v_s + t_off * VS + vc + (lane >> 4) * 8);
+        mma_bf16(y[mt * 2], ph, b[0], b[1]); mma_bf16(y[mt * 2 + 1], ph, b[2], b[3]);
+        mma_bf16(y[mt * 2], pl, b[0], b[1]); mma_bf16(y[mt * 2 + 1], pl, b[2], b[3]);
+      }
+    }
+    // ---- the new state
+    if constexpr (MODE == MODE_SSD) {
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int nt = 0; nt < 2 * KN; ++nt) {
+          S[mt][nt][0] *= c_end; S[mt][nt][1] *= c_end; S[mt][nt][2] *= c_end; S[mt][nt][3] *= c_end;
+        }
+    }
+    uint32_t va[MT][4];
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {
+      const int vc = v0 + mt * 16;
+      va[mt][0] = va[mt][1] = va[mt][2] = va[mt][3] = 0u;
+      if (vc < V) ldsm_x4_t(va[mt], v_s + ((lane & 7) + (lane >> 4) * 8) * VS + vc + ((lane >> 3) & 1) * 8);
+    }
+#pragma unroll
+    for (int ks = 0; ks < KN; ++ks) {
+      uint32_t b[4], bl[4];
+      ldsm_x4_t(b, k_hi + t_off * NS + ks * 16 + (lane >> 4) * 8);
+      ldsm_x4_t(bl, k_lo + t_off * NS + ks * 16 + (lane >> 4) * 8);
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt) {
+        mma_bf16(S[mt][2 * ks], va[mt], b[0], b[1]);
+        mma_bf16(S[mt][2 * ks + 1], va[mt], b[2], b[3]);
+        mma_bf16(S[mt][2 * ks], va[mt], bl[0], bl[1]);
+        mma_bf16(S[mt][2 * ks + 1], va[mt], bl[2], bl[3]);
+      }
+    }
+    if constexpr (MODE == MODE_FORGET) {                   // to the end of the tile
+#pragma unroll
+      for (int nt = 0; nt < 2 * KN; ++nt) {
+        const float2 e = *reinterpret_cast<const float2*>(e_s + NP + nt * 8 + qc);
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt) {
+          S[mt][nt][0] *= e.x; S[mt][nt][1] *= e.y; S[mt][nt][2] *= e.x; S[mt][nt][3] *= e.y;
+        }
+      }
+    }
+    // ---- out
+    if constexpr (MODE == MODE_SSD) {
+#pragma unroll
+      for (int i = 0; i < MT * 2; ++i) {
+        const int v = v0 + i * 8 + qc;
+        if (v < V)
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            const int t = gr + r * 8;
+            if (t < L) {
+              const float2 x = Num<bf16>::unpack(*reinterpret_cast<const uint32_t*>(v_s + t * VS + v));
+              *reinterpret_cast<float2*>(a.raw + (size_t)(tc + t) * a.H * V + (size_t)h * V + v) =
+                  make_float2(y[i][2 * r] + skip * x.x, y[i][2 * r + 1] + skip * x.y);
+            }
+          }
+      }
+      __syncthreads();                                     // the tile's rows are done with
+    } else {
+#pragma unroll
+      for (int i = 0; i < MT * 2; ++i) {
+        const int v = v0 + i * 8 + qc;
+        if (v < V) {
+          *reinterpret_cast<float2*>(o_s + gr * OS + v) = make_float2(y[i][0], y[i][1]);
+          *reinterpret_cast<float2*>(o_s + (gr + 8) * OS + v) = make_float2(y[i][2], y[i][3]);
+        }
+      }
+      __syncthreads();                                     // the read-outs stand; the tile's rows are done with
+      for (int t = warp; t < L; t += n_warps) {
+        const float* ot = o_s + t * OS;
+        float ss = 0.0f;
+        for (int c = lane * 2; c < V; c += 64) {
+          const float2 o = *reinterpret_cast<const float2*>(ot + c);
+          ss += o.x * o.x + o.y * o.y;
+        }
+        ss = warp_sum(ss);
+        const float inv = a.mul / sqrtf(ss / (float)V + a.eps);
+        bf16* dst = a.out + (size_t)(tc + t) * a.ldo + (size_t)h * V;
+        for (int c = lane * 2; c < V; c += 64) {
+          const float2 o = *reinterpret_cast<const float2*>(ot + c);
+          *reinterpret_cast<uint32_t*>(dst + c) = Num<bf16>::pack(o.x * inv * a.norm_w[c], o.y * inv * a.norm_w[c + 1]);
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < 2 * KN; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = nt * 8 + qc + (e & 1), v = v0 + mt * 16 + gr + (e >> 1) * 8;
+        if (n < N && v < V) Sg[(size_t)n * V + v] = S[mt][nt][e];
+      }
+}
+
+template <int MODE, int KN, int MT>
+int launch_scan_tc_n(const ScanArgs<__nv_bfloat16>& a, int64_t n_seq, cudaStream_t st) {
+  const int warps = (a.V + 16 * MT - 1) / (16 * MT);
+  size_t smem = ((size_t)TileRows<KN>::kRows + (size_t)kTile * (a.V + 8)) * sizeof(__nv_bfloat16);
+  smem += (MODE == MODE_FORGET ? (size_t)4 * 16 * KN + (size_t)kTile * (a.V + 4) : (size_t)2 * kTile) * sizeof(float);
+  auto kern = linear_scan_tc_kernel<MODE, KN, MT>;
+  if (smem > 48 * 1024)
+    B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  kern<<<dim3((unsigned)n_seq, (unsigned)a.H), warps * 32, smem, st>>>(a);
+  B200_LAUNCH_OK("linear_scan_tc_kernel");
+  return B200_OK;
+}
+
+template <int MODE>
+int launch_scan_tc(const ScanArgs<__nv_bfloat16>& a, int64_t n_seq, cudaStream_t st) {
+  const bool two = a.V > 64;                              // 16 value rows a warp, or 32
+  if (a.N <= 32) return two ? launch_scan_tc_n<MODE, 2, 2>(a, n_seq, st) : launch_scan_tc_n<MODE, 2, 1>(a, n_seq, st);
+  if (a.N <= 64) return two ? launch_scan_tc_n<MODE, 4, 2>(a, n_seq, st) : launch_scan_tc_n<MODE, 4, 1>(a, n_seq, st);
+  return two ? launch_scan_tc_n<MODE, 8, 2>(a, n_seq, st) : launch_scan_tc_n<MODE, 8, 1>(a, n_seq, st);
+}
+
+template <int MODE>
+int launch_scan_tc(const ScanArgs<float>&, int64_t, cudaStream_t) {
+  return set_error(B200_ERR_UNSUPPORTED, "linear_scan: the tensor-core form takes bf16");
+}
+
+bool scan_tc_fits(int64_t N, int64_t V, int dtype) {
+  return dtype == B200_BF16 && N > 0 && N % 8 == 0 && N <= 128 && V > 0 && V % 16 == 0 && V <= 32 * kScanWarps;
+}
+
 }  // namespace
 }  // namespace b200
 
@@ -382,18 +844,23 @@ extern "C" {
 
 int b200_linear_scan_parts(int64_t N, int64_t V) { return scan_col_parts((int)N, (int)V); }
 
+int b200_linear_scan_tc_supported(int64_t N, int64_t V, int dtype) { return scan_tc_fits(N, V, dtype); }
+
 int b200_forget_scan(void* out, int64_t ldo, const void* q, const void* f, const void* v, int64_t ld,
                      const float* f_bias, const float* f_low, const float* norm_weight, float* state,
                      const int32_t* q_cu_lens, const int32_t* positions, const int32_t* state_slots, int64_t n_seq,
                      int64_t q_max, int64_t rows, int64_t H, int64_t N, int64_t V, float eps, float mul, float* raw,
-                     int dtype, b200_stream_t stream) {
+                     int tensor_cores, int dtype, b200_stream_t stream) {
   if (rows == 0 || n_seq == 0) return B200_OK;
   B200_CHECK_ARG(out && q && f && v && f_bias && f_low && norm_weight && state && q_cu_lens && positions && state_slots,
                  "forget_scan: null pointer");
   B200_CHECK_ARG(rows > 0 && n_seq > 0 && q_max > 0 && H > 0 && H <= 65535 && N > 0 && N <= 512 && V > 0 && V <= 4096 &&
                      ldo >= H * V && ld >= H * (N > V ? N : V),
                  "forget_scan: bad shape (key size <= 512)");
-  B200_CHECK_ARG(raw || scan_col_parts((int)N, (int)V) == 1, "forget_scan: heads in several column parts need a workspace");
+  B200_CHECK_ARG(!tensor_cores || (scan_tc_fits(N, V, dtype) && ld % 8 == 0 && ldo % 2 == 0 && is_aligned(q, 4) &&
+                                   is_aligned(f, 4) && is_aligned(v, 16) && is_aligned(out, 4)),
+                 "forget_scan: sizes or alignment do not fit the tensor-core tiles");
+  B200_CHECK_ARG(tensor_cores || raw || scan_col_parts((int)N, (int)V) == 1, "forget_scan: heads in several column parts need a workspace");
   auto st = static_cast<cudaStream_t>(stream);
   SCAN_DISPATCH(dtype, {
     ScanArgs<T> a{};
@@ -405,6 +872,7 @@ int b200_forget_scan(void* out, int64_t ldo, const void* q, const void* f, const
     a.vec_in = N % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && is_aligned(q, 4 * sizeof(T)) && is_aligned(f, 4 * sizeof(T)) &&
                is_aligned(v, 4 * sizeof(T));
     a.vec_state = V % 4 == 0 && is_aligned(state, 16);
+    if (tensor_cores) return launch_scan_tc<MODE_FORGET>(a, n_seq, st);
     const int rc = launch_scan<T, MODE_FORGET>(a, n_seq, q_max, st);
     if (rc != B200_OK) return rc;
     if (raw) {
@@ -420,13 +888,16 @@ int b200_forget_scan(void* out, int64_t ldo, const void* q, const void* f, const
 int b200_ssd_scan(float* y, const void* x, const void* B, const void* Cm, int64_t ld, const void* dt, int64_t ld_dt,
                   const float* dt_bias, const float* a_log, const float* skip, float* state, const int32_t* q_cu_lens,
                   const int32_t* positions, const int32_t* state_slots, int64_t n_seq, int64_t q_max, int64_t rows,
-                  int64_t H, int64_t G, int64_t N, int64_t V, int dtype, b200_stream_t stream) {
+                  int64_t H, int64_t G, int64_t N, int64_t V, int tensor_cores, int dtype, b200_stream_t stream) {
   if (rows == 0 || n_seq == 0) return B200_OK;
   B200_CHECK_ARG(y && x && B && Cm && dt && dt_bias && a_log && skip && state && q_cu_lens && positions && state_slots,
                  "ssd_scan: null pointer");
   B200_CHECK_ARG(rows > 0 && n_seq > 0 && q_max > 0 && H > 0 && H <= 65535 && G > 0 && H % G == 0 && N > 0 && N <= 512 &&
                      V > 0 && V <= 4096 && ld >= H * V && ld >= G * N && ld_dt >= H,
                  "ssd_scan: bad shape (state size <= 512, heads a multiple of groups)");
+  B200_CHECK_ARG(!tensor_cores || (scan_tc_fits(N, V, dtype) && ld % 8 == 0 && is_aligned(x, 16) && is_aligned(B, 16) &&
+                                   is_aligned(Cm, 16) && is_aligned(y, 8)),
+                 "ssd_scan: sizes or alignment do not fit the tensor-core tiles");
   auto st = static_cast<cudaStream_t>(stream);
   SCAN_DISPATCH(dtype, {
     ScanArgs<T> a{};
@@ -438,6 +909,7 @@ int b200_ssd_scan(float* y, const void* x, const void* B, const void* Cm, int64_
     a.vec_in = N % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && is_aligned(x, 4 * sizeof(T)) && is_aligned(B, 4 * sizeof(T)) &&
                is_aligned(Cm, 4 * sizeof(T));
     a.vec_state = V % 4 == 0 && is_aligned(state, 16);
+    if (tensor_cores) return launch_scan_tc<MODE_SSD>(a, n_seq, st);
     return (launch_scan<T, MODE_SSD>(a, n_seq, q_max, st));
   });
   return B200_OK;

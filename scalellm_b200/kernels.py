@@ -1607,6 +1607,17 @@ def causal_filter(x: torch.Tensor, filter: torch.Tensor, bias: Optional[torch.Te
     return out
 
 
+# a step whose longest portion has at least this many tokens walks the recurrences 16 tokens at a time on the tensor
+# cores (bf16, fitting sizes; B200_SCAN_IMPL=simt: never)
+SCAN_TC_MIN_ROWS = 8
+
+
+def _scan_tc(q_max: int, N: int, V: int, ld: int, *blocks: torch.Tensor) -> bool:
+    return (q_max >= SCAN_TC_MIN_ROWS and os.environ.get("B200_SCAN_IMPL") != "simt" and ld % 8 == 0
+            and all(t.data_ptr() % 16 == 0 for t in blocks)
+            and bool(_lib.load().b200_linear_scan_tc_supported(N, V, _dt(blocks[0]))))
+
+
 def forget_scan(q: torch.Tensor, f: torch.Tensor, v: torch.Tensor, f_bias: torch.Tensor, f_low: torch.Tensor,
                 norm_weight: torch.Tensor, state: torch.Tensor, q_cu: torch.Tensor, positions: torch.Tensor,
                 state_slots: torch.Tensor, n_seq: int, q_max: int, eps: float, out_mul: float = 1.0,
@@ -1625,10 +1636,12 @@ def forget_scan(q: torch.Tensor, f: torch.Tensor, v: torch.Tensor, f_bias: torch
         out = torch.empty((rows, H * V), dtype=q.dtype, device=q.device)
     assert out.shape == (rows, H * V) and out.stride(1) == 1 and out.dtype == q.dtype
     lib = _lib.load()
-    raw = torch.empty((rows, H * V), dtype=torch.float32, device=q.device) if lib.b200_linear_scan_parts(N, V) > 1 else None
+    tc = _scan_tc(q_max, N, V, ld, q, f, v) and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0
+    raw = (torch.empty((rows, H * V), dtype=torch.float32, device=q.device)
+           if not tc and lib.b200_linear_scan_parts(N, V) > 1 else None)
     check(lib.b200_forget_scan(_p(out), out.stride(0), _p(q), _p(f), _p(v), ld, _p(f_bias), _p(f_low), _p(norm_weight),
                                _p(state), _p(q_cu), _p(positions), _p(state_slots), n_seq, q_max, rows, H, N, V, eps,
-                               out_mul, _p(raw), _dt(q), _stream()))
+                               out_mul, _p(raw), 1 if tc else 0, _dt(q), _stream()))
     return out
 
 
@@ -1648,7 +1661,7 @@ def ssd_scan(x: torch.Tensor, B: torch.Tensor, C_: torch.Tensor, dt: torch.Tenso
     y = torch.empty((rows, H * V), dtype=torch.float32, device=x.device)
     check(_lib.load().b200_ssd_scan(_p(y), _p(x), _p(B), _p(C_), ld, _p(dt), dt.stride(0), _p(dt_bias), _p(a_log),
                                     _p(skip), _p(state), _p(q_cu), _p(positions), _p(state_slots), n_seq, q_max, rows,
-                                    H, groups, N, V, _dt(x), _stream()))
+                                    H, groups, N, V, 1 if _scan_tc(q_max, N, V, ld, x, B, C_) else 0, _dt(x), _stream()))
     return y
 
 

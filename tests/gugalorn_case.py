@@ -116,8 +116,8 @@ CONFIGS = {
     "odd": config([
         (mamba(5, 6, 7, 5, 3, conv=1), 30),
         (pair(left(3, 3, 10, 7, 2), right(1, 9, 15), 1.3, 0.5), 22),
-        (mamba(1, 13, 18, 1, 13, conv=5), None),
-        (pair(left(5, 1, 6, 5, 6), right(5, 6, 3), 0.7, 0.7), None),
+        (mamba(1, 13, 18, 1, 1, conv=5), None),
+        (pair(left(5, 1, 6, 5, 6), right(5, 6, 11), 0.7, 0.7), None),
     ], width=42, vocab=61, taps=1, embed_scale=1.0),
     # more taps than most portions have tokens, key and value sizes of several column and row parts
     "wide": config([

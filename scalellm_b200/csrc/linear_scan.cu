@@ -402,8 +402,7 @@ __device__ __forceinline__ void split_bf16(float x, float y, uint32_t& hi, uint3
   lo = Num<__nv_bfloat16>::pack(x - h.x, y - h.y);
 }
 
-// Shared-memory rows of a tile (bf16, 8 elements of padding per row).  forget: q hi, q lo, k hi, k lo; ssd: C, B, k hi,
-// k lo (k: B with its decay to the tile's end).
+// Shared-memory rows of a forget tile (bf16, 8 elements of padding per row): q hi, q lo, k hi, k lo.
 template <int KN>
 struct TileRows {
   static constexpr int NS = 16 * KN + 8;
@@ -480,18 +479,18 @@ __device__ __forceinline__ float2 stage_forget_half(__nv_bfloat16* rows, const _
   return r;
 }
 
-template <int MODE, int KN, int MT>
-__global__ void __launch_bounds__(MT == 1 ? 128 : kScanWarps * 32, MT == 1 ? (MODE == MODE_SSD ? 3 : 2) : 1)
-linear_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
+template <int KN, int MT>
+__global__ void __launch_bounds__(MT == 1 ? 128 : kScanWarps * 32, MT == 1 ? 2 : 1)
+forget_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
   using bf16 = __nv_bfloat16;
   constexpr int NP = 16 * KN, NS = TileRows<KN>::NS;
   extern __shared__ __align__(16) unsigned char smraw[];
   const int N = a.N, V = a.V, VS = V + 8, OS = V + 4;
   bf16* rows = reinterpret_cast<bf16*>(smraw);            // [4][16][NS]
   bf16* v_s = rows + TileRows<KN>::kRows;                 // [16][VS]
-  float* e_s = reinterpret_cast<float*>(v_s + kTile * VS);   // forget: [2][NP] half products; ssd: [16] c_i, [16] d_i
-  float* c_s = e_s + (MODE == MODE_FORGET ? 2 * NP : 2 * kTile);   // forget: [2][NP] bias, lower bound
-  float* o_s = c_s + (MODE == MODE_FORGET ? 2 * NP : 0);           // forget: [16][OS]
+  float* e_s = reinterpret_cast<float*>(v_s + kTile * VS);   // [2][NP] products of the two halves
+  float* c_s = e_s + 2 * NP;                              // [2][NP] bias, lower bound
+  float* o_s = c_s + 2 * NP;                              // [16][OS]
   const int seq = blockIdx.x, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
   const int t0 = a.q_cu[seq], t1 = a.q_cu[seq + 1];
@@ -510,93 +509,39 @@ linear_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
         const int n = nt * 8 + qc + (e & 1), v = v0 + mt * 16 + gr + (e >> 1) * 8;
         S[mt][nt][e] = (!fresh && n < N && v < V) ? Sg[(size_t)n * V + v] : 0.0f;
       }
-  const int g = MODE == MODE_SSD ? h / (a.H / a.G) : h;
-  float neg_a = 0.0f, dbias = 0.0f, skip = 0.0f;
-  if constexpr (MODE == MODE_SSD) {
-    neg_a = -expf(a.a_log[h]);
-    dbias = a.dt_bias[h];
-    skip = a.skip[h];
-  } else {
-    for (int i = threadIdx.x; i < NP; i += blockDim.x) {
-      c_s[i] = i < N ? a.f_bias[h * N + i] : 0.0f;
-      c_s[NP + i] = i < N ? a.f_low[h * N + i] : 1.0f;
-    }
-    __syncthreads();
+  for (int i = threadIdx.x; i < NP; i += blockDim.x) {
+    c_s[i] = i < N ? a.f_bias[h * N + i] : 0.0f;
+    c_s[NP + i] = i < N ? a.f_low[h * N + i] : 1.0f;
   }
+  __syncthreads();
   int L = 0;
   for (int tc = t0; tc < t1; tc += L) {
     L = t1 - tc < kTile ? t1 - tc : kTile;
     // ---- stage the tile
     const bf16* vg = a.v + (size_t)tc * a.ld + (size_t)h * V;
-    if constexpr (MODE == MODE_FORGET) {
-      const bf16* qg = a.q + (size_t)tc * a.ld + (size_t)h * N;
-      const bf16* fg = a.k + (size_t)tc * a.ld + (size_t)h * N;
-      while (true) {
-        const int HA = (L + 1) / 2;
-        bool bad = false;
-        for (int u = threadIdx.x; u < NP; u += blockDim.x) {
-          const bool before = u < NP / 2;
-          const int c = (before ? u : u - NP / 2) * 2;
-          const bool live = c < N;
-          const float2 bias = *reinterpret_cast<const float2*>(c_s + c), low = *reinterpret_cast<const float2*>(c_s + NP + c);
-          float2 r;
-          if (L == kTile) {
-            r = before ? stage_forget_half<KN, true, true>(rows, qg, fg, a.ld, c, live, bias, low, HA, L)
-                       : stage_forget_half<KN, false, true>(rows, qg, fg, a.ld, c, live, bias, low, HA, L);
-          } else {
-            r = before ? stage_forget_half<KN, true, false>(rows, qg, fg, a.ld, c, live, bias, low, HA, L)
-                       : stage_forget_half<KN, false, false>(rows, qg, fg, a.ld, c, live, bias, low, HA, L);
-          }
-          *reinterpret_cast<float2*>(e_s + (before ? 0 : NP) + c) = r;
-          bad |= live && !(fminf(r.x, r.y) >= kMinSpan);
+    const bf16* qg = a.q + (size_t)tc * a.ld + (size_t)h * N;
+    const bf16* fg = a.k + (size_t)tc * a.ld + (size_t)h * N;
+    while (true) {
+      const int HA = (L + 1) / 2;
+      bool bad = false;
+      for (int u = threadIdx.x; u < NP; u += blockDim.x) {
+        const bool before = u < NP / 2;
+        const int c = (before ? u : u - NP / 2) * 2;
+        const bool live = c < N;
+        const float2 bias = *reinterpret_cast<const float2*>(c_s + c), low = *reinterpret_cast<const float2*>(c_s + NP + c);
+        float2 r;
+        if (L == kTile) {
+          r = before ? stage_forget_half<KN, true, true>(rows, qg, fg, a.ld, c, live, bias, low, HA, L)
+                     : stage_forget_half<KN, false, true>(rows, qg, fg, a.ld, c, live, bias, low, HA, L);
+        } else {
+          r = before ? stage_forget_half<KN, true, false>(rows, qg, fg, a.ld, c, live, bias, low, HA, L)
+                     : stage_forget_half<KN, false, false>(rows, qg, fg, a.ld, c, live, bias, low, HA, L);
         }
-        if (L == 1 || !__syncthreads_or(bad)) break;
-        L = L > 4 ? 4 : 1;
+        *reinterpret_cast<float2*>(e_s + (before ? 0 : NP) + c) = r;
+        bad |= live && !(fminf(r.x, r.y) >= kMinSpan);
       }
-    } else {
-      // the tile's decay exponents, by every warp for itself: lane t < 16 holds token t
-      const bool tok_ok = lane < L;
-      float d = 0.0f;
-      if (tok_ok) d = softplus_f(Num<bf16>::to_f(a.dt[(size_t)(tc + lane) * a.ld_dt + h]) + dbias);
-      float c = neg_a * d;
-#pragma unroll
-      for (int s = 1; s < kTile; s <<= 1) {
-        const float up = __shfl_up_sync(0xffffffffu, c, s);
-        if (lane >= s) c += up;
-      }
-      const float c_last = __shfl_sync(0xffffffffu, c, kTile - 1);     // (tokens past L add nothing)
-      if (warp == 0 && lane < kTile) {
-        e_s[lane] = c;
-        e_s[kTile + lane] = d;
-      }
-      const float wgt = d * expf(c_last - c);
-      const bf16* cg = a.q + (size_t)tc * a.ld + (size_t)g * N;
-      const bf16* bg = a.k + (size_t)tc * a.ld + (size_t)g * N;
-#pragma unroll 4
-      for (int t = warp; t < kTile; t += n_warps) {
-        const float wt = __shfl_sync(0xffffffffu, wgt, t);
-        for (int x = lane; x < NP / 4; x += 32) {          // 8 channels of C, or of B
-          const bool is_b = x >= NP / 8;
-          const int ch = (is_b ? x - NP / 8 : x) * 8;
-          uint4 raw = make_uint4(0u, 0u, 0u, 0u);
-          if (t < L && ch < N) raw = *reinterpret_cast<const uint4*>((is_b ? bg : cg) + (size_t)t * a.ld + ch);
-          bf16* dst = rows + (size_t)t * NS + ch;
-          if (!is_b) {
-            *reinterpret_cast<uint4*>(dst) = raw;
-          } else {
-            *reinterpret_cast<uint4*>(dst + kTile * NS) = raw;
-            const uint32_t in[4] = {raw.x, raw.y, raw.z, raw.w};
-            uint32_t hi[4], lo[4];
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-              const float2 b = Num<bf16>::unpack(in[i]);
-              split_bf16(b.x * wt, b.y * wt, hi[i], lo[i]);
-            }
-            *reinterpret_cast<uint4*>(dst + 2 * kTile * NS) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-            *reinterpret_cast<uint4*>(dst + 3 * kTile * NS) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-          }
-        }
-      }
+      if (L == 1 || !__syncthreads_or(bad)) break;
+      L = L > 4 ? 4 : 1;
     }
     for (int x = threadIdx.x; x < kTile * (V / 8); x += blockDim.x) {
       const int t = x / (V / 8), ch = (x - t * (V / 8)) * 8;
@@ -607,17 +552,15 @@ linear_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
     __syncthreads();
     // ---- products
     const bf16* q_hi = rows;
-    const bf16* q_lo = rows + kTile * NS;                  // ssd: B
+    const bf16* q_lo = rows + kTile * NS;
     const bf16* k_hi = rows + 2 * kTile * NS;
     const bf16* k_lo = rows + 3 * kTile * NS;
-    if constexpr (MODE == MODE_FORGET) {                   // to the middle of the tile
 #pragma unroll
-      for (int nt = 0; nt < 2 * KN; ++nt) {
-        const float2 e = *reinterpret_cast<const float2*>(e_s + nt * 8 + qc);
+    for (int nt = 0; nt < 2 * KN; ++nt) {                  // to the middle of the tile
+      const float2 e = *reinterpret_cast<const float2*>(e_s + nt * 8 + qc);
 #pragma unroll
-        for (int mt = 0; mt < MT; ++mt) {
-          S[mt][nt][0] *= e.x; S[mt][nt][1] *= e.y; S[mt][nt][2] *= e.x; S[mt][nt][3] *= e.y;
-        }
+      for (int mt = 0; mt < MT; ++mt) {
+        S[mt][nt][0] *= e.x; S[mt][nt][1] *= e.y; S[mt][nt][2] *= e.x; S[mt][nt][3] *= e.y;
       }
     }
     float sc[2][4], y[MT * 2][4];
@@ -631,62 +574,30 @@ linear_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
     for (int ks = 0; ks < KN; ++ks) {
       uint32_t ah[4], b[4];
       ldsm_x4(ah, q_hi + a_off + ks * 16);
-      if constexpr (MODE == MODE_FORGET) {
-        uint32_t al[4], bl[4];
-        ldsm_x4(al, q_lo + a_off + ks * 16);
-        ldsm_x4(b, k_hi + b_off + ks * 16);
-        ldsm_x4(bl, k_lo + b_off + ks * 16);
-        mma_bf16(sc[0], ah, b[0], b[1]);  mma_bf16(sc[1], ah, b[2], b[3]);
-        mma_bf16(sc[0], ah, bl[0], bl[1]); mma_bf16(sc[1], ah, bl[2], bl[3]);
-        mma_bf16(sc[0], al, b[0], b[1]);  mma_bf16(sc[1], al, b[2], b[3]);
+      uint32_t al[4], bl[4];
+      ldsm_x4(al, q_lo + a_off + ks * 16);
+      ldsm_x4(b, k_hi + b_off + ks * 16);
+      ldsm_x4(bl, k_lo + b_off + ks * 16);
+      mma_bf16(sc[0], ah, b[0], b[1]);  mma_bf16(sc[1], ah, b[2], b[3]);
+      mma_bf16(sc[0], ah, bl[0], bl[1]); mma_bf16(sc[1], ah, bl[2], bl[3]);
+      mma_bf16(sc[0], al, b[0], b[1]);  mma_bf16(sc[1], al, b[2], b[3]);
 #pragma unroll
-        for (int mt = 0; mt < MT; ++mt)
+      for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-          for (int hf = 0; hf < 2; ++hf) {
-            uint32_t h0, l0, h1, l1;
-            split_bf16(S[mt][2 * ks][2 * hf], S[mt][2 * ks][2 * hf + 1], h0, l0);
-            split_bf16(S[mt][2 * ks + 1][2 * hf], S[mt][2 * ks + 1][2 * hf + 1], h1, l1);
-            mma_bf16(y[mt * 2 + hf], ah, h0, h1);
-            mma_bf16(y[mt * 2 + hf], ah, l0, l1);
-            mma_bf16(y[mt * 2 + hf], al, h0, h1);
-          }
-      } else {
-        ldsm_x4(b, q_lo + b_off + ks * 16);
-        mma_bf16(sc[0], ah, b[0], b[1]);
-        mma_bf16(sc[1], ah, b[2], b[3]);
-#pragma unroll
-        for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-          for (int hf = 0; hf < 2; ++hf) {
-            uint32_t h0, l0, h1, l1;
-            split_bf16(S[mt][2 * ks][2 * hf], S[mt][2 * ks][2 * hf + 1], h0, l0);
-            split_bf16(S[mt][2 * ks + 1][2 * hf], S[mt][2 * ks + 1][2 * hf + 1], h1, l1);
-            mma_bf16(y[mt * 2 + hf], ah, h0, h1);
-            mma_bf16(y[mt * 2 + hf], ah, l0, l1);
-          }
-      }
-    }
-    float c_end = 0.0f;
-    if constexpr (MODE == MODE_SSD) {
-      const float ci[2] = {e_s[gr], e_s[gr + 8]};
-      const float gi[2] = {expf(ci[0]), expf(ci[1])};
-      c_end = expf(e_s[kTile - 1]);
-#pragma unroll
-      for (int i = 0; i < MT * 2; ++i) { y[i][0] *= gi[0]; y[i][1] *= gi[0]; y[i][2] *= gi[1]; y[i][3] *= gi[1]; }
-#pragma unroll
-      for (int n = 0; n < 2; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int i = gr + (e >> 1) * 8, j = n * 8 + qc + (e & 1);
-          sc[n][e] = j <= i ? sc[n][e] * (expf(ci[e >> 1] - e_s[j]) * e_s[kTile + j]) : 0.0f;
+        for (int hf = 0; hf < 2; ++hf) {
+          uint32_t h0, l0, h1, l1;
+          split_bf16(S[mt][2 * ks][2 * hf], S[mt][2 * ks][2 * hf + 1], h0, l0);
+          split_bf16(S[mt][2 * ks + 1][2 * hf], S[mt][2 * ks + 1][2 * hf + 1], h1, l1);
+          mma_bf16(y[mt * 2 + hf], ah, h0, h1);
+          mma_bf16(y[mt * 2 + hf], ah, l0, l1);
+          mma_bf16(y[mt * 2 + hf], al, h0, h1);
         }
-    } else {
-#pragma unroll
-      for (int n = 0; n < 2; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e)
-          if (n * 8 + qc + (e & 1) > gr + (e >> 1) * 8) sc[n][e] = 0.0f;
     }
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (n * 8 + qc + (e & 1) > gr + (e >> 1) * 8) sc[n][e] = 0.0f;
     uint32_t ph[4], pl[4];
 #pragma unroll
     for (int n = 0; n < 2; ++n) {
@@ -705,14 +616,6 @@ linear_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
       }
     }
     // ---- the new state
-    if constexpr (MODE == MODE_SSD) {
-#pragma unroll
-      for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-        for (int nt = 0; nt < 2 * KN; ++nt) {
-          S[mt][nt][0] *= c_end; S[mt][nt][1] *= c_end; S[mt][nt][2] *= c_end; S[mt][nt][3] *= c_end;
-        }
-    }
     uint32_t va[MT][4];
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
@@ -733,57 +636,37 @@ linear_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
         mma_bf16(S[mt][2 * ks + 1], va[mt], bl[2], bl[3]);
       }
     }
-    if constexpr (MODE == MODE_FORGET) {                   // to the end of the tile
 #pragma unroll
-      for (int nt = 0; nt < 2 * KN; ++nt) {
-        const float2 e = *reinterpret_cast<const float2*>(e_s + NP + nt * 8 + qc);
+    for (int nt = 0; nt < 2 * KN; ++nt) {                  // to the end of the tile
+      const float2 e = *reinterpret_cast<const float2*>(e_s + NP + nt * 8 + qc);
 #pragma unroll
-        for (int mt = 0; mt < MT; ++mt) {
-          S[mt][nt][0] *= e.x; S[mt][nt][1] *= e.y; S[mt][nt][2] *= e.x; S[mt][nt][3] *= e.y;
-        }
+      for (int mt = 0; mt < MT; ++mt) {
+        S[mt][nt][0] *= e.x; S[mt][nt][1] *= e.y; S[mt][nt][2] *= e.x; S[mt][nt][3] *= e.y;
       }
     }
     // ---- out
-    if constexpr (MODE == MODE_SSD) {
 #pragma unroll
-      for (int i = 0; i < MT * 2; ++i) {
-        const int v = v0 + i * 8 + qc;
-        if (v < V)
-#pragma unroll
-          for (int r = 0; r < 2; ++r) {
-            const int t = gr + r * 8;
-            if (t < L) {
-              const float2 x = Num<bf16>::unpack(*reinterpret_cast<const uint32_t*>(v_s + t * VS + v));
-              *reinterpret_cast<float2*>(a.raw + (size_t)(tc + t) * a.H * V + (size_t)h * V + v) =
-                  make_float2(y[i][2 * r] + skip * x.x, y[i][2 * r + 1] + skip * x.y);
-            }
-          }
+    for (int i = 0; i < MT * 2; ++i) {
+      const int v = v0 + i * 8 + qc;
+      if (v < V) {
+        *reinterpret_cast<float2*>(o_s + gr * OS + v) = make_float2(y[i][0], y[i][1]);
+        *reinterpret_cast<float2*>(o_s + (gr + 8) * OS + v) = make_float2(y[i][2], y[i][3]);
       }
-      __syncthreads();                                     // the tile's rows are done with
-    } else {
-#pragma unroll
-      for (int i = 0; i < MT * 2; ++i) {
-        const int v = v0 + i * 8 + qc;
-        if (v < V) {
-          *reinterpret_cast<float2*>(o_s + gr * OS + v) = make_float2(y[i][0], y[i][1]);
-          *reinterpret_cast<float2*>(o_s + (gr + 8) * OS + v) = make_float2(y[i][2], y[i][3]);
-        }
+    }
+    __syncthreads();                                     // the read-outs stand; the tile's rows are done with
+    for (int t = warp; t < L; t += n_warps) {
+      const float* ot = o_s + t * OS;
+      float ss = 0.0f;
+      for (int c = lane * 2; c < V; c += 64) {
+        const float2 o = *reinterpret_cast<const float2*>(ot + c);
+        ss += o.x * o.x + o.y * o.y;
       }
-      __syncthreads();                                     // the read-outs stand; the tile's rows are done with
-      for (int t = warp; t < L; t += n_warps) {
-        const float* ot = o_s + t * OS;
-        float ss = 0.0f;
-        for (int c = lane * 2; c < V; c += 64) {
-          const float2 o = *reinterpret_cast<const float2*>(ot + c);
-          ss += o.x * o.x + o.y * o.y;
-        }
-        ss = warp_sum(ss);
-        const float inv = a.mul / sqrtf(ss / (float)V + a.eps);
-        bf16* dst = a.out + (size_t)(tc + t) * a.ldo + (size_t)h * V;
-        for (int c = lane * 2; c < V; c += 64) {
-          const float2 o = *reinterpret_cast<const float2*>(ot + c);
-          *reinterpret_cast<uint32_t*>(dst + c) = Num<bf16>::pack(o.x * inv * a.norm_w[c], o.y * inv * a.norm_w[c + 1]);
-        }
+      ss = warp_sum(ss);
+      const float inv = a.mul / sqrtf(ss / (float)V + a.eps);
+      bf16* dst = a.out + (size_t)(tc + t) * a.ldo + (size_t)h * V;
+      for (int c = lane * 2; c < V; c += 64) {
+        const float2 o = *reinterpret_cast<const float2*>(ot + c);
+        *reinterpret_cast<uint32_t*>(dst + c) = Num<bf16>::pack(o.x * inv * a.norm_w[c], o.y * inv * a.norm_w[c + 1]);
       }
     }
   }
@@ -798,29 +681,251 @@ linear_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
       }
 }
 
-template <int MODE, int KN, int MT>
-int launch_scan_tc_n(const ScanArgs<__nv_bfloat16>& a, int64_t n_seq, cudaStream_t st) {
+__device__ __forceinline__ void cp_async16(void* smem_dst, const void* gsrc, bool valid) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(smem_dst)), "l"(gsrc), "r"(valid ? 16 : 0)
+               : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+
+// A tile's C, B and x rows are copied one tile ahead (two buffers); its decay exponents are worked out one tile ahead by
+// one warp, which takes turns.
+template <int KN, int MT>
+__global__ void __launch_bounds__(MT == 1 ? 128 : kScanWarps * 32, MT == 1 ? 3 : 1)
+ssd_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
+  using bf16 = __nv_bfloat16;
+  constexpr int NP = 16 * KN, NS = TileRows<KN>::NS, PIECES = NP / 8;
+  extern __shared__ __align__(16) unsigned char smraw[];
+  const int N = a.N, V = a.V, VS = V + 8;
+  bf16* cb_s = reinterpret_cast<bf16*>(smraw);            // [2 buffers][C, B][16][NS]
+  bf16* k_s = cb_s + 4 * kTile * NS;                      // [hi, lo][16][NS]: B with its step size and decay to the end
+  bf16* v_s = k_s + 2 * kTile * NS;                       // [2 buffers][16][VS]
+  float* e_s = reinterpret_cast<float*>(v_s + 2 * kTile * VS);   // [2 buffers][c_i | d_i | d_i exp(c_last - c_i)][16]
+  const int seq = blockIdx.x, h = blockIdx.y, g = h / (a.H / a.G);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+  const int t0 = a.q_cu[seq], t1 = a.q_cu[seq + 1];
+  if (t0 >= t1) return;
+  const int gr = lane >> 2, qc = (lane & 3) * 2;
+  const int v0 = warp * 16 * MT;                          // this warp's value rows v0 .. v0 + 16 MT - 1
+  const float neg_a = -expf(a.a_log[h]), dbias = a.dt_bias[h], skip = a.skip[h];
+  const int n_tiles = (t1 - t0 + kTile - 1) / kTile;
+  const bf16* cg = a.q + (size_t)g * N;
+  const bf16* bg = a.k + (size_t)g * N;
+  const bf16* vg = a.v + (size_t)h * V;
+  const int vp = V / 8;
+  auto copy_tile = [&](int it) {
+    const int buf = it & 1, tc = t0 + it * kTile;
+    bf16* dst = cb_s + buf * 2 * kTile * NS;
+    for (int x = threadIdx.x; x < 2 * kTile * PIECES; x += blockDim.x) {
+      const int t = x / (2 * PIECES), p = x % (2 * PIECES);
+      const bool is_b = p >= PIECES;
+      const int ch = (is_b ? p - PIECES : p) * 8;
+      const bool ok = tc + t < t1 && ch < N;
+      const bf16* src = is_b ? bg : cg;
+      cp_async16(dst + ((is_b ? kTile : 0) + t) * NS + ch, ok ? src + (size_t)(tc + t) * a.ld + ch : src, ok);
+    }
+    bf16* vd = v_s + buf * kTile * VS;
+    for (int t = warp; t < kTile; t += n_warps)
+      for (int p = lane; p < vp; p += 32) {
+        const bool ok = tc + t < t1;
+        cp_async16(vd + t * VS + p * 8, ok ? vg + (size_t)(tc + t) * a.ld + p * 8 : vg, ok);
+      }
+    cp_async_commit();
+  };
+  auto load_dt = [&](int it) {                            // lane t holds token t of the tile (-inf: no step)
+    const int t = t0 + it * kTile + lane;
+    return lane < kTile && t < t1 ? Num<bf16>::to_f(a.dt[(size_t)t * a.ld_dt + h]) + dbias : -INFINITY;
+  };
+  auto exponents = [&](int it, float z) {
+    const float d = z == -INFINITY ? 0.0f : softplus_f(z);
+    float c = neg_a * d;
+#pragma unroll
+    for (int s = 1; s < kTile; s <<= 1) {
+      const float up = __shfl_up_sync(0xffffffffu, c, s);
+      if (lane >= s) c += up;
+    }
+    const float c_last = __shfl_sync(0xffffffffu, c, kTile - 1);
+    if (lane < kTile) {
+      float* e = e_s + (it & 1) * 3 * kTile;
+      e[lane] = c;
+      e[kTile + lane] = d;
+      e[2 * kTile + lane] = d * expf(c_last - c);
+    }
+  };
+  copy_tile(0);
+  if (warp == 0) exponents(0, load_dt(0));
+  float* Sg = a.state + (((size_t)a.state_slots[seq] * a.H + h) * N) * V;
+  const bool fresh = a.positions[t0] == 0;
+  float S[MT][2 * KN][4];
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < 2 * KN; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = nt * 8 + qc + (e & 1), v = v0 + mt * 16 + gr + (e >> 1) * 8;
+        S[mt][nt][e] = (!fresh && n < N && v < V) ? Sg[(size_t)n * V + v] : 0.0f;
+      }
+  const int a_off = (lane & 15) * NS + (lane >> 4) * 8;
+  const int b_off = ((lane & 7) + (lane >> 4) * 8) * NS + ((lane >> 3) & 1) * 8;
+  const int t_off = (lane & 7) + ((lane >> 3) & 1) * 8;
+  for (int it = 0; it < n_tiles; ++it) {
+    const int buf = it & 1;
+    cp_async_wait_all();
+    __syncthreads();                                       // tile `it` stands; everyone is done with the tile before
+    const bool ahead = it + 1 < n_tiles, mine = ahead && it % n_warps == warp;
+    float z = -INFINITY;
+    if (ahead) copy_tile(it + 1);
+    if (mine) z = load_dt(it + 1);
+    const bf16* c_t = cb_s + buf * 2 * kTile * NS;
+    const bf16* b_t = c_t + kTile * NS;
+    const bf16* v_t = v_s + buf * kTile * VS;
+    const float* e = e_s + buf * 3 * kTile;
+    for (int x = threadIdx.x; x < kTile * PIECES; x += blockDim.x) {
+      const int t = x / PIECES, ch = (x % PIECES) * 8;
+      const uint4 raw = *reinterpret_cast<const uint4*>(b_t + t * NS + ch);
+      const float wt = e[2 * kTile + t];
+      const uint32_t in[4] = {raw.x, raw.y, raw.z, raw.w};
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 bv = Num<bf16>::unpack(in[i]);
+        split_bf16(bv.x * wt, bv.y * wt, hi[i], lo[i]);
+      }
+      *reinterpret_cast<uint4*>(k_s + t * NS + ch) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(k_s + (kTile + t) * NS + ch) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
+    // ---- read-outs: C . S and the scores C . B
+    float sc[2][4], y[MT * 2][4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.0f;
+#pragma unroll
+    for (int i = 0; i < MT * 2; ++i) y[i][0] = y[i][1] = y[i][2] = y[i][3] = 0.0f;
+#pragma unroll
+    for (int ks = 0; ks < KN; ++ks) {
+      uint32_t ca[4], b[4];
+      ldsm_x4(ca, c_t + a_off + ks * 16);
+      ldsm_x4(b, b_t + b_off + ks * 16);
+      mma_bf16(sc[0], ca, b[0], b[1]);
+      mma_bf16(sc[1], ca, b[2], b[3]);
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf) {
+          uint32_t h0, l0, h1, l1;
+          split_bf16(S[mt][2 * ks][2 * hf], S[mt][2 * ks][2 * hf + 1], h0, l0);
+          split_bf16(S[mt][2 * ks + 1][2 * hf], S[mt][2 * ks + 1][2 * hf + 1], h1, l1);
+          mma_bf16(y[mt * 2 + hf], ca, h0, h1);
+          mma_bf16(y[mt * 2 + hf], ca, l0, l1);
+        }
+    }
+    const float ci[2] = {e[gr], e[gr + 8]};
+    const float gi[2] = {__expf(ci[0]), __expf(ci[1])}, c_end = __expf(e[kTile - 1]);
+#pragma unroll
+    for (int i = 0; i < MT * 2; ++i) { y[i][0] *= gi[0]; y[i][1] *= gi[0]; y[i][2] *= gi[1]; y[i][3] *= gi[1]; }
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+      const float2 cj = *reinterpret_cast<const float2*>(e + n * 8 + qc);
+      const float2 dj = *reinterpret_cast<const float2*>(e + kTile + n * 8 + qc);
+#pragma unroll
+      for (int r = 0; r < 4; ++r) {
+        const int i = gr + (r >> 1) * 8, j = n * 8 + qc + (r & 1);
+        const float w = __expf(ci[r >> 1] - (r & 1 ? cj.y : cj.x)) * (r & 1 ? dj.y : dj.x);
+        sc[n][r] = j <= i ? sc[n][r] * w : 0.0f;
+      }
+    }
+    uint32_t ph[4], pl[4];
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+      split_bf16(sc[n][0], sc[n][1], ph[n * 2], pl[n * 2]);
+      split_bf16(sc[n][2], sc[n][3], ph[n * 2 + 1], pl[n * 2 + 1]);
+    }
+    uint32_t va[MT][4];
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {
+      const int vc = v0 + mt * 16;
+      va[mt][0] = va[mt][1] = va[mt][2] = va[mt][3] = 0u;
+      if (vc < V) {                                        // (the same for the whole warp)
+        uint32_t b[4];
+        ldsm_x4_t(b, v_t + t_off * VS + vc + (lane >> 4) * 8);
+        ldsm_x4_t(va[mt], v_t + ((lane & 7) + (lane >> 4) * 8) * VS + vc + ((lane >> 3) & 1) * 8);
+        mma_bf16(y[mt * 2], ph, b[0], b[1]); mma_bf16(y[mt * 2 + 1], ph, b[2], b[3]);
+        mma_bf16(y[mt * 2], pl, b[0], b[1]); mma_bf16(y[mt * 2 + 1], pl, b[2], b[3]);
+      }
+    }
+    const int tc = t0 + it * kTile;
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int t = gr + r * 8;
+      if (tc + t < t1) {
+        float* dst = a.raw + ((size_t)(tc + t) * a.H + h) * V + v0 + qc;
+        const bf16* xr = v_t + t * VS + v0 + qc;
+#pragma unroll
+        for (int i = 0; i < MT * 2; ++i)
+          if (v0 + i * 8 < V) {
+            const float2 x = Num<bf16>::unpack(*reinterpret_cast<const uint32_t*>(xr + i * 8));
+            *reinterpret_cast<float2*>(dst + i * 8) = make_float2(y[i][2 * r] + skip * x.x, y[i][2 * r + 1] + skip * x.y);
+          }
+      }
+    }
+    // ---- the new state
+    __syncthreads();                                       // k_s stands
+#pragma unroll
+    for (int ks = 0; ks < KN; ++ks) {
+      uint32_t b[4], bl[4];
+      ldsm_x4_t(b, k_s + t_off * NS + ks * 16 + (lane >> 4) * 8);
+      ldsm_x4_t(bl, k_s + (kTile + t_off) * NS + ks * 16 + (lane >> 4) * 8);
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt) {
+#pragma unroll
+        for (int r = 0; r < 4; ++r) {
+          S[mt][2 * ks][r] *= c_end;
+          S[mt][2 * ks + 1][r] *= c_end;
+        }
+        mma_bf16(S[mt][2 * ks], va[mt], b[0], b[1]);
+        mma_bf16(S[mt][2 * ks + 1], va[mt], b[2], b[3]);
+        mma_bf16(S[mt][2 * ks], va[mt], bl[0], bl[1]);
+        mma_bf16(S[mt][2 * ks + 1], va[mt], bl[2], bl[3]);
+      }
+    }
+    if (mine) exponents(it + 1, z);
+  }
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < 2 * KN; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = nt * 8 + qc + (e & 1), v = v0 + mt * 16 + gr + (e >> 1) * 8;
+        if (n < N && v < V) Sg[(size_t)n * V + v] = S[mt][nt][e];
+      }
+}
+
+template <int KN, int MT>
+int launch_tc_n(bool forget, const ScanArgs<__nv_bfloat16>& a, int64_t n_seq, cudaStream_t st) {
   const int warps = (a.V + 16 * MT - 1) / (16 * MT);
-  size_t smem = ((size_t)TileRows<KN>::kRows + (size_t)kTile * (a.V + 8)) * sizeof(__nv_bfloat16);
-  smem += (MODE == MODE_FORGET ? (size_t)4 * 16 * KN + (size_t)kTile * (a.V + 4) : (size_t)2 * kTile) * sizeof(float);
-  auto kern = linear_scan_tc_kernel<MODE, KN, MT>;
+  constexpr int NS = TileRows<KN>::NS;
+  size_t smem;
+  if (forget)
+    smem = (size_t)(4 * kTile * NS + kTile * (a.V + 8)) * sizeof(__nv_bfloat16) +
+           (size_t)(4 * 16 * KN + kTile * (a.V + 4)) * sizeof(float);
+  else
+    smem = (size_t)(6 * kTile * NS + 2 * kTile * (a.V + 8)) * sizeof(__nv_bfloat16) + 6 * kTile * sizeof(float);
+  auto kern = forget ? forget_scan_tc_kernel<KN, MT> : ssd_scan_tc_kernel<KN, MT>;
   if (smem > 48 * 1024)
     B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   kern<<<dim3((unsigned)n_seq, (unsigned)a.H), warps * 32, smem, st>>>(a);
-  B200_LAUNCH_OK("linear_scan_tc_kernel");
+  B200_LAUNCH_OK("scan_tc_kernel");
   return B200_OK;
 }
 
-template <int MODE>
-int launch_scan_tc(const ScanArgs<__nv_bfloat16>& a, int64_t n_seq, cudaStream_t st) {
+int launch_scan_tc(bool forget, const ScanArgs<__nv_bfloat16>& a, int64_t n_seq, cudaStream_t st) {
   const bool two = a.V > 64;                              // 16 value rows a warp, or 32
-  if (a.N <= 32) return two ? launch_scan_tc_n<MODE, 2, 2>(a, n_seq, st) : launch_scan_tc_n<MODE, 2, 1>(a, n_seq, st);
-  if (a.N <= 64) return two ? launch_scan_tc_n<MODE, 4, 2>(a, n_seq, st) : launch_scan_tc_n<MODE, 4, 1>(a, n_seq, st);
-  return two ? launch_scan_tc_n<MODE, 8, 2>(a, n_seq, st) : launch_scan_tc_n<MODE, 8, 1>(a, n_seq, st);
+  if (a.N <= 32) return two ? launch_tc_n<2, 2>(forget, a, n_seq, st) : launch_tc_n<2, 1>(forget, a, n_seq, st);
+  if (a.N <= 64) return two ? launch_tc_n<4, 2>(forget, a, n_seq, st) : launch_tc_n<4, 1>(forget, a, n_seq, st);
+  return two ? launch_tc_n<8, 2>(forget, a, n_seq, st) : launch_tc_n<8, 1>(forget, a, n_seq, st);
 }
-
-template <int MODE>
-int launch_scan_tc(const ScanArgs<float>&, int64_t, cudaStream_t) {
+int launch_scan_tc(bool, const ScanArgs<float>&, int64_t, cudaStream_t) {
   return set_error(B200_ERR_UNSUPPORTED, "linear_scan: the tensor-core form takes bf16");
 }
 
@@ -872,7 +977,7 @@ int b200_forget_scan(void* out, int64_t ldo, const void* q, const void* f, const
     a.vec_in = N % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && is_aligned(q, 4 * sizeof(T)) && is_aligned(f, 4 * sizeof(T)) &&
                is_aligned(v, 4 * sizeof(T));
     a.vec_state = V % 4 == 0 && is_aligned(state, 16);
-    if (tensor_cores) return launch_scan_tc<MODE_FORGET>(a, n_seq, st);
+    if (tensor_cores) return launch_scan_tc(true, a, n_seq, st);
     const int rc = launch_scan<T, MODE_FORGET>(a, n_seq, q_max, st);
     if (rc != B200_OK) return rc;
     if (raw) {
@@ -909,7 +1014,7 @@ int b200_ssd_scan(float* y, const void* x, const void* B, const void* Cm, int64_
     a.vec_in = N % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && is_aligned(x, 4 * sizeof(T)) && is_aligned(B, 4 * sizeof(T)) &&
                is_aligned(Cm, 4 * sizeof(T));
     a.vec_state = V % 4 == 0 && is_aligned(state, 16);
-    if (tensor_cores) return launch_scan_tc<MODE_SSD>(a, n_seq, st);
+    if (tensor_cores) return launch_scan_tc(false, a, n_seq, st);
     return (launch_scan<T, MODE_SSD>(a, n_seq, q_max, st));
   });
   return B200_OK;

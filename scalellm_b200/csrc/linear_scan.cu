@@ -409,6 +409,13 @@ struct TileRows {
   static constexpr int kRows = 4 * kTile * NS;            // the four key-channel arrays
 };
 
+__device__ __forceinline__ void cp_async16(void* smem_dst, const void* gsrc, bool valid) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(smem_dst)), "l"(gsrc), "r"(valid ? 16 : 0)
+               : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+
 // One token of two neighbouring key channels of a forget tile: gates a, written shares k and silu(q) from the raw pairs.
 __device__ __forceinline__ void forget_token(uint32_t qraw, uint32_t fraw, float2 bias, float2 low, float2& q, float2& a,
                                              float2& k) {
@@ -424,21 +431,22 @@ __device__ __forceinline__ void forget_token(uint32_t qraw, uint32_t fraw, float
   q = make_float2(__fdividef(qv.x, 1.0f + __expf(-qv.x)), __fdividef(qv.y, 1.0f + __expf(-qv.y)));
 }
 
-// Channels c, c + 1 of one half of a forget tile of L tokens whose middle is after token HA - 1.  BEFORE: tokens
-// HA - 1 .. 0, else tokens HA .. 15 (zeros from L on).  FULL: HA = 8, L = 16, all loads in flight together.  Returns the
-// product of the half's gates.
+// Channels c, c + 1 of one half of a forget tile of L tokens from row o on, whose middle is after token o + HA - 1.
+// BEFORE: rows o + HA - 1 .. 0, else rows o + HA .. 15 (zeros outside the tile).  FULL: o = 0, HA = 8, L = 16.  raw: the
+// window's query and forget logits [2][16][16 KN].  Returns the product of the half's gates.
 template <int KN, bool BEFORE, bool FULL>
-__device__ __forceinline__ float2 stage_forget_half(__nv_bfloat16* rows, const __nv_bfloat16* __restrict__ q,
-                                                    const __nv_bfloat16* __restrict__ f, int64_t ld, int c, bool live,
-                                                    float2 bias, float2 low, int HA_rt, int L_rt) {
-  constexpr int NS = TileRows<KN>::NS;
-  const int HA = FULL ? 8 : HA_rt, L = FULL ? kTile : L_rt;
+__device__ __forceinline__ float2 stage_forget_half(__nv_bfloat16* rows, const __nv_bfloat16* raw, int c, float2 bias,
+                                                    float2 low, int o_rt, int HA_rt, int L_rt) {
+  constexpr int NS = TileRows<KN>::NS, NP = 16 * KN;
+  const int o = FULL ? 0 : o_rt, HA = FULL ? 8 : HA_rt, L = FULL ? kTile : L_rt;
   float2 r = make_float2(1.0f, 1.0f);
-  auto put = [&](int t, uint32_t qraw, uint32_t fraw, bool ok) {
+  auto put = [&](int t) {
     uint32_t qh = 0u, ql = 0u, kh = 0u, kl = 0u;
-    if (ok) {
+    if (FULL || (t >= o && t < o + L)) {
+      const __nv_bfloat16* src = raw + t * NP + c;
       float2 qs, a, k;
-      forget_token(qraw, fraw, bias, low, qs, a, k);
+      forget_token(*reinterpret_cast<const uint32_t*>(src), *reinterpret_cast<const uint32_t*>(src + kTile * NP), bias,
+                   low, qs, a, k);
       if constexpr (BEFORE) {
         split_bf16(__fdividef(qs.x, r.x), __fdividef(qs.y, r.y), qh, ql);
         split_bf16(k.x * r.x, k.y * r.y, kh, kl);
@@ -451,45 +459,38 @@ __device__ __forceinline__ float2 stage_forget_half(__nv_bfloat16* rows, const _
         split_bf16(__fdividef(k.x, r.x), __fdividef(k.y, r.y), kh, kl);
       }
     }
-    __nv_bfloat16* dst = rows + (size_t)t * NS + c;
+    __nv_bfloat16* dst = rows + t * NS + c;
     *reinterpret_cast<uint32_t*>(dst) = qh;
     *reinterpret_cast<uint32_t*>(dst + kTile * NS) = ql;
     *reinterpret_cast<uint32_t*>(dst + 2 * kTile * NS) = kh;
     *reinterpret_cast<uint32_t*>(dst + 3 * kTile * NS) = kl;
   };
   if constexpr (FULL) {
-    uint32_t qraw[8], fraw[8];
 #pragma unroll
-    for (int s = 0; s < 8; ++s) {
-      const int t = BEFORE ? 7 - s : 8 + s;
-      qraw[s] = live ? *reinterpret_cast<const uint32_t*>(q + (int64_t)t * ld + c) : 0u;
-      fraw[s] = live ? *reinterpret_cast<const uint32_t*>(f + (int64_t)t * ld + c) : 0u;
-    }
-#pragma unroll
-    for (int s = 0; s < 8; ++s) put(BEFORE ? 7 - s : 8 + s, qraw[s], fraw[s], live);
+    for (int s = 0; s < 8; ++s) put(BEFORE ? 7 - s : 8 + s);
+  } else if constexpr (BEFORE) {
+    for (int t = o + HA - 1; t >= 0; --t) put(t);
   } else {
-    const int n = BEFORE ? HA : kTile - HA;
-    for (int s = 0; s < n; ++s) {
-      const int t = BEFORE ? HA - 1 - s : HA + s;
-      const bool ok = live && t < L;
-      put(t, ok ? *reinterpret_cast<const uint32_t*>(q + (int64_t)t * ld + c) : 0u,
-          ok ? *reinterpret_cast<const uint32_t*>(f + (int64_t)t * ld + c) : 0u, ok);
-    }
+    for (int t = o + HA; t < kTile; ++t) put(t);
   }
   return r;
 }
 
+// The walk goes by windows of 16 tokens, whose raw rows are copied one window ahead (two buffers); a window is one tile
+// unless its gates are too small.  The decay to the end of a tile is applied together with the next tile's decay to the
+// middle.
 template <int KN, int MT>
 __global__ void __launch_bounds__(MT == 1 ? 128 : kScanWarps * 32, MT == 1 ? 2 : 1)
 forget_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
   using bf16 = __nv_bfloat16;
-  constexpr int NP = 16 * KN, NS = TileRows<KN>::NS;
+  constexpr int NP = 16 * KN, NS = TileRows<KN>::NS, PIECES = NP / 8;
   extern __shared__ __align__(16) unsigned char smraw[];
   const int N = a.N, V = a.V, VS = V + 8, OS = V + 4;
-  bf16* rows = reinterpret_cast<bf16*>(smraw);            // [4][16][NS]
-  bf16* v_s = rows + TileRows<KN>::kRows;                 // [16][VS]
-  float* e_s = reinterpret_cast<float*>(v_s + kTile * VS);   // [2][NP] products of the two halves
-  float* c_s = e_s + 2 * NP;                              // [2][NP] bias, lower bound
+  bf16* rows = reinterpret_cast<bf16*>(smraw);            // [q hi, q lo, k hi, k lo][16][NS]
+  bf16* raw_s = rows + TileRows<KN>::kRows;               // [2 buffers][q, f][16][NP]
+  bf16* v_s = raw_s + 4 * kTile * NP;                     // [2 buffers][16][VS]
+  float* e_s = reinterpret_cast<float*>(v_s + 2 * kTile * VS);   // [NP] to the middle, [2][NP] to the end (two tiles')
+  float* c_s = e_s + 3 * NP;                              // [2][NP] bias, lower bound
   float* o_s = c_s + 2 * NP;                              // [16][OS]
   const int seq = blockIdx.x, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
@@ -497,6 +498,31 @@ forget_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
   if (t0 >= t1) return;
   const int gr = lane >> 2, qc = (lane & 3) * 2;
   const int v0 = warp * 16 * MT;                          // this warp's value rows v0 .. v0 + 16 MT - 1
+  const int n_windows = (t1 - t0 + kTile - 1) / kTile;
+  const bf16* qg = a.q + (size_t)h * N;
+  const bf16* fg = a.k + (size_t)h * N;
+  const bf16* vg = a.v + (size_t)h * V;
+  const int vp = V / 8;
+  auto copy_window = [&](int it) {
+    const int buf = it & 1, tc = t0 + it * kTile;
+    bf16* dst = raw_s + buf * 2 * kTile * NP;
+    for (int x = threadIdx.x; x < 2 * kTile * PIECES; x += blockDim.x) {
+      const int t = x / (2 * PIECES), p = x % (2 * PIECES);
+      const bool is_f = p >= PIECES;
+      const int ch = (is_f ? p - PIECES : p) * 8;
+      const bool ok = tc + t < t1 && ch < N;              // (channels past N: zeros make q = k = 0, the gate 1)
+      const bf16* src = is_f ? fg : qg;
+      cp_async16(dst + ((is_f ? kTile : 0) + t) * NP + ch, ok ? src + (size_t)(tc + t) * a.ld + ch : src, ok);
+    }
+    bf16* vd = v_s + buf * kTile * VS;
+    for (int t = warp; t < kTile; t += n_warps)
+      for (int p = lane; p < vp; p += 32) {
+        const bool ok = tc + t < t1;
+        cp_async16(vd + t * VS + p * 8, ok ? vg + (size_t)(tc + t) * a.ld + p * 8 : vg, ok);
+      }
+    cp_async_commit();
+  };
+  copy_window(0);
   float* Sg = a.state + (((size_t)a.state_slots[seq] * a.H + h) * N) * V;
   const bool fresh = a.positions[t0] == 0;
   float S[MT][2 * KN][4];
@@ -512,181 +538,175 @@ forget_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
   for (int i = threadIdx.x; i < NP; i += blockDim.x) {
     c_s[i] = i < N ? a.f_bias[h * N + i] : 0.0f;
     c_s[NP + i] = i < N ? a.f_low[h * N + i] : 1.0f;
+    e_s[NP + i] = 1.0f;                                    // the first tile's decay from a tile before it
   }
-  __syncthreads();
-  int L = 0;
-  for (int tc = t0; tc < t1; tc += L) {
-    L = t1 - tc < kTile ? t1 - tc : kTile;
-    // ---- stage the tile
-    const bf16* vg = a.v + (size_t)tc * a.ld + (size_t)h * V;
-    const bf16* qg = a.q + (size_t)tc * a.ld + (size_t)h * N;
-    const bf16* fg = a.k + (size_t)tc * a.ld + (size_t)h * N;
-    while (true) {
-      const int HA = (L + 1) / 2;
-      bool bad = false;
-      for (int u = threadIdx.x; u < NP; u += blockDim.x) {
-        const bool before = u < NP / 2;
-        const int c = (before ? u : u - NP / 2) * 2;
-        const bool live = c < N;
-        const float2 bias = *reinterpret_cast<const float2*>(c_s + c), low = *reinterpret_cast<const float2*>(c_s + NP + c);
-        float2 r;
-        if (L == kTile) {
-          r = before ? stage_forget_half<KN, true, true>(rows, qg, fg, a.ld, c, live, bias, low, HA, L)
-                     : stage_forget_half<KN, false, true>(rows, qg, fg, a.ld, c, live, bias, low, HA, L);
-        } else {
-          r = before ? stage_forget_half<KN, true, false>(rows, qg, fg, a.ld, c, live, bias, low, HA, L)
-                     : stage_forget_half<KN, false, false>(rows, qg, fg, a.ld, c, live, bias, low, HA, L);
+  const int a_off = (lane & 15) * NS + (lane >> 4) * 8;
+  const int b_off = ((lane & 7) + (lane >> 4) * 8) * NS + ((lane >> 3) & 1) * 8;
+  const int t_off = (lane & 7) + ((lane >> 3) & 1) * 8;
+  const bf16* q_hi = rows;
+  const bf16* q_lo = rows + kTile * NS;
+  const bf16* k_hi = rows + 2 * kTile * NS;
+  const bf16* k_lo = rows + 3 * kTile * NS;
+  int par = 0;                                             // which of the two end decays is the tile before's
+  for (int it = 0; it < n_windows; ++it) {
+    const int tc = t0 + it * kTile, nt_w = t1 - tc < kTile ? t1 - tc : kTile;
+    const bf16* raw = raw_s + (it & 1) * 2 * kTile * NP;
+    const bf16* v_t = v_s + (it & 1) * kTile * VS;
+    cp_async_wait_all();
+    __syncthreads();                                       // the window's raw rows stand
+    if (it + 1 < n_windows) copy_window(it + 1);
+    int L = 0;
+    for (int o = 0; o < nt_w; o += L) {
+      // ---- stage the tile: rows o .. o + L - 1 of the window
+      L = nt_w - o;
+      while (true) {
+        const int HA = (L + 1) / 2;
+        bool bad = false;
+        for (int u = threadIdx.x; u < NP; u += blockDim.x) {
+          const bool before = u < NP / 2;
+          const int c = (before ? u : u - NP / 2) * 2;
+          const float2 bias = *reinterpret_cast<const float2*>(c_s + c), low = *reinterpret_cast<const float2*>(c_s + NP + c);
+          float2 r;
+          if (L == kTile) {
+            r = before ? stage_forget_half<KN, true, true>(rows, raw, c, bias, low, o, HA, L)
+                       : stage_forget_half<KN, false, true>(rows, raw, c, bias, low, o, HA, L);
+          } else {
+            r = before ? stage_forget_half<KN, true, false>(rows, raw, c, bias, low, o, HA, L)
+                       : stage_forget_half<KN, false, false>(rows, raw, c, bias, low, o, HA, L);
+          }
+          *reinterpret_cast<float2*>(e_s + (before ? 0 : NP + (par ^ 1) * NP) + c) = r;
+          bad |= !(fminf(r.x, r.y) >= kMinSpan);
         }
-        *reinterpret_cast<float2*>(e_s + (before ? 0 : NP) + c) = r;
-        bad |= live && !(fminf(r.x, r.y) >= kMinSpan);
+        const int any_bad = __syncthreads_or(bad);         // (also: the tile stands)
+        if (L == 1 || !any_bad) break;
+        L = L > 4 ? 4 : 1;
       }
-      if (L == 1 || !__syncthreads_or(bad)) break;
-      L = L > 4 ? 4 : 1;
-    }
-    for (int x = threadIdx.x; x < kTile * (V / 8); x += blockDim.x) {
-      const int t = x / (V / 8), ch = (x - t * (V / 8)) * 8;
-      uint4 raw = make_uint4(0u, 0u, 0u, 0u);
-      if (t < L) raw = *reinterpret_cast<const uint4*>(vg + (size_t)t * a.ld + ch);
-      *reinterpret_cast<uint4*>(v_s + t * VS + ch) = raw;
-    }
-    __syncthreads();
-    // ---- products
-    const bf16* q_hi = rows;
-    const bf16* q_lo = rows + kTile * NS;
-    const bf16* k_hi = rows + 2 * kTile * NS;
-    const bf16* k_lo = rows + 3 * kTile * NS;
+      // ---- products
 #pragma unroll
-    for (int nt = 0; nt < 2 * KN; ++nt) {                  // to the middle of the tile
-      const float2 e = *reinterpret_cast<const float2*>(e_s + nt * 8 + qc);
+      for (int nt = 0; nt < 2 * KN; ++nt) {                // from the tile before to the middle of this one
+        float2 e = *reinterpret_cast<const float2*>(e_s + nt * 8 + qc);
+        const float2 ep = *reinterpret_cast<const float2*>(e_s + NP + par * NP + nt * 8 + qc);
+        e.x *= ep.x;
+        e.y *= ep.y;
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt) {
-        S[mt][nt][0] *= e.x; S[mt][nt][1] *= e.y; S[mt][nt][2] *= e.x; S[mt][nt][3] *= e.y;
-      }
-    }
-    float sc[2][4], y[MT * 2][4];
-#pragma unroll
-    for (int i = 0; i < 2; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.0f;
-#pragma unroll
-    for (int i = 0; i < MT * 2; ++i) y[i][0] = y[i][1] = y[i][2] = y[i][3] = 0.0f;
-    const int a_off = (lane & 15) * NS + (lane >> 4) * 8;
-    const int b_off = ((lane & 7) + (lane >> 4) * 8) * NS + ((lane >> 3) & 1) * 8;
-#pragma unroll
-    for (int ks = 0; ks < KN; ++ks) {
-      uint32_t ah[4], b[4];
-      ldsm_x4(ah, q_hi + a_off + ks * 16);
-      uint32_t al[4], bl[4];
-      ldsm_x4(al, q_lo + a_off + ks * 16);
-      ldsm_x4(b, k_hi + b_off + ks * 16);
-      ldsm_x4(bl, k_lo + b_off + ks * 16);
-      mma_bf16(sc[0], ah, b[0], b[1]);  mma_bf16(sc[1], ah, b[2], b[3]);
-      mma_bf16(sc[0], ah, bl[0], bl[1]); mma_bf16(sc[1], ah, bl[2], bl[3]);
-      mma_bf16(sc[0], al, b[0], b[1]);  mma_bf16(sc[1], al, b[2], b[3]);
-#pragma unroll
-      for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-        for (int hf = 0; hf < 2; ++hf) {
-          uint32_t h0, l0, h1, l1;
-          split_bf16(S[mt][2 * ks][2 * hf], S[mt][2 * ks][2 * hf + 1], h0, l0);
-          split_bf16(S[mt][2 * ks + 1][2 * hf], S[mt][2 * ks + 1][2 * hf + 1], h1, l1);
-          mma_bf16(y[mt * 2 + hf], ah, h0, h1);
-          mma_bf16(y[mt * 2 + hf], ah, l0, l1);
-          mma_bf16(y[mt * 2 + hf], al, h0, h1);
+        for (int mt = 0; mt < MT; ++mt) {
+          S[mt][nt][0] *= e.x; S[mt][nt][1] *= e.y; S[mt][nt][2] *= e.x; S[mt][nt][3] *= e.y;
         }
-    }
-#pragma unroll
-    for (int n = 0; n < 2; ++n)
-#pragma unroll
-      for (int e = 0; e < 4; ++e)
-        if (n * 8 + qc + (e & 1) > gr + (e >> 1) * 8) sc[n][e] = 0.0f;
-    uint32_t ph[4], pl[4];
-#pragma unroll
-    for (int n = 0; n < 2; ++n) {
-      split_bf16(sc[n][0], sc[n][1], ph[n * 2], pl[n * 2]);
-      split_bf16(sc[n][2], sc[n][3], ph[n * 2 + 1], pl[n * 2 + 1]);
-    }
-    const int t_off = ((lane & 7) + ((lane >> 3) & 1) * 8);
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt) {
-      const int vc = v0 + mt * 16;
-      if (vc < V) {                                        // (the same for the whole warp)
-        uint32_t b[4];
-        ldsm_x4_t(b, v_s + t_off * VS + vc + (lane >> 4) * 8);
-        mma_bf16(y[mt * 2], ph, b[0], b[1]); mma_bf16(y[mt * 2 + 1], ph, b[2], b[3]);
-        mma_bf16(y[mt * 2], pl, b[0], b[1]); mma_bf16(y[mt * 2 + 1], pl, b[2], b[3]);
       }
-    }
-    // ---- the new state
-    uint32_t va[MT][4];
+      par ^= 1;
+      float sc[2][4], y[MT * 2][4];
 #pragma unroll
-    for (int mt = 0; mt < MT; ++mt) {
-      const int vc = v0 + mt * 16;
-      va[mt][0] = va[mt][1] = va[mt][2] = va[mt][3] = 0u;
-      if (vc < V) ldsm_x4_t(va[mt], v_s + ((lane & 7) + (lane >> 4) * 8) * VS + vc + ((lane >> 3) & 1) * 8);
-    }
+      for (int i = 0; i < 2; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.0f;
 #pragma unroll
-    for (int ks = 0; ks < KN; ++ks) {
-      uint32_t b[4], bl[4];
-      ldsm_x4_t(b, k_hi + t_off * NS + ks * 16 + (lane >> 4) * 8);
-      ldsm_x4_t(bl, k_lo + t_off * NS + ks * 16 + (lane >> 4) * 8);
+      for (int i = 0; i < MT * 2; ++i) y[i][0] = y[i][1] = y[i][2] = y[i][3] = 0.0f;
+#pragma unroll
+      for (int ks = 0; ks < KN; ++ks) {
+        uint32_t ah[4], b[4];
+        ldsm_x4(ah, q_hi + a_off + ks * 16);
+        uint32_t al[4], bl[4];
+        ldsm_x4(al, q_lo + a_off + ks * 16);
+        ldsm_x4(b, k_hi + b_off + ks * 16);
+        ldsm_x4(bl, k_lo + b_off + ks * 16);
+        mma_bf16(sc[0], ah, b[0], b[1]);  mma_bf16(sc[1], ah, b[2], b[3]);
+        mma_bf16(sc[0], ah, bl[0], bl[1]); mma_bf16(sc[1], ah, bl[2], bl[3]);
+        mma_bf16(sc[0], al, b[0], b[1]);  mma_bf16(sc[1], al, b[2], b[3]);
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+          for (int hf = 0; hf < 2; ++hf) {
+            uint32_t h0, l0, h1, l1;
+            split_bf16(S[mt][2 * ks][2 * hf], S[mt][2 * ks][2 * hf + 1], h0, l0);
+            split_bf16(S[mt][2 * ks + 1][2 * hf], S[mt][2 * ks + 1][2 * hf + 1], h1, l1);
+            mma_bf16(y[mt * 2 + hf], ah, h0, h1);
+            mma_bf16(y[mt * 2 + hf], ah, l0, l1);
+            mma_bf16(y[mt * 2 + hf], al, h0, h1);
+          }
+      }
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (n * 8 + qc + (e & 1) > gr + (e >> 1) * 8) sc[n][e] = 0.0f;
+      uint32_t ph[4], pl[4];
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        split_bf16(sc[n][0], sc[n][1], ph[n * 2], pl[n * 2]);
+        split_bf16(sc[n][2], sc[n][3], ph[n * 2 + 1], pl[n * 2 + 1]);
+      }
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt) {
-        mma_bf16(S[mt][2 * ks], va[mt], b[0], b[1]);
-        mma_bf16(S[mt][2 * ks + 1], va[mt], b[2], b[3]);
-        mma_bf16(S[mt][2 * ks], va[mt], bl[0], bl[1]);
-        mma_bf16(S[mt][2 * ks + 1], va[mt], bl[2], bl[3]);
+        const int vc = v0 + mt * 16;
+        if (vc < V) {                                        // (the same for the whole warp)
+          uint32_t b[4];
+          ldsm_x4_t(b, v_t + t_off * VS + vc + (lane >> 4) * 8);
+          mma_bf16(y[mt * 2], ph, b[0], b[1]); mma_bf16(y[mt * 2 + 1], ph, b[2], b[3]);
+          mma_bf16(y[mt * 2], pl, b[0], b[1]); mma_bf16(y[mt * 2 + 1], pl, b[2], b[3]);
+        }
       }
-    }
-#pragma unroll
-    for (int nt = 0; nt < 2 * KN; ++nt) {                  // to the end of the tile
-      const float2 e = *reinterpret_cast<const float2*>(e_s + NP + nt * 8 + qc);
+      // ---- the new state
+      uint32_t va[MT][4];
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt) {
-        S[mt][nt][0] *= e.x; S[mt][nt][1] *= e.y; S[mt][nt][2] *= e.x; S[mt][nt][3] *= e.y;
+        const int vc = v0 + mt * 16;
+        va[mt][0] = va[mt][1] = va[mt][2] = va[mt][3] = 0u;
+        if (vc < V) ldsm_x4_t(va[mt], v_t + ((lane & 7) + (lane >> 4) * 8) * VS + vc + ((lane >> 3) & 1) * 8);
       }
-    }
-    // ---- out
 #pragma unroll
-    for (int i = 0; i < MT * 2; ++i) {
-      const int v = v0 + i * 8 + qc;
-      if (v < V) {
-        *reinterpret_cast<float2*>(o_s + gr * OS + v) = make_float2(y[i][0], y[i][1]);
-        *reinterpret_cast<float2*>(o_s + (gr + 8) * OS + v) = make_float2(y[i][2], y[i][3]);
+      for (int ks = 0; ks < KN; ++ks) {
+        uint32_t b[4], bl[4];
+        ldsm_x4_t(b, k_hi + t_off * NS + ks * 16 + (lane >> 4) * 8);
+        ldsm_x4_t(bl, k_lo + t_off * NS + ks * 16 + (lane >> 4) * 8);
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt) {
+          mma_bf16(S[mt][2 * ks], va[mt], b[0], b[1]);
+          mma_bf16(S[mt][2 * ks + 1], va[mt], b[2], b[3]);
+          mma_bf16(S[mt][2 * ks], va[mt], bl[0], bl[1]);
+          mma_bf16(S[mt][2 * ks + 1], va[mt], bl[2], bl[3]);
+        }
       }
-    }
-    __syncthreads();                                     // the read-outs stand; the tile's rows are done with
-    for (int t = warp; t < L; t += n_warps) {
-      const float* ot = o_s + t * OS;
-      float ss = 0.0f;
-      for (int c = lane * 2; c < V; c += 64) {
-        const float2 o = *reinterpret_cast<const float2*>(ot + c);
-        ss += o.x * o.x + o.y * o.y;
+      // ---- out: eight lanes a token
+#pragma unroll
+      for (int i = 0; i < MT * 2; ++i) {
+        const int v = v0 + i * 8 + qc;
+        if (v < V) {
+          *reinterpret_cast<float2*>(o_s + gr * OS + v) = make_float2(y[i][0], y[i][1]);
+          *reinterpret_cast<float2*>(o_s + (gr + 8) * OS + v) = make_float2(y[i][2], y[i][3]);
+        }
       }
-      ss = warp_sum(ss);
-      const float inv = a.mul / sqrtf(ss / (float)V + a.eps);
-      bf16* dst = a.out + (size_t)(tc + t) * a.ldo + (size_t)h * V;
-      for (int c = lane * 2; c < V; c += 64) {
-        const float2 o = *reinterpret_cast<const float2*>(ot + c);
-        *reinterpret_cast<uint32_t*>(dst + c) = Num<bf16>::pack(o.x * inv * a.norm_w[c], o.y * inv * a.norm_w[c + 1]);
+      __syncthreads();                                     // the read-outs stand; the tile's rows are done with
+      for (int tb = o + warp * 4; tb < o + L; tb += n_warps * 4) {
+        const int t = tb + (lane >> 3), sub = lane & 7;
+        const bool ok = t < o + L;
+        const float* ot = o_s + (ok ? t : o) * OS;
+        float ss = 0.0f;
+        for (int c = sub * 2; c < V; c += 16) {
+          const float2 w = *reinterpret_cast<const float2*>(ot + c);
+          ss += w.x * w.x + w.y * w.y;
+        }
+#pragma unroll
+        for (int d = 1; d < 8; d <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+        if (!ok) continue;
+        const float inv = a.mul / sqrtf(ss / (float)V + a.eps);
+        bf16* dst = a.out + (size_t)(tc + t) * a.ldo + (size_t)h * V;
+        for (int c = sub * 2; c < V; c += 16) {
+          const float2 w = *reinterpret_cast<const float2*>(ot + c), nw = *reinterpret_cast<const float2*>(a.norm_w + c);
+          *reinterpret_cast<uint32_t*>(dst + c) = Num<bf16>::pack(w.x * inv * nw.x, w.y * inv * nw.y);
+        }
       }
     }
   }
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-    for (int nt = 0; nt < 2 * KN; ++nt)
+    for (int nt = 0; nt < 2 * KN; ++nt) {
+      const float2 ep = *reinterpret_cast<const float2*>(e_s + NP + par * NP + nt * 8 + qc);   // the last tile's end
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int n = nt * 8 + qc + (e & 1), v = v0 + mt * 16 + gr + (e >> 1) * 8;
-        if (n < N && v < V) Sg[(size_t)n * V + v] = S[mt][nt][e];
+        if (n < N && v < V) Sg[(size_t)n * V + v] = S[mt][nt][e] * (e & 1 ? ep.y : ep.x);
       }
+    }
 }
-
-__device__ __forceinline__ void cp_async16(void* smem_dst, const void* gsrc, bool valid) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(smem_dst)), "l"(gsrc), "r"(valid ? 16 : 0)
-               : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
 
 // A tile's C, B and x rows are copied one tile ahead (two buffers); its decay exponents are worked out one tile ahead by
 // one warp, which takes turns.
@@ -907,8 +927,8 @@ int launch_tc_n(bool forget, const ScanArgs<__nv_bfloat16>& a, int64_t n_seq, cu
   constexpr int NS = TileRows<KN>::NS;
   size_t smem;
   if (forget)
-    smem = (size_t)(4 * kTile * NS + kTile * (a.V + 8)) * sizeof(__nv_bfloat16) +
-           (size_t)(4 * 16 * KN + kTile * (a.V + 4)) * sizeof(float);
+    smem = (size_t)(4 * kTile * (NS + 16 * KN) + 2 * kTile * (a.V + 8)) * sizeof(__nv_bfloat16) +
+           (size_t)(5 * 16 * KN + kTile * (a.V + 4)) * sizeof(float);
   else
     smem = (size_t)(6 * kTile * NS + 2 * kTile * (a.V + 8)) * sizeof(__nv_bfloat16) + 6 * kTile * sizeof(float);
   auto kern = forget ? forget_scan_tc_kernel<KN, MT> : ssd_scan_tc_kernel<KN, MT>;
@@ -962,8 +982,9 @@ int b200_forget_scan(void* out, int64_t ldo, const void* q, const void* f, const
   B200_CHECK_ARG(rows > 0 && n_seq > 0 && q_max > 0 && H > 0 && H <= 65535 && N > 0 && N <= 512 && V > 0 && V <= 4096 &&
                      ldo >= H * V && ld >= H * (N > V ? N : V),
                  "forget_scan: bad shape (key size <= 512)");
-  B200_CHECK_ARG(!tensor_cores || (scan_tc_fits(N, V, dtype) && ld % 8 == 0 && ldo % 2 == 0 && is_aligned(q, 4) &&
-                                   is_aligned(f, 4) && is_aligned(v, 16) && is_aligned(out, 4)),
+  B200_CHECK_ARG(!tensor_cores || (scan_tc_fits(N, V, dtype) && ld % 8 == 0 && ldo % 2 == 0 && is_aligned(q, 16) &&
+                                   is_aligned(f, 16) && is_aligned(v, 16) && is_aligned(out, 4) &&
+                                   is_aligned(norm_weight, 8)),
                  "forget_scan: sizes or alignment do not fit the tensor-core tiles");
   B200_CHECK_ARG(tensor_cores || raw || scan_col_parts((int)N, (int)V) == 1, "forget_scan: heads in several column parts need a workspace");
   auto st = static_cast<cudaStream_t>(stream);

@@ -99,21 +99,14 @@ linear_scan_kernel(const ScanArgs<T> a) {
   const int c0 = cq * 4;                                  // this thread's columns c0 .. c0 + 3 of the part
   float* Sg = a.state + (((size_t)a.state_slots[seq] * a.H + h) * N) * V + cb0;
   const bool fresh = a.positions[t0] == 0;
-  f32x2 S[RL / 2][4];                                     // pairs of key rows
+  // the state is asked for first and made into pairs of key rows only after the first tokens are staged, so that its
+  // latency and theirs overlap (a decoded token's step is little else)
+  float raw[RL][4];
 #pragma unroll
-  for (int i = 0; i < RL / 4; ++i) {
-    const int n0 = p * 4 + i * 4 * LP;
-#pragma unroll
-    for (int jj = 0; jj < 2; ++jj) {
-      float lo[4] = {0.0f, 0.0f, 0.0f, 0.0f}, hi[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-      const int n = n0 + jj * 2;
-      if (!fresh && c0 < ncol) {
-        if (n < N) get4c<float>(Sg + (size_t)n * V + c0, lo, ncol - c0, a.vec_state);
-        if (n + 1 < N) get4c<float>(Sg + (size_t)(n + 1) * V + c0, hi, ncol - c0, a.vec_state);
-      }
-#pragma unroll
-      for (int c = 0; c < 4; ++c) S[i * 2 + jj][c] = pack2(lo[c], hi[c]);
-    }
+  for (int i = 0; i < RL; ++i) {
+    const int n = p * 4 + (i / 4) * 4 * LP + (i & 3);
+    raw[i][0] = raw[i][1] = raw[i][2] = raw[i][3] = 0.0f;
+    if (!fresh && c0 < ncol && n < N) get4c<float>(Sg + (size_t)n * V + c0, raw[i], ncol - c0, a.vec_state);
   }
   const int g = MODE == MODE_SSD ? h / (a.H / a.G) : h;
   float neg_a = 0.0f, dbias = 0.0f, skip = 0.0f;
@@ -122,9 +115,7 @@ linear_scan_kernel(const ScanArgs<T> a) {
     dbias = a.dt_bias[h];
     skip = a.skip[h];
   }
-  for (int tc = t0; tc < t1; tc += CH) {
-    const int nt = t1 - tc < CH ? t1 - tc : CH;
-    __syncthreads();                                      // the read-outs and rows of the chunk before are done with
+  auto stage = [&](int tc, int nt) {
     for (int tok = warp; tok < nt; tok += n_warps) {
       const size_t row = (size_t)(tc + tok);
       const T* qr = a.q + row * a.ld + (size_t)g * N;
@@ -167,6 +158,19 @@ linear_scan_kernel(const ScanArgs<T> a) {
         if (c < ncol) get4c<T>(vr + c, vv, ncol - c, a.vec_in);
         *reinterpret_cast<float4*>(v_s + tok * CBP + c) = make_float4(vv[0], vv[1], vv[2], vv[3]);
       }
+    }
+  };
+  stage(t0, t1 - t0 < CH ? t1 - t0 : CH);
+  f32x2 S[RL / 2][4];
+#pragma unroll
+  for (int i = 0; i < RL / 2; ++i)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) S[i][c] = pack2(raw[2 * i][c], raw[2 * i + 1][c]);
+  for (int tc = t0; tc < t1; tc += CH) {
+    const int nt = t1 - tc < CH ? t1 - tc : CH;
+    if (tc != t0) {
+      __syncthreads();                                    // the read-outs and rows of the chunk before are done with
+      stage(tc, nt);
     }
     __syncthreads();
     for (int tok = 0; tok < nt; ++tok) {

@@ -218,6 +218,7 @@ def test_forget_gate_recurrence_over_portions(H, N, V, dtype):
     g = torch.Generator().manual_seed(H * N + V)
     fb, low = torch.randn(H * N, generator=g) * 3.0, torch.rand(H * N, generator=g) ** 0.3
     low[::5] = 0.0
+    fb[::35] = -60.0                                             # with a lower bound of 0: nothing is kept at all
     nw = 0.5 + torch.rand(V, generator=g)
     n, nv = H * N, H * V
     data = {s: (torch.randn(total(s), 2 * n + nv, generator=g).mul(2.0).to(dtype),) for s in PLANS}

@@ -185,6 +185,125 @@ __global__ void __launch_bounds__(kPnThreads) prenorm_filter_kernel(const Prenor
     }
 }
 
+// The same for filters of at most TP taps on rows of whole 4-channel groups: the last TP - 1 normalised rows stay in
+// registers (thread t owns groups t, t + threads, ...: NG of them), and R rows at a time are loaded and summed, so that
+// their loads are in flight together and share a barrier.
+template <typename T, int SRC, int TP, int NG, int R>
+__global__ void __launch_bounds__(512) prenorm_walk_kernel(const PrenormArgs a) {
+  __shared__ float red[2][R][16];
+  const int W = a.W, taps = a.taps, seq = blockIdx.y, nt = blockDim.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = nt >> 5;
+  const int q0 = a.q_cu[seq], n = a.q_cu[seq + 1] - q0;
+  const int r0 = (int)blockIdx.x * a.chunk;
+  if (r0 >= n) return;
+  const int r1 = r0 + a.chunk < n ? r0 + a.chunk : n;
+  const int pos0 = a.positions[q0];
+  float* st = a.state + (size_t)a.state_slots[seq] * (taps - 1) * W;
+  const int first = r0 - (taps - 1) > 0 ? r0 - (taps - 1) : 0;
+  float win[TP - 1][NG][4];                              // rows r - (TP - 1) .. r - 1
+#pragma unroll
+  for (int j = 0; j < TP - 1; ++j) {
+    const int r = first - (TP - 1) + j;                  // (rows of the step before `first` are not looked at)
+    const int e = taps - 1 + r;                          // state entry of a row before the step
+#pragma unroll
+    for (int g = 0; g < NG; ++g) {
+      const int i = (threadIdx.x + g * nt) * 4;
+      win[j][g][0] = win[j][g][1] = win[j][g][2] = win[j][g][3] = 0.0f;
+      if (r < 0 && e >= 0 && pos0 + r >= 0 && i < W) load4<float>(st + (size_t)e * W + i, win[j][g]);
+    }
+  }
+  int par = 0;
+  for (int rb = first; rb < r1; rb += R, par ^= 1) {
+    float v[R][NG][4], ss[R];
+#pragma unroll
+    for (int k = 0; k < R; ++k) {
+      const size_t row = (size_t)q0 + rb + k;
+#pragma unroll
+      for (int g = 0; g < NG; ++g) {
+        const int i = (threadIdx.x + g * nt) * 4;
+        v[k][g][0] = v[k][g][1] = v[k][g][2] = v[k][g][3] = 0.0f;
+        if (i < W && rb + k < r1) load4<float>(a.x_in + row * W + i, v[k][g]);
+      }
+    }
+    if constexpr (SRC == SRC_ROWS) {
+      float y[R][NG][4];
+#pragma unroll
+      for (int k = 0; k < R; ++k)
+#pragma unroll
+        for (int g = 0; g < NG; ++g) {
+          const int i = (threadIdx.x + g * nt) * 4;
+          y[k][g][0] = y[k][g][1] = y[k][g][2] = y[k][g][3] = 0.0f;
+          if (i < W && rb + k < r1)
+            load4<T>(static_cast<const T*>(a.y) + ((size_t)q0 + rb + k) * a.ldy + i, y[k][g]);
+        }
+#pragma unroll
+      for (int k = 0; k < R; ++k)
+#pragma unroll
+        for (int g = 0; g < NG; ++g) {
+          const int i = (threadIdx.x + g * nt) * 4;
+#pragma unroll
+          for (int c = 0; c < 4; ++c) v[k][g][c] += y[k][g][c];
+          if (i < W && rb + k < r1 && rb + k >= r0) put4<float>(a.x_out + ((size_t)q0 + rb + k) * W + i, v[k][g], 4, true);
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < R; ++k) {
+      ss[k] = 0.0f;
+#pragma unroll
+      for (int g = 0; g < NG; ++g)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) ss[k] += v[k][g][c] * v[k][g][c];
+      ss[k] = warp_sum(ss[k]);
+      if (lane == 0) red[par][k][warp] = ss[k];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < R; ++k)
+      ss[k] = 1.0f / sqrtf(warp_sum(lane < n_warps ? red[par][k][lane] : 0.0f) / (float)W + a.eps);
+#pragma unroll
+    for (int g = 0; g < NG; ++g) {
+      const int i = (threadIdx.x + g * nt) * 4;
+      if (i >= W) continue;
+      float w[4], co[TP][4];
+      load4<float>(a.w + i, w);
+#pragma unroll
+      for (int j = 0; j < TP; ++j) {
+        const int tap = j - (TP - taps);                 // negative: none
+        co[j][0] = co[j][1] = co[j][2] = co[j][3] = 0.0f;
+        if (tap >= 0) load4<float>(a.filt + (size_t)tap * W + i, co[j]);
+      }
+#pragma unroll
+      for (int k = 0; k < R; ++k) {
+        if (rb + k >= r1) break;
+        float acc[4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const float nv = v[k][g][c] * (ss[k] * w[c]);
+          acc[c] = nv + co[TP - 1][c] * nv;
+#pragma unroll
+          for (int j = 0; j < TP - 1; ++j) acc[c] += co[j][c] * win[j][g][c];
+#pragma unroll
+          for (int j = 0; j + 1 < TP - 1; ++j) win[j][g][c] = win[j + 1][g][c];
+          win[TP - 2][g][c] = nv;
+        }
+        if (rb + k >= r0) put4<T>(static_cast<T*>(a.h_out) + ((size_t)q0 + rb + k) * W + i, acc, 4, true);
+      }
+    }
+  }
+  if (a.write_state) {
+#pragma unroll
+    for (int j = 0; j < TP - 1; ++j) {
+      const int e = j - (TP - taps);
+      if (e < 0) continue;
+#pragma unroll
+      for (int g = 0; g < NG; ++g) {
+        const int i = (threadIdx.x + g * nt) * 4;
+        if (i < W) put4<float>(st + (size_t)e * W + i, win[j][g], 4, true);
+      }
+    }
+  }
+}
+
 template <typename T, int SRC>
 int launch_prenorm(PrenormArgs& a, int64_t rows, int64_t n_seq, int64_t q_max, cudaStream_t st) {
   if (!a.filt) {
@@ -201,13 +320,32 @@ int launch_prenorm(PrenormArgs& a, int64_t rows, int64_t n_seq, int64_t q_max, c
   if (smem > 48 * 1024)
     B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   // long chunks redo fewer rows, short ones fill the SMs
-  int chunk = rows >= 64 * sm_count() ? 16 : (rows >= 16 * sm_count() ? 8 : 4);
+  int chunk = rows >= 64 * sm_count() ? 29 : (rows >= 16 * sm_count() ? 13 : 5);
   if (q_max <= chunk) chunk = (int)q_max;
   const unsigned n_chunks = (unsigned)((q_max + chunk - 1) / chunk);
   a.chunk = chunk;
   a.carry = 0;
   a.write_state = a.taps > 1 && n_chunks == 1;
-  kern<<<dim3(n_chunks, (unsigned)n_seq), kPnThreads, smem, st>>>(a);
+  bool walked = false;
+  if constexpr (SRC != SRC_PARTIALS) {
+    const int groups = a.W / 4;
+    if (a.vec && a.taps <= 4 && groups <= 4 * 512) {
+      const int ng = groups <= 256 ? 1 : (groups <= 1024 ? 2 : 4);
+      const int threads = ((groups + ng - 1) / ng + 31) / 32 * 32;
+      const dim3 grid(n_chunks, (unsigned)n_seq);
+#define PN_WALK(TP)                                                                  \
+  do {                                                                               \
+    if (ng == 1) prenorm_walk_kernel<T, SRC, TP, 1, 4><<<grid, threads, 0, st>>>(a);     \
+    else if (ng == 2) prenorm_walk_kernel<T, SRC, TP, 2, 2><<<grid, threads, 0, st>>>(a); \
+    else prenorm_walk_kernel<T, SRC, TP, 4, 1><<<grid, threads, 0, st>>>(a);             \
+  } while (0)
+      if (a.taps <= 2) PN_WALK(2);
+      else PN_WALK(4);
+#undef PN_WALK
+      walked = true;
+    }
+  }
+  if (!walked) kern<<<dim3(n_chunks, (unsigned)n_seq), kPnThreads, smem, st>>>(a);
   B200_LAUNCH_OK("prenorm_filter_kernel");
   if (a.taps > 1 && n_chunks > 1) {
     // the last taps - 1 rows of every portion again, from the stored sums (the same numbers in the same order)
@@ -227,6 +365,13 @@ int dispatch_prenorm(PrenormArgs& a, int64_t rows, int64_t n_seq, int64_t q_max,
   if (a.partials) return launch_prenorm<T, SRC_PARTIALS>(a, rows, n_seq, q_max, st);
   if (a.y) return launch_prenorm<T, SRC_ROWS>(a, rows, n_seq, q_max, st);
   return launch_prenorm<T, SRC_NONE>(a, rows, n_seq, q_max, st);
+}
+
+// silu of an fp32 sum; where the result is rounded to 16 bits at once the fast exponential and division do
+template <typename T>
+__device__ __forceinline__ float silu_for(float x) {
+  if constexpr (sizeof(T) == 4) return x / (1.0f + expf(-x));
+  else return __fdividef(x, 1.0f + __expf(-x));
 }
 
 // ------------------------------------------------------------------------------------------------------------
@@ -282,7 +427,7 @@ causal_filter_kernel(T* __restrict__ out, int64_t ldo, const T* __restrict__ in,
       float acc = b[v];
 #pragma unroll
       for (int j = 0; j < TP; ++j) acc += co[j][v] * win[j][v];
-      o[v] = silu ? acc / (1.0f + expf(-acc)) : acc;
+      o[v] = silu ? silu_for<T>(acc) : acc;
 #pragma unroll
       for (int j = 0; j + 1 < TP; ++j) win[j][v] = win[j + 1][v];
     }

@@ -296,7 +296,10 @@ gated_part_norm_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict
     get4c<T>(z + row * ldz + i, zv, n - i, vec);
 #pragma unroll
     for (int k = 0; k < 4; ++k)
-      if (i + k < n) u_s[i + k] = yv[k] * zv[k] * sigmoid_f(zv[k]);
+      if (i + k < n) {
+        if constexpr (sizeof(T) == 4) u_s[i + k] = yv[k] * zv[k] * sigmoid_f(zv[k]);
+        else u_s[i + k] = yv[k] * __fdividef(zv[k], 1.0f + __expf(-zv[k]));
+      }
   }
   __syncthreads();
   const int ps = n / parts;
@@ -321,8 +324,14 @@ gated_part_norm_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict
   for (int i = threadIdx.x * 4; i < n; i += kPartThreads * 4) {
     float wv[4], o[4];
     get4c<float>(w + i, wv, n - i, vec);
+    if (ps % 4 == 0) {                                    // four channels of one part
+      const float r = r_s[i / ps * per];
+      const float4 u = *reinterpret_cast<const float4*>(u_s + i);
+      o[0] = u.x * r * wv[0]; o[1] = u.y * r * wv[1]; o[2] = u.z * r * wv[2]; o[3] = u.w * r * wv[3];
+    } else {
 #pragma unroll
-    for (int k = 0; k < 4; ++k) o[k] = i + k < n ? u_s[i + k] * r_s[(i + k) / ps * per] * wv[k] : 0.0f;
+      for (int k = 0; k < 4; ++k) o[k] = i + k < n ? u_s[i + k] * r_s[(i + k) / ps * per] * wv[k] : 0.0f;
+    }
     T* dst = out + row * ldo + i;
     if (vec) {
       if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);

@@ -22,7 +22,7 @@ Notation (W = width, norm(x, w) = x / sqrt(mean(x^2) + eps) * w):
     right       : q = silu(Wq h), f = l + (1 - l) sigmoid(Wf h + b), v = Wv h ; per head
                   S <- diag(f) S + (1 - f) v^T ; o = S^T q ; result Wo concat_h(norm(o, w))
     ff "dense"  : Wd (silu(Wg h) * (Wu h))
-    output      : embed norm(x, final)      (the embedding table itself, unscaled)
+    output      : embed norm(x, final)      (tied weights)
 """
 from __future__ import annotations
 

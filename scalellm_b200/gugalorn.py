@@ -11,7 +11,7 @@
                          gate
                  right — layers.ForgetWriteMixer: forget gate with a lower bound per channel, per-head norm of the read-out
     feed-forward: "dense" (layers.GatedMLP with silu)
-    output     : norm(x, "final.norm"), then the embedding table itself (unscaled) as the vocabulary projection.
+    output     : norm(x, "final.norm"), then the vocabulary projection with the weights of embed.
 
 Every size and constant is read from config.json or a tensor's shape.  Tensor names: "embed", "final.norm", and per
 layer i "l<i>.norm1|norm2|canon1", "l<i>.mix.in|conv|conv.b|dt_bias|A_log|D|norm|o" (mamba2),

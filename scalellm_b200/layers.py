@@ -1236,7 +1236,7 @@ class GroupLimitedMoE:
 
 # ---------------------------------------------------------------------------
 # Layers of pre-norm decoders whose mixers read their input through a short causal filter and mix tokens with a
-# state-space recurrence, or with softmax attention beside a recurrence whose forget gate also decides what is written.
+# state-space recurrence, or with softmax attention beside a recurrence that writes what it forgets.
 # ---------------------------------------------------------------------------
 class PreNormInput:
     """x <- x + y on an fp32 residual, then what the next sublayer reads: h = n = x / rms(x) * w, or with a filter
@@ -1298,7 +1298,7 @@ class TurnedSinkAttention:
 
 
 class ForgetWriteMixer:
-    """Linear recurrence whose forget gate also decides what is written (csrc/linear_scan.cu):
+    """Linear recurrence that writes in every key channel the share it forgets (csrc/linear_scan.cu):
         q = silu(Wq h), f = low + (1 - low) sigmoid(Wf h + b), v = Wv h ;
         S <- diag(f) S + (1 - f) v^T ; o = S^T q per head (S [dim, vdim], fp32, one per sequence slot) ;
         result = concat_h(o / rms(o) * norm) (before the output map, which belongs to the caller)."""

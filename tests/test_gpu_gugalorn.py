@@ -212,9 +212,11 @@ FORGET = [(3, 20, 12), (1, 9, 15), (2, 64, 64), (2, 128, 128), (1, 150, 136), (4
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,N,V", FORGET)
-def test_forget_gate_recurrence_over_portions(H, N, V, dtype):
+@pytest.mark.parametrize("form", ["", "simt"])
+def test_forget_gate_recurrence_over_portions(H, N, V, dtype, form, monkeypatch):
     """Gates from nearly all forgotten to nearly all kept, lower bounds at 0 and near 1; scaled into a column block."""
     from scalellm_b200 import kernels
+    monkeypatch.setenv("B200_SCAN_IMPL", form)                   # portions on the tensor cores where they fit, or never
     g = torch.Generator().manual_seed(H * N + V)
     fb, low = torch.randn(H * N, generator=g) * 3.0, torch.rand(H * N, generator=g) ** 0.3
     low[::5] = 0.0
@@ -249,8 +251,10 @@ SSD = [(6, 3, 24, 10), (1, 1, 18, 13), (4, 2, 64, 32), (2, 1, 128, 64), (2, 2, 1
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,G,N,V", SSD)
-def test_state_space_recurrence_over_portions(H, G, N, V, dtype):
+@pytest.mark.parametrize("form", ["", "simt"])
+def test_state_space_recurrence_over_portions(H, G, N, V, dtype, form, monkeypatch):
     from scalellm_b200 import kernels
+    monkeypatch.setenv("B200_SCAN_IMPL", form)
     g = torch.Generator().manual_seed(H * N + V)
     ch = H * V + 2 * G * N
     a_log, dtb, D = torch.log(0.05 + 8.0 * torch.rand(H, generator=g)), -4.0 + 5.0 * torch.rand(H, generator=g), torch.randn(H, generator=g)

@@ -85,7 +85,7 @@ def test_recurrences_by_hand():
     y = og.ssd_scan(x, B, torch.ones(2, 2, 1, dtype=torch.float64), dt, A, torch.tensor([0.0, 5.0], dtype=torch.float64), S)
     assert torch.allclose(y[:, 0, 0], torch.tensor([1.0, 1.5], dtype=torch.float64))
     assert torch.allclose(y[:, 1, 0], torch.tensor([25.0, 30.0], dtype=torch.float64))
-    # the gate comes before the norm, and every part has its own root mean square
+    # gated first, normalised after, part by part
     u = og.gated_part_norm(torch.tensor([[1.0, 1.0, 100.0, 100.0]], dtype=torch.float64),
                            torch.tensor([[5.0, 5.0, 1.0, 1.0]], dtype=torch.float64), torch.ones(4, dtype=torch.float64), 2, 0.0)
     assert torch.allclose(u, torch.ones(1, 4, dtype=torch.float64))

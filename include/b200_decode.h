@@ -626,6 +626,18 @@ B200_API int b200_mingru_scan_chunked(void* out, int64_t ldo, const void* proj, 
                                       const int32_t* q_cu_lens, const int32_t* positions, const int32_t* state_slots,
                                       int64_t n_seq, int64_t width, int64_t q_max, int64_t chunk_len, float* workspace,
                                       int64_t workspace_floats, int dtype, b200_stream_t stream);
+/* Real-gated linear recurrence per channel c of block b:  r = sigmoid(gates_r + r_bias), i = sigmoid(gates_i + i_bias) ;
+ * log a = rate * r * softplus(lam) ; S <- a S + sqrt(1 - a^2) i u (fp32, one value per slot and channel) ;
+ * out = S * gelu_tanh(y + y_bias).  u, y: rows of T; gates fp32 [blocks][rows][2 width / blocks], r before i; biases and
+ * lam fp32 [width].  chunk_len 0: one walk per sequence and channel; else portions in chunks side by side (workspace as
+ * ..._mingru_chunked_workspace_floats). */
+B200_API int b200_real_gated_scan(void* out, int64_t ldo, const void* u, int64_t ld_u, const void* y, int64_t ld_y,
+                                  const float* gates, int64_t rows, int64_t blocks, const float* r_bias,
+                                  const float* i_bias, const float* lam, const float* y_bias /*nullable*/, float rate,
+                                  float* state, const int32_t* q_cu_lens, const int32_t* positions,
+                                  const int32_t* state_slots, int64_t n_seq, int64_t width, int64_t q_max,
+                                  int64_t chunk_len, float* workspace /*nullable*/, int64_t workspace_floats, int dtype,
+                                  b200_stream_t stream);
 /* Differential attention, per token (see diff_attn.cu): RMS norm + rotation of the H * 2 query maps into q_out
  * (fp32 [rows, H, 2, dim]) and, when k_in is given, of the G * 2 key maps into k_cache[slot] ([slots, G, 2 * dim])
  * with v_in copied to v_cache[slot] ([slots, G, vdim]).  q_in / k_in / v_in: rows of stride ld. */
@@ -705,15 +717,28 @@ B200_API int b200_sink_attn_prepare_turned(float* q_out, const void* q_in, const
                                            const int32_t* positions, const int32_t* slots, int64_t rows, int64_t H,
                                            int64_t G, int64_t dim, int64_t vdim, int64_t rot_dims, float eps, int dtype,
                                            b200_stream_t stream);
+/* Per token, optional parts all nullable: q = q_in + q_bias, k = k_in + k_bias; per head q / sqrt(mean(q^2) + eps) *
+ * q_weight[dim], k likewise with k_weight; the half-pair turn of the entry above; q times 1 + temp_coef
+ * ln(floor((pos + 1) / temp_every) + 1) (temp_every 0: none).  q_out fp32 [rows, H, dim]; k, and v_in + v_bias where the
+ * projection has values, go to the cache rows `slots`. */
+B200_API int b200_sink_attn_prepare_heads(float* q_out, const void* q_in, const void* k_in, const void* v_in /*nullable*/,
+                                          int64_t ld, const float* q_bias /*nullable*/,
+                                          const float* k_bias /*nullable*/, const float* v_bias /*nullable*/,
+                                          const float* q_weight /*nullable*/, const float* k_weight /*nullable*/,
+                                          const float* inv_freq /*nullable*/, void* k_cache, void* v_cache /*nullable*/,
+                                          const int32_t* positions, const int32_t* slots, int64_t rows, int64_t H,
+                                          int64_t G, int64_t dim, int64_t vdim, int64_t rot_dims, float eps,
+                                          float temp_coef, int64_t temp_every, int dtype, b200_stream_t stream);
 /* out[row, h] = sum_j p_j v_j over the cached rows j <= position i of the row (paged), p_j = exp(s_j) /
  * (exp(sink[h]) + sum_j' exp(s_j')), s_j = scale q . k_j - r1[h] ln(1 + r2[h] (i - j)).  r1 / r2 (both or
  * neither) and sink are fp32 [H], nullable.  What is stored is out_mul * out * sigmoid(gate[row, h * vdim + c]) (gate:
- * rows of type T with stride ld_gate, nullable).  q fp32 [rows, H, dim]; caches [slots, G, dim] and [slots, G, vdim]
+ * rows of type T with stride ld_gate, nullable; gate_heads: gate[row, h], one number per head).  window > 0: only the keys
+ * j > i - window.  v_cache may be k_cache itself (dim == vdim: the values are the keys).  q fp32 [rows, H, dim]; caches [slots, G, dim] and [slots, G, vdim]
  * of type `dtype`; CUDA cores, any sizes. */
 B200_API int b200_sink_attn(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache,
                             const float* r1 /*nullable*/, const float* r2 /*nullable*/,
                             const float* sink /*nullable*/, const void* gate /*nullable*/, int64_t ld_gate,
-                            float out_mul, const int32_t* q_cu_lens, const int32_t* kv_cu_lens,
+                            float out_mul, int gate_heads, int64_t window, const int32_t* q_cu_lens, const int32_t* kv_cu_lens,
                             const int32_t* block_tables, const int32_t* cu_block_lens, const int32_t* token_seq,
                             int64_t rows, int64_t H, int64_t G, int64_t dim, int64_t vdim, int64_t block_size,
                             float scale, int dtype, b200_stream_t stream);
@@ -723,7 +748,7 @@ B200_API int b200_sink_attn_prefill_supported(int64_t dim, int64_t vdim, int dty
 B200_API int b200_sink_attn_prefill(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache,
                                     const float* r1 /*nullable*/, const float* r2 /*nullable*/,
                                     const float* sink /*nullable*/, const void* gate /*nullable*/, int64_t ld_gate,
-                                    float out_mul, const int32_t* q_cu_lens, const int32_t* kv_cu_lens, const int32_t* block_tables,
+                                    float out_mul, int gate_heads, int64_t window, const int32_t* q_cu_lens, const int32_t* kv_cu_lens, const int32_t* block_tables,
                                     const int32_t* cu_block_lens, int64_t n_seq, int64_t q_max, int64_t H, int64_t G,
                                     int64_t dim, int64_t vdim, int64_t block_size, float scale, int dtype,
                                     b200_stream_t stream);
@@ -735,7 +760,7 @@ B200_API int b200_sink_attn_prefill(void* out, int64_t ldo, const float* q, cons
 B200_API int b200_sink_attn_decode_tc(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache,
                                       const float* r1 /*nullable*/, const float* r2 /*nullable*/,
                                       const float* sink /*nullable*/, const void* gate /*nullable*/, int64_t ld_gate,
-                                      float out_mul, const int32_t* q_cu_lens, const int32_t* kv_cu_lens, const int32_t* block_tables,
+                                      float out_mul, int gate_heads, int64_t window, const int32_t* q_cu_lens, const int32_t* kv_cu_lens, const int32_t* block_tables,
                                       const int32_t* cu_block_lens, const int32_t* token_seq, int64_t rows, int64_t H,
                                       int64_t G, int64_t dim, int64_t vdim, int64_t block_size, float scale,
                                       int64_t n_splits, float* workspace /*nullable*/, int64_t workspace_floats,
@@ -816,6 +841,12 @@ B200_API int b200_moe_route_softmax(int32_t* expert_ids, float* weights, float* 
                                     const float* extra_weight /*nullable*/, int64_t rows, int64_t W, int64_t E,
                                     int64_t top, int64_t n_groups, int64_t keep_groups, float weight_eps, int dtype,
                                     b200_stream_t stream);
+/* The choice from router logits z (fp32 rows of stride ld): s = sigmoid(z) ; the E outputs form n_groups equal runs of
+ * neighbours, a run scores the sum of its group_best largest s, only outputs of the keep_groups best runs can be chosen ;
+ * the `top` largest s are chosen ; weights = factor * s / (sum of the chosen s + weight_eps). */
+B200_API int b200_moe_route_sigmoid(int32_t* expert_ids, float* weights, const float* logits, int64_t ld, int64_t rows,
+                                    int64_t E, int64_t top, int64_t n_groups, int64_t keep_groups, int64_t group_best,
+                                    float weight_eps, float factor, b200_stream_t stream);
 /* out[row] = sum_k pair_weights[row, k] * (expert_ids[row, k] < n_real ? Y[pos_of_pair[row, k]] : h[row])
  * (+ addend_gate[row] * addend[row]; gate nullable: 1). */
 B200_API int b200_moe_combine_weighted(void* out, const void* Y, int64_t ldy, const int32_t* pos_of_pair,
@@ -824,13 +855,14 @@ B200_API int b200_moe_combine_weighted(void* out, const void* Y, int64_t ldy, co
                                        const void* addend /*nullable*/, int64_t ld_add,
                                        const float* addend_gate /*nullable*/, int dtype, b200_stream_t stream);
 /* m = 1/2 (a / rms(a) * weight_a + b / rms(b) * weight_b), or m = a / rms(a) * weight_a without b, or m = a without
- * weight_a;  x_out = x_in + m / rms(m) * weight;  h_out (nullable) = x_out / rms(x_out) * weight_next as T, or x_out
+ * weight_a (bias_a, nullable, joins a first);  x_out = x_in + m / rms(m) * weight, or x_in + m without weight;  h_out (nullable) = x_out / rms(x_out) * weight_next as T, or x_out
  * as T without weight_next.  x fp32 [rows, W]; a, b of type T with row strides lda, ldb. */
 B200_API int b200_branch_norm_residual(float* x_out, void* h_out /*nullable*/, const float* x_in, const void* a,
-                                       int64_t lda, const void* b /*nullable*/, int64_t ldb,
-                                       const float* weight_a /*nullable*/, const float* weight_b /*nullable*/,
-                                       const float* weight, const float* weight_next /*nullable*/, int64_t rows,
-                                       int64_t W, float eps, int dtype, b200_stream_t stream);
+                                       int64_t lda, const float* bias_a /*nullable*/, const void* b /*nullable*/,
+                                       int64_t ldb, const float* weight_a /*nullable*/,
+                                       const float* weight_b /*nullable*/, const float* weight /*nullable*/,
+                                       const float* weight_next /*nullable*/, int64_t rows, int64_t W, float eps,
+                                       int dtype, b200_stream_t stream);
 /* out [rows, n] = max(in, 0)^2 for the first n columns of rows with stride ld_in. */
 B200_API int b200_relu_squared(void* out, const void* in, int64_t rows, int64_t n, int64_t ld_in, int dtype,
                                b200_stream_t stream);
@@ -841,20 +873,22 @@ B200_API int b200_relu_squared(void* out, const void* in, int64_t rows, int64_t 
  * first; q_max: the longest portion of the step; n_seq: its sequences. ---- */
 /* x_out = x_in + y ; n = x_out / sqrt(mean(x_out^2) + eps) * weight ; h_out[t] = n_t (filter null), or n_t +
  * sum_i filter[i] n_{t - (taps - 1) + i} per channel with zeros before the start of the sequence (filter [taps, W]).
- * y: rows of T (stride ldy), or the split-K partials [n_slots][rows][W] of the product that makes it (plan6:
+ * weight may be absent without a filter: h_out = x_out.  h_out: rows of stride ldh (W with a filter).
+ * y: rows of T (stride ldy; 0 without a filter: one row for all), or the split-K partials [n_slots][rows][W] of the product that makes it (plan6:
  * b200_dense_splitk_plan; their sum is rounded to T first), or neither (then x_in is normalised and x_out unused).
  * x_out must not be x_in. */
-B200_API int b200_prenorm(float* x_out /*nullable*/, void* h_out, const float* x_in, const void* y /*nullable*/,
-                          int64_t ldy, const float* partials /*nullable*/, int64_t n_slots,
-                          const int32_t* plan6 /*nullable*/, const float* weight, const float* filter /*nullable*/,
-                          int64_t taps, float* filter_state /*nullable*/, const int32_t* q_cu_lens /*nullable*/,
+B200_API int b200_prenorm(float* x_out /*nullable*/, void* h_out, int64_t ldh, const float* x_in,
+                          const void* y /*nullable*/, int64_t ldy, const float* partials /*nullable*/, int64_t n_slots,
+                          const int32_t* plan6 /*nullable*/, const float* weight /*nullable*/,
+                          const float* filter /*nullable*/, int64_t taps, float* filter_state /*nullable*/, const int32_t* q_cu_lens /*nullable*/,
                           const int32_t* positions /*nullable*/, const int32_t* state_slots /*nullable*/,
                           int64_t n_seq, int64_t q_max, int64_t rows, int64_t W, float eps, int dtype,
                           b200_stream_t stream);
-/* out_t = act(bias + sum_i filter[i] in_{t - (taps - 1) + i}) per channel; silu: 1 for act = silu, 0 for none.
- * filter [taps, channels]. */
+/* out_t = act(bias + sum_i filter[i] (in + in_bias)_{t - (taps - 1) + i}) per channel; silu: 1 for act = silu, 0 for none.
+ * filter [taps, channels]; the state keeps in + in_bias. */
 B200_API int b200_causal_filter(void* out, int64_t ldo, const void* in, int64_t ld, const float* filter,
-                                const float* bias /*nullable*/, int64_t taps, float* filter_state /*nullable*/,
+                                const float* in_bias /*nullable*/, const float* bias /*nullable*/, int64_t taps,
+                                float* filter_state /*nullable*/,
                                 const int32_t* q_cu_lens, const int32_t* positions, const int32_t* state_slots,
                                 int64_t n_seq, int64_t q_max, int64_t rows, int64_t channels, int silu, int dtype,
                                 b200_stream_t stream);
@@ -880,10 +914,21 @@ B200_API int b200_ssd_scan(float* y, const void* x, const void* B, const void* C
                            const int32_t* q_cu_lens, const int32_t* positions, const int32_t* state_slots,
                            int64_t n_seq, int64_t q_max, int64_t rows, int64_t H, int64_t G, int64_t N, int64_t V,
                            int tensor_cores, int dtype, b200_stream_t stream);
-/* u = y silu(z) ; out = u / sqrt(mean_part(u^2) + eps) * weight, the row of n channels in `parts` equal parts.  y fp32
- * [rows, n]; z rows of T (stride ldz).  bf16 or fp32. */
+/* Matrix memory with exponential gates, per head and token (S [N x V] in state[slot, h], n [N] and m in key_sum, fp32):
+ * f = log sigmoid(cap tanh((f_logits + f_bias) / cap)), i = cap tanh((i_logits + i_bias) / cap) ; m' = max(f + m, i) from
+ * m = 0 ; (S, n) <- exp(f + m - m') (S, n) + exp(i - m') k (v^T, 1) ; q' = q_scale q ;
+ * y[row, h] = S^T q' / (max(|n . q'|, exp(-m')) + 1e-6)  (fp32 [rows, H * V]).  q / k / v: column blocks of one matrix
+ * (row stride ld); gate logits fp32, rows of stride ld_g, [H]; key_sum [slot][H][b200_linear_scan_parts][N + 1]. */
+B200_API int b200_memory_scan(float* y, const void* q, const void* k, const void* v, int64_t ld, const float* i_logits,
+                              const float* f_logits, int64_t ld_g, const float* i_bias, const float* f_bias, float cap,
+                              float q_scale, float* state, float* key_sum, const int32_t* q_cu_lens,
+                              const int32_t* positions, const int32_t* state_slots, int64_t n_seq, int64_t q_max,
+                              int64_t rows, int64_t H, int64_t N, int64_t V, int tensor_cores, int dtype,
+                              b200_stream_t stream);
+/* u = y silu(z) ; out = u / sqrt(mean_part(u^2) + eps) * weight, the row of n channels in `parts` equal parts; with
+ * gate_after u = y and out is multiplied by sigmoid(z).  y fp32 [rows, n]; z rows of T (stride ldz).  bf16 or fp32. */
 B200_API int b200_gated_part_norm(void* out, int64_t ldo, const float* y, const void* z, int64_t ldz,
-                                  const float* weight, int64_t rows, int64_t n, int64_t parts, float eps, int dtype,
+                                  const float* weight, int64_t rows, int64_t n, int64_t parts, float eps, int gate_after, int dtype,
                                   b200_stream_t stream);
 
 #ifdef __cplusplus

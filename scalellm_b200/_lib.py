@@ -136,6 +136,8 @@ SIGNATURES = {
     "b200_mingru_chunked_workspace_floats": (_i64, [_i64, _i64, _i64, _i64]),
     "b200_mingru_scan_chunked": (_int, [_vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _vp,
                                         _i64, _int, _vp]),
+    "b200_real_gated_scan": (_int, [_vp, _i64, _vp, _i64, _vp, _i64, _vp, _i64, _i64, _vp, _vp, _vp, _vp, _f32, _vp, _vp,
+                                    _vp, _vp, _i64, _i64, _i64, _i64, _vp, _i64, _int, _vp]),
     "b200_diff_attn_prepare": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _f32, _vp, _vp, _i64, _i64,
                                       _i64, _i64, _i64, _i64, _f32, _int, _vp]),
     "b200_diff_attn": (_int, [_vp, _i64, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64,
@@ -155,13 +157,15 @@ SIGNATURES = {
                                       _i64, _i64, _f32, _f32, _i64, _int, _vp]),
     "b200_sink_attn_prepare_turned": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64,
                                              _i64, _i64, _i64, _i64, _f32, _int, _vp]),
-    "b200_sink_attn": (_int, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _f32, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64,
-                              _i64, _i64, _f32, _int, _vp]),
+    "b200_sink_attn_prepare_heads": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp,
+                                            _i64, _i64, _i64, _i64, _i64, _i64, _f32, _f32, _i64, _int, _vp]),
+    "b200_sink_attn": (_int, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _f32, _int, _i64, _vp, _vp, _vp, _vp, _vp,
+                              _i64, _i64, _i64, _i64, _i64, _i64, _f32, _int, _vp]),
     "b200_sink_attn_prefill_supported": (_int, [_i64, _i64, _int]),
-    "b200_sink_attn_decode_tc": (_int, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _f32, _vp, _vp, _vp, _vp, _vp, _i64, _i64,
-                                        _i64, _i64, _i64, _i64, _f32, _i64, _vp, _i64, _int, _vp]),
-    "b200_sink_attn_prefill": (_int, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _f32, _vp, _vp, _vp, _vp, _i64, _i64, _i64,
-                                      _i64, _i64, _i64, _i64, _f32, _int, _vp]),
+    "b200_sink_attn_decode_tc": (_int, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _f32, _int, _i64, _vp, _vp, _vp,
+                                        _vp, _vp, _i64, _i64, _i64, _i64, _i64, _i64, _f32, _i64, _vp, _i64, _int, _vp]),
+    "b200_sink_attn_prefill": (_int, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _f32, _int, _i64, _vp, _vp, _vp,
+                                      _vp, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _f32, _int, _vp]),
     # sigmoid attention in blocks of positions with a head mix, gated delta rule with input filters, softmax router
     # with group limits, branch norms (sigmoid_attn.cu, delta_rule.cu, moe.cu, postnorm.cu)
     "b200_sigmoid_attn_prepare": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64,
@@ -178,15 +182,16 @@ SIGNATURES = {
                                      _i64, _i64, _i64, _i64, _f32, _vp, _i64, _int, _vp]),
     "b200_moe_route_softmax": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _i64, _i64,
                                       _f32, _int, _vp]),
+    "b200_moe_route_sigmoid": (_int, [_vp, _vp, _vp, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _f32, _f32, _vp]),
     "b200_moe_combine_weighted": (_int, [_vp, _vp, _i64, _vp, _vp, _vp, _i64, _vp, _i64, _i64, _i64, _i64, _vp, _i64,
                                          _vp, _int, _vp]),
-    "b200_branch_norm_residual": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i64, _f32,
+    "b200_branch_norm_residual": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i64, _f32,
                                          _int, _vp]),
     "b200_relu_squared": (_int, [_vp, _vp, _i64, _i64, _i64, _int, _vp]),
     # pre-norm input side with short causal filters, linear recurrences with a matrix state (filters.cu, linear_scan.cu)
-    "b200_prenorm": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i64,
+    "b200_prenorm": (_int, [_vp, _vp, _i64, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i64,
                             _i64, _i64, _f32, _int, _vp]),
-    "b200_causal_filter": (_int, [_vp, _i64, _vp, _i64, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _int,
+    "b200_causal_filter": (_int, [_vp, _i64, _vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _int,
                                   _int, _vp]),
     "b200_linear_scan_parts": (_int, [_i64, _i64]),
     "b200_linear_scan_tc_supported": (_int, [_i64, _i64, _int]),
@@ -194,7 +199,9 @@ SIGNATURES = {
                                 _i64, _i64, _i64, _f32, _f32, _vp, _int, _int, _vp]),
     "b200_ssd_scan": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64,
                              _i64, _i64, _i64, _i64, _int, _int, _vp]),
-    "b200_gated_part_norm": (_int, [_vp, _i64, _vp, _vp, _i64, _vp, _i64, _i64, _i64, _f32, _int, _vp]),
+    "b200_memory_scan": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _vp, _i64, _vp, _vp, _f32, _f32, _vp, _vp, _vp, _vp, _vp,
+                                _i64, _i64, _i64, _i64, _i64, _i64, _int, _int, _vp]),
+    "b200_gated_part_norm": (_int, [_vp, _i64, _vp, _vp, _i64, _vp, _i64, _i64, _i64, _f32, _int, _int, _vp]),
 }
 
 # Which source files a partial library needs for a group of entry points.  The whole library

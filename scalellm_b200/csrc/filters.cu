@@ -2,8 +2,8 @@
 //
 //   prenorm : x' = x + y (y: the result of the sublayer before, optional) ; n = x' / sqrt(mean(x'^2) + eps) * w ;
 //             h = n, or with an input filter  h_t = n_t + sum_i c[i] n_{t - (taps - 1) + i}   per channel, zeros before
-//             the start of the sequence: residual sum, norm and filter in one launch
-//   filter  : out = act(b + sum_i c[i] in_{t - (taps - 1) + i})                               act: none or silu
+//             the start of the sequence: residual sum, norm and filter in one launch.  Without w: h = x' itself.
+//   filter  : out = act(b + sum_i c[i] (in + in_bias)_{t - (taps - 1) + i})                   act: none or silu
 //
 // The residual, norms, filter sums and filter states are fp32; T is the activation type of y, in, h and out.  Per
 // sequence slot a filter keeps its last taps - 1 inputs [slot, taps - 1, channels] (fp32).  A portion that starts at
@@ -48,13 +48,14 @@ __device__ __forceinline__ void put4(T* __restrict__ p, const float (&v)[4], int
 struct PrenormArgs {
   float* x_out;            // nullable (no y, or nobody needs the sum)
   void* h_out;
+  int64_t ldh;
   const float* x_in;
-  const void* y;           // SRC_ROWS: rows of T with stride ldy
+  const void* y;           // SRC_ROWS: rows of T with stride ldy (0: the same row for all)
   int64_t ldy;
   const float* partials;   // SRC_PARTIALS: fp32 [slots][rows][W]
   int64_t slot_stride;
   W4Plan plan;
-  const float* w;
+  const float* w;          // nullable without a filter: no norm
   const float* filt;       // [taps][W], oldest tap first
   float* state;            // [slot][taps - 1][W]
   const int *q_cu, *positions, *state_slots;
@@ -111,13 +112,15 @@ __global__ void __launch_bounds__(kPnThreads) prenorm_kernel(const PrenormArgs a
   const size_t row = blockIdx.x;
   const float ss = block_sum<kPnThreads>(residual_row<T, SRC>(a, sm, row, a.x_out != nullptr), red);
   const float r = 1.0f / sqrtf(ss / (float)a.W + a.eps);
-  T* h = static_cast<T*>(a.h_out) + row * a.W;
+  T* h = static_cast<T*>(a.h_out) + row * a.ldh;
   for (int i = threadIdx.x * 4; i < a.W; i += kPnThreads * 4) {
     float v[4], w[4];
     get4<float>(sm + i, v, a.W - i, a.vec);
-    get4<float>(a.w + i, w, a.W - i, a.vec);
+    if (a.w) {
+      get4<float>(a.w + i, w, a.W - i, a.vec);
 #pragma unroll
-    for (int k = 0; k < 4; ++k) v[k] *= r * w[k];
+      for (int k = 0; k < 4; ++k) v[k] *= r * w[k];
+    }
     put4<T>(h + i, v, a.W - i, a.vec);
   }
 }
@@ -383,8 +386,8 @@ constexpr int kFiThreads = 128;
 template <typename T, int TP, int V>
 __global__ void __launch_bounds__(kFiThreads)
 causal_filter_kernel(T* __restrict__ out, int64_t ldo, const T* __restrict__ in, int64_t ld,
-                     const float* __restrict__ filt, const float* __restrict__ bias, float* __restrict__ state,
-                     const int* __restrict__ q_cu, const int* __restrict__ positions,
+                     const float* __restrict__ filt, const float* __restrict__ in_bias, const float* __restrict__ bias,
+                     float* __restrict__ state, const int* __restrict__ q_cu, const int* __restrict__ positions,
                      const int* __restrict__ state_slots, int C, int taps, int chunk, int silu, int write_state) {
   const int seq = blockIdx.z;
   const int q0 = q_cu[seq], n = q_cu[seq + 1] - q0;
@@ -395,7 +398,9 @@ causal_filter_kernel(T* __restrict__ out, int64_t ldo, const T* __restrict__ in,
   if (c0 >= C) return;
   const int pos0 = positions[q0];
   float* st = state + (size_t)state_slots[seq] * (taps - 1) * C + c0;
-  float win[TP][V], co[TP][V], b[V];                     // win[0]: the oldest
+  float win[TP][V], co[TP][V], b[V], ib[V];              // win[0]: the oldest
+#pragma unroll
+  for (int v = 0; v < V; ++v) ib[v] = in_bias ? in_bias[c0 + v] : 0.0f;
 #pragma unroll
   for (int j = 0; j < TP; ++j) {
     const int tap = j - (TP - taps);                     // filter column; negative: none
@@ -406,7 +411,7 @@ causal_filter_kernel(T* __restrict__ out, int64_t ldo, const T* __restrict__ in,
     for (int v = 0; v < V; ++v) {
       win[j][v] = 0.0f;
       if (tap >= 0 && j < TP - 1 && pos0 + r >= 0)
-        win[j][v] = r >= 0 ? Num<T>::to_f(in[(size_t)(q0 + r) * ld + c0 + v]) : st[(size_t)(taps - 1 + r) * C + v];
+        win[j][v] = r >= 0 ? Num<T>::to_f(in[(size_t)(q0 + r) * ld + c0 + v]) + ib[v] : st[(size_t)(taps - 1 + r) * C + v];
     }
   }
 #pragma unroll
@@ -418,9 +423,9 @@ causal_filter_kernel(T* __restrict__ out, int64_t ldo, const T* __restrict__ in,
       float x[4];
       load4<T>(in + (size_t)(q0 + r) * ld + c0, x);
 #pragma unroll
-      for (int v = 0; v < 4; ++v) win[TP - 1][v] = x[v];
+      for (int v = 0; v < 4; ++v) win[TP - 1][v] = x[v] + ib[v];
     } else {
-      win[TP - 1][0] = Num<T>::to_f(in[(size_t)(q0 + r) * ld + c0]);
+      win[TP - 1][0] = Num<T>::to_f(in[(size_t)(q0 + r) * ld + c0]) + ib[0];
     }
 #pragma unroll
     for (int v = 0; v < V; ++v) {
@@ -453,6 +458,7 @@ causal_filter_kernel(T* __restrict__ out, int64_t ldo, const T* __restrict__ in,
 // state[slot, e] <- the input at in-step row n - (taps - 1) + e, or the old entry e + n where that is before the step
 template <typename T>
 __global__ void causal_filter_carry_kernel(float* __restrict__ state, const T* __restrict__ in, int64_t ld,
+                                           const float* __restrict__ in_bias,
                                            const int* __restrict__ q_cu, const int* __restrict__ positions,
                                            const int* __restrict__ state_slots, int C, int taps) {
   const int seq = blockIdx.y;
@@ -465,27 +471,27 @@ __global__ void causal_filter_carry_kernel(float* __restrict__ state, const T* _
   for (int e = 0; e < taps - 1; ++e) {                   // ascending: entry e reads entry e + n > e of the old state
     const int r = n - (taps - 1) + e;
     float v = 0.0f;
-    if (r >= 0) v = Num<T>::to_f(in[(size_t)(q0 + r) * ld + c]);
+    if (r >= 0) v = Num<T>::to_f(in[(size_t)(q0 + r) * ld + c]) + (in_bias ? in_bias[c] : 0.0f);
     else if (pos0 + r >= 0) v = st[(size_t)(e + n) * C];
     st[(size_t)e * C] = v;
   }
 }
 
 template <typename T, int TP, int V>
-int launch_filter(void* out, int64_t ldo, const void* in, int64_t ld, const float* filt, const float* bias,
-                  float* state, const int* q_cu, const int* positions, const int* slots, int64_t rows, int64_t n_seq,
+int launch_filter(void* out, int64_t ldo, const void* in, int64_t ld, const float* filt, const float* in_bias,
+                  const float* bias, float* state, const int* q_cu, const int* positions, const int* slots, int64_t rows, int64_t n_seq,
                   int64_t q_max, int C, int taps, int silu, cudaStream_t st) {
   const unsigned cy = (unsigned)((C + kFiThreads * V - 1) / (kFiThreads * V));
   int chunk = rows * cy >= 64 * sm_count() * 4 ? 32 : 8;
   if (q_max <= chunk) chunk = (int)q_max;
   const unsigned n_chunks = (unsigned)((q_max + chunk - 1) / chunk);
   causal_filter_kernel<T, TP, V><<<dim3(n_chunks, cy, (unsigned)n_seq), kFiThreads, 0, st>>>(
-      static_cast<T*>(out), ldo, static_cast<const T*>(in), ld, filt, bias, state, q_cu, positions, slots, C, taps, chunk,
+      static_cast<T*>(out), ldo, static_cast<const T*>(in), ld, filt, in_bias, bias, state, q_cu, positions, slots, C, taps, chunk,
       silu, taps > 1 && n_chunks == 1);
   B200_LAUNCH_OK("causal_filter_kernel");
   if (taps > 1 && n_chunks > 1) {
     causal_filter_carry_kernel<T><<<dim3((unsigned)((C + 255) / 256), (unsigned)n_seq), 256, 0, st>>>(
-        state, static_cast<const T*>(in), ld, q_cu, positions, slots, C, taps);
+        state, static_cast<const T*>(in), ld, in_bias, q_cu, positions, slots, C, taps);
     B200_LAUNCH_OK("causal_filter_carry_kernel");
   }
   return B200_OK;
@@ -506,13 +512,14 @@ using namespace b200;
 
 extern "C" {
 
-int b200_prenorm(float* x_out, void* h_out, const float* x_in, const void* y, int64_t ldy, const float* partials,
+int b200_prenorm(float* x_out, void* h_out, int64_t ldh, const float* x_in, const void* y, int64_t ldy, const float* partials,
                  int64_t n_slots, const int32_t* plan6, const float* weight, const float* filter, int64_t taps,
                  float* filter_state, const int32_t* q_cu_lens, const int32_t* positions, const int32_t* state_slots,
                  int64_t n_seq, int64_t q_max, int64_t rows, int64_t W, float eps, int dtype, b200_stream_t stream) {
   if (rows == 0) return B200_OK;
-  B200_CHECK_ARG(h_out && x_in && weight, "prenorm: null pointer");
-  B200_CHECK_ARG(rows > 0 && W > 0 && !(y && partials) && (!y || ldy >= W) && (W + 4) * 4 <= 200 * 1024,
+  B200_CHECK_ARG(h_out && x_in && (weight || !filter), "prenorm: null pointer");
+  B200_CHECK_ARG(rows > 0 && W > 0 && !(y && partials) && (!y || ldy >= W || (ldy == 0 && !filter)) &&
+                     (filter ? ldh == W : ldh >= W) && (W + 4) * 4 <= 200 * 1024,
                  "prenorm: bad shape (at most ~50K channels), or rows and partials both given");
   B200_CHECK_ARG(!(y || partials) || (x_out && x_out != x_in), "prenorm: the sum goes to a buffer of its own");
   B200_CHECK_ARG(!partials || (plan6 && W % 8 == 0 && n_slots == plan6[4] && n_slots <= W4_MAX_SLOTS &&
@@ -524,7 +531,7 @@ int b200_prenorm(float* x_out, void* h_out, const float* x_in, const void* y, in
                  "prenorm: bad filter (1 to 16 taps, taps * channels at most ~50K)");
   PrenormArgs a{};
   a.x_out = (y || partials) ? x_out : nullptr;
-  a.h_out = h_out; a.x_in = x_in; a.y = y; a.ldy = ldy; a.partials = partials; a.slot_stride = rows * W;
+  a.h_out = h_out; a.ldh = ldh; a.x_in = x_in; a.y = y; a.ldy = ldy; a.partials = partials; a.slot_stride = rows * W;
   if (plan6 && partials) {
     a.plan.units = plan6[0]; a.plan.P = plan6[1]; a.plan.KT = plan6[2]; a.plan.NT = plan6[3]; a.plan.slots = plan6[4];
     a.plan.nsub_log2 = plan6[5];
@@ -532,15 +539,15 @@ int b200_prenorm(float* x_out, void* h_out, const float* x_in, const void* y, in
   a.w = weight; a.filt = filter; a.state = filter_state; a.q_cu = q_cu_lens; a.positions = positions;
   a.state_slots = state_slots; a.W = (int)W; a.taps = (int)taps; a.eps = eps;
   a.vec = W % 4 == 0 && is_aligned(x_in, 16) && (!a.x_out || is_aligned(x_out, 16)) && is_aligned(h_out, 16) &&
-          (!y || (ldy % 4 == 0 && is_aligned(y, 16))) && is_aligned(weight, 16) &&
+          ldh % 4 == 0 && (!y || (ldy % 4 == 0 && is_aligned(y, 16))) && (!weight || is_aligned(weight, 16)) &&
           (!filter || (is_aligned(filter, 16) && (taps == 1 || is_aligned(filter_state, 16))));
   auto st = static_cast<cudaStream_t>(stream);
   FILTERS_DISPATCH(dtype, return dispatch_prenorm<T>(a, rows, n_seq, q_max, st));
   return B200_OK;
 }
 
-int b200_causal_filter(void* out, int64_t ldo, const void* in, int64_t ld, const float* filter, const float* bias,
-                       int64_t taps, float* filter_state, const int32_t* q_cu_lens, const int32_t* positions,
+int b200_causal_filter(void* out, int64_t ldo, const void* in, int64_t ld, const float* filter,
+                       const float* in_bias, const float* bias, int64_t taps, float* filter_state, const int32_t* q_cu_lens, const int32_t* positions,
                        const int32_t* state_slots, int64_t n_seq, int64_t q_max, int64_t rows, int64_t channels, int silu,
                        int dtype, b200_stream_t stream) {
   if (rows == 0 || n_seq == 0) return B200_OK;
@@ -553,7 +560,7 @@ int b200_causal_filter(void* out, int64_t ldo, const void* in, int64_t ld, const
   const size_t esz = dtype == B200_FP32 ? 4 : 2;
   const bool vec = channels % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 && is_aligned(in, 4 * esz) && is_aligned(out, 4 * esz);
 #define CF_CALL(TP, V)                                                                                          \
-  return (launch_filter<T, TP, V>(out, ldo, in, ld, filter, bias, filter_state, q_cu_lens, positions, state_slots, \
+  return (launch_filter<T, TP, V>(out, ldo, in, ld, filter, in_bias, bias, filter_state, q_cu_lens, positions, state_slots, \
                                   rows, n_seq, q_max, (int)channels, (int)taps, silu, st))
   FILTERS_DISPATCH(dtype, {
     if (vec) {

@@ -6,6 +6,9 @@
 //            out = mul * o / sqrt(mean_head(o^2) + eps) * w                              (what is forgotten is written)
 //   ssd    : a = exp(-exp(A_h) d) for the whole head, k = d B, q = C (one B, C per group of heads),
 //            d = softplus(dl + bias_h);  y = o + D_h v                                   (state-space duality form)
+//   memory : f = log sigmoid(cap tanh((fl + bf_h) / cap)), i = cap tanh((il + bi_h) / cap), m' = max(f + m, i) from m = 0 ;
+//            a = exp(f + m - m'), k = exp(i - m') kl, q = c ql ; a sum of keys n <- a n + k goes along ;
+//            y = o / (max(|n . q|, exp(-m')) + 1e-6)                                     (matrix memory with exponential gates)
 //
 // The elements of S do not meet except in o's sum over the key channels, so a thread keeps a tile of RL key rows x 4
 // value columns in registers (packed pairs of key rows: two multiply-adds an instruction) and LP neighbouring lanes
@@ -15,6 +18,9 @@
 // A portion that starts at position 0 starts from S = 0 instead of reading the slot.
 //
 //   part_norm : out = u / sqrt(mean_part(u^2) + eps) * w, u = y silu(z), the row in equal parts    (after the ssd walk)
+//               or u = y and sigmoid(z) on the way out                                             (after the memory walk)
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace b200 {
@@ -23,8 +29,16 @@ namespace {
 constexpr int kScanTokens = 16;
 constexpr int kScanWarps = 8;
 
-enum { MODE_FORGET = 0, MODE_SSD = 1 };
+constexpr float kMemoryDenEps = 1e-6f;
 
+enum { MODE_FORGET = 0, MODE_SSD = 1, MODE_MEMORY = 2 };
+
+// Column parts a head is walked in (the walk on CUDA cores).
+__host__ __device__ constexpr int scan_col_parts(int N, int V) {
+  const int lp = N <= 128 ? 4 : (N <= 256 ? 8 : 16);
+  const int warps = (V + 128 / lp - 1) / (128 / lp);
+  return (warps + kScanWarps - 1) / kScanWarps;
+}
 typedef unsigned long long f32x2;
 __device__ __forceinline__ f32x2 pack2(float lo, float hi) {
   f32x2 r;
@@ -49,6 +63,7 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
+__device__ __forceinline__ float log_sigmoid_f(float x) { return fminf(x, 0.0f) - log1pf(expf(-fabsf(x))); }
 
 template <typename T>
 struct ScanArgs {
@@ -61,6 +76,11 @@ struct ScanArgs {
   const T* dt;
   int64_t ld_dt;
   const float *dt_bias, *a_log, *skip;
+  const float *gi, *gf;    // memory: gate logits, fp32 rows of stride ld_g; one bias per head each
+  int64_t ld_g;
+  const float *gi_bias, *gf_bias;
+  float cap, q_scale;
+  float* key_sum;          // memory: [slot][H][column part][N + 1]: n, then m (one copy per column part of the walk)
   float* state;            // [slot][H][N][V]
   const int *q_cu, *positions, *state_slots;
   int H, G, N, V, CB, chunk;
@@ -86,8 +106,9 @@ linear_scan_kernel(const ScanArgs<T> a) {
   const int CH = a.chunk, CBP = (int)(blockDim.x >> 5) * (128 / LP);
   float* k_s = sm;                                        // [CH][NP]
   float* q_s = k_s + CH * NP;                             // [CH][NP]
-  float* a_s = q_s + CH * NP;                             // forget: [CH][NP]; ssd: [CH] (rounded up to 4)
-  float* v_s = a_s + (MODE == MODE_FORGET ? CH * NP : (CH + 3) / 4 * 4);   // [CH][CBP]
+  float* a_s = q_s + CH * NP;                             // forget: [CH][NP]; ssd: [CH]; memory: log gates f, i [2][CH4]
+  const int CH4 = (CH + 3) / 4 * 4;
+  float* v_s = a_s + (MODE == MODE_FORGET ? CH * NP : (MODE == MODE_MEMORY ? 2 * CH4 : CH4));   // [CH][CBP]
   float* o_s = v_s + CH * CBP;                            // [CH][CBP]
   const int seq = blockIdx.x, h = blockIdx.y, cb0 = (int)blockIdx.z * a.CB;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
@@ -108,6 +129,18 @@ linear_scan_kernel(const ScanArgs<T> a) {
     raw[i][0] = raw[i][1] = raw[i][2] = raw[i][3] = 0.0f;
     if (!fresh && c0 < ncol && n < N) get4c<float>(Sg + (size_t)n * V + c0, raw[i], ncol - c0, a.vec_state);
   }
+  float* key_sum = nullptr;
+  float m = 0.0f;
+  float raw_n[MODE == MODE_MEMORY ? RL : 1];
+  if constexpr (MODE == MODE_MEMORY) {
+    key_sum = a.key_sum + (((size_t)a.state_slots[seq] * a.H + h) * gridDim.z + blockIdx.z) * (N + 1);
+    if (!fresh) m = key_sum[N];
+#pragma unroll
+    for (int i = 0; i < RL; ++i) {
+      const int n = p * 4 + (i / 4) * 4 * LP + (i & 3);
+      raw_n[i] = !fresh && n < N ? key_sum[n] : 0.0f;
+    }
+  }
   const int g = MODE == MODE_SSD ? h / (a.H / a.G) : h;
   float neg_a = 0.0f, dbias = 0.0f, skip = 0.0f;
   if constexpr (MODE == MODE_SSD) {
@@ -124,6 +157,13 @@ linear_scan_kernel(const ScanArgs<T> a) {
       if constexpr (MODE == MODE_SSD) {
         dt = softplus_f(Num<T>::to_f(a.dt[row * a.ld_dt + h]) + dbias);
         if (lane == 0) a_s[tok] = expf(neg_a * dt);
+      }
+      if constexpr (MODE == MODE_MEMORY) {
+        if (lane < 2) {
+          const float z = lane == 0 ? a.gf[row * a.ld_g + h] + a.gf_bias[h] : a.gi[row * a.ld_g + h] + a.gi_bias[h];
+          const float t = a.cap * tanhf(z / a.cap);
+          a_s[lane * CH4 + tok] = lane == 0 ? log_sigmoid_f(t) : t;
+        }
       }
       for (int c = lane * 4; c < NP; c += 128) {
         float qv[4] = {0.0f, 0.0f, 0.0f, 0.0f}, kv[4] = {0.0f, 0.0f, 0.0f, 0.0f}, av[4] = {0.0f, 0.0f, 0.0f, 0.0f};
@@ -142,7 +182,7 @@ linear_scan_kernel(const ScanArgs<T> a) {
                 kv[i] = (1.0f - l) * (z >= 0.0f ? small : big);
                 qv[i] = qv[i] * sigmoid_f(qv[i]);
               }
-            } else {
+            } else if constexpr (MODE == MODE_SSD) {
               kv[i] *= dt;
             }
           }
@@ -166,6 +206,11 @@ linear_scan_kernel(const ScanArgs<T> a) {
   for (int i = 0; i < RL / 2; ++i)
 #pragma unroll
     for (int c = 0; c < 4; ++c) S[i][c] = pack2(raw[2 * i][c], raw[2 * i + 1][c]);
+  f32x2 n2[MODE == MODE_MEMORY ? RL / 2 : 1];             // every column group keeps the sum of keys of its rows
+  if constexpr (MODE == MODE_MEMORY) {
+#pragma unroll
+    for (int i = 0; i < RL / 2; ++i) n2[i] = pack2(raw_n[2 * i], raw_n[2 * i + 1]);
+  }
   for (int tc = t0; tc < t1; tc += CH) {
     const int nt = t1 - tc < CH ? t1 - tc : CH;
     if (tc != t0) {
@@ -174,13 +219,21 @@ linear_scan_kernel(const ScanArgs<T> a) {
     }
     __syncthreads();
     for (int tok = 0; tok < nt; ++tok) {
-      const float4 vv = *reinterpret_cast<const float4*>(v_s + tok * CBP + c0);
+      float4 vv = *reinterpret_cast<const float4*>(v_s + tok * CBP + c0);
+      f32x2 da = 0ull, w2 = 0ull, nq2 = 0ull;
+      if constexpr (MODE == MODE_SSD) da = pack2(a_s[tok], a_s[tok]);
+      if constexpr (MODE == MODE_MEMORY) {
+        const float fm = a_s[tok] + m, li = a_s[CH4 + tok];
+        m = fmaxf(fm, li);
+        const float keep = expf(fm - m), write = expf(li - m);
+        da = pack2(keep, keep);
+        w2 = pack2(write, write);
+        vv.x *= write; vv.y *= write; vv.z *= write; vv.w *= write;
+      }
       const f32x2 v2[4] = {pack2(vv.x, vv.x), pack2(vv.y, vv.y), pack2(vv.z, vv.z), pack2(vv.w, vv.w)};
       f32x2 o2[4];
 #pragma unroll
       for (int c = 0; c < 4; ++c) o2[c] = 0ull;
-      f32x2 da = 0ull;
-      if constexpr (MODE == MODE_SSD) da = pack2(a_s[tok], a_s[tok]);
 #pragma unroll
       for (int i = 0; i < RL / 4; ++i) {
         const int n0 = tok * NP + p * 4 + i * 4 * LP;
@@ -195,6 +248,12 @@ linear_scan_kernel(const ScanArgs<T> a) {
           o2[c] = fma2(S[i * 2][c], q2.x, o2[c]);
           S[i * 2 + 1][c] = fma2(f2.y, S[i * 2 + 1][c], mul2(k2.y, v2[c]));
           o2[c] = fma2(S[i * 2 + 1][c], q2.y, o2[c]);
+        }
+        if constexpr (MODE == MODE_MEMORY) {
+          n2[i * 2] = fma2(da, n2[i * 2], mul2(k2.x, w2));
+          nq2 = fma2(n2[i * 2], q2.x, nq2);
+          n2[i * 2 + 1] = fma2(da, n2[i * 2 + 1], mul2(k2.y, w2));
+          nq2 = fma2(n2[i * 2 + 1], q2.y, nq2);
         }
       }
       float o[4];
@@ -213,6 +272,13 @@ linear_scan_kernel(const ScanArgs<T> a) {
       r += __shfl_xor_sync(0xffffffffu, s, 2);
 #pragma unroll
       for (int d = 4; d < LP; d <<= 1) r += __shfl_xor_sync(0xffffffffu, r, d);
+      if constexpr (MODE == MODE_MEMORY) {
+        const float2 t = unpack2(nq2);
+        float nq = t.x + t.y;
+#pragma unroll
+        for (int d = 1; d < LP; d <<= 1) nq += __shfl_xor_sync(0xffffffffu, nq, d);
+        r = r * a.q_scale / (fmaxf(fabsf(nq * a.q_scale), expf(-m)) + kMemoryDenEps);
+      }
       if (p < 4) o_s[tok * CBP + c0 + (b0 ? 2 : 0) + (b1 ? 1 : 0)] = r;
     }
     __syncthreads();
@@ -222,7 +288,7 @@ linear_scan_kernel(const ScanArgs<T> a) {
       if constexpr (MODE == MODE_SSD) {
         float* dst = a.raw + row * (size_t)a.H * V + (size_t)h * V + cb0;
         for (int c = lane; c < ncol; c += 32) dst[c] = ot[c] + skip * v_s[tok * CBP + c];
-      } else if (a.raw) {
+      } else if (MODE == MODE_MEMORY || a.raw) {
         float* dst = a.raw + row * (size_t)a.H * V + (size_t)h * V + cb0;
         for (int c = lane; c < ncol; c += 32) dst[c] = ot[c];
       } else {
@@ -232,6 +298,18 @@ linear_scan_kernel(const ScanArgs<T> a) {
         const float inv = a.mul / sqrtf(ss / (float)V + a.eps);
         T* dst = a.out + row * a.ldo + (size_t)h * V;
         for (int c = lane; c < V; c += 32) dst[c] = Num<T>::from_f(ot[c] * inv * a.norm_w[c]);
+      }
+    }
+  }
+  if constexpr (MODE == MODE_MEMORY) {
+    if (cq == 0) {                                        // LP threads, each with the rows of its p
+      if (p == 0) key_sum[N] = m;
+#pragma unroll
+      for (int i = 0; i < RL / 2; ++i) {
+        const int n = p * 4 + (i / 2) * 4 * LP + (i & 1) * 2;
+        const float2 t = unpack2(n2[i]);
+        if (n < N) key_sum[n] = t.x;
+        if (n + 1 < N) key_sum[n + 1] = t.y;
       }
     }
   }
@@ -277,10 +355,10 @@ head_norm_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict__ raw
   for (int i = lane; i < V; i += 32) out[(size_t)row * ldo + (size_t)h * V + i] = Num<T>::from_f(r[i] * inv * w[i]);
 }
 
-// out = u / sqrt(mean_part(u^2) + eps) * w, u = y silu(z); one CTA per row, the row in `parts` equal parts.  With
-// fewer parts than warps several warps share a part.
+// out = u / sqrt(mean_part(u^2) + eps) * w, u = y silu(z), or (GATE_AFTER) out = y / sqrt(mean_part(y^2) + eps) * w *
+// sigmoid(z); one CTA per row, the row in `parts` equal parts.  With fewer parts than warps several warps share a part.
 constexpr int kPartThreads = 256;
-template <typename T>
+template <typename T, bool GATE_AFTER>
 __global__ void __launch_bounds__(kPartThreads)
 gated_part_norm_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict__ y, const T* __restrict__ z,
                        int64_t ldz, const float* __restrict__ w, int n, int parts, float eps, int vec) {
@@ -293,11 +371,12 @@ gated_part_norm_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict
   for (int i = threadIdx.x * 4; i < n; i += kPartThreads * 4) {
     float yv[4], zv[4];
     get4c<float>(y + row * n + i, yv, n - i, vec);
-    get4c<T>(z + row * ldz + i, zv, n - i, vec);
+    if constexpr (!GATE_AFTER) get4c<T>(z + row * ldz + i, zv, n - i, vec);
 #pragma unroll
     for (int k = 0; k < 4; ++k)
       if (i + k < n) {
-        if constexpr (sizeof(T) == 4) u_s[i + k] = yv[k] * zv[k] * sigmoid_f(zv[k]);
+        if constexpr (GATE_AFTER) u_s[i + k] = yv[k];
+        else if constexpr (sizeof(T) == 4) u_s[i + k] = yv[k] * zv[k] * sigmoid_f(zv[k]);
         else u_s[i + k] = yv[k] * __fdividef(zv[k], 1.0f + __expf(-zv[k]));
       }
   }
@@ -332,6 +411,15 @@ gated_part_norm_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict
 #pragma unroll
       for (int k = 0; k < 4; ++k) o[k] = i + k < n ? u_s[i + k] * r_s[(i + k) / ps * per] * wv[k] : 0.0f;
     }
+    if constexpr (GATE_AFTER) {
+      float zv[4];
+      get4c<T>(z + row * ldz + i, zv, n - i, vec);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        if constexpr (sizeof(T) == 4) o[k] *= sigmoid_f(zv[k]);
+        else o[k] = __fdividef(o[k], 1.0f + __expf(-zv[k]));
+      }
+    }
     T* dst = out + row * ldo + i;
     if (vec) {
       if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
@@ -344,12 +432,6 @@ gated_part_norm_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict
   }
 }
 
-int scan_col_parts(int N, int V) {
-  const int lp = N <= 128 ? 4 : (N <= 256 ? 8 : 16);
-  const int warps = (V + 128 / lp - 1) / (128 / lp);
-  return (warps + kScanWarps - 1) / kScanWarps;
-}
-
 template <typename T, int MODE, int RL, int LP>
 int launch_scan_n(ScanArgs<T>& a, int64_t n_seq, int64_t q_max, cudaStream_t st) {
   constexpr int CW = 128 / LP;                            // columns of a warp
@@ -360,7 +442,8 @@ int launch_scan_n(ScanArgs<T>& a, int64_t n_seq, int64_t q_max, cudaStream_t st)
   a.chunk = q_max < kScanTokens ? (int)q_max : kScanTokens;
   constexpr int NP = RL * LP;
   const size_t smem = ((size_t)a.chunk * (NP * (MODE == MODE_FORGET ? 3 : 2) + 2 * a.CB) +
-                       (MODE == MODE_FORGET ? 0 : (a.chunk + 3) / 4 * 4)) * sizeof(float);
+                       (MODE == MODE_FORGET ? 0 : (a.chunk + 3) / 4 * 4 * (MODE == MODE_MEMORY ? 2 : 1))) *
+                      sizeof(float);
   auto kern = linear_scan_kernel<T, MODE, RL, LP>;
   if (smem > 48 * 1024)
     B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
@@ -388,6 +471,11 @@ int launch_scan(ScanArgs<T>& a, int64_t n_seq, int64_t q_max, cudaStream_t st) {
 // they are.
 //   ssd    : with c_i = sum_{t <= i} log a_t inside the tile,  o_i = exp(c_i) (C_i . S) + sum_{j <= i} (C_i . B_j)
 //            exp(c_i - c_j) d_j x_j ;  S <- exp(c_last) S + sum_j exp(c_last - c_j) d_j B_j x_j^T    (exponents <= 0)
+//   memory : with F_t = sum of the tile's log forget gates up to t, u_t = i_t - F_t and M_t = max(m, u_1 .. u_t) the running
+//            maximum is m_t = F_t + M_t, the decay since the tile's start exp(m - M_t) and the weight of token j in row t
+//            exp(u_j - M_t) (exponents <= 0): the ssd form with other exponents.  n rides along in shared memory: n . q
+//            of the state before the tile is 16 dot products shared out over the CTA, the tile's own part the sum of a
+//            row of weighted scores
 //   forget : everything relative to the middle of the tile, per key channel: with r_t the product of the gates between
 //            token t and the middle, q and k become q / r, k r before it and q r, k / r after it; S is decayed to the
 //            middle, o = q . S + (masked q k^T) v, S <- S + k v^T, and S is decayed to the end.  Where a product of a
@@ -721,10 +809,10 @@ forget_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
     }
 }
 
-// A tile's C, B and x rows are copied one tile ahead (two buffers); its decay exponents are worked out one tile ahead by
+// The ssd walk, and (MEM) the matrix memory's with C = q, B = k, x = v.  A tile's C, B and x rows are copied one tile ahead (two buffers); its decay exponents are worked out one tile ahead by
 // one warp, which takes turns.
-template <int KN, int MT>
-__global__ void __launch_bounds__(MT == 1 ? 128 : kScanWarps * 32, MT == 1 ? 3 : 1)
+template <int KN, int MT, bool MEM>
+__global__ void __launch_bounds__(MT == 1 ? 128 : kScanWarps * 32, MT == 1 ? (MEM ? 2 : 3) : 1)
 ssd_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
   using bf16 = __nv_bfloat16;
   constexpr int NP = 16 * KN, NS = TileRows<KN>::NS, PIECES = NP / 8;
@@ -733,14 +821,25 @@ ssd_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
   bf16* cb_s = reinterpret_cast<bf16*>(smraw);            // [2 buffers][C, B][16][NS]
   bf16* k_s = cb_s + 4 * kTile * NS;                      // [hi, lo][16][NS]: B with its step size and decay to the end
   bf16* v_s = k_s + 2 * kTile * NS;                       // [2 buffers][16][VS]
-  float* e_s = reinterpret_cast<float*>(v_s + 2 * kTile * VS);   // [2 buffers][c_i | d_i | d_i exp(c_last - c_i)][16]
+  float* e_s = reinterpret_cast<float*>(v_s + 2 * kTile * VS);   // ssd: [2 buffers][c_i | d_i | d_i exp(c_last - c_i)][16]
+  constexpr int ES = MEM ? 5 : 3;                         // memory: [2][M_i | u_i | exp(u_i - M_last) | exp(-m_i) | m, m'][16]
+  float* n_s = e_s + 2 * ES * kTile;                      // memory: [NP] the sum of keys before the tile
+  float* nq_s = n_s + NP;                                 // memory: [16] its products with the tile's queries
   const int seq = blockIdx.x, h = blockIdx.y, g = h / (a.H / a.G);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
   const int t0 = a.q_cu[seq], t1 = a.q_cu[seq + 1];
   if (t0 >= t1) return;
   const int gr = lane >> 2, qc = (lane & 3) * 2;
   const int v0 = warp * 16 * MT;                          // this warp's value rows v0 .. v0 + 16 MT - 1
-  const float neg_a = -expf(a.a_log[h]), dbias = a.dt_bias[h], skip = a.skip[h];
+  float neg_a = 0.0f, dbias = 0.0f, skip = 0.0f, ibias = 0.0f;
+  if constexpr (MEM) {
+    dbias = a.gf_bias[h];
+    ibias = a.gi_bias[h];
+  } else {
+    neg_a = -expf(a.a_log[h]);
+    dbias = a.dt_bias[h];
+    skip = a.skip[h];
+  }
   const int n_tiles = (t1 - t0 + kTile - 1) / kTile;
   const bf16* cg = a.q + (size_t)g * N;
   const bf16* bg = a.k + (size_t)g * N;
@@ -767,9 +866,44 @@ ssd_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
   };
   auto load_dt = [&](int it) {                            // lane t holds token t of the tile (-inf: no step)
     const int t = t0 + it * kTile + lane;
-    return lane < kTile && t < t1 ? Num<bf16>::to_f(a.dt[(size_t)t * a.ld_dt + h]) + dbias : -INFINITY;
+    const bool ok = lane < kTile && t < t1;
+    if constexpr (MEM)
+      return make_float2(ok ? a.gf[(size_t)t * a.ld_g + h] + dbias : -INFINITY,
+                         ok ? a.gi[(size_t)t * a.ld_g + h] + ibias : 0.0f);
+    else
+      return ok ? Num<bf16>::to_f(a.dt[(size_t)t * a.ld_dt + h]) + dbias : -INFINITY;
   };
-  auto exponents = [&](int it, float z) {
+  using Gate = typename std::conditional<MEM, float2, float>::type;
+  auto exponents_mem = [&](int it, float2 z, float m) {   // m: the running maximum before the tile
+    const bool ok = z.x != -INFINITY;
+    const float ft = a.cap * tanhf((ok ? z.x : 0.0f) / a.cap), iv = a.cap * tanhf(z.y / a.cap);
+    float F = ok ? log_sigmoid_f(ft) : 0.0f;
+#pragma unroll
+    for (int s = 1; s < kTile; s <<= 1) {
+      const float up = __shfl_up_sync(0xffffffffu, F, s);
+      if (lane >= s) F += up;
+    }
+    const float u = ok ? iv - F : -INFINITY;
+    float M = fmaxf(m, u);
+#pragma unroll
+    for (int s = 1; s < kTile; s <<= 1) {
+      const float up = __shfl_up_sync(0xffffffffu, M, s);
+      if (lane >= s) M = fmaxf(M, up);
+    }
+    const float M_last = __shfl_sync(0xffffffffu, M, kTile - 1);
+    if (lane < kTile) {
+      float* e = e_s + (it & 1) * ES * kTile;
+      e[lane] = M;
+      e[kTile + lane] = u;
+      e[2 * kTile + lane] = expf(u - M_last);
+      e[3 * kTile + lane] = expf(-(F + M));
+      if (lane == kTile - 1) {
+        e[4 * kTile] = m;
+        e[4 * kTile + 1] = F + M;
+      }
+    }
+  };
+  auto exponents_ssd = [&](int it, float z) {
     const float d = z == -INFINITY ? 0.0f : softplus_f(z);
     float c = neg_a * d;
 #pragma unroll
@@ -779,16 +913,23 @@ ssd_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
     }
     const float c_last = __shfl_sync(0xffffffffu, c, kTile - 1);
     if (lane < kTile) {
-      float* e = e_s + (it & 1) * 3 * kTile;
+      float* e = e_s + (it & 1) * ES * kTile;
       e[lane] = c;
       e[kTile + lane] = d;
       e[2 * kTile + lane] = d * expf(c_last - c);
     }
   };
   copy_tile(0);
-  if (warp == 0) exponents(0, load_dt(0));
-  float* Sg = a.state + (((size_t)a.state_slots[seq] * a.H + h) * N) * V;
   const bool fresh = a.positions[t0] == 0;
+  float* key_sum = nullptr;
+  if constexpr (MEM) {
+    key_sum = a.key_sum + ((size_t)a.state_slots[seq] * a.H + h) * scan_col_parts(N, V) * (N + 1);
+    if (warp == 0) exponents_mem(0, load_dt(0), fresh ? 0.0f : key_sum[N]);
+    for (int i = threadIdx.x; i < NP; i += blockDim.x) n_s[i] = !fresh && i < N ? key_sum[i] : 0.0f;
+  } else {
+    if (warp == 0) exponents_ssd(0, load_dt(0));
+  }
+  float* Sg = a.state + (((size_t)a.state_slots[seq] * a.H + h) * N) * V;
   float S[MT][2 * KN][4];
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
@@ -807,13 +948,13 @@ ssd_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
     cp_async_wait_all();
     __syncthreads();                                       // tile `it` stands; everyone is done with the tile before
     const bool ahead = it + 1 < n_tiles, mine = ahead && it % n_warps == warp;
-    float z = -INFINITY;
+    Gate z{};
     if (ahead) copy_tile(it + 1);
     if (mine) z = load_dt(it + 1);
     const bf16* c_t = cb_s + buf * 2 * kTile * NS;
     const bf16* b_t = c_t + kTile * NS;
     const bf16* v_t = v_s + buf * kTile * VS;
-    const float* e = e_s + buf * 3 * kTile;
+    const float* e = e_s + buf * ES * kTile;
     for (int x = threadIdx.x; x < kTile * PIECES; x += blockDim.x) {
       const int t = x / PIECES, ch = (x % PIECES) * 8;
       const uint4 raw = *reinterpret_cast<const uint4*>(b_t + t * NS + ch);
@@ -827,6 +968,20 @@ ssd_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
       }
       *reinterpret_cast<uint4*>(k_s + t * NS + ch) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
       *reinterpret_cast<uint4*>(k_s + (kTile + t) * NS + ch) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
+    if constexpr (MEM) {
+      // n . q: eight lanes a token
+      for (int t = threadIdx.x >> 3; t < kTile; t += blockDim.x >> 3) {
+        float s = 0.0f;
+        for (int c = (threadIdx.x & 7) * 2; c < NP; c += 16) {
+          const float2 qv = Num<bf16>::unpack(*reinterpret_cast<const uint32_t*>(c_t + t * NS + c));
+          const float2 nv = *reinterpret_cast<const float2*>(n_s + c);
+          s += qv.x * nv.x + qv.y * nv.y;
+        }
+#pragma unroll
+        for (int d = 1; d < 8; d <<= 1) s += __shfl_xor_sync(0xffffffffu, s, d);
+        if ((threadIdx.x & 7) == 0) nq_s[t] = s;
+      }
     }
     // ---- read-outs: C . S and the scores C . B
     float sc[2][4], y[MT * 2][4];
@@ -853,7 +1008,17 @@ ssd_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
         }
     }
     const float ci[2] = {e[gr], e[gr + 8]};
-    const float gi[2] = {__expf(ci[0]), __expf(ci[1])}, c_end = __expf(e[kTile - 1]);
+    float gi[2], c_end, rs[2] = {0.0f, 0.0f};               // rs: row sums of the weighted scores
+    if constexpr (MEM) {
+      const float m = e[4 * kTile];
+      gi[0] = expf(m - ci[0]);
+      gi[1] = expf(m - ci[1]);
+      c_end = expf(m - e[kTile - 1]);
+    } else {
+      gi[0] = __expf(ci[0]);
+      gi[1] = __expf(ci[1]);
+      c_end = __expf(e[kTile - 1]);
+    }
 #pragma unroll
     for (int i = 0; i < MT * 2; ++i) { y[i][0] *= gi[0]; y[i][1] *= gi[0]; y[i][2] *= gi[1]; y[i][3] *= gi[1]; }
 #pragma unroll
@@ -863,8 +1028,13 @@ ssd_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
 #pragma unroll
       for (int r = 0; r < 4; ++r) {
         const int i = gr + (r >> 1) * 8, j = n * 8 + qc + (r & 1);
-        const float w = __expf(ci[r >> 1] - (r & 1 ? cj.y : cj.x)) * (r & 1 ? dj.y : dj.x);
-        sc[n][r] = j <= i ? sc[n][r] * w : 0.0f;
+        if constexpr (MEM) {
+          sc[n][r] = j <= i ? sc[n][r] * expf((r & 1 ? dj.y : dj.x) - ci[r >> 1]) : 0.0f;
+          rs[r >> 1] += sc[n][r];
+        } else {
+          const float w = __expf(ci[r >> 1] - (r & 1 ? cj.y : cj.x)) * (r & 1 ? dj.y : dj.x);
+          sc[n][r] = j <= i ? sc[n][r] * w : 0.0f;
+        }
       }
     }
     uint32_t ph[4], pl[4];
@@ -887,22 +1057,44 @@ ssd_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
       }
     }
     const int tc = t0 + it * kTile;
+    auto write_out = [&]() {
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      const int t = gr + r * 8;
-      if (tc + t < t1) {
-        float* dst = a.raw + ((size_t)(tc + t) * a.H + h) * V + v0 + qc;
-        const bf16* xr = v_t + t * VS + v0 + qc;
+      for (int r = 0; r < 2; ++r) {
+        const int t = gr + r * 8;
+        float f = 1.0f;
+        if constexpr (MEM) {
+          rs[r] += __shfl_xor_sync(0xffffffffu, rs[r], 1);
+          rs[r] += __shfl_xor_sync(0xffffffffu, rs[r], 2);
+          f = a.q_scale / (fmaxf(fabsf((gi[r] * nq_s[t] + rs[r]) * a.q_scale), e[3 * kTile + t]) + kMemoryDenEps);
+        }
+        if (tc + t < t1) {
+          float* dst = a.raw + ((size_t)(tc + t) * a.H + h) * V + v0 + qc;
+          const bf16* xr = v_t + t * VS + v0 + qc;
 #pragma unroll
-        for (int i = 0; i < MT * 2; ++i)
-          if (v0 + i * 8 < V) {
-            const float2 x = Num<bf16>::unpack(*reinterpret_cast<const uint32_t*>(xr + i * 8));
-            *reinterpret_cast<float2*>(dst + i * 8) = make_float2(y[i][2 * r] + skip * x.x, y[i][2 * r + 1] + skip * x.y);
-          }
+          for (int i = 0; i < MT * 2; ++i)
+            if (v0 + i * 8 < V) {
+              if constexpr (MEM) {
+                *reinterpret_cast<float2*>(dst + i * 8) = make_float2(y[i][2 * r] * f, y[i][2 * r + 1] * f);
+              } else {
+                const float2 x = Num<bf16>::unpack(*reinterpret_cast<const uint32_t*>(xr + i * 8));
+                *reinterpret_cast<float2*>(dst + i * 8) = make_float2(y[i][2 * r] + skip * x.x, y[i][2 * r + 1] + skip * x.y);
+              }
+            }
+        }
+      }
+    };
+    if constexpr (!MEM) write_out();
+    // ---- the new state
+    __syncthreads();                                       // k_s stands (memory: and n . q)
+    if constexpr (MEM) {
+      write_out();
+      for (int c = threadIdx.x; c < NP; c += blockDim.x) {
+        float n = n_s[c] * c_end;
+#pragma unroll 4
+        for (int t = 0; t < kTile; ++t) n += Num<bf16>::to_f(b_t[t * NS + c]) * e[2 * kTile + t];
+        n_s[c] = n;
       }
     }
-    // ---- the new state
-    __syncthreads();                                       // k_s stands
 #pragma unroll
     for (int ks = 0; ks < KN; ++ks) {
       uint32_t b[4], bl[4];
@@ -921,7 +1113,19 @@ ssd_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
         mma_bf16(S[mt][2 * ks + 1], va[mt], bl[2], bl[3]);
       }
     }
-    if (mine) exponents(it + 1, z);
+    if (mine) {
+      if constexpr (MEM) exponents_mem(it + 1, z, e[4 * kTile + 1]);
+      else exponents_ssd(it + 1, z);
+    }
+  }
+  if constexpr (MEM) {
+    __syncthreads();                                       // n stands
+    const float* e = e_s + ((n_tiles - 1) & 1) * ES * kTile;
+    const int parts = scan_col_parts(N, V);                // every copy: a walk of another form may follow
+    for (int i = threadIdx.x; i < parts * (N + 1); i += blockDim.x) {
+      const int c = i % (N + 1);
+      key_sum[i] = c < N ? n_s[c] : e[4 * kTile + 1];
+    }
   }
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
@@ -935,16 +1139,18 @@ ssd_scan_tc_kernel(const ScanArgs<__nv_bfloat16> a) {
 }
 
 template <int KN, int MT>
-int launch_tc_n(bool forget, const ScanArgs<__nv_bfloat16>& a, int64_t n_seq, cudaStream_t st) {
+int launch_tc_n(int mode, const ScanArgs<__nv_bfloat16>& a, int64_t n_seq, cudaStream_t st) {
   const int warps = (a.V + 16 * MT - 1) / (16 * MT);
   constexpr int NS = TileRows<KN>::NS;
   size_t smem;
-  if (forget)
+  if (mode == MODE_FORGET)
     smem = (size_t)(4 * kTile * (NS + 16 * KN) + 2 * kTile * (a.V + 8)) * sizeof(__nv_bfloat16) +
            (size_t)(5 * 16 * KN + kTile * (a.V + 4)) * sizeof(float);
   else
-    smem = (size_t)(6 * kTile * NS + 2 * kTile * (a.V + 8)) * sizeof(__nv_bfloat16) + 6 * kTile * sizeof(float);
-  auto kern = forget ? forget_scan_tc_kernel<KN, MT> : ssd_scan_tc_kernel<KN, MT>;
+    smem = (size_t)(6 * kTile * NS + 2 * kTile * (a.V + 8)) * sizeof(__nv_bfloat16) +
+           (mode == MODE_SSD ? 6 * kTile : 11 * kTile + 16 * KN) * sizeof(float);
+  auto kern = mode == MODE_FORGET ? forget_scan_tc_kernel<KN, MT>
+                                  : (mode == MODE_SSD ? ssd_scan_tc_kernel<KN, MT, false> : ssd_scan_tc_kernel<KN, MT, true>);
   if (smem > 48 * 1024)
     B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   kern<<<dim3((unsigned)n_seq, (unsigned)a.H), warps * 32, smem, st>>>(a);
@@ -952,13 +1158,13 @@ int launch_tc_n(bool forget, const ScanArgs<__nv_bfloat16>& a, int64_t n_seq, cu
   return B200_OK;
 }
 
-int launch_scan_tc(bool forget, const ScanArgs<__nv_bfloat16>& a, int64_t n_seq, cudaStream_t st) {
+int launch_scan_tc(int mode, const ScanArgs<__nv_bfloat16>& a, int64_t n_seq, cudaStream_t st) {
   const bool two = a.V > 64;                              // 16 value rows a warp, or 32
-  if (a.N <= 32) return two ? launch_tc_n<2, 2>(forget, a, n_seq, st) : launch_tc_n<2, 1>(forget, a, n_seq, st);
-  if (a.N <= 64) return two ? launch_tc_n<4, 2>(forget, a, n_seq, st) : launch_tc_n<4, 1>(forget, a, n_seq, st);
-  return two ? launch_tc_n<8, 2>(forget, a, n_seq, st) : launch_tc_n<8, 1>(forget, a, n_seq, st);
+  if (a.N <= 32) return two ? launch_tc_n<2, 2>(mode, a, n_seq, st) : launch_tc_n<2, 1>(mode, a, n_seq, st);
+  if (a.N <= 64) return two ? launch_tc_n<4, 2>(mode, a, n_seq, st) : launch_tc_n<4, 1>(mode, a, n_seq, st);
+  return two ? launch_tc_n<8, 2>(mode, a, n_seq, st) : launch_tc_n<8, 1>(mode, a, n_seq, st);
 }
-int launch_scan_tc(bool, const ScanArgs<float>&, int64_t, cudaStream_t) {
+int launch_scan_tc(int, const ScanArgs<float>&, int64_t, cudaStream_t) {
   return set_error(B200_ERR_UNSUPPORTED, "linear_scan: the tensor-core form takes bf16");
 }
 
@@ -1011,7 +1217,7 @@ int b200_forget_scan(void* out, int64_t ldo, const void* q, const void* f, const
     a.vec_in = N % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && is_aligned(q, 4 * sizeof(T)) && is_aligned(f, 4 * sizeof(T)) &&
                is_aligned(v, 4 * sizeof(T));
     a.vec_state = V % 4 == 0 && is_aligned(state, 16);
-    if (tensor_cores) return launch_scan_tc(true, a, n_seq, st);
+    if (tensor_cores) return launch_scan_tc(MODE_FORGET, a, n_seq, st);
     const int rc = launch_scan<T, MODE_FORGET>(a, n_seq, q_max, st);
     if (rc != B200_OK) return rc;
     if (raw) {
@@ -1048,14 +1254,47 @@ int b200_ssd_scan(float* y, const void* x, const void* B, const void* Cm, int64_
     a.vec_in = N % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && is_aligned(x, 4 * sizeof(T)) && is_aligned(B, 4 * sizeof(T)) &&
                is_aligned(Cm, 4 * sizeof(T));
     a.vec_state = V % 4 == 0 && is_aligned(state, 16);
-    if (tensor_cores) return launch_scan_tc(false, a, n_seq, st);
+    if (tensor_cores) return launch_scan_tc(MODE_SSD, a, n_seq, st);
     return (launch_scan<T, MODE_SSD>(a, n_seq, q_max, st));
   });
   return B200_OK;
 }
 
+int b200_memory_scan(float* y, const void* q, const void* k, const void* v, int64_t ld, const float* i_logits,
+                     const float* f_logits, int64_t ld_g, const float* i_bias, const float* f_bias, float cap,
+                     float q_scale, float* state, float* key_sum, const int32_t* q_cu_lens, const int32_t* positions,
+                     const int32_t* state_slots, int64_t n_seq, int64_t q_max, int64_t rows, int64_t H, int64_t N,
+                     int64_t V, int tensor_cores, int dtype, b200_stream_t stream) {
+  if (rows == 0 || n_seq == 0) return B200_OK;
+  B200_CHECK_ARG(y && q && k && v && i_logits && f_logits && i_bias && f_bias && state && key_sum && q_cu_lens &&
+                     positions && state_slots,
+                 "memory_scan: null pointer");
+  B200_CHECK_ARG(rows > 0 && n_seq > 0 && q_max > 0 && H > 0 && H <= 65535 && N > 0 && N <= 512 && V > 0 && V <= 4096 &&
+                     ld >= H * (N > V ? N : V) && ld_g >= H && cap > 0.0f,
+                 "memory_scan: bad shape (key size <= 512)");
+  B200_CHECK_ARG(!tensor_cores || (scan_tc_fits(N, V, dtype) && ld % 8 == 0 && is_aligned(q, 16) && is_aligned(k, 16) &&
+                                   is_aligned(v, 16) && is_aligned(y, 8)),
+                 "memory_scan: sizes or alignment do not fit the tensor-core tiles");
+  auto st = static_cast<cudaStream_t>(stream);
+  SCAN_DISPATCH(dtype, {
+    ScanArgs<T> a{};
+    a.raw = y;
+    a.q = static_cast<const T*>(q); a.k = static_cast<const T*>(k); a.v = static_cast<const T*>(v); a.ld = ld;
+    a.gi = i_logits; a.gf = f_logits; a.ld_g = ld_g; a.gi_bias = i_bias; a.gf_bias = f_bias; a.cap = cap;
+    a.q_scale = q_scale; a.key_sum = key_sum;
+    a.state = state; a.q_cu = q_cu_lens; a.positions = positions; a.state_slots = state_slots;
+    a.H = (int)H; a.G = (int)H; a.N = (int)N; a.V = (int)V; a.mul = 1.0f;
+    a.vec_in = N % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && is_aligned(q, 4 * sizeof(T)) && is_aligned(k, 4 * sizeof(T)) &&
+               is_aligned(v, 4 * sizeof(T));
+    a.vec_state = V % 4 == 0 && is_aligned(state, 16);
+    if (tensor_cores) return launch_scan_tc(MODE_MEMORY, a, n_seq, st);
+    return (launch_scan<T, MODE_MEMORY>(a, n_seq, q_max, st));
+  });
+  return B200_OK;
+}
+
 int b200_gated_part_norm(void* out, int64_t ldo, const float* y, const void* z, int64_t ldz, const float* weight,
-                         int64_t rows, int64_t n, int64_t parts, float eps, int dtype, b200_stream_t stream) {
+                         int64_t rows, int64_t n, int64_t parts, float eps, int gate_after, int dtype, b200_stream_t stream) {
   if (rows == 0) return B200_OK;
   B200_CHECK_ARG(out && y && z && weight, "gated_part_norm: null pointer");
   B200_CHECK_ARG(rows > 0 && n > 0 && parts > 0 && n % parts == 0 && ldo >= n && ldz >= n && (n + parts + 16) * 4 <= 200 * 1024,
@@ -1065,11 +1304,11 @@ int b200_gated_part_norm(void* out, int64_t ldo, const float* y, const void* z, 
   SCAN_DISPATCH(dtype, {
     const int vec = n % 4 == 0 && ldo % 4 == 0 && ldz % 4 == 0 && is_aligned(out, 4 * sizeof(T)) &&
                     is_aligned(z, 4 * sizeof(T)) && is_aligned(y, 16) && is_aligned(weight, 16);
+    auto kern = gate_after ? gated_part_norm_kernel<T, true> : gated_part_norm_kernel<T, false>;
     if (smem > 48 * 1024)
-      B200_CUDA_OK(cudaFuncSetAttribute(gated_part_norm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    gated_part_norm_kernel<T><<<(unsigned)rows, kPartThreads, smem, st>>>(static_cast<T*>(out), ldo, y,
-                                                                          static_cast<const T*>(z), ldz, weight, (int)n,
-                                                                          (int)parts, eps, vec);
+      B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    kern<<<(unsigned)rows, kPartThreads, smem, st>>>(static_cast<T*>(out), ldo, y, static_cast<const T*>(z), ldz, weight,
+                                                     (int)n, (int)parts, eps, vec);
   });
   B200_LAUNCH_OK("gated_part_norm_kernel");
   return B200_OK;

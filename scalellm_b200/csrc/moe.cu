@@ -361,6 +361,89 @@ moe_route_softmax_kernel(int* __restrict__ ids, float* __restrict__ weights, flo
   }
 }
 
+// The choice alone, from router logits that a matrix product left in fp32: one warp per row.
+//     s = sigmoid(z) ; the E outputs form n_groups equal runs of neighbours, a run scores the sum of its `group_best`
+//     largest s, and only outputs of the keep_groups best runs can be chosen ; the `top` largest s are chosen (first
+//     index wins a tie) ; weight = factor * s / (sum of the chosen s + weight_eps)
+constexpr int kChoiceWarps = 4;
+
+__device__ __forceinline__ int warp_argmax(float v, int idx) {       // smallest index among the largest v
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float u = __shfl_xor_sync(0xffffffffu, v, o);
+    const int j = __shfl_xor_sync(0xffffffffu, idx, o);
+    if (u > v || (u == v && j < idx)) { v = u; idx = j; }
+  }
+  return idx;
+}
+
+__global__ void __launch_bounds__(kChoiceWarps * 32)
+moe_route_sigmoid_kernel(int* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ logits,
+                         int64_t ld, int64_t rows, int E, int top, int n_groups, int keep_groups, int group_best,
+                         float weight_eps, float factor) {
+  extern __shared__ float route_sm[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* s_s = route_sm + (size_t)warp * (E + n_groups);   // [E] scores; what cannot be chosen (any more) becomes -1
+  float* g_s = s_s + E;                                    // [n_groups]
+  const int64_t row = (int64_t)blockIdx.x * kChoiceWarps + warp;
+  if (row >= rows) return;
+  for (int e = lane; e < E; e += 32) s_s[e] = 1.0f / (1.0f + expf(-logits[row * ld + e]));
+  __syncwarp();
+  if (keep_groups < n_groups) {
+    const int gs = E / n_groups;
+    for (int g = lane; g < n_groups; g += 32) {
+      float total = 0.0f, below = INFINITY;                // the group_best largest, one at a time
+      int used_at = -1;
+      for (int k = 0; k < group_best && k < gs; ++k) {
+        float best = -1.0f;
+        int at = -1;
+        for (int j = 0; j < gs; ++j) {
+          const float s = s_s[g * gs + j];
+          if ((s < below || (s == below && j > used_at)) && s > best) { best = s; at = j; }
+        }
+        total += best;
+        below = best;
+        used_at = at;
+      }
+      g_s[g] = total;
+    }
+    __syncwarp();
+    for (int k = 0; k < keep_groups; ++k) {                // the kept groups' scores become negative
+      float bz = -INFINITY;
+      int best = 0x7fffffff;
+      for (int g = lane; g < n_groups; g += 32)
+        if (g_s[g] >= 0.0f && g_s[g] > bz) { bz = g_s[g]; best = g; }
+      best = warp_argmax(bz, best);
+      if (lane == 0) g_s[best] = -1.0f;
+      __syncwarp();
+    }
+    for (int e = lane; e < E; e += 32)
+      if (g_s[e / gs] >= 0.0f) s_s[e] = -1.0f;
+    __syncwarp();
+  }
+  float sum = 0.0f, mine = 0.0f;                           // lane k keeps the k-th choice (top <= 32)
+  int mine_id = 0;
+  for (int k = 0; k < top; ++k) {
+    float bz = -2.0f;
+    int best = 0x7fffffff;
+    for (int e = lane; e < E; e += 32) {
+      const float s = s_s[e];
+      if (s > bz) { bz = s; best = e; }
+    }
+    best = warp_argmax(bz, best);
+    const float s = s_s[best];
+    __syncwarp();
+    if (lane == 0) s_s[best] = -1.0f;
+    if (lane == k) { mine = s; mine_id = best; }
+    sum += s;
+    __syncwarp();
+  }
+  if (lane < top) {
+    ids[row * top + lane] = mine_id;
+    weights[row * top + lane] = factor * mine / (sum + weight_eps);
+  }
+}
+
 // out[row] = sum_k w[row, k] * (ids[row, k] < n_real ? Y[pos_of_pair[row, k]] : h[row])   (outputs from n_real on pass
 // their input through) + addend_gate[row] * addend[row] (a result every token gets, scaled per token)
 template <typename T>
@@ -533,6 +616,25 @@ int b200_moe_route_softmax(int32_t* expert_ids, float* weights, float* extra_out
                           expert_ids, weights, extra_out, static_cast<const T*>(h), ldh, router_weight, correction,
                           extra_weight, (int)W, (int)E, (int)top, (int)n_groups, (int)keep_groups, weight_eps)));
   B200_LAUNCH_OK("moe_route_softmax_kernel");
+  return B200_OK;
+}
+
+int b200_moe_route_sigmoid(int32_t* expert_ids, float* weights, const float* logits, int64_t ld, int64_t rows, int64_t E,
+                           int64_t top, int64_t n_groups, int64_t keep_groups, int64_t group_best, float weight_eps,
+                           float factor, b200_stream_t stream) {
+  if (rows == 0) return B200_OK;
+  B200_CHECK_ARG(expert_ids && weights && logits, "moe_route_sigmoid: null pointer");
+  B200_CHECK_ARG(rows > 0 && E >= 1 && E <= kMaxExperts && ld >= E && top >= 1 && top <= kMaxTop && n_groups >= 1 &&
+                     E % n_groups == 0 && keep_groups >= 1 && keep_groups <= n_groups && group_best >= 1 &&
+                     top <= keep_groups * (E / n_groups),
+                 "moe_route_sigmoid: bad shape (outputs <= 1024 in equal groups, top <= min(32, outputs of the kept "
+                 "groups))");
+  const size_t smem = (size_t)kChoiceWarps * (E + n_groups) * sizeof(float);
+  moe_route_sigmoid_kernel<<<(unsigned)((rows + kChoiceWarps - 1) / kChoiceWarps), kChoiceWarps * 32, smem,
+                             static_cast<cudaStream_t>(stream)>>>(
+      expert_ids, weights, logits, ld, rows, (int)E, (int)top, (int)n_groups, (int)keep_groups, (int)group_best,
+      weight_eps, factor);
+  B200_LAUNCH_OK("moe_route_sigmoid_kernel");
   return B200_OK;
 }
 

@@ -341,8 +341,9 @@ group_rms_norm_kernel(T* __restrict__ out, const float* __restrict__ x, const fl
 template <typename T>
 __global__ void __launch_bounds__(kRowThreads)
 branch_norm_residual_kernel(float* __restrict__ x_out, T* __restrict__ h_out, const float* __restrict__ x_in,
-                            const T* __restrict__ a, int64_t lda, const T* __restrict__ b, int64_t ldb,
-                            const float* __restrict__ wa, const float* __restrict__ wb, const float* __restrict__ w,
+                            const T* __restrict__ a, int64_t lda, const float* __restrict__ bias_a,
+                            const T* __restrict__ b, int64_t ldb, const float* __restrict__ wa,
+                            const float* __restrict__ wb, const float* __restrict__ w,
                             const float* __restrict__ w_next, int W, float eps) {
   extern __shared__ __align__(16) float sm[];
   float* m_s = sm;          // [W]
@@ -351,7 +352,8 @@ branch_norm_residual_kernel(float* __restrict__ x_out, T* __restrict__ h_out, co
   const int row = blockIdx.x;
   float sa = 0.0f, sb = 0.0f;
   for (int i = threadIdx.x; i < W; i += kRowThreads) {
-    const float av = Num<T>::to_f(a[(size_t)row * lda + i]);
+    float av = Num<T>::to_f(a[(size_t)row * lda + i]);
+    if (bias_a) av += bias_a[i];
     m_s[i] = av;
     sa += av * av;
     if (b) {
@@ -378,11 +380,14 @@ branch_norm_residual_kernel(float* __restrict__ x_out, T* __restrict__ h_out, co
   } else {
     sm2 = sa;
   }
-  sm2 = block_sum<kRowThreads>(sm2, red[2]);
-  const float rm = 1.0f / sqrtf(sm2 / (float)W + eps);
+  float rm = 1.0f;
+  if (w) {
+    sm2 = block_sum<kRowThreads>(sm2, red[2]);
+    rm = 1.0f / sqrtf(sm2 / (float)W + eps);
+  }
   float sx = 0.0f;
   for (int i = threadIdx.x; i < W; i += kRowThreads) {
-    const float r = x_in[(size_t)row * W + i] + m_s[i] * rm * w[i];
+    const float r = x_in[(size_t)row * W + i] + (w ? m_s[i] * rm * w[i] : m_s[i]);
     x_out[(size_t)row * W + i] = r;
     m_s[i] = r;
     sx += r * r;
@@ -737,12 +742,12 @@ int b200_token_gated_gelu(void* out, const void* in, int64_t ld_in, const void* 
   return B200_OK;
 }
 
-int b200_branch_norm_residual(float* x_out, void* h_out, const float* x_in, const void* a, int64_t lda, const void* b,
-                              int64_t ldb, const float* weight_a, const float* weight_b, const float* weight,
+int b200_branch_norm_residual(float* x_out, void* h_out, const float* x_in, const void* a, int64_t lda,
+                              const float* bias_a, const void* b, int64_t ldb, const float* weight_a, const float* weight_b, const float* weight,
                               const float* weight_next, int64_t rows, int64_t W, float eps, int dtype,
                               b200_stream_t stream) {
   if (rows == 0) return B200_OK;
-  B200_CHECK_ARG(x_out && x_in && a && weight, "branch_norm_residual: null pointer");
+  B200_CHECK_ARG(x_out && x_in && a, "branch_norm_residual: null pointer");
   B200_CHECK_ARG(!b || (weight_a && weight_b), "branch_norm_residual: two branches take both branch weights");
   B200_CHECK_ARG(rows > 0 && W > 0 && lda >= W && (!b || ldb >= W) && 2 * W * 4 <= 200 * 1024,
                  "branch_norm_residual: bad shape (at most ~25K channels)");
@@ -753,8 +758,8 @@ int b200_branch_norm_residual(float* x_out, void* h_out, const float* x_in, cons
       B200_CUDA_OK(cudaFuncSetAttribute(branch_norm_residual_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                         (int)smem));
     branch_norm_residual_kernel<T><<<(unsigned)rows, kRowThreads, smem, st>>>(
-        x_out, static_cast<T*>(h_out), x_in, static_cast<const T*>(a), lda, static_cast<const T*>(b), ldb, weight_a,
-        weight_b, weight, weight_next, (int)W, eps);
+        x_out, static_cast<T*>(h_out), x_in, static_cast<const T*>(a), lda, bias_a, static_cast<const T*>(b), ldb,
+        weight_a, weight_b, weight, weight_next, (int)W, eps);
   });
   B200_LAUNCH_OK("branch_norm_residual_kernel");
   return B200_OK;

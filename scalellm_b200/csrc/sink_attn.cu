@@ -6,14 +6,18 @@
 //     s_ij = scale q_i . k_j - r1_h ln(1 + r2_h (i - j))               j <= i                 (r1 absent: no bias)
 //     p_ij = exp(s_ij) / (exp(sink_h) + sum_j' exp(s_ij'))             the sink has no key and no value
 //     o_i  = sum_j p_ij v_j
-// On the way out a head's result may be multiplied by a number and, element by element, with sigmoid(gate): an output
-// gate and a branch weight cost no launch of their own.
+// A window > 0 limits row i to the keys i - window < j <= i.  Where the values ARE the keys (both cache pointers the
+// same) a staged tile serves both products.  On the way out a head's result may be multiplied by a number and with
+// sigmoid(gate), the gate one number per channel or one per head: an output gate and a branch weight cost no launch of
+// their own.
 // Query head h reads key/value head h / (H / G).  Values may be blended with the values another layer made of the
 // same token before they are cached:  v <- (1 - lam) v + lam v_other.
 //
 //   turned prepare : instead of unit heads and the temperature, one root mean square over ALL heads of the queries (and
 //             one over all of the keys) with a weight per channel, then a rotary turn of the first rot_dims channels of
 //             every head: channel t with t + rot_dims / 2, angle position * inv_freq[t] (fp32)
+//   heads prepare : optional biases, optional RMS norms per head with a weight [dim] shared by all heads, an optional
+//             half-pair turn as above and the query temperature; without values in the projection only keys are cached
 //   prepare : q rows -> fp32 [rows, H, dim]; k rows -> K cache [slots, G, dim]; v rows -> V cache [slots, G, vdim]
 //             (cache entries have the activation type T)
 //   attend  : CUDA cores, any type and size: one CTA per (row, key/value head, chunk of query heads); its warps are
@@ -178,6 +182,121 @@ int launch_prepare_turned(float* q_out, const void* q_in, const void* k_in, cons
   return B200_OK;
 }
 
+// Queries and keys of one row: biases, RMS norms per head (one weight [dim] for all heads), turn, temperature; queries
+// to q_out, keys (and values, where the projection has them) into the cache.  One CTA per row.
+struct HeadsPrepare {
+  float* q_out;
+  const void *q_in, *k_in, *v_in;          // column blocks of stride ld; v_in nullable: nothing but keys is cached
+  int64_t ld;
+  const float *q_bias, *k_bias, *v_bias;   // nullable
+  const float *q_w, *k_w;                  // [dim], nullable: no norms
+  const float* inv_freq;
+  void *k_cache, *v_cache;
+  const int *positions, *slots;
+  int H, G, dim, vdim, rot_dims;
+  float eps, temp_coef;
+  int temp_every;
+};
+
+template <typename T, int V>
+__global__ void __launch_bounds__(kTurnThreads) sink_attn_prepare_heads_kernel(const HeadsPrepare a) {
+  extern __shared__ __align__(16) float sm[];
+  const int H = a.H, G = a.G, dim = a.dim, nq = H * dim, nk = G * dim, nv = G * a.vdim, half = a.rot_dims / 2;
+  float* x_s = sm;                                       // [nq + nk] projected rows with their biases
+  float* r_s = x_s + (nq + nk + 3) / 4 * 4;              // [H + G] one factor per head
+  float* cos_s = r_s + (H + G + 3) / 4 * 4;              // [half]
+  float* sin_s = cos_s + (half + 3) / 4 * 4;             // [half]
+  const size_t row = blockIdx.x;
+  const int pos = a.positions[row], warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const size_t slot = (size_t)a.slots[row];
+  const T* q_in = static_cast<const T*>(a.q_in) + row * a.ld;
+  const T* k_in = static_cast<const T*>(a.k_in) + row * a.ld;
+  for (int i = threadIdx.x; i < half; i += kTurnThreads) sincosf((float)pos * a.inv_freq[i], &sin_s[i], &cos_s[i]);
+  for (int e = threadIdx.x * V; e < nq + nk; e += kTurnThreads * V) {
+    const bool is_q = e < nq;
+    const T* src = is_q ? q_in + e : k_in + (e - nq);
+    const float* b = is_q ? a.q_bias : a.k_bias;
+    const int be = is_q ? e : e - nq;
+    float x[V];
+    if constexpr (V == 4) load4<T>(src, x);
+    else x[0] = Num<T>::to_f(src[0]);
+#pragma unroll
+    for (int k = 0; k < V; ++k) x_s[e + k] = b ? x[k] + b[be + k] : x[k];
+  }
+  float temp = 1.0f;
+  if (a.temp_coef != 0.0f && a.temp_every > 0)
+    temp = 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.0f);
+  __syncthreads();
+  for (int u = warp; u < H + G; u += kTurnThreads / 32) {
+    float r = 1.0f;
+    if (a.q_w) {
+      const float* x = x_s + (size_t)u * dim;
+      float ss = 0.0f;
+      for (int i = lane; i < dim; i += 32) ss += x[i] * x[i];
+      r = 1.0f / sqrtf(warp_sum(ss) / (float)dim + a.eps);
+    }
+    if (lane == 0) r_s[u] = u < H ? r * temp : r;
+  }
+  __syncthreads();
+  for (int e = threadIdx.x * V; e < nq + nk; e += kTurnThreads * V) {
+    const bool is_q = e < nq;
+    const int u = e / dim, d = e - u * dim;
+    const float r = r_s[u];
+    const float* w = is_q ? a.q_w : a.k_w;
+    auto at = [&](int i, int t) { return w ? x_s[i] * r * w[t] : x_s[i] * r; };
+    float y[V];
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      const int t = d + k;
+      float v = at(e + k, t);
+      if (t < half) v = v * cos_s[t] - at(e + k + half, t + half) * sin_s[t];
+      else if (t < 2 * half) v = v * cos_s[t - half] + at(e + k - half, t - half) * sin_s[t - half];
+      y[k] = v;
+    }
+    if (is_q) {
+      float* dst = a.q_out + row * nq + e;
+      if constexpr (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1], y[2], y[3]);
+      else dst[0] = y[0];
+    } else {
+      T* dst = static_cast<T*>(a.k_cache) + slot * nk + (e - nq);
+      if constexpr (V == 4 && sizeof(T) == 4) *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1], y[2], y[3]);
+      else if constexpr (V == 4)
+        *reinterpret_cast<uint2*>(dst) = make_uint2(Num<T>::pack(y[0], y[1]), Num<T>::pack(y[2], y[3]));
+      else dst[0] = Num<T>::from_f(y[0]);
+    }
+  }
+  if (!a.v_in) return;
+  const T* vs = static_cast<const T*>(a.v_in) + row * a.ld;
+  T* vd = static_cast<T*>(a.v_cache) + slot * nv;
+  if (a.v_bias) {
+    for (int i = threadIdx.x; i < nv; i += kTurnThreads) vd[i] = Num<T>::from_f(Num<T>::to_f(vs[i]) + a.v_bias[i]);
+  } else if constexpr (V == 4) {
+    using U = typename std::conditional<sizeof(T) == 4, uint4, uint2>::type;
+    for (int i = threadIdx.x * 4; i < nv; i += kTurnThreads * 4)
+      *reinterpret_cast<U*>(vd + i) = *reinterpret_cast<const U*>(vs + i);
+  } else {
+    for (int i = threadIdx.x; i < nv; i += kTurnThreads) vd[i] = vs[i];
+  }
+}
+
+template <typename T>
+int launch_prepare_heads(const HeadsPrepare& a, int64_t rows, cudaStream_t st) {
+  const size_t smem = ((size_t)((a.H + a.G) * a.dim + 3) / 4 * 4 + (size_t)(a.H + a.G + 3) / 4 * 4 +
+                       (size_t)(a.rot_dims / 2 + 3) / 4 * 8) * sizeof(float);
+  B200_CHECK_ARG(smem <= 200 * 1024, "sink_attn_prepare_heads: %d + %d heads of %d do not fit in shared memory", a.H, a.G,
+                 a.dim);
+  const bool vec = a.dim % 4 == 0 && (!a.v_in || (a.vdim % 4 == 0 && is_aligned(a.v_in, 4 * sizeof(T)) &&
+                                                  is_aligned(a.v_cache, 16))) &&
+                   a.ld % 4 == 0 && is_aligned(a.q_in, 4 * sizeof(T)) && is_aligned(a.k_in, 4 * sizeof(T)) &&
+                   is_aligned(a.k_cache, 16) && is_aligned(a.q_out, 16);
+  auto kern = vec ? sink_attn_prepare_heads_kernel<T, 4> : sink_attn_prepare_heads_kernel<T, 1>;
+  if (smem > 48 * 1024)
+    B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  kern<<<(unsigned)rows, kTurnThreads, smem, st>>>(a);
+  B200_LAUNCH_OK("sink_attn_prepare_heads_kernel");
+  return B200_OK;
+}
+
 // The end of a head's walk: its softmax denominator takes the sink, a term exp(sink) with no value.
 __device__ __forceinline__ float sink_scale(float m, float l, const float* sink, int h) {
   // returns f with o_final = o * f, o accumulated relative to the running maximum m with sum l
@@ -186,6 +305,16 @@ __device__ __forceinline__ float sink_scale(float m, float l, const float* sink,
   const float M = fmaxf(m, s);
   const float c = expf(m - M);
   return c / (l * c + expf(s - M));
+}
+
+// A row's first visible key under a window (0: no window).
+__device__ __forceinline__ int first_key(int i, int window) {
+  return window > 0 && i >= window ? i - window + 1 : 0;
+}
+
+// Where head h's gate numbers start and how far apart the numbers of neighbouring channels are.
+__device__ __forceinline__ size_t gate_base(size_t row, int64_t ld_gate, int h, int vdim, int gate_heads) {
+  return row * (size_t)ld_gate + (gate_heads ? (size_t)h : (size_t)h * vdim);
 }
 
 // What leaves the kernels: mul * o * sigmoid(gate[i]) (gate absent: mul * o).
@@ -202,7 +331,7 @@ __global__ void __launch_bounds__(kMaxWarps * 32)
 sink_attn_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict__ q, const T* __restrict__ k_cache,
                  const T* __restrict__ v_cache, const float* __restrict__ r1, const float* __restrict__ r2,
                  const float* __restrict__ sink, const T* __restrict__ gate, int64_t ld_gate, float out_mul,
-                 const int* __restrict__ q_cu, const int* __restrict__ kv_cu,
+                 int gate_heads, int window, const int* __restrict__ q_cu, const int* __restrict__ kv_cu,
                  const int* __restrict__ block_tables, const int* __restrict__ cu_block_lens,
                  const int* __restrict__ token_seq, int H, int G, int dim, int vdim, int block_size, float scale,
                  int RH, int S) {
@@ -233,10 +362,11 @@ sink_attn_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict__ q, 
   float acc[NC];
 #pragma unroll
   for (int c = 0; c < NC; ++c) acc[c] = 0.0f;
-  for (int n0 = sp * 32; n0 <= i; n0 += S * 32) {
+  const int j_lo = first_key(i, window);
+  for (int n0 = j_lo / 32 * 32 + sp * 32; n0 <= i; n0 += S * 32) {
     const int j = n0 + lane;
-    const bool live = j <= i;
-    // lanes past the last key point at the row's own position (always written) with weight 0
+    const bool live = j <= i && j >= j_lo;
+    // lanes outside the row's keys point at the row's own position (always written) with weight 0
     const int jj = live ? j : i;
     const int slot = table[jj / block_size] + jj % block_size;
     float s = -INFINITY;
@@ -250,7 +380,7 @@ sink_attn_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict__ q, 
     float t = s;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) t = fmaxf(t, __shfl_xor_sync(0xffffffffu, t, o));
-    const float nm = fmaxf(m, t);            // finite: lane 0 of a started group is live
+    const float nm = fmaxf(m, t);            // finite: a started group holds a live lane
     const float corr = expf(m - nm);
     const float p = live ? expf(s - nm) : 0.0f;
     l = l * corr + warp_sum(p);
@@ -302,14 +432,15 @@ sink_attn_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict__ q, 
     const int col = lane + 32 * c;
     if (col < vdim)
       out[(size_t)row * ldo + (size_t)h * vdim + col] =
-          Num<T>::from_f(gated_out(o[c] * f, gate, (size_t)row * ld_gate + (size_t)h * vdim + col, out_mul));
+          Num<T>::from_f(gated_out(o[c] * f, gate, gate_base(row, ld_gate, h, vdim, gate_heads) + (gate_heads ? 0 : col),
+                                   out_mul));
   }
 }
 
 template <typename T, int NC>
 int launch_simt(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache, const float* r1,
-                const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul, const int* q_cu,
-                const int* kv_cu, const int* tables, const int* blk_cu, const int* token_seq, int64_t rows, int H, int G,
+                const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul, int gate_heads,
+                int window, const int* q_cu, const int* kv_cu, const int* tables, const int* blk_cu, const int* token_seq, int64_t rows, int H, int G,
                 int dim, int vdim, int block_size, float scale, cudaStream_t st) {
   const int R = H / G;
   const int RH = R < kMaxWarps ? R : kMaxWarps;
@@ -325,19 +456,19 @@ int launch_simt(void* out, int64_t ldo, const float* q, const void* k_cache, con
   dim3 grid((unsigned)rows, (unsigned)G, (unsigned)chunks);
   kern<<<grid, n_warps * 32, smem, st>>>(static_cast<T*>(out), ldo, q, static_cast<const T*>(k_cache),
                                          static_cast<const T*>(v_cache), r1, r2, sink, static_cast<const T*>(gate),
-                                         ld_gate, out_mul, q_cu, kv_cu, tables, blk_cu, token_seq, H, G, dim, vdim,
-                                         block_size, scale, RH, S);
+                                         ld_gate, out_mul, gate_heads, window, q_cu, kv_cu, tables, blk_cu, token_seq, H,
+                                         G, dim, vdim, block_size, scale, RH, S);
   B200_LAUNCH_OK("sink_attn_kernel");
   return B200_OK;
 }
 
 template <typename T>
 int dispatch_simt(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache, const float* r1,
-                  const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul, const int* q_cu,
-                  const int* kv_cu, const int* tables, const int* blk_cu, const int* token_seq, int64_t rows, int H,
+                  const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul, int gate_heads,
+                  int window, const int* q_cu, const int* kv_cu, const int* tables, const int* blk_cu, const int* token_seq, int64_t rows, int H,
                   int G, int dim, int vdim, int block_size, float scale, cudaStream_t st) {
-#define SA_ARGS out, ldo, q, k_cache, v_cache, r1, r2, sink, gate, ld_gate, out_mul, q_cu, kv_cu, tables, blk_cu, \
-                token_seq, rows, H, G, dim, vdim, block_size, scale, st
+#define SA_ARGS out, ldo, q, k_cache, v_cache, r1, r2, sink, gate, ld_gate, out_mul, gate_heads, window, q_cu, kv_cu, \
+                tables, blk_cu, token_seq, rows, H, G, dim, vdim, block_size, scale, st
   const int nc = (vdim + 31) / 32;
   if (nc <= 1) return launch_simt<T, 1>(SA_ARGS);
   if (nc <= 2) return launch_simt<T, 2>(SA_ARGS);
@@ -390,8 +521,8 @@ __global__ void __launch_bounds__(128, EXACT ? 4 : 1)
 sink_attn_prefill_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const float* __restrict__ q,
                          const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
                          const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink,
-                         const __nv_bfloat16* __restrict__ gate, int64_t ld_gate, float out_mul,
-                         const int* __restrict__ q_cu, const int* __restrict__ kv_cu,
+                         const __nv_bfloat16* __restrict__ gate, int64_t ld_gate, float out_mul, int gate_heads,
+                         int window, const int* __restrict__ q_cu, const int* __restrict__ kv_cu,
                          const int* __restrict__ block_tables, const int* __restrict__ cu_block_lens, int H, int G,
                          int dim_rt, int vdim_rt, int block_size, float scale, int RW, int chunks) {
   extern __shared__ __align__(16) unsigned char smraw[];
@@ -399,7 +530,8 @@ sink_attn_prefill_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const flo
   const int KROW = dim + 8, VROW = vdim + 8;            // bf16 elements per staged row (16 bytes of padding)
   __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(smraw);     // [4][16][KROW]
   __nv_bfloat16* Ks = Qs + 4 * 16 * KROW;                          // [2][kBK][KROW]
-  __nv_bfloat16* Vs = Ks + 2 * kBK * KROW;                         // [2][kBK][VROW]
+  const bool shared_kv = k_cache == v_cache;                       // the values are the keys: one tile for both
+  __nv_bfloat16* Vs = shared_kv ? Ks : Ks + 2 * kBK * KROW;        // [2][kBK][VROW]
   const int seq = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = blockIdx.z / chunks, chunk = blockIdx.z % chunks;
   const int R = H / G, TW = 4 / RW, BQ = 16 * TW;
@@ -424,6 +556,7 @@ sink_attn_prefill_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const flo
   }
   const int P1 = first_pos + (t0 + BQ < q_len ? t0 + BQ : q_len) - 1;   // last position of the CTA's tokens
   const int n_tiles = P1 / kBK + 1;
+  const int tile0 = first_key(first_pos + t0, window) / kBK;            // tiles before it lie outside every row's window
   const size_t k_stride = (size_t)G * dim, v_stride = (size_t)G * vdim;
   auto load_tile = [&](int idx, int buf) {
     const int key = threadIdx.x >> 2, sub = threadIdx.x & 3;
@@ -436,9 +569,10 @@ sink_attn_prefill_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const flo
     __nv_bfloat16* kd = Ks + ((size_t)buf * kBK + key) * KROW;
     __nv_bfloat16* vd = Vs + ((size_t)buf * kBK + key) * VROW;
     for (int c = sub; c < dim / 8; c += 4) cp_async16(kd + c * 8, kr + c * 8, ok);
-    for (int c = sub; c < vdim / 8; c += 4) cp_async16(vd + c * 8, vr + c * 8, ok);
+    if (!shared_kv)
+      for (int c = sub; c < vdim / 8; c += 4) cp_async16(vd + c * 8, vr + c * 8, ok);
   };
-  load_tile(0, 0);
+  load_tile(tile0, tile0 & 1);
   cp_async_commit();
 
   const int gr = lane >> 2, qc = (lane & 3) * 2;        // fragment row within 8, first column of the pair
@@ -455,7 +589,7 @@ sink_attn_prefill_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const flo
 #pragma unroll
   for (int n = 0; n < VT_MAX * 2; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.0f;
   const __nv_bfloat16* qw = Qs + warp * 16 * KROW;
-  for (int it = 0; it < n_tiles; ++it) {
+  for (int it = tile0; it < n_tiles; ++it) {
     const int buf = it & 1;
     cp_async_wait_all();
     __syncthreads();                                    // tile `it` has landed; everyone is done with tile it - 1
@@ -463,7 +597,8 @@ sink_attn_prefill_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const flo
     cp_async_commit();
     const int j0 = it * kBK;
     if (j0 > wpos0 + 15) continue;                      // the whole tile lies after this warp's last row
-    const bool full_tile = warp_rows_valid && j0 + kBK - 1 <= wpos0;
+    if (window > 0 && j0 + kBK + window <= wpos0 + 1) continue;       // ... or before its first row's window
+    const bool full_tile = warp_rows_valid && j0 + kBK - 1 <= wpos0 && (window <= 0 || wpos0 + 15 - j0 < window);
     const __nv_bfloat16* kt = Ks + (size_t)buf * kBK * KROW;
     const __nv_bfloat16* vt = Vs + (size_t)buf * kBK * VROW;
     float sc[4][4];
@@ -491,7 +626,7 @@ sink_attn_prefill_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const flo
         const int j = j0 + n * 8 + qc + (e & 1), i = pos[e >> 1];
         float v = sc[n][e] * scale;
         if (biased) v -= b1 * __logf(1.0f + b2 * (float)(i - j));     // (a NaN of an unseen key is replaced below)
-        if (!full_tile && j > i) v = -INFINITY;
+        if (!full_tile && (j > i || (window > 0 && i - j >= window))) v = -INFINITY;
         sc[n][e] = v;
         rmax[e >> 1] = fmaxf(rmax[e >> 1], v);
       }
@@ -558,34 +693,38 @@ sink_attn_prefill_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const flo
     const float f = sink_scale(mx[r2i], ls[r2i], sink, h);
     const size_t row = (size_t)q0 + row_t[r2i];
     __nv_bfloat16* dst = out + row * ldo + (size_t)h * vdim;
-    const size_t gi = row * ld_gate + (size_t)h * vdim + qc;
+    const size_t gi = gate_base(row, ld_gate, h, vdim, gate_heads) + (gate_heads ? 0 : qc);
+    // (one gate number for the head joins the factor; the loop below then has none to read)
+    const __nv_bfloat16* ge = gate_heads ? nullptr : gate;
+    const float fm = gate_heads ? gated_out(f, gate, gi, out_mul) : f, mul = gate_heads ? 1.0f : out_mul;
 #pragma unroll
     for (int n = 0; n < VT_MAX * 2; ++n)
       if (n < VT * 2)
         *reinterpret_cast<uint32_t*>(dst + n * 8 + qc) =
-            Num<__nv_bfloat16>::pack(gated_out(o[n][r2i * 2] * f, gate, gi + n * 8, out_mul),
-                                     gated_out(o[n][r2i * 2 + 1] * f, gate, gi + n * 8 + 1, out_mul));
+            Num<__nv_bfloat16>::pack(gated_out(o[n][r2i * 2] * fm, ge, gi + n * 8, mul),
+                                     gated_out(o[n][r2i * 2 + 1] * fm, ge, gi + n * 8 + 1, mul));
   }
 }
 
 template <int KS_MAX, int VT_MAX, bool EXACT>
 int launch_prefill(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache, const float* r1,
-                   const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul, const int* q_cu, const int* kv_cu, const int* tables,
-                   const int* blk_cu, int64_t n_seq, int64_t q_max, int H, int G, int dim, int vdim, int block_size,
-                   float scale, cudaStream_t st) {
+                   const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul, int gate_heads,
+                   int window, const int* q_cu, const int* kv_cu, const int* tables, const int* blk_cu,
+                   int64_t n_seq, int64_t q_max, int H, int G, int dim, int vdim, int block_size, float scale, cudaStream_t st) {
   const int R = H / G;
   const int RW = R >= 4 ? 4 : (R >= 2 ? 2 : 1);
   const int chunks = (R + RW - 1) / RW;
   const int BQ = 16 * (4 / RW);
-  const size_t smem = ((size_t)(4 * 16 + 2 * kBK) * (dim + 8) + (size_t)2 * kBK * (vdim + 8)) * sizeof(__nv_bfloat16);
+  const size_t smem = ((size_t)(4 * 16 + 2 * kBK) * (dim + 8) + (k_cache == v_cache ? 0 : (size_t)2 * kBK * (vdim + 8))) *
+                      sizeof(__nv_bfloat16);
   auto kern = sink_attn_prefill_kernel<KS_MAX, VT_MAX, EXACT>;
   if (smem > 48 * 1024)
     B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   dim3 grid((unsigned)((q_max + BQ - 1) / BQ), (unsigned)n_seq, (unsigned)(G * chunks));
   kern<<<grid, 128, smem, st>>>(static_cast<__nv_bfloat16*>(out), ldo, q, static_cast<const __nv_bfloat16*>(k_cache),
                                 static_cast<const __nv_bfloat16*>(v_cache), r1, r2, sink,
-                                static_cast<const __nv_bfloat16*>(gate), ld_gate, out_mul, q_cu, kv_cu, tables, blk_cu,
-                                H, G, dim, vdim, block_size, scale, RW, chunks);
+                                static_cast<const __nv_bfloat16*>(gate), ld_gate, out_mul, gate_heads, window, q_cu,
+                                kv_cu, tables, blk_cu, H, G, dim, vdim, block_size, scale, RW, chunks);
   B200_LAUNCH_OK("sink_attn_prefill_kernel");
   return B200_OK;
 }
@@ -607,8 +746,8 @@ __global__ void __launch_bounds__(128)
 sink_attn_decode_tc_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const float* __restrict__ q,
                            const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
                            const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink,
-                           const __nv_bfloat16* __restrict__ gate, int64_t ld_gate, float out_mul,
-                           const int* __restrict__ q_cu, const int* __restrict__ kv_cu,
+                           const __nv_bfloat16* __restrict__ gate, int64_t ld_gate, float out_mul, int gate_heads,
+                           int window, const int* __restrict__ q_cu, const int* __restrict__ kv_cu,
                            const int* __restrict__ block_tables, const int* __restrict__ cu_block_lens,
                            const int* __restrict__ token_seq, int H, int G, int dim, int vdim, int block_size,
                            float scale, int n_splits, float* __restrict__ ws) {
@@ -620,7 +759,8 @@ sink_attn_decode_tc_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const f
   int* slot_s = reinterpret_cast<int*>(b_s + 2 * 16);              // [2][kDK] cache rows of the keys of two tiles
   unsigned char* big = reinterpret_cast<unsigned char*>(slot_s + 2 * kDK);
   __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(big);       // [kDS][kDK][KROW]
-  __nv_bfloat16* Vs = Ks + kDS * kDK * KROW;                       // [kDS][kDK][VROW]
+  const bool shared_kv = k_cache == v_cache;                       // the values are the keys: one tile for both
+  __nv_bfloat16* Vs = shared_kv ? Ks : Ks + kDS * kDK * KROW;      // [kDS][kDK][VROW]
   float* o_s = reinterpret_cast<float*>(big);                      // after the walk: [4 warps][16][vdim]
   const int row = blockIdx.x / n_splits, split = blockIdx.x % n_splits, g = blockIdx.y, warp = threadIdx.x >> 5,
             lane = threadIdx.x & 31;
@@ -642,11 +782,13 @@ sink_attn_decode_tc_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const f
     b_s[threadIdx.x] = ok ? r1[g * R + h_base + threadIdx.x] : 0.0f;
     b_s[16 + threadIdx.x] = ok ? r2[g * R + h_base + threadIdx.x] : 0.0f;
   }
-  const int all_tiles = i / kDK + 1;
+  const int j_lo = first_key(i, window), tile_lo = j_lo / kDK;
+  const int all_tiles = i / kDK + 1 - tile_lo;
   // this CTA's share of the row's tiles (n_splits CTAs per row; an empty share hands on sums of zero)
   const int per = (all_tiles + n_splits - 1) / n_splits;
-  const int tile0 = split * per;
-  const int n_tiles = all_tiles - tile0 < per ? (all_tiles - tile0 > 0 ? all_tiles - tile0 : 0) : per;
+  const int left = all_tiles - split * per;
+  const int tile0 = tile_lo + split * per;
+  const int n_tiles = left < per ? (left > 0 ? left : 0) : per;
   const size_t k_stride = (size_t)G * dim, v_stride = (size_t)G * vdim;
   // The cache rows of a tile's keys are looked up in the block table one tile ahead of their copy (threads 0..63, one
   // key each, into slot_s), so that the lookup's latency is off the walk's critical path; the copy itself runs with
@@ -667,7 +809,7 @@ sink_attn_decode_tc_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const f
       cp_async16(Ks + ((size_t)buf * kDK + key) * KROW + c * 8,
                  k_cache + (size_t)(slot < 0 ? 0 : slot) * k_stride + (size_t)g * dim + c * 8, slot >= 0);
     }
-    for (int id = threadIdx.x; id < kDK * CV; id += 128) {
+    if (!shared_kv) for (int id = threadIdx.x; id < kDK * CV; id += 128) {
       const int key = id / CV, c = id - key * CV;
       const int slot = sl[key];
       cp_async16(Vs + ((size_t)buf * kDK + key) * VROW + c * 8,
@@ -694,7 +836,7 @@ sink_attn_decode_tc_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const f
     lookup(it + 2);                                        // into the half of slot_s that tile `it` has left
     if (it == 0) { hb1[0] = b_s[gr]; hb1[1] = b_s[gr + 8]; hb2[0] = b_s[16 + gr]; hb2[1] = b_s[16 + gr + 8]; }
     const int j0 = (tile0 + it) * kDK + warp * 16;       // this warp's 16 keys of the tile
-    if (j0 > i) continue;                                // all after the row's position
+    if (j0 > i || j0 + 15 < j_lo) continue;              // all after the row's position, or before its window
     const __nv_bfloat16* kt = Ks + ((size_t)buf * kDK + warp * 16) * KROW;
     const __nv_bfloat16* vt = Vs + ((size_t)buf * kDK + warp * 16) * VROW;
     float sc[2][4];
@@ -718,7 +860,7 @@ sink_attn_decode_tc_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const f
         const int j = j0 + n * 8 + qc + (e & 1);
         float v = sc[n][e] * scale;
         if (biased) v -= hb1[e >> 1] * __logf(1.0f + hb2[e >> 1] * (float)(i - j));
-        if (j > i) v = -INFINITY;
+        if (j > i || j < j_lo) v = -INFINITY;
         sc[n][e] = v;
         rmax[e >> 1] = fmaxf(rmax[e >> 1], v);
       }
@@ -820,7 +962,7 @@ sink_attn_decode_tc_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const f
       const int col = lane + 32 * c;
       if (col < vdim)
         out[(size_t)row * ldo + (size_t)h * vdim + col] = __float2bfloat16_rn(
-            gated_out(x[c] * fo, gate, (size_t)row * ld_gate + (size_t)h * vdim + col, out_mul));
+            gated_out(x[c] * fo, gate, gate_base(row, ld_gate, h, vdim, gate_heads) + (gate_heads ? 0 : col), out_mul));
     }
   }
 }
@@ -830,7 +972,7 @@ sink_attn_decode_tc_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const f
 __global__ void __launch_bounds__(128)
 sink_attn_merge_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const float* __restrict__ ws,
                        const float* __restrict__ sink, const __nv_bfloat16* __restrict__ gate, int64_t ld_gate,
-                       float out_mul, int64_t n_pairs, int H, int vdim, int n_splits) {
+                       float out_mul, int gate_heads, int64_t n_pairs, int H, int vdim, int n_splits) {
   const int64_t pair = (int64_t)blockIdx.x * 4 + (threadIdx.x >> 5);      // row * H + head
   const int lane = threadIdx.x & 31;
   if (pair >= n_pairs) return;
@@ -855,17 +997,18 @@ sink_attn_merge_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const float
     const int col = lane + 32 * c;
     if (col < vdim)
       out[row * ldo + (size_t)h * vdim + col] = __float2bfloat16_rn(
-          gated_out(x[c] * fo, gate, (size_t)row * ld_gate + (size_t)h * vdim + col, out_mul));
+          gated_out(x[c] * fo, gate, gate_base(row, ld_gate, h, vdim, gate_heads) + (gate_heads ? 0 : col), out_mul));
   }
 }
 
 template <int KS_MAX, int VT_MAX>
 int launch_decode_tc(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache, const float* r1,
-                     const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul,
-                     const int* q_cu, const int* kv_cu, const int* tables, const int* blk_cu, const int* token_seq, int64_t rows, int H, int G, int dim, int vdim,
-                     int block_size, float scale, int n_splits, float* ws, cudaStream_t st) {
+                     const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul, int gate_heads,
+                     int window, const int* q_cu, const int* kv_cu, const int* tables, const int* blk_cu,
+                     const int* token_seq, int64_t rows, int H, int G, int dim, int vdim, int block_size, float scale, int n_splits, float* ws, cudaStream_t st) {
   const int R = H / G;
-  const size_t tiles = ((size_t)kDS * kDK * (dim + 8) + (size_t)kDS * kDK * (vdim + 8)) * sizeof(__nv_bfloat16);
+  const size_t tiles = ((size_t)kDS * kDK * (dim + 8) + (k_cache == v_cache ? 0 : (size_t)kDS * kDK * (vdim + 8))) *
+                       sizeof(__nv_bfloat16);
   const size_t sums = (size_t)4 * 16 * vdim * sizeof(float);
   const size_t smem = (size_t)16 * (dim + 8) * sizeof(__nv_bfloat16) + (4 * 2 * 16 + 2 * 16) * sizeof(float) +
                       2 * kDK * sizeof(int) + (tiles > sums ? tiles : sums);
@@ -875,14 +1018,14 @@ int launch_decode_tc(void* out, int64_t ldo, const float* q, const void* k_cache
   dim3 grid((unsigned)(rows * n_splits), (unsigned)G, (unsigned)((R + 15) / 16));
   kern<<<grid, 128, smem, st>>>(static_cast<__nv_bfloat16*>(out), ldo, q, static_cast<const __nv_bfloat16*>(k_cache),
                                 static_cast<const __nv_bfloat16*>(v_cache), r1, r2, sink,
-                                static_cast<const __nv_bfloat16*>(gate), ld_gate, out_mul, q_cu, kv_cu, tables, blk_cu,
-                                token_seq, H, G, dim, vdim, block_size, scale, n_splits, n_splits > 1 ? ws : nullptr);
+                                static_cast<const __nv_bfloat16*>(gate), ld_gate, out_mul, gate_heads, window, q_cu,
+                                kv_cu, tables, blk_cu, token_seq, H, G, dim, vdim, block_size, scale, n_splits, n_splits > 1 ? ws : nullptr);
   B200_LAUNCH_OK("sink_attn_decode_tc_kernel");
   if (n_splits > 1) {
     const int64_t n_pairs = rows * H;
     sink_attn_merge_kernel<<<(unsigned)((n_pairs + 3) / 4), 128, 0, st>>>(
-        static_cast<__nv_bfloat16*>(out), ldo, ws, sink, static_cast<const __nv_bfloat16*>(gate), ld_gate, out_mul, n_pairs,
-        H, vdim, n_splits);
+        static_cast<__nv_bfloat16*>(out), ldo, ws, sink, static_cast<const __nv_bfloat16*>(gate), ld_gate, out_mul,
+        gate_heads, n_pairs, H, vdim, n_splits);
     B200_LAUNCH_OK("sink_attn_merge_kernel");
   }
   return B200_OK;
@@ -947,23 +1090,51 @@ int b200_sink_attn_prepare_turned(float* q_out, const void* q_in, const void* k_
 #undef SPT_CALL
 }
 
+int b200_sink_attn_prepare_heads(float* q_out, const void* q_in, const void* k_in, const void* v_in, int64_t ld,
+                                 const float* q_bias, const float* k_bias, const float* v_bias, const float* q_weight,
+                                 const float* k_weight, const float* inv_freq, void* k_cache, void* v_cache,
+                                 const int32_t* positions, const int32_t* slots, int64_t rows, int64_t H, int64_t G,
+                                 int64_t dim, int64_t vdim, int64_t rot_dims, float eps, float temp_coef,
+                                 int64_t temp_every, int dtype, b200_stream_t stream) {
+  if (rows == 0) return B200_OK;
+  B200_CHECK_ARG(q_out && q_in && k_in && k_cache && positions && slots && (!v_in || v_cache) &&
+                     (q_weight == nullptr) == (k_weight == nullptr) && (v_in || !v_bias),
+                 "sink_attn_prepare_heads: null pointer, or a norm for queries or keys only");
+  B200_CHECK_ARG(rows > 0 && H > 0 && G > 0 && H % G == 0 && dim > 0 && vdim > 0 && ld >= H * dim &&
+                     (!v_in || ld >= G * vdim) && rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim &&
+                     (rot_dims == 0 || inv_freq) && temp_every >= 0 && temp_every < (1ll << 31),
+                 "sink_attn_prepare_heads: bad shape (an even number of turned channels, at most the head's)");
+  HeadsPrepare a{q_out, q_in, k_in, v_in, ld, q_bias, k_bias, v_bias, q_weight, k_weight, inv_freq, k_cache, v_cache,
+                 positions, slots, (int)H, (int)G, (int)dim, (int)vdim, (int)rot_dims, eps, temp_coef, (int)temp_every};
+  auto st = static_cast<cudaStream_t>(stream);
+  switch (dtype) {
+    case B200_BF16: return launch_prepare_heads<__nv_bfloat16>(a, rows, st);
+    case B200_FP16: return launch_prepare_heads<__half>(a, rows, st);
+    case B200_FP32: return launch_prepare_heads<float>(a, rows, st);
+    default: return set_error(B200_ERR_INVALID_ARG, "bad dtype %d", dtype);
+  }
+}
+
 int b200_sink_attn(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache, const float* r1,
-                   const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul,
-                   const int32_t* q_cu_lens, const int32_t* kv_cu_lens, const int32_t* block_tables, const int32_t* cu_block_lens, const int32_t* token_seq, int64_t rows,
-                   int64_t H, int64_t G, int64_t dim, int64_t vdim, int64_t block_size, float scale, int dtype,
+                   const float* r2, const float* sink, const void* gate, int64_t ld_gate, float out_mul, int gate_heads,
+                   int64_t window, const int32_t* q_cu_lens, const int32_t* kv_cu_lens, const int32_t* block_tables,
+                   const int32_t* cu_block_lens, const int32_t* token_seq, int64_t rows, int64_t H,
+                   int64_t G, int64_t dim, int64_t vdim, int64_t block_size, float scale, int dtype,
                    b200_stream_t stream) {
   if (rows == 0) return B200_OK;
   B200_CHECK_ARG(out && q && k_cache && v_cache && q_cu_lens && kv_cu_lens && block_tables && cu_block_lens && token_seq,
                  "sink_attn: null pointer");
   B200_CHECK_ARG((r1 == nullptr) == (r2 == nullptr), "sink_attn: the distance bias takes both of its numbers");
-  B200_CHECK_ARG(!gate || ld_gate >= H * vdim, "sink_attn: gate rows shorter than the heads");
+  B200_CHECK_ARG(!gate || ld_gate >= (gate_heads ? H : H * vdim), "sink_attn: gate rows shorter than the heads");
+  B200_CHECK_ARG(window >= 0 && window < (1ll << 30) && (k_cache != v_cache || dim == vdim),
+                 "sink_attn: bad window, or shared keys and values of different sizes");
   B200_CHECK_ARG(rows > 0 && H > 0 && G > 0 && G <= 65535 && H % G == 0 && dim > 0 && vdim > 0 && vdim <= kMaxVdim &&
                      block_size > 0 && ldo >= H * vdim,
                  "sink_attn: bad shape (value heads of at most %d channels)", kMaxVdim);
   auto st = static_cast<cudaStream_t>(stream);
 #define SA_CALL(T)                                                                                                 \
-  return dispatch_simt<T>(out, ldo, q, k_cache, v_cache, r1, r2, sink, gate, ld_gate, out_mul, q_cu_lens, kv_cu_lens, \
-                          block_tables, cu_block_lens, token_seq, rows, (int)H, (int)G, (int)dim, (int)vdim, (int)block_size, scale, st)
+  return dispatch_simt<T>(out, ldo, q, k_cache, v_cache, r1, r2, sink, gate, ld_gate, out_mul, gate_heads, (int)window, \
+                          q_cu_lens, kv_cu_lens, block_tables, cu_block_lens, token_seq, rows, (int)H, (int)G, (int)dim, (int)vdim, (int)block_size, scale, st)
   switch (dtype) {
     case B200_BF16: SA_CALL(__nv_bfloat16);
     case B200_FP16: SA_CALL(__half);
@@ -979,14 +1150,17 @@ int b200_sink_attn_prefill_supported(int64_t dim, int64_t vdim, int dtype) {
 
 int b200_sink_attn_prefill(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache,
                            const float* r1, const float* r2, const float* sink, const void* gate, int64_t ld_gate,
-                           float out_mul, const int32_t* q_cu_lens, const int32_t* kv_cu_lens, const int32_t* block_tables, const int32_t* cu_block_lens,
+                           float out_mul, int gate_heads, int64_t window, const int32_t* q_cu_lens,
+                           const int32_t* kv_cu_lens, const int32_t* block_tables, const int32_t* cu_block_lens,
                            int64_t n_seq, int64_t q_max, int64_t H, int64_t G, int64_t dim, int64_t vdim,
                            int64_t block_size, float scale, int dtype, b200_stream_t stream) {
   if (n_seq == 0 || q_max == 0) return B200_OK;
   B200_CHECK_ARG(out && q && k_cache && v_cache && q_cu_lens && kv_cu_lens && block_tables && cu_block_lens,
                  "sink_attn_prefill: null pointer");
   B200_CHECK_ARG((r1 == nullptr) == (r2 == nullptr), "sink_attn_prefill: the distance bias takes both of its numbers");
-  B200_CHECK_ARG(!gate || ld_gate >= H * vdim, "sink_attn_prefill: gate rows shorter than the heads");
+  B200_CHECK_ARG(!gate || ld_gate >= (gate_heads ? H : H * vdim), "sink_attn_prefill: gate rows shorter than the heads");
+  B200_CHECK_ARG(window >= 0 && window < (1ll << 30) && (k_cache != v_cache || dim == vdim),
+                 "sink_attn_prefill: bad window, or shared keys and values of different sizes");
   B200_CHECK_ARG(b200_sink_attn_prefill_supported(dim, vdim, dtype),
                  "sink_attn_prefill: bf16 with head sizes that are multiples of 16 and at most 128");
   B200_CHECK_ARG(n_seq > 0 && n_seq <= 65535 && q_max > 0 && H > 0 && G > 0 && H % G == 0 && block_size > 0 &&
@@ -994,8 +1168,8 @@ int b200_sink_attn_prefill(void* out, int64_t ldo, const float* q, const void* k
                      is_aligned(v_cache, 16) && G * ((H / G + 3) / 4) <= 65535,
                  "sink_attn_prefill: bad shape or alignment");
   auto st = static_cast<cudaStream_t>(stream);
-#define SPF_ARGS out, ldo, q, k_cache, v_cache, r1, r2, sink, gate, ld_gate, out_mul, q_cu_lens, kv_cu_lens, \
-                 block_tables, cu_block_lens, n_seq, q_max, (int)H, (int)G, (int)dim, (int)vdim, (int)block_size, scale, st
+#define SPF_ARGS out, ldo, q, k_cache, v_cache, r1, r2, sink, gate, ld_gate, out_mul, gate_heads, (int)window, \
+                 q_cu_lens, kv_cu_lens, block_tables, cu_block_lens, n_seq, q_max, (int)H, (int)G, (int)dim, (int)vdim, (int)block_size, scale, st
   if (dim == 64 && vdim == 64) return launch_prefill<4, 4, true>(SPF_ARGS);
   if (dim == 128 && vdim == 128) return launch_prefill<8, 8, true>(SPF_ARGS);
   if (dim <= 64 && vdim <= 64) return launch_prefill<4, 4, false>(SPF_ARGS);
@@ -1005,7 +1179,8 @@ int b200_sink_attn_prefill(void* out, int64_t ldo, const float* q, const void* k
 
 int b200_sink_attn_decode_tc(void* out, int64_t ldo, const float* q, const void* k_cache, const void* v_cache,
                              const float* r1, const float* r2, const float* sink, const void* gate, int64_t ld_gate,
-                             float out_mul, const int32_t* q_cu_lens, const int32_t* kv_cu_lens, const int32_t* block_tables, const int32_t* cu_block_lens,
+                             float out_mul, int gate_heads, int64_t window, const int32_t* q_cu_lens,
+                             const int32_t* kv_cu_lens, const int32_t* block_tables, const int32_t* cu_block_lens,
                              const int32_t* token_seq, int64_t rows, int64_t H, int64_t G, int64_t dim, int64_t vdim,
                              int64_t block_size, float scale, int64_t n_splits, float* workspace,
                              int64_t workspace_floats, int dtype, b200_stream_t stream) {
@@ -1013,7 +1188,9 @@ int b200_sink_attn_decode_tc(void* out, int64_t ldo, const float* q, const void*
   B200_CHECK_ARG(out && q && k_cache && v_cache && q_cu_lens && kv_cu_lens && block_tables && cu_block_lens && token_seq,
                  "sink_attn_decode_tc: null pointer");
   B200_CHECK_ARG((r1 == nullptr) == (r2 == nullptr), "sink_attn_decode_tc: the distance bias takes both of its numbers");
-  B200_CHECK_ARG(!gate || ld_gate >= H * vdim, "sink_attn_decode_tc: gate rows shorter than the heads");
+  B200_CHECK_ARG(!gate || ld_gate >= (gate_heads ? H : H * vdim), "sink_attn_decode_tc: gate rows shorter than the heads");
+  B200_CHECK_ARG(window >= 0 && window < (1ll << 30) && (k_cache != v_cache || dim == vdim),
+                 "sink_attn_decode_tc: bad window, or shared keys and values of different sizes");
   B200_CHECK_ARG(b200_sink_attn_prefill_supported(dim, vdim, dtype),
                  "sink_attn_decode_tc: bf16 with head sizes that are multiples of 16 and at most 128");
   B200_CHECK_ARG(rows > 0 && H > 0 && G > 0 && G <= 65535 && H % G == 0 && block_size > 0 && ldo >= H * vdim &&
@@ -1022,8 +1199,8 @@ int b200_sink_attn_decode_tc(void* out, int64_t ldo, const float* q, const void*
   B200_CHECK_ARG(n_splits == 1 || (workspace && workspace_floats >= rows * H * n_splits * (2 + vdim)),
                  "sink_attn_decode_tc: workspace of rows * H * n_splits * (2 + vdim) floats required");
   auto st = static_cast<cudaStream_t>(stream);
-#define SDT_ARGS out, ldo, q, k_cache, v_cache, r1, r2, sink, gate, ld_gate, out_mul, q_cu_lens, kv_cu_lens, \
-                 block_tables, cu_block_lens, token_seq, rows, (int)H, (int)G, (int)dim, (int)vdim, (int)block_size, scale, (int)n_splits, workspace, st
+#define SDT_ARGS out, ldo, q, k_cache, v_cache, r1, r2, sink, gate, ld_gate, out_mul, gate_heads, (int)window, \
+                 q_cu_lens, kv_cu_lens, block_tables, cu_block_lens, token_seq, rows, (int)H, (int)G, (int)dim, (int)vdim, (int)block_size, scale, (int)n_splits, workspace, st
   if (dim <= 64 && vdim <= 64) return launch_decode_tc<4, 4>(SDT_ARGS);
   return launch_decode_tc<8, 8>(SDT_ARGS);
 #undef SDT_ARGS

@@ -803,6 +803,17 @@ def delta_rule(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay_logits: 
     return out
 
 
+def matmul_f32(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """x W^T with fp32 results: 16-bit factors are multiplied exactly and summed in fp32 by the library product, fp32
+    ones in true fp32.  x [rows, K] with weight [N, K], or x [blocks, rows, K] (any strides) with weight [blocks, N, K]."""
+    _cuda(x, weight)
+    if x.dtype == torch.float32:
+        return torch.matmul(x, weight.transpose(-1, -2))
+    if x.dim() == 3:
+        return torch.bmm(x, weight.transpose(1, 2), out_dtype=torch.float32)
+    return torch.mm(x, weight.t(), out_dtype=torch.float32)
+
+
 # ---------------------------------------------------------------------------
 # mixture of experts (csrc/moe.cu)
 # ---------------------------------------------------------------------------
@@ -1084,6 +1095,35 @@ def mingru_scan(proj: torch.Tensor, z_bias: Optional[torch.Tensor], x_bias: Opti
     return out
 
 
+def real_gated_scan(u: torch.Tensor, y: torch.Tensor, gates: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor,
+                    lam: torch.Tensor, y_bias: Optional[torch.Tensor], rate: float, state: torch.Tensor,
+                    q_cu: torch.Tensor, positions: torch.Tensor, state_slots: torch.Tensor, n_seq: int, q_max: int = 0,
+                    chunk_len: int = 0) -> torch.Tensor:
+    """log a = rate sigmoid(gate_r + r_bias) softplus(lam) ; S <- a S + sqrt(1 - a^2) sigmoid(gate_i + i_bias) u ;
+    S * gelu_tanh(y + y_bias) per channel, [rows, width].  gates fp32 [blocks, rows, 2 width / blocks] (r before i); state
+    fp32 [slots, width].  Long portions run as chunks side by side, as in mingru_scan."""
+    _cuda(u, y, gates, state)
+    _f32(gates, r_bias, i_bias, lam, y_bias, state)
+    _check_i32(q_cu, positions, state_slots)
+    rows, width = u.shape
+    blocks = gates.shape[0]
+    assert u.stride(1) == 1 and y.stride(1) == 1 and y.shape == (rows, width) and y.dtype == u.dtype
+    assert gates.shape == (blocks, rows, 2 * width // blocks) and gates.is_contiguous() and state.shape[1] == width
+    assert r_bias.numel() == i_bias.numel() == lam.numel() == width
+    out = torch.empty((rows, width), dtype=u.dtype, device=u.device)
+    L, ws = 0, None
+    if chunk_len > 0 or q_max >= MINGRU_CHUNKED_MIN_ROWS:
+        L = chunk_len or MINGRU_CHUNK
+        q_max = q_max or rows
+        ws = torch.empty(_lib.load().b200_mingru_chunked_workspace_floats(n_seq, width, q_max, L), dtype=torch.float32,
+                         device=u.device)
+    check(_lib.load().b200_real_gated_scan(_p(out), width, _p(u), u.stride(0), _p(y), y.stride(0), _p(gates), rows, blocks,
+                                           _p(r_bias), _p(i_bias), _p(lam), _p(y_bias), rate, _p(state), _p(q_cu),
+                                           _p(positions), _p(state_slots), n_seq, width, q_max, L, _p(ws),
+                                           ws.numel() if ws is not None else 0, _dt(u), _stream()))
+    return out
+
+
 # ---------------------------------------------------------------------------
 # differential sliding-window attention (csrc/diff_attn.cu)
 # ---------------------------------------------------------------------------
@@ -1262,6 +1302,41 @@ def sink_attn_prepare_turned(q_in: torch.Tensor, k_in: torch.Tensor, v_in: torch
     return q
 
 
+def sink_attn_prepare_heads(q_in: torch.Tensor, k_in: torch.Tensor, v_in: Optional[torch.Tensor], k_cache: torch.Tensor,
+                            v_cache: Optional[torch.Tensor], positions: torch.Tensor, slots: torch.Tensor, H: int, G: int,
+                            dim: int, q_bias: Optional[torch.Tensor] = None, k_bias: Optional[torch.Tensor] = None,
+                            v_bias: Optional[torch.Tensor] = None, q_weight: Optional[torch.Tensor] = None,
+                            k_weight: Optional[torch.Tensor] = None, inv_freq: Optional[torch.Tensor] = None,
+                            rot_dims: int = 0, eps: float = 0.0, temp_coef: float = 0.0,
+                            temp_every: int = 0) -> torch.Tensor:
+    """Queries (fp32 [rows, H, dim]) and keys with optional biases, RMS norms per head (weights [dim]), half-pair turn of
+    the first rot_dims channels and query temperature; keys, and values where the projection has them, go to the cache
+    rows `slots`.  q_in, k_in, v_in: column blocks of one projection matrix."""
+    _cuda(q_in, k_in, v_in, k_cache, v_cache)
+    _f32(q_bias, k_bias, v_bias, q_weight, k_weight, inv_freq)
+    _check_i32(positions, slots)
+    rows, ld = q_in.shape[0], q_in.stride(0)
+    assert q_in.shape[1] == H * dim and k_in.shape[1] == G * dim and k_cache.shape[1:] == (G, dim)
+    assert q_bias is None or q_bias.numel() == H * dim
+    assert k_bias is None or k_bias.numel() == G * dim
+    assert q_weight is None or (q_weight.numel() == dim and k_weight.numel() == dim)
+    assert rot_dims == 0 or inv_freq.numel() == rot_dims // 2
+    vdim = dim
+    if v_in is not None:
+        vdim = v_cache.shape[2]
+        assert v_in.shape[1] == G * vdim and v_cache.shape[1] == G and v_cache.is_contiguous()
+        assert v_bias is None or v_bias.numel() == G * vdim
+    for t in (q_in, k_in) + ((v_in,) if v_in is not None else ()):
+        assert t.stride(1) == 1 and t.stride(0) == ld and t.dtype == k_cache.dtype
+    assert k_cache.is_contiguous()
+    q = torch.empty((rows, H, dim), dtype=torch.float32, device=q_in.device)
+    check(_lib.load().b200_sink_attn_prepare_heads(_p(q), _p(q_in), _p(k_in), _p(v_in), ld, _p(q_bias), _p(k_bias),
+                                                   _p(v_bias), _p(q_weight), _p(k_weight), _p(inv_freq), _p(k_cache),
+                                                   _p(v_cache), _p(positions), _p(slots), rows, H, G, dim, vdim, rot_dims,
+                                                   eps, temp_coef, temp_every, _dt(q_in), _stream()))
+    return q
+
+
 # a step whose longest portion has at least this many tokens runs the tensor-core kernel (bf16, fitting head sizes)
 SINK_ATTN_PREFILL_MIN_ROWS = 4
 # single tokens in bf16 with at least this many query heads per key/value head run as tensor-core tiles of heads
@@ -1273,14 +1348,15 @@ def sink_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, r1:
               block_tables: torch.Tensor, cu_block_lens: torch.Tensor, token_seq: torch.Tensor, block_size: int,
               scale: float, n_seq: int = 0, q_max: int = 0, kv_max: int = 0, n_splits: int = 0,
               gate: Optional[torch.Tensor] = None, out_mul: float = 1.0,
-              out: Optional[torch.Tensor] = None) -> torch.Tensor:
+              out: Optional[torch.Tensor] = None, window: int = 0) -> torch.Tensor:
     """[rows, H * vdim] in the cache's dtype (into `out` where given): causal softmax attention with the score scale q . k - r1 ln(1 + r2
     (i - j)) and exp(sink) added to the denominator (r1 / r2 / sink fp32 [H] or None).  With n_seq and q_max (the
     step's sequence count and longest portion, host numbers) a step with prompt portions in bf16 runs on the tensor
     cores where the head sizes allow it; single tokens in bf16 with grouped heads run as tensor-core tiles of heads,
     their keys shared out over several CTAs per row when the step has few rows (kv_max: an upper bound of the cached
     lengths, sizes the split; n_splits forces it); fp32 and odd sizes run the CUDA-core kernel.  What is stored is
-    out_mul * result * sigmoid(gate) (gate [rows, H * vdim], a column block, or None)."""
+    out_mul * result * sigmoid(gate) (gate [rows, H * vdim] or, one number per head, [rows, H], a column block, or None).
+    window > 0: row i sees the keys j > i - window only.  v_cache may be k_cache itself: the values are the keys."""
     _cuda(q, k_cache, v_cache, r1, r2, sink, gate, out)
     _f32(q, r1, r2, sink)
     _check_i32(q_cu, kv_cu, block_tables, cu_block_lens, token_seq)
@@ -1289,7 +1365,8 @@ def sink_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, r1:
     if out is None:
         out = torch.empty((rows, H * vdim), dtype=k_cache.dtype, device=q.device)
     assert out.shape == (rows, H * vdim) and out.stride(1) == 1 and out.dtype == k_cache.dtype
-    assert gate is None or (gate.shape == out.shape and gate.stride(1) == 1 and gate.dtype == out.dtype)
+    assert gate is None or (gate.shape in (out.shape, (rows, H)) and gate.stride(1) == 1 and gate.dtype == out.dtype)
+    gate_heads = 1 if gate is not None and gate.shape[1] == H and vdim > 1 else 0
     ldo, ldg = out.stride(0), gate.stride(0) if gate is not None else 0
     lib = _lib.load()
     impl = os.environ.get("B200_SINK_ATTN_IMPL")      # "simt": CUDA cores throughout; "simt_decode": for single tokens
@@ -1297,8 +1374,8 @@ def sink_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, r1:
             and ldo % 2 == 0 and out.data_ptr() % 4 == 0
             and lib.b200_sink_attn_prefill_supported(dim, vdim, _dt(k_cache))):
         check(lib.b200_sink_attn_prefill(_p(out), ldo, _p(q), _p(k_cache), _p(v_cache), _p(r1), _p(r2), _p(sink),
-                                         _p(gate), ldg, out_mul, _p(q_cu), _p(kv_cu), _p(block_tables), _p(cu_block_lens), n_seq, q_max, H, G,
-                                         dim, vdim, block_size, scale, _dt(k_cache), _stream()))
+                                         _p(gate), ldg, out_mul, gate_heads, window, _p(q_cu), _p(kv_cu),
+                                         _p(block_tables), _p(cu_block_lens), n_seq, q_max, H, G, dim, vdim, block_size, scale, _dt(k_cache), _stream()))
         return out
     if (impl not in ("simt", "simt_decode") and H // G >= SINK_ATTN_DECODE_TC_MIN_GROUP
             and lib.b200_sink_attn_prefill_supported(dim, vdim, _dt(k_cache))):
@@ -1306,20 +1383,21 @@ def sink_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, r1:
             # steps with fewer CTAs than SMs are split to about two CTAs per SM; walks of 32 tiles (2 048 keys) and
             # more are cut in four whatever the step's size (measured: a CTA's walk is bound by its own latency, and
             # four shorter walks per row keep three CTAs resident per SM); never fewer than two 64-key tiles a share
-            tiles = max(1, -(-kv_max // 64))
+            seen = min(kv_max, window + 63) if window > 0 else kv_max
+            tiles = max(1, -(-seen // 64))
             ctas = rows * G * -(-(H // G) // 16)
             n_splits = max(1, min(max(296 // ctas, 4 if tiles >= 32 else 1), tiles // 2, 64))
         ws = None
         if n_splits > 1:
             ws = torch.empty(rows * H * n_splits * (2 + vdim), dtype=torch.float32, device=q.device)
         check(lib.b200_sink_attn_decode_tc(_p(out), ldo, _p(q), _p(k_cache), _p(v_cache), _p(r1), _p(r2), _p(sink),
-                                           _p(gate), ldg, out_mul, _p(q_cu), _p(kv_cu), _p(block_tables), _p(cu_block_lens), _p(token_seq),
-                                           rows, H, G, dim, vdim, block_size, scale, n_splits, _p(ws),
+                                           _p(gate), ldg, out_mul, gate_heads, window, _p(q_cu), _p(kv_cu),
+                                           _p(block_tables), _p(cu_block_lens), _p(token_seq), rows, H, G, dim, vdim, block_size, scale, n_splits, _p(ws),
                                            ws.numel() if ws is not None else 0, _dt(k_cache), _stream()))
         return out
     check(lib.b200_sink_attn(_p(out), ldo, _p(q), _p(k_cache), _p(v_cache), _p(r1), _p(r2), _p(sink), _p(gate), ldg,
-                             out_mul, _p(q_cu), _p(kv_cu), _p(block_tables), _p(cu_block_lens), _p(token_seq), rows, H, G, dim, vdim,
-                             block_size, scale, _dt(k_cache), _stream()))
+                             out_mul, gate_heads, window, _p(q_cu), _p(kv_cu), _p(block_tables), _p(cu_block_lens),
+                             _p(token_seq), rows, H, G, dim, vdim, block_size, scale, _dt(k_cache), _stream()))
     return out
 
 
@@ -1497,6 +1575,21 @@ def moe_route_softmax(h: torch.Tensor, router_weight: torch.Tensor, correction: 
     return ids, wts, extra
 
 
+def moe_route_sigmoid(logits: torch.Tensor, top: int, n_groups: int = 1, keep_groups: int = 1, group_best: int = 1,
+                      weight_eps: float = 0.0, factor: float = 1.0):
+    """(ids [rows, top] int32, weights [rows, top] fp32) from router logits (fp32 [rows, E]): s = sigmoid(logits); runs of
+    neighbours score the sum of their group_best largest s and the keep_groups best of n_groups runs stay; the `top`
+    largest s are chosen; weights = factor * s / (sum of the chosen s + weight_eps)."""
+    _cuda(logits)
+    rows, E = logits.shape
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1
+    ids = torch.empty((rows, top), dtype=torch.int32, device=logits.device)
+    wts = torch.empty((rows, top), dtype=torch.float32, device=logits.device)
+    check(_lib.load().b200_moe_route_sigmoid(_p(ids), _p(wts), _p(logits), logits.stride(0), rows, E, top, n_groups,
+                                             keep_groups, group_best, weight_eps, factor, _stream()))
+    return ids, wts
+
+
 def moe_combine_weighted(y: torch.Tensor, pos_of_pair: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
                          n_real: int, h: torch.Tensor, addend: Optional[torch.Tensor] = None,
                          addend_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -1519,20 +1612,21 @@ def moe_combine_weighted(y: torch.Tensor, pos_of_pair: torch.Tensor, ids: torch.
 
 
 def branch_norm_residual(x: torch.Tensor, a: torch.Tensor, b: Optional[torch.Tensor], weight_a: Optional[torch.Tensor],
-                         weight_b: Optional[torch.Tensor], weight: torch.Tensor, weight_next: Optional[torch.Tensor],
-                         eps: float, x_out: Optional[torch.Tensor] = None, want_h: bool = True):
-    """m = (norm(a) weight_a + norm(b) weight_b) / 2 (one branch: norm(a) weight_a; no branch weight: a itself);
-    x_out (default: x, in place) = x + norm(m) weight; h = norm(x_out) weight_next, or x_out itself without
+                         weight_b: Optional[torch.Tensor], weight: Optional[torch.Tensor],
+                         weight_next: Optional[torch.Tensor], eps: float, x_out: Optional[torch.Tensor] = None,
+                         want_h: bool = True, bias_a: Optional[torch.Tensor] = None):
+    """m = (norm(a) weight_a + norm(b) weight_b) / 2 (one branch: norm(a) weight_a; no branch weight: a itself; bias_a [W]
+    joins a first); x_out (default: x, in place) = x + norm(m) weight, or x + m without weight; h = norm(x_out) weight_next, or x_out itself without
     weight_next, in a's dtype.  norm(z) = z / sqrt(mean(z^2) + eps).  Returns (x_out, h or None)."""
-    _cuda(x, a, b, weight_a, weight_b, weight, weight_next)
-    _f32(x, weight_a, weight_b, weight, weight_next)
+    _cuda(x, a, b, weight_a, weight_b, weight, weight_next, bias_a)
+    _f32(x, weight_a, weight_b, weight, weight_next, bias_a)
     rows, W = x.shape
     assert a.shape == (rows, W) and a.stride(1) == 1
     assert b is None or (b.shape == (rows, W) and b.stride(1) == 1 and b.dtype == a.dtype)
     out = x if x_out is None else x_out
     _f32(out)
     h = torch.empty((rows, W), dtype=a.dtype, device=x.device) if want_h else None
-    check(_lib.load().b200_branch_norm_residual(_p(out), _p(h), _p(x), _p(a), a.stride(0), _p(b),
+    check(_lib.load().b200_branch_norm_residual(_p(out), _p(h), _p(x), _p(a), a.stride(0), _p(bias_a), _p(b),
                                                 b.stride(0) if b is not None else 0, _p(weight_a), _p(weight_b),
                                                 _p(weight), _p(weight_next), rows, W, eps, _dt(a), _stream()))
     return out, h
@@ -1551,12 +1645,14 @@ def relu_squared(x: torch.Tensor) -> torch.Tensor:
 # pre-norm input side with short causal filters (csrc/filters.cu), linear recurrences with a matrix state
 # (csrc/linear_scan.cu)
 # ---------------------------------------------------------------------------
-def prenorm(x: torch.Tensor, y, weight: torch.Tensor, eps: float, dtype: torch.dtype,
+def prenorm(x: torch.Tensor, y, weight: Optional[torch.Tensor], eps: float, dtype: torch.dtype,
             filter: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None,
             q_cu: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None,
-            state_slots: Optional[torch.Tensor] = None, n_seq: int = 0, q_max: int = 0):
-    """x' = x + y (y: the rows of the sublayer before, the split-K partials of the product that makes them, or None),
-    h = x' / rms(x') * weight in `dtype`; with filter [taps, W] (fp32) h_t = n_t + sum_i filter[i] n_{t - taps + 1 + i}
+            state_slots: Optional[torch.Tensor] = None, n_seq: int = 0, q_max: int = 0,
+            out: Optional[torch.Tensor] = None):
+    """x' = x + y (y: the rows of the sublayer before, one row [W] for all, the split-K partials of the product that
+    makes them, or None), h = x' / rms(x') * weight in `dtype` (no weight: x' itself; `out`: where h goes, rows of any
+    stride); with filter [taps, W] (fp32) h_t = n_t + sum_i filter[i] n_{t - taps + 1 + i}
     over each sequence's rows, the lags before the step from state [slots, taps - 1, W] (which then takes the step's
     last rows).  Returns (x' — x itself where y is None —, h)."""
     partials = y.data if isinstance(y, W4Partials) else None
@@ -1564,9 +1660,11 @@ def prenorm(x: torch.Tensor, y, weight: torch.Tensor, eps: float, dtype: torch.d
     _cuda(x, rows_y, partials, weight, filter, state)
     _f32(x, weight, filter, state, partials)
     rows, W = x.shape
-    assert x.is_contiguous() and weight.numel() == W
+    assert x.is_contiguous() and (weight is None or weight.numel() == W)
+    ldy = 0
     if rows_y is not None:
-        assert rows_y.shape == (rows, W) and rows_y.stride(1) == 1 and rows_y.dtype == dtype
+        assert rows_y.shape in ((rows, W), (W,)) and rows_y.stride(-1) == 1 and rows_y.dtype == dtype
+        ldy = rows_y.stride(0) if rows_y.dim() == 2 else 0
     if partials is not None:
         assert partials.shape[1:] == (rows, W)
     taps = 0
@@ -1575,33 +1673,34 @@ def prenorm(x: torch.Tensor, y, weight: torch.Tensor, eps: float, dtype: torch.d
         taps = filter.shape[0]
         assert filter.shape == (taps, W) and filter.is_contiguous() and n_seq > 0 and q_max > 0
         assert taps == 1 or (state.shape[1:] == (taps - 1, W) and state.is_contiguous())
-    out = torch.empty_like(x) if y is not None else x
-    h = torch.empty((rows, W), dtype=dtype, device=x.device)
-    check(_lib.load().b200_prenorm(_p(out) if y is not None else None, _p(h), _p(x), _p(rows_y),
-                                   rows_y.stride(0) if rows_y is not None else 0, _p(partials),
+    x_out = torch.empty_like(x) if y is not None else x
+    h = out if out is not None else torch.empty((rows, W), dtype=dtype, device=x.device)
+    assert h.shape == (rows, W) and h.stride(1) == 1 and h.dtype == dtype
+    check(_lib.load().b200_prenorm(_p(x_out) if y is not None else None, _p(h), h.stride(0), _p(x), _p(rows_y), ldy,
+                                   _p(partials),
                                    partials.shape[0] if partials is not None else 0,
                                    splitk_plan(W, y.K) if partials is not None else None, _p(weight), _p(filter), taps,
                                    _p(state), _p(q_cu), _p(positions), _p(state_slots), n_seq, q_max, rows, W, eps,
                                    _DT[dtype], _stream()))
-    return out, h
+    return x_out, h
 
 
 def causal_filter(x: torch.Tensor, filter: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor,
                   q_cu: torch.Tensor, positions: torch.Tensor, state_slots: torch.Tensor, n_seq: int, q_max: int,
-                  silu: bool) -> torch.Tensor:
-    """act(bias + sum_i filter[i] x_{t - taps + 1 + i}) per channel over each sequence's rows (filter [taps, channels]
+                  silu: bool, in_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """act(bias + sum_i filter[i] (x + in_bias)_{t - taps + 1 + i}) per channel over each sequence's rows (filter [taps, channels]
     fp32); the lags before the step come from state [slots, taps - 1, channels] fp32, which then takes the step's last
     rows.  x may be a column block."""
-    _cuda(x, filter, bias, state)
-    _f32(filter, bias, state)
+    _cuda(x, filter, bias, in_bias, state)
+    _f32(filter, bias, in_bias, state)
     _check_i32(q_cu, positions, state_slots)
     rows, ch = x.shape
     taps = filter.shape[0]
     assert x.stride(1) == 1 and filter.shape == (taps, ch) and filter.is_contiguous()
-    assert bias is None or bias.numel() == ch
+    assert (bias is None or bias.numel() == ch) and (in_bias is None or in_bias.numel() == ch)
     assert taps == 1 or (state.shape[1:] == (taps - 1, ch) and state.is_contiguous())
     out = torch.empty((rows, ch), dtype=x.dtype, device=x.device)
-    check(_lib.load().b200_causal_filter(_p(out), ch, _p(x), x.stride(0), _p(filter), _p(bias), taps, _p(state),
+    check(_lib.load().b200_causal_filter(_p(out), ch, _p(x), x.stride(0), _p(filter), _p(in_bias), _p(bias), taps, _p(state),
                                          _p(q_cu), _p(positions), _p(state_slots), n_seq, q_max, rows, ch,
                                          1 if silu else 0, _dt(x), _stream()))
     return out
@@ -1665,13 +1764,47 @@ def ssd_scan(x: torch.Tensor, B: torch.Tensor, C_: torch.Tensor, dt: torch.Tenso
     return y
 
 
-def gated_part_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, parts: int, eps: float) -> torch.Tensor:
-    """u = y silu(z) ; u / rms_part(u) * weight with one root mean square per equal part of the row, in z's dtype."""
+def memory_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, i_logits: torch.Tensor, f_logits: torch.Tensor,
+                i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, q_scale: float, state: torch.Tensor,
+                key_sum: torch.Tensor, q_cu: torch.Tensor, positions: torch.Tensor, state_slots: torch.Tensor,
+                n_seq: int, q_max: int) -> torch.Tensor:
+    """Matrix memory with exponential gates: f = log sigmoid(cap tanh((f_logits + f_bias) / cap)), i = cap tanh((i_logits
+    + i_bias) / cap), m' = max(f + m, i), (S, n) <- exp(f + m - m') (S, n) + exp(i - m') k (v^T, 1), read out at q_scale q
+    and divided by max(|n . q|, exp(-m')) + 1e-6; fp32 [rows, H * V].  state [slots, H, N, V] (S) and key_sum
+    [slots, H, memory_parts(N, V), N + 1] (n and m) fp32; gate logits fp32 [rows, H] of one matrix."""
+    _cuda(q, k, v, i_logits, f_logits, i_bias, f_bias, state, key_sum)
+    _f32(i_bias, f_bias, state, key_sum)
+    _check_i32(q_cu, positions, state_slots)
+    H, N, V = state.shape[1:]
+    rows, ld = q.shape[0], q.stride(0)
+    for t, n in ((q, H * N), (k, H * N), (v, H * V)):
+        assert t.shape == (rows, n) and t.stride(1) == 1 and t.stride(0) == ld and t.dtype == q.dtype
+    for t in (i_logits, f_logits):
+        assert t.shape == (rows, H) and t.dtype == torch.float32 and t.stride(1) == 1 and t.stride(0) == i_logits.stride(0)
+    assert i_bias.numel() == f_bias.numel() == H and state.is_contiguous() and key_sum.is_contiguous()
+    assert key_sum.shape[1:] == (H, memory_parts(N, V), N + 1)
+    y = torch.empty((rows, H * V), dtype=torch.float32, device=q.device)
+    check(_lib.load().b200_memory_scan(_p(y), _p(q), _p(k), _p(v), ld, _p(i_logits), _p(f_logits), i_logits.stride(0),
+                                       _p(i_bias), _p(f_bias), cap, q_scale, _p(state), _p(key_sum), _p(q_cu),
+                                       _p(positions), _p(state_slots), n_seq, q_max, rows, H, N, V,
+                                       1 if _scan_tc(q_max, N, V, ld, q, k, v) else 0, _dt(q), _stream()))
+    return y
+
+
+def memory_parts(N: int, V: int) -> int:
+    """Copies of n and m a matrix memory of these sizes keeps (column parts of its walk)."""
+    return int(_lib.load().b200_linear_scan_parts(N, V))
+
+
+def gated_part_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, parts: int, eps: float,
+                    gate_after: bool = False) -> torch.Tensor:
+    """u = y silu(z) ; u / rms_part(u) * weight with one root mean square per equal part of the row, in z's dtype;
+    gate_after: y / rms_part(y) * weight * sigmoid(z)."""
     _cuda(y, z, weight)
     _f32(y, weight)
     rows, n = y.shape
     assert y.is_contiguous() and z.shape == (rows, n) and z.stride(1) == 1 and weight.numel() == n
     out = torch.empty((rows, n), dtype=z.dtype, device=z.device)
     check(_lib.load().b200_gated_part_norm(_p(out), n, _p(y), _p(z), z.stride(0), _p(weight), rows, n, parts, eps,
-                                           _dt(z), _stream()))
+                                           1 if gate_after else 0, _dt(z), _stream()))
     return out

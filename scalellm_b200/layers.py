@@ -60,12 +60,13 @@ class KVCache:
     """Per-layer K and V tensors [n_blocks*block_size, n_kv_heads, head_dim] (kv_cache.cpp:15-27)."""
 
     def __init__(self, n_blocks: int, block_size: int, n_kv_heads: int, head_dim: int,
-                 dtype: torch.dtype, device, value_dim: Optional[int] = None):
-        """value_dim: width of a value head where it differs from the key head's (default: the same)."""
+                 dtype: torch.dtype, device, value_dim: Optional[int] = None, shared: bool = False):
+        """value_dim: width of a value head where it differs from the key head's (default: the same).  shared: the
+        values are the keys, one tensor serves as both."""
         self._block_size = block_size
         self.key_cache = torch.empty((n_blocks * block_size, n_kv_heads, head_dim), dtype=dtype,
                                      device=device)
-        self.value_cache = (torch.empty_like(self.key_cache) if value_dim is None else
+        self.value_cache = (self.key_cache if shared else torch.empty_like(self.key_cache) if value_dim is None else
                             torch.empty((n_blocks * block_size, n_kv_heads, value_dim), dtype=dtype, device=device))
 
     def block_size(self) -> int:
@@ -629,6 +630,39 @@ class Linear:
     __call__ = forward
 
 
+class LinearF32:
+    """y = x W^T with fp32 results whatever the model dtype is (routers, gates of recurrences): a weight that 16 bits
+    hold exactly meets the 16-bit rows as it is (exact products, fp32 sums), any other one in fp32.  weight [out, in], or
+    [blocks, out, in] for a block-diagonal map of rows x [rows, blocks * in] -> [blocks, rows, out]."""
+
+    def __init__(self, weight: torch.Tensor, dtype: torch.dtype):
+        w = weight.to(dtype)
+        self.weight = (w if torch.equal(w.to(torch.float32), weight.to(torch.float32)) else weight.to(torch.float32)).contiguous()
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        if self.weight.dim() == 3:
+            nb, _, k = self.weight.shape
+            x = x.reshape(x.shape[0], nb, k).transpose(0, 1)
+        return kernels.matmul_f32(x.to(self.weight.dtype), self.weight)
+
+    __call__ = forward
+
+
+def stack_rows(parts, multiple: int = 1) -> torch.Tensor:
+    """Weights [out_i, in] one below the other, filled up with rows of zeros to a multiple of `multiple`."""
+    n = sum(p.shape[0] for p in parts)
+    pad = -n % multiple
+    if pad:
+        parts = list(parts) + [torch.zeros((pad, parts[0].shape[1]), dtype=parts[0].dtype, device=parts[0].device)]
+    return torch.cat(list(parts), dim=0)
+
+
+def input_rows_multiple(n: int) -> int:
+    """What the rows of an input product are padded to: whole 128-row tiles where that costs little (the stream kernel of
+    decode-sized steps takes no others), else 8, which keeps the products' rows on 16 bytes."""
+    return 128 if n >= 1024 else 8
+
+
 class LatentKVCache:
     """One row [latent (rank) | rotary key (rot_dim)] per cached token: [n_blocks * block_size, rank + rot_dim]."""
 
@@ -1042,20 +1076,21 @@ class TableMoE:
 # tokens to experts with a softmax router under group limits.
 # ---------------------------------------------------------------------------
 class BranchNormResidual:
-    """x <- x + norm(m) w on an fp32 residual, where m is a sublayer's result, or the average of two results each
-    normalised with its own weight first: m = (norm(a) wa + norm(b) wb) / 2.  norm(z) = z / sqrt(mean(z^2) + eps).
-    The new residual is handed on under the next sublayer's input norm (next_weight) or as it is."""
+    """x <- x + norm(m) w (no w: x + m) on an fp32 residual, where m is a sublayer's result, or the average of two results
+    each normalised with its own weight first: m = (norm(a + bias_a) wa + norm(b) wb) / 2.  norm(z) = z / sqrt(mean(z^2) +
+    eps).  The new residual is handed on under the next sublayer's input norm (next_weight) or as it is."""
 
-    def __init__(self, weight: torch.Tensor, eps: float, weight_a: Optional[torch.Tensor] = None,
-                 weight_b: Optional[torch.Tensor] = None):
+    def __init__(self, weight: Optional[torch.Tensor], eps: float, weight_a: Optional[torch.Tensor] = None,
+                 weight_b: Optional[torch.Tensor] = None, bias_a: Optional[torch.Tensor] = None):
         f = lambda t: None if t is None else t.to(torch.float32).contiguous()
+        self.bias_a = f(bias_a)
         self.weight, self.weight_a, self.weight_b, self.eps = f(weight), f(weight_a), f(weight_b), eps
 
     def forward(self, x: torch.Tensor, a: torch.Tensor, b: Optional[torch.Tensor] = None,
                 next_weight: Optional[torch.Tensor] = None, want_h: bool = True):
         """Returns (new x fp32, the rows the next matrix product reads in a's dtype, or None if not wanted)."""
         return kernels.branch_norm_residual(x, a, b, self.weight_a, self.weight_b if b is not None else None,
-                                            self.weight, next_weight, self.eps, want_h=want_h)
+                                            self.weight, next_weight, self.eps, want_h=want_h, bias_a=self.bias_a)
 
     __call__ = forward
 
@@ -1165,17 +1200,18 @@ class GatedDeltaMixer:
 class ParallelMixer:
     """Two mixers side by side on the same rows: an attention-like one with a paged cache (`left`) and a recurrent one
     with state slots (`right`).  Everything that reads h is ONE matrix product; the results come back as a pair (the
-    caller's BranchNormResidual normalises and averages them)."""
+    caller's BranchNormResidual normalises and averages them).  rows_multiple: what that product's rows are padded to.
+    right_args of a step go to the right half (its state where the layer does not hold it, h)."""
 
-    def __init__(self, left, right):
+    def __init__(self, left, right, rows_multiple: int = 1):
         self.left, self.right = left, right
-        self.in_proj = Linear(torch.cat([left.in_weight, right.in_weight], dim=0))
+        self.in_proj = Linear(stack_rows([left.in_weight, right.in_weight], rows_multiple))
 
-    def forward(self, h: torch.Tensor, positions: torch.Tensor, cache: KVCache, params: InputParameters):
+    def forward(self, h: torch.Tensor, positions: torch.Tensor, cache: KVCache, params: InputParameters, *right_args):
         proj = self.in_proj(h)
         n = self.left.n_in
         return (self.left.run(proj[:, :n], positions, cache, params),
-                self.right.run(proj[:, n:], positions, params))
+                self.right.run(proj[:, n: n + self.right.n_in], positions, params, *right_args))
 
     __call__ = forward
 
@@ -1376,5 +1412,205 @@ class StateSpaceMixer:
                              self.dt_bias, self.a_log, self.skip, self.state, *step, self.groups)
         return self.o_proj.forward_fusable(kernels.gated_part_norm(y, proj[:, :inner], self.norm_weight, self.parts,
                                                                    self.eps))
+
+    __call__ = forward
+
+
+# ---------------------------------------------------------------------------
+# Layers of decoders that run some of their layers several times: weights are held once, so every class below leaves its
+# state per sequence (new_state) to the caller, one for each run.
+# ---------------------------------------------------------------------------
+class LoopInput:
+    """What a pass over looped layers starts from: x <- W_in [x ; x0], x0 a row kept from before (fp32 residuals; the
+    product reads 16-bit rows in a 16-bit model and leaves fp32)."""
+
+    def __init__(self, weight: torch.Tensor, dtype: torch.dtype):
+        self.proj, self.dtype, self.width = LinearF32(weight, dtype), dtype, weight.shape[0]
+
+    def start(self, x0: torch.Tensor) -> torch.Tensor:
+        """The step's rows [x ; x0], with x0 in place."""
+        both = torch.empty((x0.shape[0], 2 * self.width), dtype=self.dtype, device=x0.device)
+        kernels.prenorm(x0, None, None, 0.0, self.dtype, out=both[:, self.width:])
+        return both
+
+    def forward(self, x: torch.Tensor, y, both: torch.Tensor):
+        """y: what the sublayer before made.  Returns (x + y, the pass's first x)."""
+        x, _ = kernels.prenorm(x, y, None, 0.0, self.dtype, out=both[:, : self.width])
+        return x, self.proj(both)
+
+    __call__ = forward
+
+
+class SharedKVAttention:
+    """Causal softmax attention whose values are its keys (csrc/sink_attn.cu; cache: KVCache(shared=True)):
+        q, k = affine maps of h, q_i *= 1 + temp_coef ln(floor((i + 1) / temp_every) + 1)        (temp_every 0: none)
+        p_j = exp(scale q . k_j) / (exp(sink_h) + sum_j' exp(scale q . k_j'))                    ("sink" [H], optional)
+        result = Wo concat_h(sigmoid(Wg h)_h sum_j p_j k_j),  H / G query heads per key/value head, no rotary turn.
+    The output map's bias ("o.b") belongs to the caller.  `in_weight` [n_in, W] is everything that reads h (see
+    SigmoidBlockAttention)."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], n_heads: int, n_kv_heads: int, dim: int, scale: float,
+                 temp_coef: float, temp_every: int, dtype: torch.dtype, device):
+        self.H, self.G, self.dim, self.scale = n_heads, n_kv_heads, dim, scale
+        self.temp_coef, self.temp_every = temp_coef, temp_every
+        self.q_end = n_heads * dim
+        self.k_end = self.q_end + n_kv_heads * dim
+        self.in_weight = stack_rows([w["q"], w["k"], w["g"]], 8)
+        self.n_in = self.in_weight.shape[0]
+        f = lambda name: w[name].to(torch.float32).to(device).contiguous() if name in w else None
+        self.q_bias, self.k_bias, self.sink = f("q.b"), f("k.b"), f("sink")
+        self.o_proj = Linear(w["o"])
+
+    def run(self, proj: torch.Tensor, positions: torch.Tensor, cache: KVCache, params: InputParameters) -> torch.Tensor:
+        """proj [rows, n_in]: this mixer's column block of the input product (without biases)."""
+        q = kernels.sink_attn_prepare_heads(proj[:, : self.q_end], proj[:, self.q_end: self.k_end], None, cache.key_cache,
+                                            None, positions, params.new_cache_slots, self.H, self.G, self.dim,
+                                            self.q_bias, self.k_bias, temp_coef=self.temp_coef,
+                                            temp_every=self.temp_every)
+        o = kernels.sink_attn(q, cache.key_cache, cache.value_cache, None, None, self.sink, params.q_cu_seq_lens,
+                              params.kv_cu_seq_lens, params.block_tables, params.cu_block_lens, params.token_seq,
+                              cache.block_size(), self.scale, params.num_sequences, params.q_max_seq_len,
+                              params.kv_max_seq_len, gate=proj[:, self.k_end: self.k_end + self.H])
+        return self.o_proj(o)
+
+
+class MatrixMemoryMixer:
+    """Matrix memory with exponential gates and a running maximum (csrc/linear_scan.cu):
+        q, k [heads x dim], v [heads x vdim] = maps of h ; i = cap tanh((Wi h + bi) / cap) ,
+        f = log sigmoid(cap tanh((Wf h + bf) / cap)) ; m' = max(f + m, i) ;
+        (S, n) <- exp(f + m - m') (S, n) + exp(i - m') k (v^T, 1) ; o = S^T q' / (max(|n . q'|, exp(-m')) + 1e-6), q' = q / sqrt(dim)
+        result = Wo (concat_h(o / rms(o)) * norm * sigmoid(Wg h)).
+    The gate logits are fp32 products.  State per slot: S, and n with m."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], n_heads: int, dim: int, vdim: int, cap: float, eps: float,
+                 dtype: torch.dtype, device):
+        self.H, self.dim, self.vd, self.cap, self.eps, self.device = n_heads, dim, vdim, cap, eps, device
+        self.in_weight = torch.cat([w["q"], w["k"], w["v"], w["g"]], dim=0)
+        self.n_in = self.in_weight.shape[0]
+        self.gates = LinearF32(torch.cat([w["i"], w["f"]], dim=0), dtype)
+        f = lambda name: w[name].to(torch.float32).to(device).contiguous()
+        self.i_bias, self.f_bias, self.norm_weight = f("i.b"), f("f.b"), f("norm")
+        self.o_proj = Linear(w["o"])
+
+    def new_state(self, n_slots: int):
+        parts = kernels.memory_parts(self.dim, self.vd)
+        return (torch.zeros((n_slots, self.H, self.dim, self.vd), dtype=torch.float32, device=self.device),
+                torch.zeros((n_slots, self.H, parts, self.dim + 1), dtype=torch.float32, device=self.device))
+
+    def run(self, proj: torch.Tensor, positions: torch.Tensor, params: InputParameters, h: torch.Tensor,
+            state) -> torch.Tensor:
+        """proj [rows, n_in]: this mixer's column block of the input product; h: the rows it was made from."""
+        n, nv = self.H * self.dim, self.H * self.vd
+        z = self.gates(h)
+        o = kernels.memory_scan(proj[:, :n], proj[:, n: 2 * n], proj[:, 2 * n: 2 * n + nv], z[:, : self.H], z[:, self.H:],
+                                self.i_bias, self.f_bias, self.cap, self.dim ** -0.5, state[0], state[1],
+                                params.q_cu_seq_lens, positions, params.state_slots, params.num_sequences,
+                                params.q_max_seq_len)
+        return self.o_proj(kernels.gated_part_norm(o, proj[:, 2 * n + nv: self.n_in], self.norm_weight, self.H, self.eps,
+                                                   gate_after=True))
+
+
+class RealGatedMixer:
+    """Real-gated linear recurrence behind a short filter (csrc/mingru.cu, csrc/filters.cu):
+        y = gelu_tanh(Wy h + by) ; u = filter(Wx h + bx) + bc, filter [channels, taps] causal ;
+        r, i = sigmoid(R u + br), sigmoid(I u + bi) with R and I block-diagonal ("ra", "ri" [blocks, n, n]) ;
+        log a = rate r softplus(lam) ; S <- a S + sqrt(1 - a^2) i u per channel ; result = Wo (S y).
+    The gates' logits are fp32 products.  State per slot: the last taps - 1 filter inputs, and S."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], rate: float, dtype: torch.dtype, device):
+        self.width, self.rate, self.device = w["y"].shape[0], rate, device
+        self.in_proj = Linear(stack_rows([w["y"], w["x"]], input_rows_multiple(2 * self.width)))
+        f = lambda name: w[name].to(torch.float32).to(device).contiguous()
+        self.y_bias, self.x_bias, self.filter_bias, self.lam = f("y.b"), f("x.b"), f("conv.b"), f("lam")
+        self.filter = f("conv").t().contiguous()
+        self.gates = LinearF32(torch.cat([w["ra"], w["ri"]], dim=1), dtype)            # [blocks, 2 n, n]
+        self.r_bias, self.i_bias = f("ra.b").reshape(-1), f("ri.b").reshape(-1)
+        self.o_proj = Linear(w["o"])
+
+    def new_state(self, n_slots: int):
+        return (torch.zeros((n_slots, self.filter.shape[0] - 1, self.width), dtype=torch.float32, device=self.device),
+                torch.zeros((n_slots, self.width), dtype=torch.float32, device=self.device))
+
+    def forward(self, h: torch.Tensor, positions: torch.Tensor, params: InputParameters, state):
+        """The result, or the output product's split-K partials where a fused consumer can take them."""
+        proj, n = self.in_proj(h), self.width
+        u = kernels.causal_filter(proj[:, n: 2 * n], self.filter, self.filter_bias, state[0], params.q_cu_seq_lens,
+                                  positions, params.state_slots, params.num_sequences, params.q_max_seq_len, silu=False,
+                                  in_bias=self.x_bias)
+        o = kernels.real_gated_scan(u, proj[:, :n], self.gates(u), self.r_bias, self.i_bias, self.lam, self.y_bias,
+                                    self.rate, state[1], params.q_cu_seq_lens, positions, params.state_slots,
+                                    params.num_sequences, params.q_max_seq_len)
+        return self.o_proj.forward_fusable(o)
+
+    __call__ = forward
+
+
+class FilteredWindowAttention:
+    """Softmax attention inside a sliding window on filtered projections (csrc/filters.cu, csrc/sink_attn.cu):
+        q, k, v = filter(W h + b), one causal filter [channels, taps] each ; q and k under RMS norms per head ("q.norm",
+        "k.norm" [dim]) ; the first rot_dims channels of every q and k head turn with the position (channel t with
+        t + rot_dims / 2) ; softmax of scale q . k over the keys j > i - window (window 0: all) ; result = Wo concat_h(.).
+    State per slot: the last taps - 1 projected rows."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], n_heads: int, n_kv_heads: int, dim: int, vdim: int, scale: float,
+                 window: int, inv_freq: Optional[torch.Tensor], rot_dims: int, eps: float, dtype: torch.dtype, device):
+        self.H, self.G, self.dim, self.vd = n_heads, n_kv_heads, dim, vdim
+        self.scale, self.window, self.rot_dims, self.eps, self.device = scale, window, rot_dims, eps, device
+        self.inv_freq = None if inv_freq is None else inv_freq.to(torch.float32).to(device).contiguous()
+        self.q_end = n_heads * dim
+        self.k_end = self.q_end + n_kv_heads * dim
+        self.v_end = self.k_end + n_kv_heads * vdim
+        self.in_proj = Linear(stack_rows([w["q"], w["k"], w["v"]], input_rows_multiple(self.v_end)))
+        f = lambda t: t.to(torch.float32).to(device).contiguous()
+        self.in_bias = f(torch.cat([w["q.b"], w["k.b"], w["v.b"]]))
+        self.filter = f(torch.cat([w["q.conv"], w["k.conv"], w["v.conv"]], dim=0).t())
+        self.q_norm, self.k_norm = f(w["q.norm"]), f(w["k.norm"])
+        self.o_proj = Linear(w["o"])
+
+    def new_state(self, n_slots: int):
+        return torch.zeros((n_slots, self.filter.shape[0] - 1, self.v_end), dtype=torch.float32, device=self.device)
+
+    def forward(self, h: torch.Tensor, positions: torch.Tensor, cache: KVCache, params: InputParameters, state):
+        """The result, or the output product's split-K partials where a fused consumer can take them."""
+        z = kernels.causal_filter(self.in_proj(h)[:, : self.v_end], self.filter, None, state, params.q_cu_seq_lens,
+                                  positions, params.state_slots, params.num_sequences, params.q_max_seq_len, silu=False,
+                                  in_bias=self.in_bias)
+        q = kernels.sink_attn_prepare_heads(z[:, : self.q_end], z[:, self.q_end: self.k_end], z[:, self.k_end:],
+                                            cache.key_cache, cache.value_cache, positions, params.new_cache_slots, self.H,
+                                            self.G, self.dim, q_weight=self.q_norm, k_weight=self.k_norm,
+                                            inv_freq=self.inv_freq, rot_dims=self.rot_dims, eps=self.eps)
+        o = kernels.sink_attn(q, cache.key_cache, cache.value_cache, None, None, None, params.q_cu_seq_lens,
+                              params.kv_cu_seq_lens, params.block_tables, params.cu_block_lens, params.token_seq,
+                              cache.block_size(), self.scale, params.num_sequences, params.q_max_seq_len,
+                              params.kv_max_seq_len, window=self.window)
+        return self.o_proj.forward_fusable(o)
+
+    __call__ = forward
+
+
+class GroupSigmoidMoE:
+    """Token-choice squared-ReLU experts behind a sigmoid router (csrc/moe.cu):
+        s = sigmoid(R h) in fp32 ; the experts form n_groups equal runs of neighbours, a run scores the sum of its
+        group_best largest s, only experts of the keep_groups best runs can be chosen ; the `top` largest s are chosen ;
+        weight = factor * s / (sum of the chosen s + weight_eps) ; out = sum weight * down_e(max(up_e h, 0)^2) (+ shared(h)).
+    Expert weights are stacked [E, ...]; pairs are grouped by expert on the device (no host sync)."""
+
+    def __init__(self, router: torch.Tensor, up: torch.Tensor, down: torch.Tensor, top: int, n_groups: int,
+                 keep_groups: int, group_best: int, weight_eps: float, factor: float, dtype: torch.dtype,
+                 shared: Optional["ReluSquaredMLP"] = None):
+        self.router = LinearF32(router, dtype)
+        self.up, self.down = up.contiguous(), down.contiguous()        # [E, ff, W], [E, W, ff]
+        self.E, self.top, self.n_groups, self.keep_groups = up.shape[0], top, n_groups, keep_groups
+        self.group_best, self.weight_eps, self.factor, self.shared = group_best, weight_eps, factor, shared
+
+    def forward(self, h: torch.Tensor) -> torch.Tensor:
+        ids, wts = kernels.moe_route_sigmoid(self.router(h), self.top, self.n_groups, self.keep_groups, self.group_best,
+                                             self.weight_eps, self.factor)
+        offsets, sorted_pair, pos_of_pair = kernels.moe_plan(ids, self.E)
+        n = h.shape[0] * self.top
+        u = kernels.grouped_gemm(h, self.up, offsets, n, sorted_pair, None, self.top)
+        y = kernels.grouped_gemm(kernels.relu_squared(u), self.down, offsets, n)
+        shared = self.shared(h) if self.shared is not None else None
+        return kernels.moe_combine_weighted(y, pos_of_pair, ids, wts, self.E, h, shared)
 
     __call__ = forward

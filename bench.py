@@ -60,9 +60,9 @@ def parse():
     ap.add_argument("--layers", type=int, default=None, help="debug only; the default is the named config")
     ap.add_argument("--no-graph", action="store_true")
     ap.add_argument("--skip-cpu-baseline", action="store_true")
-    ap.add_argument("--arch", default="llama", choices=["llama", "kigalix", "pokadra", "zomurax", "fesupel", "gugalorn"],
-                    help="kigalix / pokadra / zomurax / fesupel / gugalorn: prefill / decode throughput of that design beside the Llama "
-                         "decoder (zomurax and fesupel also beside kigalix, gugalorn beside fesupel) at equal size through the serving engine (scalellm_b200/arch_bench.py); the default "
+    ap.add_argument("--arch", default="llama", choices=["llama", "kigalix", "pokadra", "zomurax", "fesupel", "gugalorn", "palulorn"],
+                    help="kigalix / pokadra / zomurax / fesupel / gugalorn / palulorn: prefill / decode throughput of that design beside the Llama "
+                         "decoder (zomurax and fesupel also beside kigalix, gugalorn beside fesupel, palulorn beside fesupel, gugalorn and pokadra) at equal size through the serving engine (scalellm_b200/arch_bench.py); the default "
                          "workload and its JSON line are untouched")
     ap.add_argument("--arch-size", default="all", choices=["all", "w2048", "w4096"])
     ap.add_argument("--arch-batch", type=int, default=16)
@@ -714,6 +714,10 @@ def main():
     if a.arch == "gugalorn":
         from scalellm_b200 import arch_bench
         arch_bench.run_gugalorn(a)
+        return
+    if a.arch == "palulorn":
+        from scalellm_b200 import arch_bench
+        arch_bench.run_palulorn(a)
         return
     if a.arch == "pokadra":
         from scalellm_b200 import arch_bench

@@ -1,6 +1,6 @@
-"""Prefill and decode throughput of the Kigalix, Pokadra, Zomurax, Fesupel and Gugalorn designs beside the Llama decoder
-(Zomurax and Fesupel also beside Kigalix, Gugalorn beside Fesupel: the designs nearest to them) at equal size (`bench.py
---arch kigalix|pokadra|zomurax|fesupel|gugalorn`), all through the serving engine, random weights, bf16.
+"""Prefill and decode throughput of the Kigalix, Pokadra, Zomurax, Fesupel, Gugalorn and Palulorn designs beside the Llama
+decoder (Zomurax and Fesupel also beside Kigalix, Gugalorn beside Fesupel, Palulorn beside Fesupel, Gugalorn and Pokadra:
+the designs nearest to them) at equal size (`bench.py --arch kigalix|pokadra|zomurax|fesupel|gugalorn|palulorn`), all through the serving engine, random weights, bf16.
 
 Per size: tokens/s of a prompt step (B sequences of L tokens in one batch) and of decode steps (B sequences
 with L cached tokens, one token each), timed with CUDA events after warm-up; and, per kind of kernel, the
@@ -54,11 +54,14 @@ class KernelTimer:
         self.events: Dict[str, List] = {}
         self._undo: List = []
 
-    def wrap(self, owner, names: List[str], label: Callable[[str], str] = lambda n: n) -> None:
+    def wrap(self, owner, names: List[str], label: Callable[[str], str] = lambda n: n,
+             tag: Callable[[str, tuple, dict], str] = lambda n, a, k: "") -> None:
+        """tag(name, args, kwargs) is added to the label: calls of one function with different jobs are kept apart."""
         for n in names:
             fn = getattr(owner, n)
 
-            def timed(*a, __fn=fn, __l=label(n), **k):
+            def timed(*a, __fn=fn, __n=n, __l=label(n), **k):
+                __l = __l + tag(__n, a, k)
                 e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
                 e0.record()
                 out = __fn(*a, **k)
@@ -78,6 +81,12 @@ class KernelTimer:
         out = {k: sum(a.elapsed_time(b) for a, b in v) for k, v in self.events.items()}
         self.events = {}
         return out
+
+
+def _job(name: str, args: tuple, kwargs: dict) -> str:
+    if name == "matmul_f32":
+        return " " + "x".join(str(n) for n in args[1].shape)
+    return " (window)" if kwargs.get("window") else ""
 
 
 def _time_steps(fn: Callable[[], None], warmup: int, steps: int) -> float:
@@ -129,7 +138,7 @@ def _run_model(config: dict, batch: int, seqlen: int, warmup: int, steps: int, k
     res["decode"] = {"ms_per_step": ms, "tokens_per_s": batch / ms * 1e3}
     # per-kernel device time of one prompt step and one decode step
     timer = KernelTimer()
-    timer.wrap(kernels, kernel_names)
+    timer.wrap(kernels, kernel_names, tag=_job)
     timer.wrap(kernels, ["dense_gemm", "dense_gemm_splitk"], lambda n: "linear (dense GEMMs)")
     timer.wrap(torch.nn.functional, ["linear"], lambda n: "linear (dense GEMMs)")
     timer.wrap(torch, ["bmm"], lambda n: "bmm (per-head key / value maps)")
@@ -992,5 +1001,211 @@ def run_gugalorn(args) -> None:
         out["sizes"][name] = {"shape": s, "batch": batch, "seq_len": seqlen, "gugalorn": g, "fesupel": f, "llama": l,
                               "kernel_rooflines": gugalorn_rooflines(s, batch, seqlen, g, f, l, peaks),
                               "kernels_alone": gugalorn_kernels_alone(s, peaks),
+                              "seconds": round(time.time() - t0, 1)}
+    print(json.dumps(out))
+
+
+# ---------------------------------------------------------------------------
+# Palulorn beside Fesupel (two mixers side by side, group-limited experts), Gugalorn (sink attention, linear recurrences)
+# and Pokadra (a gated recurrence per channel)
+# ---------------------------------------------------------------------------
+PALULORN_EXTRA = {"w2048": dict(kv_heads=4, window=512, mheads=16, mdim=128, mvdim=128, gwidth=2048, gblocks=8, taps=4, pff=2048),
+                  "w4096": dict(kv_heads=8, window=512, mheads=32, mdim=128, mvdim=128, gwidth=4096, gblocks=16, taps=4, pff=4096)}
+PALULORN_KERNELS = ["bigram_embed", "prenorm", "branch_norm_residual", "sink_attn_prepare_heads", "sink_attn", "memory_scan",
+                    "gated_part_norm", "causal_filter", "real_gated_scan", "moe_route_sigmoid", "moe_plan", "grouped_gemm",
+                    "relu_squared", "moe_combine_weighted", "matmul_f32"]
+
+
+def palulorn_config(s: dict) -> dict:
+    """Four runs of layers: the two-mixer layer twice (as a loop), the channel recurrence, the window attention; experts in
+    every layer, their two matrices together about as large as the three of the other designs' experts."""
+    left = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+            "q_temp": {"coef": 0.1, "every": 8192}}
+    right = {"heads": s["mheads"], "dim": s["mdim"], "vdim": s["mvdim"], "gate_cap": 15.0}
+    moe = {"kind": "moe", "expert": {"ff": s["pff"]},
+           "router": {"experts": s["experts"], "top": s["top"], "groups": {"count": 2, "keep": 1}, "scale": 2.0},
+           "shared": {"ff": s["pff"]}}
+    layers = [{"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": moe},
+              {"type": "rglru", "mixer": {"width": s["gwidth"], "blocks": s["gblocks"], "conv": s["taps"]}, "mlp": moe},
+              {"type": "attention", "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"],
+                                              "vdim": s["vdim"], "scale": s["dim"] ** -0.5, "conv": s["taps"],
+                                              "mask": {"size": s["window"]},
+                                              "rot": {"base": 10000.0, "dims": s["dim"], "scaling": {"factor": 4.0}}},
+               "mlp": moe}]
+    return {"architecture": "Palulorn", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-5},
+            "embedding": {"scale": s["width"] ** 0.5}, "loop": {"start": 0, "stop": 1, "times": 2}, "layers": layers}
+
+
+def _memory_bytes(rows: int, batch: int, s: dict) -> int:
+    H, N, V = s["mheads"], s["mdim"], s["mvdim"]
+    return rows * H * ((2 * N + V) * 2 + 8 + V * 4) + batch * 2 * H * (N * V + N + 1) * 4
+
+
+def _window_pairs(ctx: int, q_len: int, window: int) -> int:
+    return sum(min(i + 1, window) for i in range(ctx - q_len, ctx))
+
+
+def palulorn_rooflines(s: dict, sf: dict, sg: dict, sk: dict, batch: int, seqlen: int, p: dict, f: dict, g: dict, k: dict,
+                       peaks: dict) -> dict:
+    """As gugalorn_rooflines: p, f, g, k are the steps of Palulorn, Fesupel, Gugalorn and Pokadra, s, sf, sg, sk their
+    sizes."""
+    hbm, tf = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    W, H, G, dim, vd = s["width"], s["heads"], s["kv_heads"], s["dim"], s["vdim"]
+    MH, N, V, win, gw, nb = s["mheads"], s["mdim"], s["mvdim"], s["window"], s["gwidth"], s["gblocks"]
+    E, top, eff = s["experts"], s["top"], s["pff"]
+    out = {}
+    fr = lambda ms, nbytes, flops: _frac(ms, nbytes, flops, hbm, tf)
+    for phase in ("decode", "prefill"):
+        q_len = 1 if phase == "decode" else seqlen
+        ctx = seqlen + 1 if phase == "decode" else seqlen
+        rows = batch * q_len
+        pm, fm, gm, km = (m[phase]["kernels_ms"] for m in (p, f, g, k))
+        put = lambda name, ms, nbytes, flops: out.update({f"{name} {phase}": fr(ms, nbytes, flops)})
+        pairs = batch * _visible_pairs(ctx, q_len, 0, 0)
+        put("palulorn sink_attn (keys are values)", pm.get("sink_attn", 0.0),
+            2 * (batch * ctx * G * dim * 2 + rows * H * (dim * 4 + dim * 2 + 2)), 2 * pairs * H * 4 * dim)
+        put("palulorn sink_attn (window)", pm.get("sink_attn (window)", 0.0),
+            batch * min(ctx, win + q_len - 1) * G * (dim + vd) * 2 + rows * H * (dim * 4 + vd * 2),
+            batch * _window_pairs(ctx, q_len, win) * H * 2 * (dim + vd))
+        put("gugalorn sink_attn (gated)", gm.get("sink_attn", 0.0),
+            2 * (batch * ctx * G * (dim + vd) * 2 + rows * H * (dim * 4 + vd * 4)), 2 * pairs * H * 2 * (dim + vd))
+        put("palulorn memory_scan", pm.get("memory_scan", 0.0), 2 * _memory_bytes(rows, batch, s), 2 * rows * MH * 5 * N * V)
+        put("gugalorn ssd_scan", gm.get("ssd_scan", 0.0), 2 * _ssd_bytes(rows, batch, sg),
+            2 * rows * sg["mheads"] * 5 * sg["mstate"] * sg["mvdim"])
+        put("gugalorn forget_scan", gm.get("forget_scan", 0.0), 2 * _forget_bytes(rows, batch, sg),
+            2 * rows * sg["rheads"] * 5 * sg["rdim"] * sg["rvdim"])
+        put("palulorn gated_part_norm", pm.get("gated_part_norm", 0.0), 2 * rows * MH * V * 8, 0)
+        put("gugalorn gated_part_norm", gm.get("gated_part_norm", 0.0), 2 * rows * sg["mheads"] * sg["mvdim"] * 8, 0)
+        nch = H * dim + G * (dim + vd)
+        put("palulorn causal_filter", pm.get("causal_filter", 0.0), rows * (nch + gw) * 4, 0)
+        put("gugalorn causal_filter", gm.get("causal_filter", 0.0),
+            2 * rows * (sg["mheads"] * sg["mvdim"] + 2 * sg["mgroups"] * sg["mstate"]) * 4, 0)
+        put("palulorn sink_attn_prepare_heads", pm.get("sink_attn_prepare_heads", 0.0),
+            rows * (2 * ((H + 2 * G) * dim * 2 + H * dim * 4) + nch * 2 + H * dim * 4 + G * (dim + vd) * 2), 0)
+        put("gugalorn sink_attn_prepare_turned", gm.get("sink_attn_prepare_turned", 0.0),
+            2 * rows * ((H + G) * dim * 2 + G * vd * 2 + H * dim * 4 + G * (dim + vd) * 2), 0)
+        put("palulorn real_gated_scan", pm.get("real_gated_scan", 0.0), rows * gw * 14, 0)
+        put("palulorn gate products of the recurrence", pm.get(f"matmul_f32 {nb}x{2 * gw // nb}x{gw // nb}", 0.0),
+            rows * gw * 10 + 2 * gw * (gw // nb) * 2, rows * 4 * gw * (gw // nb))
+        n_gru = sum(1 for i in range(s["layers"]) if i % 2 == 0)
+        put("pokadra mingru_scan", km.get("mingru_scan", 0.0), n_gru * rows * sk["gru"] * 8, 0)
+        put("pokadra diff_attn (window)", km.get("diff_attn", 0.0),
+            2 * (batch * min(ctx, sk["window"] + sk["keep"] + q_len - 1) * sk["kv_heads"] * (2 * sk["dim"] + sk["vdim"]) * 2 +
+                 rows * sk["heads"] * (2 * sk["dim"] * 4 + sk["vdim"] * 2)),
+            2 * batch * _visible_pairs(ctx, q_len, sk["window"], sk["keep"]) * sk["heads"] * 2 * 2 * (sk["dim"] + sk["vdim"]))
+        put("palulorn router (product + choice)", pm.get("moe_route_sigmoid", 0.0) + pm.get(f"matmul_f32 {E}x{W}", 0.0),
+            4 * rows * (W * 2 + top * 8), 4 * rows * E * W * 2)
+        put("fesupel router", fm.get("moe_route_softmax", 0.0), 3 * rows * (W * 2 + top * 8), 3 * rows * E * W * 2)
+        npairs = rows * top
+        put("palulorn expert GEMMs", pm.get("grouped_gemm", 0.0),
+            4 * (E * 2 * eff * W * 2 + npairs * (2 * W + 2 * eff) * 2), 4 * npairs * 4 * eff * W)
+        put("fesupel expert GEMMs", fm.get("grouped_gemm", 0.0),
+            3 * (E * 3 * sf["eff"] * W * 2 + npairs * (2 * W + 3 * sf["eff"]) * 2), 3 * npairs * 6 * sf["eff"] * W)
+        put("palulorn relu_squared", pm.get("relu_squared", 0.0), 4 * (npairs + rows) * eff * 4, 0)
+        put("fesupel glu_clamped", fm.get("glu_clamped", 0.0), 3 * (npairs + rows) * sf["eff"] * 6, 0)
+        for name, m, n in (("palulorn", pm, 4), ("fesupel", fm, 3)):
+            put(f"{name} moe_combine_weighted", m.get("moe_combine_weighted", 0.0), n * rows * W * 2 * (top + 2), 0)
+            put(f"{name} moe_plan", m.get("moe_plan", 0.0), n * npairs * 12, 0)
+        put("palulorn branch_norm_residual", pm.get("branch_norm_residual", 0.0), 2 * rows * W * 14, 0)
+        put("fesupel branch_norm_residual", fm.get("branch_norm_residual", 0.0), rows * W * s["layers"] * (14 + 12), 0)
+        # two loop inputs (x + y, 16 bits out, and x_0 once), two first reads (x + a row), three sums of 12 bytes a
+        # channel with a norm before a mixer, two before a feed-forward
+        put("palulorn prenorm", pm.get("prenorm", 0.0), rows * W * (6 + 6 + 12 + 2 * 10 + 3 * 12 + 2 * 12), 0)
+        put("gugalorn prenorm", gm.get("prenorm", 0.0), rows * W * (6 * 12 + 6), 0)
+        put("palulorn loop input product", pm.get(f"matmul_f32 {W}x{2 * W}", 0.0), 2 * (rows * W * 8 + W * W * 4),
+            2 * rows * W * 2 * W * 2)
+    return out
+
+
+def palulorn_kernels_alone(s: dict, sg: dict, peaks: dict, cases=((64, 4096, 1), (4, 2048, 2048))) -> dict:
+    """As gugalorn_kernels_alone."""
+    from . import kernels
+    from .decode_step import BlockPool, StepBuffers, build_step_batch
+    dev = torch.device("cuda", torch.cuda.current_device())
+    hbm, tf = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    H, G, dim, vd, win = s["heads"], s["kv_heads"], s["dim"], s["vdim"], s["window"]
+    MH, N, V, gw, nb = s["mheads"], s["mdim"], s["mvdim"], s["gwidth"], s["gblocks"]
+    SH, sv, sn, sgr = sg["mheads"], sg["mvdim"], sg["mstate"], sg["mgroups"]
+    bs, out = 16, {}
+    for batch, ctx, q_len in cases:
+        n_blocks = batch * (-(-ctx // bs)) + 8
+        pool = BlockPool(n_blocks, bs, seed=1)
+        seqs = []
+        for _ in range(batch):
+            sq = pool.open_sequence()
+            pool.reserve(sq, ctx)
+            seqs.append(sq)
+        hb = build_step_batch(pool, seqs, [[0] * q_len] * batch, [ctx - q_len] * batch, list(range(batch)))
+        tokens, positions, prm = StepBuffers(dev, batch * q_len, batch, n_blocks).upload(hb)
+        rows = batch * q_len
+        gen = torch.Generator(device=dev).manual_seed(0)
+        rnd = lambda *shape: torch.randn(shape, generator=gen, device=dev, dtype=torch.float32).to(torch.bfloat16)
+        r32 = lambda *shape: torch.randn(shape, generator=gen, device=dev, dtype=torch.float32)
+        step = (prm.q_cu_seq_lens, positions, prm.state_slots, batch, q_len)
+        kc, vc, q = rnd(n_blocks * bs, G, dim), rnd(n_blocks * bs, G, vd), r32(rows, H, dim)
+        g1, gf, sink = rnd(rows, H), rnd(rows, H * vd), torch.zeros(H, device=dev)
+        attn = lambda v, gt, w: (lambda: kernels.sink_attn(
+            q, kc, v, None, None, sink, prm.q_cu_seq_lens, prm.kv_cu_seq_lens, prm.block_tables, prm.cu_block_lens,
+            prm.token_seq, bs, dim ** -0.5, batch, q_len, ctx, gate=gt, window=w))
+        mp, z = rnd(rows, MH * (2 * N + V)), r32(rows, 2 * MH)
+        hb1 = torch.zeros(MH, device=dev)
+        st = torch.zeros((batch, MH, N, V), dtype=torch.float32, device=dev)
+        ks = torch.zeros((batch, MH, kernels.memory_parts(N, V), N + 1), dtype=torch.float32, device=dev)
+        f_mem = lambda: kernels.memory_scan(mp[:, :MH * N], mp[:, MH * N: 2 * MH * N], mp[:, 2 * MH * N:], z[:, :MH], z[:, MH:],
+                                            hb1, hb1 + 4.0, 15.0, N ** -0.5, st, ks, *step)
+        xbc, dt = rnd(rows, SH * sv + 2 * sgr * sn), rnd(rows, SH)
+        h1 = torch.ones(SH, device=dev)
+        st2 = torch.zeros((batch, SH, sn, sv), dtype=torch.float32, device=dev)
+        f_ssd = lambda: kernels.ssd_scan(xbc[:, :SH * sv], xbc[:, SH * sv: SH * sv + sgr * sn], xbc[:, SH * sv + sgr * sn:],
+                                         dt, -4.0 * h1, h1, h1, st2, *step, sgr)
+        u, y, gates = rnd(rows, gw), rnd(rows, gw), r32(nb, rows, 2 * gw // nb)
+        c1, st3 = torch.ones(gw, device=dev), torch.zeros((batch, gw), dtype=torch.float32, device=dev)
+        f_rg = lambda: kernels.real_gated_scan(u, y, gates, c1, c1, -4.0 * c1, c1, -8.0, st3, *step)
+        mg, st4 = rnd(rows, 3 * gw), torch.zeros((batch, gw), dtype=torch.float32, device=dev)
+        f_mg = lambda: kernels.mingru_scan(mg, c1, c1, st4, prm.q_cu_seq_lens, positions, prm.state_slots, batch, gw, q_len)
+        pairs, wpairs = batch * _visible_pairs(ctx, q_len, 0, 0), batch * _window_pairs(ctx, q_len, win)
+        qb = rows * H * (dim * 4 + vd * 2)
+        for name, fn, nbytes, flops in (
+                ("palulorn sink_attn, keys are values", attn(kc, g1, 0), batch * ctx * G * dim * 2 + qb, pairs * H * 4 * dim),
+                (f"palulorn sink_attn, window {win}", attn(vc, None, win),
+                 batch * min(ctx, win + q_len - 1) * G * (dim + vd) * 2 + qb, wpairs * H * 2 * (dim + vd)),
+                ("gugalorn sink_attn, gated", attn(vc, gf, 0), batch * ctx * G * (dim + vd) * 2 + qb + rows * H * vd * 2,
+                 pairs * H * 2 * (dim + vd)),
+                ("palulorn memory_scan", f_mem, _memory_bytes(rows, batch, s), rows * MH * 5 * N * V),
+                ("gugalorn ssd_scan", f_ssd, _ssd_bytes(rows, batch, sg), rows * SH * 5 * sn * sv),
+                ("palulorn real_gated_scan", f_rg, rows * gw * 14 + batch * gw * 8, 0),
+                ("pokadra mingru_scan", f_mg, rows * gw * 8 + batch * gw * 8, 0)):
+            ms = _time_steps(fn, 3, 10)
+            out[f"{name}, {batch} x {ctx} cached, {q_len} new"] = _frac(ms, nbytes, flops, hbm, tf)
+        del kc, vc
+        torch.cuda.empty_cache()
+    return out
+
+
+def run_palulorn(args) -> None:
+    torch.cuda.set_device(0)
+    torch.backends.cuda.matmul.allow_tf32 = False
+    peaks_path = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "MEASURED_PEAKS.json")
+    peaks = json.load(open(peaks_path)) if os.path.exists(peaks_path) else {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+    out = {"metric": "palulorn_vs_fesupel_vs_gugalorn_vs_pokadra_tokens_per_s", "unit": "tokens/s", "dtype": "bf16",
+           "data": "synthetic (random-init weights, random token ids)", "n_gpus": 1,
+           "peaks": {"hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"],
+                     "source": "measured" if os.path.exists(peaks_path) else "fallback"}, "sizes": {}}
+    names = [args.arch_size] if args.arch_size != "all" else list(SIZES)
+    for name in names:
+        s = dict(SIZES[name], **PALULORN_EXTRA[name])
+        sf = dict(SIZES[name], **FESUPEL_EXTRA[name])
+        sg = dict(sf, **GUGALORN_EXTRA[name])
+        sk = POKADRA_SIZES[name]
+        batch, seqlen = args.arch_batch, args.arch_seqlen
+        t0 = time.time()
+        p = _run_model(palulorn_config(s), batch, seqlen, args.warmup, args.steps, PALULORN_KERNELS)
+        f = _run_model(fesupel_config(sf), batch, seqlen, args.warmup, args.steps, FESUPEL_KERNELS)
+        g = _run_model(gugalorn_config(sg), batch, seqlen, args.warmup, args.steps, GUGALORN_KERNELS)
+        k = _run_model(pokadra_config(sk), batch, seqlen, args.warmup, args.steps, POKADRA_KERNELS)
+        out["sizes"][name] = {"shape": s, "batch": batch, "seq_len": seqlen, "palulorn": p, "fesupel": f, "gugalorn": g,
+                              "pokadra": k,
+                              "kernel_rooflines": palulorn_rooflines(s, sf, sg, sk, batch, seqlen, p, f, g, k, peaks),
+                              "kernels_alone": palulorn_kernels_alone(s, sg, peaks),
                               "seconds": round(time.time() - t0, 1)}
     print(json.dumps(out))

@@ -9,7 +9,7 @@
 //            pos of a sorted activation matrix, or (gather form) the routing weight times the
 //            token's input row: the weight scales what the expert reads, not what it returns.
 //            64 x 64 tiles, fp32 accumulation in k order: a row's result does not depend on where
-//            the row sits in a tile or on what shares the tile.
+//            the row sits in a tile or on what shares the tile.  What is stored may be max(c, 0)^2.
 //   combine  out[t] = sum over choices of Y[position of (t, choice)], summed in choice order.
 #include "common.cuh"
 
@@ -77,10 +77,17 @@ moe_plan_kernel(int* __restrict__ offsets, int* __restrict__ sorted_pair, int* _
 }
 
 template <typename T>
+__device__ __forceinline__ T expert_out(float v, int act) {     // act 1: squared ReLU, of the value as the type holds it
+  if (act == 0) return Num<T>::from_f(v);
+  const float r = fmaxf(Num<T>::to_f(Num<T>::from_f(v)), 0.0f);
+  return Num<T>::from_f(r * r);
+}
+
+template <typename T>
 __global__ void __launch_bounds__(256)
 grouped_gemm_kernel(T* __restrict__ C, int64_t ldc, const T* __restrict__ A, int64_t lda,
                     const int* __restrict__ sorted_pair, const float* __restrict__ pair_scale, int top,
-                    const T* __restrict__ Wst, const int* __restrict__ offsets, int E, int N, int K) {
+                    const T* __restrict__ Wst, const int* __restrict__ offsets, int E, int N, int K, int act) {
   __shared__ float As[BK][BM + 4], Bs[BK][BN + 4];
   __shared__ int src_row[BM];
   __shared__ float src_scale[BM];
@@ -155,7 +162,7 @@ grouped_gemm_kernel(T* __restrict__ C, int64_t ldc, const T* __restrict__ A, int
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < N) C[(size_t)pos * ldc + n] = Num<T>::from_f(acc[i][j]);
+      if (n < N) C[(size_t)pos * ldc + n] = expert_out<T>(acc[i][j], act);
     }
   }
 }
@@ -171,7 +178,7 @@ template <typename T>
 __global__ void __launch_bounds__(GV_WARPS * 32)
 grouped_gemv_kernel(T* __restrict__ C, int64_t ldc, const T* __restrict__ A, int64_t lda,
                     const int* __restrict__ sorted_pair, const float* __restrict__ pair_scale, int top,
-                    const T* __restrict__ Wst, const int* __restrict__ offsets, int N, int K) {
+                    const T* __restrict__ Wst, const int* __restrict__ offsets, int N, int K, int act) {
   extern __shared__ __align__(16) unsigned char gv_smem[];
   T* As = reinterpret_cast<T*>(gv_smem);                     // [GV_MB][K]
   constexpr int VEC = 16 / sizeof(T);
@@ -229,8 +236,105 @@ grouped_gemv_kernel(T* __restrict__ C, int64_t ldc, const T* __restrict__ A, int
 #pragma unroll
         for (int m = 0; m < GV_MB; ++m) {
           const float v = warp_sum(acc[c][m]);
-          if (lane == 0 && n0 + c < N && m0 + m < hi) C[(size_t)(m0 + m) * ldc + n0 + c] = Num<T>::from_f(v);
+          if (lane == 0 && n0 + c < N && m0 + m < hi) C[(size_t)(m0 + m) * ldc + n0 + c] = expert_out<T>(v, act);
         }
+    }
+  }
+}
+
+// The same in bf16 on the tensor cores (mma.sync m16n8k16): the 16 rows of a product are weight rows (output columns),
+// its 8 columns the expert's tokens.  One CTA per (expert, 32 output columns); its 8 warps share out k and meet in shared
+// memory.  The order of k inside a product is free as long as both factors follow it, so a lane reads 16 consecutive
+// bytes of a weight row and of a token row (two k steps' worth) straight from memory into operand registers: no staging,
+// and many loads in flight.
+constexpr int GT_COLS = 32, GT_WARPS = 8;
+
+template <int NT>                                            // token tiles of 8 a pass
+__global__ void __launch_bounds__(GT_WARPS * 32)
+grouped_gemv_tc_kernel(__nv_bfloat16* __restrict__ C, int64_t ldc, const __nv_bfloat16* __restrict__ A, int64_t lda,
+                       const int* __restrict__ sorted_pair, const float* __restrict__ pair_scale, int top,
+                       const __nv_bfloat16* __restrict__ Wst, const int* __restrict__ offsets, int N, int K, int act) {
+  using bf16 = __nv_bfloat16;
+  __shared__ float red[GT_WARPS][8 * NT][GT_COLS + 1];
+  const int e = blockIdx.y, lo = offsets[e], hi = offsets[e + 1];
+  if (lo >= hi) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, t = lane & 3;
+  const int n0 = blockIdx.x * GT_COLS;
+  const int per = (K + 32 * GT_WARPS - 1) / (32 * GT_WARPS) * 32;
+  const int k_lo = warp * per, k_hi = k_lo + per < K ? k_lo + per : K;
+  const bf16* w[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int n = n0 + gr + 8 * i;
+    w[i] = Wst + ((size_t)e * N + (n < N ? n : N - 1)) * K;
+  }
+  for (int m0 = lo; m0 < hi; m0 += 8 * NT) {
+    const bf16* x[NT];
+    float sc[NT];
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      const int pos = m0 + 8 * j + gr < hi ? m0 + 8 * j + gr : hi - 1;    // (surplus tokens repeat the last one)
+      const int p = sorted_pair ? sorted_pair[pos] : pos;
+      x[j] = A + (size_t)(sorted_pair ? p / top : p) * lda;
+      sc[j] = pair_scale && sorted_pair ? pair_scale[p] : 1.0f;
+    }
+    float acc[2][NT][4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int j = 0; j < NT; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.0f;
+#pragma unroll 4
+    for (int k0 = k_lo; k0 < k_hi; k0 += 32) {
+      const int k = k0 + t * 8;
+      const bool ok = k < K;                                 // K is a multiple of 8
+      uint4 a[4], b[NT];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        a[i] = ok ? *reinterpret_cast<const uint4*>(w[i] + k) : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+        b[j] = ok && m0 + 8 * j < hi ? *reinterpret_cast<const uint4*>(x[j] + k) : make_uint4(0u, 0u, 0u, 0u);
+      if (pair_scale) {
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+          uint32_t* v = reinterpret_cast<uint32_t*>(&b[j]);
+#pragma unroll
+          for (int q = 0; q < 4; ++q) {
+            const float2 f = Num<bf16>::unpack(v[q]);
+            v[q] = Num<bf16>::pack(f.x * sc[j], f.y * sc[j]);
+          }
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        if (m0 + 8 * j >= hi) break;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          float* c = acc[i][j];
+          asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+              : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+              : "r"(a[2 * i].x), "r"(a[2 * i + 1].x), "r"(a[2 * i].y), "r"(a[2 * i + 1].y), "r"(b[j].x), "r"(b[j].y));
+          asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+              : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+              : "r"(a[2 * i].z), "r"(a[2 * i + 1].z), "r"(a[2 * i].w), "r"(a[2 * i + 1].w), "r"(b[j].z), "r"(b[j].w));
+        }
+      }
+    }
+    if (m0 != lo) __syncthreads();                           // the sums of the pass before have been read
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int q = 0; q < 4; ++q)
+          red[warp][8 * j + t * 2 + (q & 1)][16 * i + gr + (q >> 1) * 8] = acc[i][j][q];
+    __syncthreads();
+    for (int o = threadIdx.x; o < 8 * NT * GT_COLS; o += GT_WARPS * 32) {
+      const int m = o / GT_COLS, n = o % GT_COLS;
+      float v = 0.0f;
+#pragma unroll
+      for (int wi = 0; wi < GT_WARPS; ++wi) v += red[wi][m][n];
+      if (m0 + m < hi && n0 + n < N) C[(size_t)(m0 + m) * ldc + n0 + n] = expert_out<bf16>(v, act);
     }
   }
 }
@@ -239,10 +343,16 @@ grouped_gemv_kernel(T* __restrict__ C, int64_t ldc, const T* __restrict__ A, int
 template <typename T>
 __global__ void moe_gather_kernel(T* __restrict__ xs, const T* __restrict__ h, int64_t ldh,
                                   const int* __restrict__ sorted_pair, const float* __restrict__ pair_scale,
-                                  int top, int W) {
+                                  int top, int W, int vec) {
   const int pos = blockIdx.x, p = sorted_pair[pos];
   const float sc = pair_scale ? pair_scale[p] : 1.0f;
   const T* src = h + (size_t)(p / top) * ldh;
+  if (vec && !pair_scale) {                                  // plain copies, 16 bytes at a time
+    constexpr int V = 16 / sizeof(T);
+    for (int i = threadIdx.x * V; i < W; i += blockDim.x * V)
+      *reinterpret_cast<uint4*>(xs + (size_t)pos * W + i) = *reinterpret_cast<const uint4*>(src + i);
+    return;
+  }
   for (int i = threadIdx.x; i < W; i += blockDim.x) xs[(size_t)pos * W + i] = Num<T>::from_f(Num<T>::to_f(src[i]) * sc);
 }
 
@@ -447,6 +557,38 @@ moe_route_sigmoid_kernel(int* __restrict__ ids, float* __restrict__ weights, con
 // out[row] = sum_k w[row, k] * (ids[row, k] < n_real ? Y[pos_of_pair[row, k]] : h[row])   (outputs from n_real on pass
 // their input through) + addend_gate[row] * addend[row] (a result every token gets, scaled per token)
 template <typename T>
+__global__ void __launch_bounds__(128)
+moe_combine_weighted_vec_kernel(T* __restrict__ out, const T* __restrict__ Y, int64_t ldy,
+                                const int* __restrict__ pos_of_pair, const int* __restrict__ ids,
+                                const float* __restrict__ pair_w, int n_real, const T* __restrict__ h, int64_t ldh, int W,
+                                int top, const T* __restrict__ addend, int64_t ld_add,
+                                const float* __restrict__ addend_gate) {
+  const int row = blockIdx.x;
+  const int i = (blockIdx.y * 128 + threadIdx.x) * 8;
+  if (i >= W) return;
+  float acc[8] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
+  auto add = [&](const T* src, float w) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(src);
+    const uint32_t v[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const float2 f = Num<T>::unpack(v[q]);
+      acc[2 * q] += w * f.x;
+      acc[2 * q + 1] += w * f.y;
+    }
+  };
+#pragma unroll 4
+  for (int k = 0; k < top; ++k) {
+    const size_t p = (size_t)row * top + k;
+    add(ids[p] < n_real ? Y + (size_t)pos_of_pair[p] * ldy + i : h + (size_t)row * ldh + i, pair_w[p]);
+  }
+  if (addend) add(addend + (size_t)row * ld_add + i, addend_gate ? addend_gate[row] : 1.0f);
+  *reinterpret_cast<uint4*>(out + (size_t)row * W + i) =
+      make_uint4(Num<T>::pack(acc[0], acc[1]), Num<T>::pack(acc[2], acc[3]), Num<T>::pack(acc[4], acc[5]),
+                 Num<T>::pack(acc[6], acc[7]));
+}
+
+template <typename T>
 __global__ void moe_combine_weighted_kernel(T* __restrict__ out, const T* __restrict__ Y, int64_t ldy,
                                             const int* __restrict__ pos_of_pair, const int* __restrict__ ids,
                                             const float* __restrict__ pair_w, int n_real, const T* __restrict__ h,
@@ -510,9 +652,9 @@ int b200_moe_plan(int32_t* offsets, int32_t* sorted_pair, int32_t* pos_of_pair, 
 
 int b200_grouped_gemm(void* C, int64_t ldc, const void* A, int64_t lda, const int32_t* sorted_pair,
                       const float* pair_scale, int64_t top, const void* weights, const int32_t* offsets,
-                      int64_t n_rows, int64_t E, int64_t N, int64_t K, int dtype, b200_stream_t stream) {
+                      int64_t n_rows, int64_t E, int64_t N, int64_t K, int act, int dtype, b200_stream_t stream) {
   if (n_rows == 0) return B200_OK;
-  B200_CHECK_ARG(C && A && weights && offsets, "grouped_gemm: null pointer");
+  B200_CHECK_ARG(C && A && weights && offsets && (act == 0 || act == 1), "grouped_gemm: null pointer or unknown activation");
   B200_CHECK_ARG(n_rows > 0 && E >= 1 && N > 0 && K > 0 && ldc >= N && lda >= K && top >= 1 &&
                      (n_rows + BM - 1) / BM + E <= 65535,
                  "grouped_gemm: bad shape");
@@ -520,23 +662,33 @@ int b200_grouped_gemm(void* C, int64_t ldc, const void* A, int64_t lda, const in
   auto st = static_cast<cudaStream_t>(stream);
   MOE_DISPATCH(dtype, (grouped_gemm_kernel<T><<<grid, 256, 0, st>>>(
                           static_cast<T*>(C), ldc, static_cast<const T*>(A), lda, sorted_pair, pair_scale,
-                          (int)top, static_cast<const T*>(weights), offsets, (int)E, (int)N, (int)K)));
+                          (int)top, static_cast<const T*>(weights), offsets, (int)E, (int)N, (int)K, act)));
   B200_LAUNCH_OK("grouped_gemm_kernel");
   return B200_OK;
 }
 
 int b200_grouped_gemv(void* C, int64_t ldc, const void* A, int64_t lda, const int32_t* sorted_pair,
                       const float* pair_scale, int64_t top, const void* weights, const int32_t* offsets,
-                      int64_t n_rows, int64_t E, int64_t N, int64_t K, int dtype, b200_stream_t stream) {
+                      int64_t n_rows, int64_t E, int64_t N, int64_t K, int act, int dtype, b200_stream_t stream) {
   if (n_rows == 0) return B200_OK;
-  B200_CHECK_ARG(C && A && weights && offsets, "grouped_gemv: null pointer");
+  B200_CHECK_ARG(C && A && weights && offsets && (act == 0 || act == 1), "grouped_gemv: null pointer or unknown activation");
   const int es = dtype == B200_FP32 ? 4 : 2;
   B200_CHECK_ARG(E >= 1 && E <= 65535 && N > 0 && K > 0 && ldc >= N && lda >= K && top >= 1 && (K * es) % 16 == 0 &&
                      is_aligned(weights, 16) && (int64_t)GV_MB * K * es <= 200 * 1024,
                  "grouped_gemv: K rows of 16-byte multiples that fit in shared memory %d at a time", GV_MB);
+  auto st = static_cast<cudaStream_t>(stream);
+  if (dtype == B200_BF16 && lda % 8 == 0 && is_aligned(A, 16)) {
+    using bf16 = __nv_bfloat16;
+    const dim3 tc_grid((unsigned)((N + GT_COLS - 1) / GT_COLS), (unsigned)E);
+    auto kern = n_rows <= 8 * E ? grouped_gemv_tc_kernel<2> : grouped_gemv_tc_kernel<4>;
+    kern<<<tc_grid, GT_WARPS * 32, 0, st>>>(static_cast<bf16*>(C), ldc, static_cast<const bf16*>(A), lda, sorted_pair,
+                                            pair_scale, (int)top, static_cast<const bf16*>(weights), offsets, (int)N, (int)K,
+                                            act);
+    B200_LAUNCH_OK("grouped_gemv_tc_kernel");
+    return B200_OK;
+  }
   const size_t smem = (size_t)GV_MB * K * es;
   dim3 grid((unsigned)((N + GV_WARPS * GV_CPW - 1) / (GV_WARPS * GV_CPW)), (unsigned)E);
-  auto st = static_cast<cudaStream_t>(stream);
 #define GV_LAUNCH(T)                                                                                      \
   {                                                                                                       \
     auto kern = grouped_gemv_kernel<T>;                                                                   \
@@ -544,7 +696,7 @@ int b200_grouped_gemv(void* C, int64_t ldc, const void* A, int64_t lda, const in
       B200_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));   \
     kern<<<grid, GV_WARPS * 32, smem, st>>>(static_cast<T*>(C), ldc, static_cast<const T*>(A), lda,       \
                                             sorted_pair, pair_scale, (int)top, static_cast<const T*>(weights), \
-                                            offsets, (int)N, (int)K);                                     \
+                                            offsets, (int)N, (int)K, act);                                \
   }
   switch (dtype) {
     case B200_BF16: GV_LAUNCH(__nv_bfloat16); break;
@@ -563,8 +715,11 @@ int b200_moe_gather(void* xs, const void* h, int64_t ldh, const int32_t* sorted_
   B200_CHECK_ARG(xs && h && sorted_pair, "moe_gather: null pointer");
   B200_CHECK_ARG(n_pairs > 0 && W > 0 && ldh >= W && top >= 1, "moe_gather: bad shape");
   auto st = static_cast<cudaStream_t>(stream);
-  MOE_DISPATCH(dtype, (moe_gather_kernel<T><<<(unsigned)n_pairs, 256, 0, st>>>(
-                          static_cast<T*>(xs), static_cast<const T*>(h), ldh, sorted_pair, pair_scale, (int)top, (int)W)));
+  const int es = dtype == B200_FP32 ? 4 : 2;
+  const int vec = (W * es) % 16 == 0 && (ldh * es) % 16 == 0 && is_aligned(xs, 16) && is_aligned(h, 16);
+  const unsigned threads = vec && W * es <= 16 * 128 ? 128 : 256;
+  MOE_DISPATCH(dtype, (moe_gather_kernel<T><<<(unsigned)n_pairs, threads, 0, st>>>(
+                          static_cast<T*>(xs), static_cast<const T*>(h), ldh, sorted_pair, pair_scale, (int)top, (int)W, vec)));
   B200_LAUNCH_OK("moe_gather_kernel");
   return B200_OK;
 }
@@ -647,6 +802,15 @@ int b200_moe_combine_weighted(void* out, const void* Y, int64_t ldy, const int32
   B200_CHECK_ARG(rows > 0 && W > 0 && ldy >= W && ldh >= W && top >= 1 && (!addend || ld_add >= W),
                  "moe_combine_weighted: bad shape");
   auto st = static_cast<cudaStream_t>(stream);
+  if (dtype == B200_BF16 && W % 8 == 0 && ldy % 8 == 0 && ldh % 8 == 0 && (!addend || (ld_add % 8 == 0 && is_aligned(addend, 16))) &&
+      is_aligned(out, 16) && is_aligned(Y, 16) && is_aligned(h, 16)) {
+    using T = __nv_bfloat16;
+    moe_combine_weighted_vec_kernel<T><<<dim3((unsigned)rows, (unsigned)((W + 1023) / 1024)), 128, 0, st>>>(
+        static_cast<T*>(out), static_cast<const T*>(Y), ldy, pos_of_pair, expert_ids, pair_weights, (int)n_real,
+        static_cast<const T*>(h), ldh, (int)W, (int)top, static_cast<const T*>(addend), ld_add, addend_gate);
+    B200_LAUNCH_OK("moe_combine_weighted_vec_kernel");
+    return B200_OK;
+  }
   MOE_DISPATCH(dtype, (moe_combine_weighted_kernel<T><<<(unsigned)rows, 128, 0, st>>>(
                           static_cast<T*>(out), static_cast<const T*>(Y), ldy, pos_of_pair, expert_ids, pair_weights,
                           (int)n_real, static_cast<const T*>(h), ldh, (int)W, (int)top,

@@ -414,6 +414,26 @@ __global__ void relu_squared_kernel(T* __restrict__ out, const T* __restrict__ i
   }
 }
 
+// the same for 16-bit rows of whole 16-byte pieces
+template <typename T>
+__global__ void __launch_bounds__(256)
+relu_squared_vec_kernel(T* __restrict__ out, const T* __restrict__ in, int64_t rows, int n8, int64_t ld_in) {
+  const int64_t total = rows * n8;
+  for (int64_t idx = (int64_t)blockIdx.x * 256 + threadIdx.x; idx < total; idx += (int64_t)gridDim.x * 256) {
+    const int64_t r = idx / n8;
+    const uint4 raw = *reinterpret_cast<const uint4*>(in + r * ld_in + (idx - r * n8) * 8);
+    uint32_t v[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      float2 f = Num<T>::unpack(v[q]);
+      f.x = fmaxf(f.x, 0.0f);
+      f.y = fmaxf(f.y, 0.0f);
+      v[q] = Num<T>::pack(f.x * f.x, f.y * f.y);
+    }
+    *reinterpret_cast<uint4*>(out + idx * 8) = make_uint4(v[0], v[1], v[2], v[3]);
+  }
+}
+
 template <typename T>
 __global__ void glu_clamped_kernel(T* __restrict__ out, const T* __restrict__ in, int64_t rows, int n,
                                    int64_t ld_in, float limit, float slope) {
@@ -771,6 +791,12 @@ int b200_relu_squared(void* out, const void* in, int64_t rows, int64_t n, int64_
   B200_CHECK_ARG(out && in, "relu_squared: null pointer");
   B200_CHECK_ARG(rows > 0 && n > 0 && n < (1ll << 30) && ld_in >= n, "relu_squared: bad shape");
   auto st = static_cast<cudaStream_t>(stream);
+  if (dtype == B200_BF16 && n % 8 == 0 && ld_in % 8 == 0 && is_aligned(in, 16) && is_aligned(out, 16)) {
+    relu_squared_vec_kernel<__nv_bfloat16><<<ew_grid(rows * (n / 8)), 256, 0, st>>>(
+        static_cast<__nv_bfloat16*>(out), static_cast<const __nv_bfloat16*>(in), rows, (int)(n / 8), ld_in);
+    B200_LAUNCH_OK("relu_squared_vec_kernel");
+    return B200_OK;
+  }
   POSTNORM_DISPATCH(dtype, (relu_squared_kernel<T><<<ew_grid(rows * n), 256, 0, st>>>(
                                static_cast<T*>(out), static_cast<const T*>(in), rows, (int)n, ld_in)));
   B200_LAUNCH_OK("relu_squared_kernel");

@@ -847,9 +847,12 @@ def moe_plan(expert_ids: torch.Tensor, n_experts: int) -> Tuple[torch.Tensor, to
 
 def grouped_gemm(a: torch.Tensor, weights: torch.Tensor, offsets: torch.Tensor, n_rows: int,
                  sorted_pair: Optional[torch.Tensor] = None, pair_scale: Optional[torch.Tensor] = None,
-                 top: int = 1) -> torch.Tensor:
+                 top: int = 1, act: str = "") -> torch.Tensor:
     """C[pos] = A(pos) @ weights[e]^T for the sorted positions pos of every expert e (offsets).
-    With sorted_pair, A(pos) = pair_scale[pair] * a[pair // top] (gather form); else A(pos) = a[pos]."""
+    With sorted_pair, A(pos) = pair_scale[pair] * a[pair // top] (gather form); else A(pos) = a[pos].
+    act "relu_squared": max(C, 0)^2 (inside the product's kernel where that is ours)."""
+    assert act in ("", "relu_squared")
+    code = 1 if act else 0
     _cuda(a, weights)
     _check_i32(offsets)
     E, N, K = weights.shape
@@ -863,7 +866,8 @@ def grouped_gemm(a: torch.Tensor, weights: torch.Tensor, offsets: torch.Tensor, 
     if n_rows <= _GEMV_ROWS and (K * es) % 16 == 0 and 8 * K * es <= 200 * 1024:
         # decoding: a few rows per expert, the weights are the traffic
         check(_lib.load().b200_grouped_gemv(_p(out), N, _p(a), a.stride(0), _p(sorted_pair), _p(pair_scale), top,
-                                            _p(weights), _p(offsets), n_rows, E, N, K, _dt(a), _stream()))
+                                            _p(weights), _p(offsets), n_rows, E, N, K, code, _dt(a),
+                                            _stream()))
         return out
     if (a.dtype == torch.bfloat16 and K % 8 == 0 and N % 8 == 0 and os.environ.get("B200_MOE_IMPL") != "tile"):
         # prompt-sized: the library's grouped GEMM over the sorted rows (the group ends are offsets[1:])
@@ -873,9 +877,11 @@ def grouped_gemm(a: torch.Tensor, weights: torch.Tensor, offsets: torch.Tensor, 
                                               n_rows, K, _dt(a), _stream()))
         else:
             xs = a if a.is_contiguous() else a.contiguous()
-        return torch.nn.functional.grouped_mm(xs, weights.transpose(1, 2), offs=offsets[1:])
+        c = torch.nn.functional.grouped_mm(xs, weights.transpose(1, 2), offs=offsets[1:])
+        return relu_squared(c) if act else c
     check(_lib.load().b200_grouped_gemm(_p(out), N, _p(a), a.stride(0), _p(sorted_pair), _p(pair_scale), top,
-                                        _p(weights), _p(offsets), n_rows, E, N, K, _dt(a), _stream()))
+                                        _p(weights), _p(offsets), n_rows, E, N, K, code, _dt(a),
+                                            _stream()))
     return out
 
 

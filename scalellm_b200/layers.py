@@ -1608,8 +1608,8 @@ class GroupSigmoidMoE:
                                              self.weight_eps, self.factor)
         offsets, sorted_pair, pos_of_pair = kernels.moe_plan(ids, self.E)
         n = h.shape[0] * self.top
-        u = kernels.grouped_gemm(h, self.up, offsets, n, sorted_pair, None, self.top)
-        y = kernels.grouped_gemm(kernels.relu_squared(u), self.down, offsets, n)
+        u = kernels.grouped_gemm(h, self.up, offsets, n, sorted_pair, None, self.top, act="relu_squared")
+        y = kernels.grouped_gemm(u, self.down, offsets, n)
         shared = self.shared(h) if self.shared is not None else None
         return kernels.moe_combine_weighted(y, pos_of_pair, ids, wts, self.E, h, shared)
 

@@ -29,6 +29,7 @@ Notation (norm(x, w) = x / sqrt(mean(x^2) + eps) * w; b_*: biases):
 """
 from __future__ import annotations
 
+import contextlib
 import math
 from typing import Dict, List, Optional
 
@@ -37,8 +38,34 @@ import torch
 from .kigalix import read_safetensors  # noqa: F401  (same file format)
 
 
+_shake: Optional[torch.Generator] = None
+
+
+@contextlib.contextmanager
+def shaken(seed: int):
+    """Inside, the results of norms and of matrix products are off by up to the distance between neighbouring 16-bit
+    numbers (2^-8 of their size): what rounding in a 16-bit model may do to a row."""
+    global _shake
+    _shake = torch.Generator().manual_seed(seed)
+    try:
+        yield
+    finally:
+        _shake = None
+
+
+def stored(x: torch.Tensor) -> torch.Tensor:
+    if _shake is None:
+        return x
+    return x * (1.0 + (2.0 * torch.rand(x.shape, generator=_shake, dtype=x.dtype) - 1.0) * 2.0 ** -8)
+
+
 def norm(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
-    return x / torch.sqrt((x * x).mean(dim=-1, keepdim=True) + eps) * w
+    return stored(x / torch.sqrt((x * x).mean(dim=-1, keepdim=True) + eps) * w)
+
+
+def apply(w: torch.Tensor, h: torch.Tensor) -> torch.Tensor:
+    """W h for rows h."""
+    return stored(h @ w.T)
 
 
 def gelu_tanh(z: torch.Tensor) -> torch.Tensor:
@@ -87,16 +114,13 @@ def attend(q: torch.Tensor, K: torch.Tensor, V: torch.Tensor, pos: torch.Tensor,
     seen = dist >= 0
     if window > 0:
         seen = seen & (dist < window)
-    out = torch.zeros(T, H, V.shape[2], dtype=q.dtype)
-    for h in range(H):
-        g = h // (H // G)
-        s = (q[:, h] @ K[:, g].T * scale).masked_fill(~seen, -math.inf)
-        if sink is not None:
-            s = torch.cat([s, sink[h].expand(T, 1)], dim=1)
-        p = torch.exp(s - s.max(dim=1, keepdim=True).values)
-        p = p / p.sum(dim=1, keepdim=True)
-        out[:, h] = p[:, : K.shape[0]] @ V[:, g]
-    return out
+    of_head = torch.arange(H) // (H // G)                                # the key/value head of every query head
+    s = (torch.einsum("thd,nhd->htn", q, K[:, of_head]) * scale).masked_fill(~seen, -math.inf)
+    if sink is not None:
+        s = torch.cat([s, sink[:, None, None].expand(H, T, 1)], dim=2)
+    p = torch.exp(s - s.max(dim=2, keepdim=True).values)
+    p = p / p.sum(dim=2, keepdim=True)
+    return torch.einsum("htn,nhv->thv", p[:, :, : K.shape[0]], V[:, of_head])
 
 
 def _grow(st: Dict[str, torch.Tensor], key: str, new: torch.Tensor) -> torch.Tensor:
@@ -107,14 +131,14 @@ def _grow(st: Dict[str, torch.Tensor], key: str, new: torch.Tensor) -> torch.Ten
 def left_half(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, pos: torch.Tensor, st: Dict) -> torch.Tensor:
     H, G, dim = int(m["heads"]), int(m["kv_heads"]), int(m["dim"])
     T = h.shape[0]
-    q = (h @ w["q"].T + w["q.b"]).reshape(T, H, dim)
-    k = (h @ w["k"].T + w["k.b"]).reshape(T, G, dim)
+    q = (apply(w["q"], h) + w["q.b"]).reshape(T, H, dim)
+    k = (apply(w["k"], h) + w["k.b"]).reshape(T, G, dim)
     if m.get("q_temp"):
         q = q * temperature(pos, float(m["q_temp"]["coef"]), int(m["q_temp"]["every"])).to(q.dtype)[:, None, None]
     K = _grow(st, "k", k)
     o = attend(q, K, K, pos, float(m["scale"]), 0, w["sink"])
-    o = o * torch.sigmoid(h @ w["g"].T)[:, :, None]
-    return o.reshape(T, H * dim) @ w["o"].T + w["o.b"]
+    o = o * torch.sigmoid(apply(w["g"], h))[:, :, None]
+    return apply(w["o"], o.reshape(T, H * dim)) + w["o.b"]
 
 
 def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, i: torch.Tensor, f: torch.Tensor, S: torch.Tensor,
@@ -136,9 +160,9 @@ def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, i: torch.Te
 def right_half(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float, st: Dict) -> torch.Tensor:
     H, dim, vd, cap = int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"])
     T = h.shape[0]
-    q = (h @ w["q"].T).reshape(T, H, dim) * dim ** -0.5
-    k = (h @ w["k"].T).reshape(T, H, dim)
-    v = (h @ w["v"].T).reshape(T, H, vd)
+    q = (apply(w["q"], h)).reshape(T, H, dim) * dim ** -0.5
+    k = (apply(w["k"], h)).reshape(T, H, dim)
+    v = (apply(w["v"], h)).reshape(T, H, vd)
     i = cap * torch.tanh((h @ w["i"].T + w["i.b"]) / cap)
     f = log_sigmoid(cap * torch.tanh((h @ w["f"].T + w["f.b"]) / cap))
     if "S" not in st:
@@ -146,7 +170,7 @@ def right_half(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float,
                                      torch.zeros(H, dtype=h.dtype))
     o = matrix_memory(q, k, v, i, f, st["S"], st["n"], st["m"])
     o = norm(o, w["norm"].reshape(H, vd), eps).reshape(T, H * vd)
-    return (o * torch.sigmoid(h @ w["g"].T)) @ w["o"].T
+    return apply(w["o"], o * torch.sigmoid(apply(w["g"], h)))
 
 
 def parallel_mixer(h, wl, wr, ml, mr, pos, eps, st) -> torch.Tensor:
@@ -172,20 +196,20 @@ def block_map(u: torch.Tensor, M: torch.Tensor, b: torch.Tensor) -> torch.Tensor
 
 
 def rglru_mixer(h: torch.Tensor, w: Dict[str, torch.Tensor], st: Dict) -> torch.Tensor:
-    y = gelu_tanh(h @ w["y"].T + w["y.b"])
-    u = short_filter(h @ w["x"].T + w["x.b"], w["conv"], st, "taps") + w["conv.b"]
+    y = gelu_tanh(apply(w["y"], h) + w["y.b"])
+    u = short_filter(apply(w["x"], h) + w["x.b"], w["conv"], st, "taps") + w["conv.b"]
     r = torch.sigmoid(block_map(u, w["ra"], w["ra.b"]))
     i = torch.sigmoid(block_map(u, w["ri"], w["ri.b"]))
     if "S" not in st:
         st["S"] = torch.zeros(u.shape[1], dtype=h.dtype)
-    return (gated_scan(u, r, i, w["lam"], st["S"]) * y) @ w["o"].T
+    return apply(w["o"], gated_scan(u, r, i, w["lam"], st["S"]) * y)
 
 
 def attention_mixer(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, pos: torch.Tensor, eps: float,
                     st: Dict) -> torch.Tensor:
     H, G, dim, vd = int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"])
     T = h.shape[0]
-    q, k, v = (short_filter(h @ w[c].T + w[c + ".b"], w[c + ".conv"], st, c + ".taps") for c in "qkv")
+    q, k, v = (short_filter(apply(w[c], h) + w[c + ".b"], w[c + ".conv"], st, c + ".taps") for c in "qkv")
     q = norm(q.reshape(T, H, dim), w["q.norm"], eps)
     k = norm(k.reshape(T, G, dim), w["k.norm"], eps)
     rot = m.get("rot")
@@ -194,7 +218,7 @@ def attention_mixer(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, pos: t
         q, k = (turn(z, pos, float(rot["base"]), int(rot["dims"]), factor) for z in (q, k))
     K, V = _grow(st, "k", k), _grow(st, "v", v.reshape(T, G, vd))
     o = attend(q, K, V, pos, float(m["scale"]), int((m.get("mask") or {}).get("size") or 0))
-    return o.reshape(T, H * vd) @ w["o"].T
+    return apply(w["o"], o.reshape(T, H * vd))
 
 
 def route(z: torch.Tensor, top: int, n_groups: int, keep: int, factor: float):
@@ -214,7 +238,7 @@ def route(z: torch.Tensor, top: int, n_groups: int, keep: int, factor: float):
 
 
 def relu_squared_ff(h: torch.Tensor, up: torch.Tensor, down: torch.Tensor) -> torch.Tensor:
-    return torch.clamp(h @ up.T, min=0.0) ** 2 @ down.T
+    return apply(down, torch.clamp(apply(up, h), min=0.0) ** 2)
 
 
 def moe_ff(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict) -> torch.Tensor:

@@ -133,7 +133,7 @@ def _run_model(config: dict, batch: int, seqlen: int, warmup: int, steps: int, k
     prefill()
 
     def decode():
-        eng.step([StepEntry(f"s{i}", [7], [0]) for i in range(batch)])
+        eng.step([StepEntry(f"s{i}", [7 + i], [0]) for i in range(batch)])
     ms = _time_steps(decode, warmup, min(steps, 48))
     res["decode"] = {"ms_per_step": ms, "tokens_per_s": batch / ms * 1e3}
     # per-kernel device time of one prompt step and one decode step

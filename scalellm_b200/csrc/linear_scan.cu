@@ -365,21 +365,18 @@ gated_part_norm_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict
   extern __shared__ __align__(16) float sm[];
   float* u_s = sm;                                        // [n]
   float* r_s = sm + (n + 3) / 4 * 4;                      // [units] partial sums of squares
-  float* g_s = r_s + (parts < 8 ? 8 : parts);             // GATE_AFTER: [n] gates, asked for with the rows they meet
   constexpr int NW = kPartThreads / 32;
   const size_t row = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int i = threadIdx.x * 4; i < n; i += kPartThreads * 4) {
     float yv[4], zv[4];
     get4c<float>(y + row * n + i, yv, n - i, vec);
-    get4c<T>(z + row * ldz + i, zv, n - i, vec);
+    if constexpr (!GATE_AFTER) get4c<T>(z + row * ldz + i, zv, n - i, vec);
 #pragma unroll
     for (int k = 0; k < 4; ++k)
       if (i + k < n) {
-        if constexpr (GATE_AFTER) {
-          u_s[i + k] = yv[k];
-          g_s[i + k] = zv[k];
-        } else if constexpr (sizeof(T) == 4) u_s[i + k] = yv[k] * zv[k] * sigmoid_f(zv[k]);
+        if constexpr (GATE_AFTER) u_s[i + k] = yv[k];
+        else if constexpr (sizeof(T) == 4) u_s[i + k] = yv[k] * zv[k] * sigmoid_f(zv[k]);
         else u_s[i + k] = yv[k] * __fdividef(zv[k], 1.0f + __expf(-zv[k]));
       }
   }
@@ -415,11 +412,12 @@ gated_part_norm_kernel(T* __restrict__ out, int64_t ldo, const float* __restrict
       for (int k = 0; k < 4; ++k) o[k] = i + k < n ? u_s[i + k] * r_s[(i + k) / ps * per] * wv[k] : 0.0f;
     }
     if constexpr (GATE_AFTER) {
+      float zv[4];
+      get4c<T>(z + row * ldz + i, zv, n - i, vec);
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
-        const float z = i + k < n ? g_s[i + k] : 0.0f;
-        if constexpr (sizeof(T) == 4) o[k] *= sigmoid_f(z);
-        else o[k] = __fdividef(o[k], 1.0f + __expf(-z));
+        if constexpr (sizeof(T) == 4) o[k] *= sigmoid_f(zv[k]);
+        else o[k] = __fdividef(o[k], 1.0f + __expf(-zv[k]));
       }
     }
     T* dst = out + row * ldo + i;
@@ -1302,8 +1300,7 @@ int b200_gated_part_norm(void* out, int64_t ldo, const float* y, const void* z, 
   B200_CHECK_ARG(rows > 0 && n > 0 && parts > 0 && n % parts == 0 && ldo >= n && ldz >= n && (n + parts + 16) * 4 <= 200 * 1024,
                  "gated_part_norm: bad shape (the row in equal parts, at most ~50K channels)");
   auto st = static_cast<cudaStream_t>(stream);
-  const size_t smem = (size_t)((n + 3) / 4 * 4 + (parts < 8 ? 8 : parts) + (gate_after ? n : 0)) * sizeof(float);
-  B200_CHECK_ARG(smem <= 200 * 1024, "gated_part_norm: rows of at most ~25K channels with the gate after the norm");
+  const size_t smem = (size_t)((n + 3) / 4 * 4 + (parts < 8 ? 8 : parts)) * sizeof(float);
   SCAN_DISPATCH(dtype, {
     const int vec = n % 4 == 0 && ldo % 4 == 0 && ldz % 4 == 0 && is_aligned(out, 4 * sizeof(T)) &&
                     is_aligned(z, 4 * sizeof(T)) && is_aligned(y, 16) && is_aligned(weight, 16);

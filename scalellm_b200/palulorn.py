@@ -289,11 +289,12 @@ class PalulornDecoder:
             if lay.ff is not None:
                 x, h = lay.read2(x, y, dt, positions, params)
                 y = lay.ff(h)
+        rows = None if last_token_idxes is None else last_token_idxes.to(torch.int64)
+        if rows is not None and layer_out is None and (y is None or isinstance(y, torch.Tensor)):
+            x, y, rows = x.index_select(0, rows), None if y is None else y.index_select(0, rows), None
         x, h = self.final(x, y, dt, positions, params)
         if layer_out is not None:
             layer_out.append(x.clone())
-        if last_token_idxes is not None:
-            h = h.index_select(0, last_token_idxes.to(torch.int64))
-        return self.head(h)
+        return self.head(h if rows is None else h.index_select(0, rows))
 
     __call__ = forward

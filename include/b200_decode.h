@@ -867,6 +867,9 @@ B200_API int b200_branch_norm_residual(float* x_out, void* h_out /*nullable*/, c
 /* out [rows, n] = max(in, 0)^2 for the first n columns of rows with stride ld_in. */
 B200_API int b200_relu_squared(void* out, const void* in, int64_t rows, int64_t n, int64_t ld_in, int dtype,
                                b200_stream_t stream);
+/* The same fed by the split-K partials [n_slots][rows][n] of the product before it (plan6: b200_dense_splitk_plan). */
+B200_API int b200_relu_squared_splitk(void* out, const float* partials, int64_t n_slots, const int32_t* plan6,
+                                      int64_t rows, int64_t n, int dtype, b200_stream_t stream);
 
 /* ---- input side of pre-norm sublayers with short causal filters, linear recurrences with a matrix state whose decay
  * does not look at the state (filters.cu, linear_scan.cu).  The reference has no such operators; each entry states its

@@ -188,6 +188,7 @@ SIGNATURES = {
     "b200_branch_norm_residual": (_int, [_vp, _vp, _vp, _vp, _i64, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i64, _f32,
                                          _int, _vp]),
     "b200_relu_squared": (_int, [_vp, _vp, _i64, _i64, _i64, _int, _vp]),
+    "b200_relu_squared_splitk": (_int, [_vp, _vp, _i64, _vp, _i64, _i64, _int, _vp]),
     # pre-norm input side with short causal filters, linear recurrences with a matrix state (filters.cu, linear_scan.cu)
     "b200_prenorm": (_int, [_vp, _vp, _i64, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i64,
                             _i64, _i64, _f32, _int, _vp]),

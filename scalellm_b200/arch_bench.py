@@ -1097,11 +1097,13 @@ def palulorn_rooflines(s: dict, sf: dict, sg: dict, sk: dict, batch: int, seqlen
             4 * rows * (W * 2 + top * 8), 4 * rows * E * W * 2)
         put("fesupel router", fm.get("moe_route_softmax", 0.0), 3 * rows * (W * 2 + top * 8), 3 * rows * E * W * 2)
         npairs = rows * top
+        # (the experts' activation is part of the call: inside the kernel for decode-sized steps, a pass for prompts)
+        apass = npairs * eff * 4 if phase == "prefill" else 0
         put("palulorn expert GEMMs", pm.get("grouped_gemm", 0.0),
-            4 * (E * 2 * eff * W * 2 + npairs * (2 * W + 2 * eff) * 2), 4 * npairs * 4 * eff * W)
+            4 * (E * 2 * eff * W * 2 + npairs * (2 * W + 2 * eff) * 2 + apass), 4 * npairs * 4 * eff * W)
         put("fesupel expert GEMMs", fm.get("grouped_gemm", 0.0),
             3 * (E * 3 * sf["eff"] * W * 2 + npairs * (2 * W + 3 * sf["eff"]) * 2), 3 * npairs * 6 * sf["eff"] * W)
-        put("palulorn relu_squared", pm.get("relu_squared", 0.0), 4 * (npairs + rows) * eff * 4, 0)
+        put("palulorn relu_squared", pm.get("relu_squared", 0.0), 4 * (apass + rows * eff * 4), 0)
         put("fesupel glu_clamped", fm.get("glu_clamped", 0.0), 3 * (npairs + rows) * sf["eff"] * 6, 0)
         for name, m, n in (("palulorn", pm, 4), ("fesupel", fm, 3)):
             put(f"{name} moe_combine_weighted", m.get("moe_combine_weighted", 0.0), n * rows * W * 2 * (top + 2), 0)

@@ -496,6 +496,26 @@ __global__ void glu_clamped_splitk_kernel(T* __restrict__ out, const float* __re
   }
 }
 
+// the squared ReLU fed by the split-K partials of the product before it
+template <typename T>
+__global__ void relu_squared_splitk_kernel(T* __restrict__ out, const float* __restrict__ partials, W4Plan plan,
+                                           int64_t slot_stride, int64_t rows, int n) {
+  const int nv = n / 8;
+  const int64_t total = rows * nv;
+  for (int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
+       idx += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t r = idx / nv;
+    const int j = (int)(idx - r * nv);
+    float u[8];
+    w4_sum_partials8(u, partials + r * n + j * 8, slot_stride, w4_contrib_col(plan, j * 8));
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float v = fmaxf(rnd<T>(u[i]), 0.0f);
+      out[r * n + j * 8 + i] = Num<T>::from_f(v * v);
+    }
+  }
+}
+
 template <typename T>
 __global__ void token_gated_gelu_kernel(T* __restrict__ out, const T* __restrict__ in, int64_t ld_in,
                                         const T* __restrict__ table, int64_t ld_table, int col0,
@@ -671,6 +691,21 @@ int b200_glu_clamped_splitk(void* out, const float* partials, int64_t n_slots, c
   POSTNORM_DISPATCH(dtype, (glu_clamped_splitk_kernel<T><<<ew_grid(rows * (n / 8)), 256, 0, st>>>(
                                static_cast<T*>(out), partials, plan, rows * 2 * n, rows, (int)n, limit, slope)));
   B200_LAUNCH_OK("glu_clamped_splitk_kernel");
+  return B200_OK;
+}
+
+int b200_relu_squared_splitk(void* out, const float* partials, int64_t n_slots, const int32_t* plan6, int64_t rows,
+                             int64_t n, int dtype, b200_stream_t stream) {
+  if (rows == 0 || n == 0) return B200_OK;
+  B200_CHECK_ARG(out && partials && plan6, "relu_squared_splitk: null pointer");
+  B200_CHECK_ARG(rows > 0 && n > 0 && n % 8 == 0 && n < (1ll << 30) && n_slots == plan6[4] && n_slots <= W4_MAX_SLOTS &&
+                     is_aligned(partials, 16),
+                 "relu_squared_splitk: bad shape, or the partials are not those of the given partition");
+  auto st = static_cast<cudaStream_t>(stream);
+  const W4Plan plan = plan_of(plan6);
+  POSTNORM_DISPATCH(dtype, (relu_squared_splitk_kernel<T><<<ew_grid(rows * (n / 8)), 256, 0, st>>>(
+                               static_cast<T*>(out), partials, plan, rows * n, rows, (int)n)));
+  B200_LAUNCH_OK("relu_squared_splitk_kernel");
   return B200_OK;
 }
 

@@ -1638,8 +1638,17 @@ def branch_norm_residual(x: torch.Tensor, a: torch.Tensor, b: Optional[torch.Ten
     return out, h
 
 
-def relu_squared(x: torch.Tensor) -> torch.Tensor:
-    """max(x, 0)^2 of a [rows, n] matrix (rows may be strided)."""
+def relu_squared(x, dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
+    """max(x, 0)^2 of a [rows, n] matrix (rows may be strided), or of a product's split-K partials (then in `dtype`)."""
+    if isinstance(x, W4Partials):
+        data = x.data
+        _cuda(data)
+        _f32(data)
+        S, rows, n = data.shape
+        out = torch.empty((rows, n), dtype=dtype, device=data.device)
+        check(_lib.load().b200_relu_squared_splitk(_p(out), _p(data), S, splitk_plan(n, x.K), rows, n, _DT[dtype],
+                                                   _stream()))
+        return out
     _cuda(x)
     assert x.dim() == 2 and x.stride(1) == 1
     out = torch.empty(x.shape, dtype=x.dtype, device=x.device)

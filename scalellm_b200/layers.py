@@ -1217,13 +1217,13 @@ class ParallelMixer:
 
 
 class ReluSquaredMLP:
-    """down(max(up h, 0)^2)."""
+    """down(max(up h, 0)^2); decode-sized bf16 steps fold the up product's reduction into the activation launch."""
 
     def __init__(self, up: torch.Tensor, down: torch.Tensor):
         self.up, self.down = Linear(up), Linear(down)
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
-        return self.down(kernels.relu_squared(self.up(h)))
+        return self.down(kernels.relu_squared(self.up.forward_fusable(h), h.dtype))
 
     __call__ = forward
 

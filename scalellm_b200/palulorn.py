@@ -290,7 +290,8 @@ class PalulornDecoder:
                 x, h = lay.read2(x, y, dt, positions, params)
                 y = lay.ff(h)
         rows = None if last_token_idxes is None else last_token_idxes.to(torch.int64)
-        if rows is not None and layer_out is None and (y is None or isinstance(y, torch.Tensor)):
+        few = rows is not None and 2 * rows.numel() <= x.shape[0]       # the last norm runs over the asked rows only
+        if few and layer_out is None and (y is None or isinstance(y, torch.Tensor)):
             x, y, rows = x.index_select(0, rows), None if y is None else y.index_select(0, rows), None
         x, h = self.final(x, y, dt, positions, params)
         if layer_out is not None:

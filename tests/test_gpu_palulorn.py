@@ -508,6 +508,21 @@ def test_experts_layer(W, f, dtype):
         close(layer(d(h)), want, dtype, rows, tol=3e-5 if dtype == torch.float32 else 3e-2)
 
 
+@pytest.mark.parametrize("rows", [1, 16, 100])
+def test_squared_relu_feed_forward_takes_split_k_partials(rows):
+    from scalellm_b200 import kernels
+    from scalellm_b200.layers import ReluSquaredMLP
+    g = torch.Generator().manual_seed(rows)
+    up, down = ((torch.randn(n, k, generator=g) / math.sqrt(k)).to(torch.bfloat16) for n, k in ((384, 256), (256, 384)))
+    h = torch.randn(rows, 256, generator=g).to(torch.bfloat16)
+    ff = ReluSquaredMLP(up.to(DEV), down.to(DEV))
+    assert ff.up.supports_partials(rows)
+    a = kernels.relu_squared(ff.up.forward_partials(h.to(DEV)), torch.bfloat16)
+    close(a, torch.clamp(h.double() @ up.double().T, min=0.0) ** 2, torch.bfloat16)
+    assert torch.equal(a, kernels.relu_squared(ff.up(h.to(DEV))))
+    close(ff(h.to(DEV)), op.relu_squared_ff(h.double(), up.double(), down.double()), torch.bfloat16)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("W", [42, 256])
 def test_two_branches_join_without_a_norm_of_their_sum(W, dtype):

@@ -1110,9 +1110,10 @@ def palulorn_rooflines(s: dict, sf: dict, sg: dict, sk: dict, batch: int, seqlen
             put(f"{name} moe_plan", m.get("moe_plan", 0.0), n * npairs * 12, 0)
         put("palulorn branch_norm_residual", pm.get("branch_norm_residual", 0.0), 2 * rows * W * 14, 0)
         put("fesupel branch_norm_residual", fm.get("branch_norm_residual", 0.0), rows * W * s["layers"] * (14 + 12), 0)
-        # two loop inputs (x + y, 16 bits out, and x_0 once), two first reads (x + a row), three sums of 12 bytes a
-        # channel with a norm before a mixer, two before a feed-forward
-        put("palulorn prenorm", pm.get("prenorm", 0.0), rows * W * (6 + 6 + 12 + 2 * 10 + 3 * 12 + 2 * 12), 0)
+        # x_0 to 16 bits once, two loop inputs (the second with a sum), two first reads of a pass (x + a row), two sums
+        # before a mixer, two before a feed-forward; the last norm takes the asked rows only
+        put("palulorn prenorm", pm.get("prenorm", 0.0),
+            rows * W * (6 + 6 + 12 + 2 * 10 + 2 * 12 + 2 * 12 + (12 if phase == "decode" else 0)), 0)
         put("gugalorn prenorm", gm.get("prenorm", 0.0), rows * W * (6 * 12 + 6), 0)
         put("palulorn loop input product", pm.get(f"matmul_f32 {W}x{2 * W}", 0.0), 2 * (rows * W * 8 + W * W * 4),
             2 * rows * W * 2 * W * 2)
@@ -1160,6 +1161,10 @@ def palulorn_kernels_alone(s: dict, sg: dict, peaks: dict, cases=((64, 4096, 1),
         st2 = torch.zeros((batch, SH, sn, sv), dtype=torch.float32, device=dev)
         f_ssd = lambda: kernels.ssd_scan(xbc[:, :SH * sv], xbc[:, SH * sv: SH * sv + sgr * sn], xbc[:, SH * sv + sgr * sn:],
                                          dt, -4.0 * h1, h1, h1, st2, *step, sgr)
+        n, nv = sg["rheads"] * sg["rdim"], sg["rheads"] * sg["rvdim"]
+        rp, fb, low, wn = rnd(rows, 2 * n + nv), r32(n), torch.rand(n, device=dev), torch.ones(sg["rvdim"], device=dev)
+        st5 = torch.zeros((batch, sg["rheads"], sg["rdim"], sg["rvdim"]), dtype=torch.float32, device=dev)
+        f_fs = lambda: kernels.forget_scan(rp[:, :n], rp[:, n:2 * n], rp[:, 2 * n:], fb, low, wn, st5, *step, 1e-5, 0.7)
         u, y, gates = rnd(rows, gw), rnd(rows, gw), r32(nb, rows, 2 * gw // nb)
         c1, st3 = torch.ones(gw, device=dev), torch.zeros((batch, gw), dtype=torch.float32, device=dev)
         f_rg = lambda: kernels.real_gated_scan(u, y, gates, c1, c1, -4.0 * c1, c1, -8.0, st3, *step)
@@ -1175,6 +1180,7 @@ def palulorn_kernels_alone(s: dict, sg: dict, peaks: dict, cases=((64, 4096, 1),
                  pairs * H * 2 * (dim + vd)),
                 ("palulorn memory_scan", f_mem, _memory_bytes(rows, batch, s), rows * MH * 5 * N * V),
                 ("gugalorn ssd_scan", f_ssd, _ssd_bytes(rows, batch, sg), rows * SH * 5 * sn * sv),
+                ("gugalorn forget_scan, same heads", f_fs, _forget_bytes(rows, batch, sg), rows * sg["rheads"] * 5 * sg["rdim"] * sg["rvdim"]),
                 ("palulorn real_gated_scan", f_rg, rows * gw * 14 + batch * gw * 8, 0),
                 ("pokadra mingru_scan", f_mg, rows * gw * 8 + batch * gw * 8, 0)):
             ms = _time_steps(fn, 3, 10)
